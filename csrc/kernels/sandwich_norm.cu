@@ -1,0 +1,149 @@
+// Residual and norm steps of decoders whose residual stream is kept in fp32 and whose sublayers are normed before and
+// after: one launch does everything between two projections,
+//   x   <- embedding row                    (first layer)    or
+//   x   <- x + rms(y) * (bias + w_post)     (y = the sublayer's output, fp32)
+//   out <- rms(x) * (bias + w_pre)          (the next sublayer's input, bf16 or fp32, columns padded with zeros)
+// `bias` is 1 for weights stored around zero and 0 for plain weights. One block per row, the row stays in registers.
+#include "../common/pk_common.cuh"
+
+namespace {
+
+using namespace pk;
+
+struct NormParams {
+  float* x;              // [rows of the step, width] residual stream
+  const int* tokens;     // first layer: embedding ids (x is written)
+  const bf16* embed;
+  int vocab;
+  const float* y;        // [rows, ldy] or null
+  int ldy;
+  const float* w_post;
+  const int* rows;       // output row r works on residual row rows[r] (null: r); x is not written then
+  int width;
+  const float* w_pre;    // null: no output
+  float bias, eps;
+  void* out;             // [M, ldo]
+  int ldo;
+};
+
+// PT = values per thread held in registers
+template <typename OutT, int PT>
+__global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams p) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float scratch[33];
+  const int r = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  const int row = p.rows ? p.rows[r] : r;
+  float* xr = p.x + (size_t)row * p.width;
+  float v[PT];
+  if (p.tokens) {
+    int t = p.tokens[row];
+    t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
+    const bf16* e = p.embed + (size_t)t * p.width;
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      v[i] = c < p.width ? __bfloat162float(e[c]) : 0.f;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      v[i] = c < p.width ? xr[c] : 0.f;
+    }
+  }
+  if (p.y) {
+    const float* yr = p.y + (size_t)row * p.ldy;
+    float u[PT], ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      u[i] = c < p.width ? yr[c] : 0.f;
+      ss = fmaf(u[i], u[i], ss);
+    }
+    const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      if (c < p.width) v[i] += u[i] * rr * (p.bias + p.w_post[c]);
+    }
+  }
+  if (p.rows == nullptr && (p.tokens || p.y)) {
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      if (c < p.width) xr[c] = v[i];
+    }
+  }
+  if (p.w_pre) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < PT; ++i) ss = fmaf(v[i], v[i], ss);
+    const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
+    OutT* o = reinterpret_cast<OutT*>(p.out) + (size_t)r * p.ldo;
+#pragma unroll
+    for (int i = 0; i < PT; ++i) {
+      const int c = tid + i * nt;
+      if (c < p.width) o[c] = (OutT)(v[i] * rr * (p.bias + p.w_pre[c]));
+    }
+    for (int c = p.width + tid; c < p.ldo; c += nt) o[c] = (OutT)0.f;
+  }
+}
+
+template <typename OutT>
+int launch_norm(const NormParams& p, int M, cudaStream_t stream) {
+  const int nt = p.width >= 256 ? 256 : ((p.width + 31) / 32) * 32;
+  const int per = (p.width + nt - 1) / nt;
+#define PK_NORM_CASE(n)                                                                            \
+  if (per <= n) {                                                                                  \
+    PK_LAUNCH_PDL((sandwich_norm_kernel<OutT, n>), dim3(M), dim3(nt), (size_t)0, stream, p);       \
+    return PK_OK;                                                                                  \
+  }
+  PK_NORM_CASE(2)
+  PK_NORM_CASE(8)
+  PK_NORM_CASE(16)
+  PK_NORM_CASE(32)
+  PK_NORM_CASE(64)
+#undef PK_NORM_CASE
+  return PK_ERR_UNSUPPORTED;
+}
+
+// ---- per-sequence feedback of greedy decoding: next token and position stay on the device ----
+
+__global__ void feed_tokens_kernel(const int* next, int n, int* tokens, int* pos, int4* seqs, int* hist, int hist_ld, const int* step) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const int t = next[i];
+  const int s = step[0];
+  if (s < hist_ld) hist[(size_t)i * hist_ld + s] = t;
+  tokens[i] = t;
+  pos[i] += 1;
+  seqs[i].w += 1;
+}
+__global__ void bump_kernel(int* step) { step[0] += 1; }
+
+}  // namespace
+
+// See the head of this file. tokens != null: x is filled from the embedding table; y != null: the normed sublayer output is
+// added first. rows != null: only the M listed rows are normed (x stays as it is). width up to 16384.
+PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int vocab, const float* y, int ldy, const float* w_post,
+                            const int* rows, int M, int width, const float* w_pre, int plus_one, float eps, void* out, int ldo,
+                            int out_f32, cudaStream_t stream) {
+  if (M < 1 || width < 1 || x == nullptr) return PK_ERR_BAD_ARG;
+  if (y != nullptr && (w_post == nullptr || ldy < width)) return PK_ERR_BAD_ARG;
+  if (tokens != nullptr && (embed == nullptr || vocab < 1)) return PK_ERR_BAD_ARG;
+  if (w_pre != nullptr && (out == nullptr || ldo < width)) return PK_ERR_BAD_ARG;
+  NormParams p{x, tokens, (const pk::bf16*)embed, vocab, y, ldy, w_post, rows, width, w_pre, plus_one ? 1.f : 0.f, eps, out, ldo};
+  return out_f32 ? launch_norm<float>(p, M, stream) : launch_norm<pk::bf16>(p, M, stream);
+}
+
+// next [n] becomes the input token of every row, pos and the
+// sequence descriptors' position advance by one, the token is kept in hist[row, step] and step advances.
+PK_API int pk_feed_tokens(const int* next, int n, int* tokens, int* pos, void* seqs, int* hist, int hist_ld, int* step, cudaStream_t stream) {
+  if (n < 1 || hist_ld < 1) return PK_ERR_BAD_ARG;
+  feed_tokens_kernel<<<(n + 127) / 128, 128, 0, stream>>>(next, n, tokens, pos, (int4*)seqs, hist, hist_ld, step);
+  PK_CHECK_LAUNCH();
+  bump_kernel<<<1, 1, 0, stream>>>(step);
+  PK_CHECK_LAUNCH();
+  return PK_OK;
+}

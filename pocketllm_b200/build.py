@@ -12,11 +12,18 @@
 
 Objects are cached by source hash under `build/`, compiled in parallel, and nothing here
 needs a GPU (nvcc cross-compiles).
+
+A program that needs only part of the kernels can ask for a named set (`KERNEL_SETS`): `ensure_kernels("mixer")` returns the
+full kernel library when it is there and current, and otherwise compiles that set alone into
+`libpocket_kernels_mixer.so` (from the same object cache).
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import contextlib
+import fcntl
 import hashlib
+import json
 import os
 import shutil
 import subprocess
@@ -34,6 +41,13 @@ COMMON = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-Xcompiler",
           "-Xcompiler", "-Wall", "-Xcudafe", "--diag_suppress=177"]
 
 
+# translation units behind `ops.mixer_ops`
+KERNEL_SETS = {
+    "mixer": ["kernels/sandwich_norm.cu", "kernels/linear_f32.cu", "kernels/linear_rows.cu", "kernels/linear_state.cu", "kernels/latent_attention.cu",
+              "kernels/latent_prefill.cu", "kernels/gemm_bf16.cu", "kernels/misc.cu", "common/pk_status.cu"],
+}
+
+
 def _headers_digest() -> str:
     h = hashlib.sha256()
     for p in sorted(list(CSRC.rglob("*.cuh")) + list(CSRC.rglob("*.h")) + list(CSRC.rglob("*.hpp")) + list(CSRC.rglob("*.inc"))):
@@ -41,16 +55,65 @@ def _headers_digest() -> str:
     return h.hexdigest()
 
 
+def _source_key(src: Path, hdr_digest: str, extra: list[str]) -> str:
+    return hashlib.sha256(src.read_bytes() + hdr_digest.encode() + " ".join(extra).encode()).hexdigest()[:16]
+
+
+def _stamp(lib: Path) -> Path:
+    return lib.with_suffix(".stamp")
+
+
+def _write_stamp(lib: Path, srcs: list[Path], hdr: str) -> None:
+    """What a library was built from: {source: key}."""
+    _stamp(lib).write_text(json.dumps({str(s.relative_to(CSRC)): _source_key(s, hdr, []) for s in srcs}))
+
+
+def _current(lib: Path, srcs: list[Path], hdr: str) -> bool:
+    """Whether `lib` exists and holds these sources as they are now."""
+    try:
+        have = json.loads(_stamp(lib).read_text())
+    except (OSError, ValueError):
+        return False
+    return lib.exists() and all(have.get(str(s.relative_to(CSRC))) == _source_key(s, hdr, []) for s in srcs)
+
+
+@contextlib.contextmanager
+def _build_lock():
+    OBJ.mkdir(parents=True, exist_ok=True)
+    with open(OBJ.parent / ".lock", "w") as f:
+        fcntl.flock(f, fcntl.LOCK_EX)
+        yield
+
+
+def ensure_kernels(name: str, verbose: bool = False) -> Path:
+    """A kernel library that holds the set `name`, compiled now if there is none."""
+    srcs = [CSRC / s for s in KERNEL_SETS[name]]
+    hdr = _headers_digest()
+    full, part = OUT / "libpocket_kernels.so", OUT / f"libpocket_kernels_{name}.so"
+    for lib in (full, part):
+        if _current(lib, srcs, hdr):
+            return lib
+    with _build_lock():
+        if _current(part, srcs, hdr):
+            return part
+        OUT.mkdir(parents=True, exist_ok=True)
+        with cf.ThreadPoolExecutor(max_workers=min(len(srcs), max(1, os.cpu_count() or 4))) as ex:
+            objs = list(ex.map(lambda s: _compile_one(s, hdr, [], verbose), srcs))
+        tmp = part.with_suffix(f".{os.getpid()}.so")
+        _link(objs, tmp, True, ["-lcudart"], verbose)
+        tmp.rename(part)
+        _write_stamp(part, srcs, hdr)
+    return part
+
+
 def _compile_one(src: Path, hdr_digest: str, extra: list[str], verbose: bool) -> Path:
-    key = hashlib.sha256(src.read_bytes() + hdr_digest.encode() + " ".join(extra).encode()).hexdigest()[:16]
-    obj = OBJ / f"{src.stem}.{key}.o"
+    obj = OBJ / f"{src.stem}.{_source_key(src, hdr_digest, extra)}.o"
     if obj.exists():
         return obj
     OBJ.mkdir(parents=True, exist_ok=True)
-    if src.suffix == ".cu":
-        cmd = [NVCC, *ARCH, *COMMON, *extra, "-c", str(src), "-o", str(obj)]
-    else:
-        cmd = [NVCC, *COMMON, *extra, "-c", str(src), "-o", str(obj)]
+    part = obj.with_suffix(f".{os.getpid()}.tmp.o")          # renamed when complete: an interrupted compile leaves no object
+    arch = ARCH if src.suffix == ".cu" else []
+    cmd = [NVCC, *arch, *COMMON, *extra, "-c", str(src), "-o", str(part)]
     if verbose:
         print(" ".join(cmd), flush=True)
     r = subprocess.run(cmd, capture_output=True, text=True)
@@ -58,6 +121,7 @@ def _compile_one(src: Path, hdr_digest: str, extra: list[str], verbose: bool) ->
         raise RuntimeError(f"compile failed: {src}\n{r.stdout}\n{r.stderr}")
     if verbose and r.stderr.strip():
         print(r.stderr)
+    part.rename(obj)
     return obj
 
 
@@ -101,6 +165,7 @@ def build(verbose: bool = False, jobs: int | None = None) -> dict[str, Path]:
     arts: dict[str, Path] = {}
     kern_so = OUT / "libpocket_kernels.so"
     _link([objs[s] for s in kernel_srcs], kern_so, True, ["-lcudart"], verbose)
+    _write_stamp(kern_so, kernel_srcs, hdr)
     arts["kernels"] = kern_so
     dbg_so = OUT / "libpocket_kernels_debug.so"
     _link([dbg_objs[s] for s in kernel_srcs], dbg_so, True, ["-lcudart"], verbose)

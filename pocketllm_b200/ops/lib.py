@@ -37,6 +37,17 @@ def load(name: str) -> ctypes.CDLL:
     return lib
 
 
+def use_kernel_set(name: str) -> Path:
+    """Serve `kernels()` from a library that holds the kernel set `name` (`build.KERNEL_SETS`): the full one when it is built
+    and current, else one with that set alone, compiled on first use. Returns its path."""
+    if "kernels" in _libs:
+        return Path(_libs["kernels"]._name)
+    from .. import build
+    path = build.ensure_kernels(name)
+    _libs["kernels"] = ctypes.CDLL(str(path), mode=ctypes.RTLD_GLOBAL)
+    return path
+
+
 def available(name: str = "kernels") -> bool:
     return lib_path(name).exists()
 
