@@ -95,7 +95,7 @@ void usage() {
                "  --weight-source DIR|FILE.gguf [--lookup NAME | --lookup-expert LAYER,EXPERT,w1|w2|w3]   tensor lookup by model name\n"
                "  --serve [--host H --port P --model-name N --tokenizer chars|hf:DIR|gguf:FILE --chat-format qwen|glm|minimax|dsv4\n"
                "           --sidecar-python EXE --fake-engine-script TEXT --allow-shutdown]\n"
-               "  --serve --model-worker dsv4|gguf|qwen --ckpt PATH [--worker-tokenizer-path DIR] [--worker-ranks N]   serve a model family whose runtime is the\n"
+               "  --serve --model-worker dsv4|gguf|qwen|mixer --ckpt PATH [--worker-tokenizer-path DIR] [--worker-ranks N]   serve a model family whose runtime is the\n"
                "                 Python one: this process is the HTTP / SSE front end, generation runs in a worker process\n"
                "                 (python -m pocketllm_b200.server.model_worker) on the GPU\n");
 }

@@ -5,7 +5,7 @@
         [--max-new-tokens N] [--temperature T] [--top-p P] [--seed S] [--mtp] [--skip-special]
 
 `safetensors` directories hold a DeepSeek-V4 checkpoint (run by the DSV4 runtime, optionally with MTP speculative
-decoding); `gguf` files go through the architecture registry (MiniMax-M2, GLM-DSA). Tokenizer: a directory with
+decoding) or one of a registered architecture such as Gidisun (chosen by config.json); `gguf` files go through the architecture registry (MiniMax-M2, GLM-DSA). Tokenizer: a directory with
 `tokenizer.json`, the GGUF's own metadata, or `chars` (one token per character, for tiny test models).
 """
 from __future__ import annotations
@@ -35,6 +35,20 @@ def _load(args):
         render = (lambda m, thinking: chat.render_glm(m, thinking=thinking)) if arch == "glm-dsa" else (lambda m, thinking: chat.render_minimax(m, thinking=thinking))
         step = lambda t: rt.decode_one(t)
         return rt.prefill, step, None, tok, [i for i in (sp["eos"], sp["eot"]) if i is not None], render
+    from ..models import registry
+    if registry.folder_architecture(args.ckpt_path):
+        import os
+        rt = registry.build_runtime(args.ckpt_path, max_context=args.max_context, max_requests=1, dtype=getattr(torch, args.dtype))
+        tok = None
+        d = args.tokenizer_path or args.ckpt_path
+        if d != "chars" and os.path.exists(os.path.join(d, "tokenizer.json")):
+            from tokenizers import Tokenizer
+            tok = Tokenizer.from_file(os.path.join(d, "tokenizer.json"))
+
+        def prefill(ids):
+            rt.reset()
+            return rt.prefill(ids)
+        return prefill, rt.decode_one, rt, tok, [], lambda m, thinking: "\n".join(dsv4._text(x.get("content")) for x in m)
     from ..models import deepseek_v4_loader as ld
     from ..models.deepseek_v4_runtime import DSV4Runtime
     cfg, W = ld.load_checkpoint(args.ckpt_path)
@@ -65,6 +79,7 @@ def main(argv=None) -> int:
     ap.add_argument("--system-prompt", default=None)
     ap.add_argument("--max-new-tokens", type=int, default=64)
     ap.add_argument("--max-context", type=int, default=4096)
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="registered Safetensors architectures: precision of the run")
     ap.add_argument("--temperature", type=float, default=0.0)
     ap.add_argument("--top-p", type=float, default=1.0)
     ap.add_argument("--seed", type=int, default=0)
@@ -87,7 +102,7 @@ def main(argv=None) -> int:
             text = render(msgs, args.thinking)
         ids = enc(text)
         t0 = time.perf_counter()
-        if args.mtp and dsv4_rt is not None and args.temperature <= 0:
+        if args.mtp and hasattr(dsv4_rt, "generate_mtp") and args.temperature <= 0:
             out, stats = dsv4_rt.generate_mtp(ids, args.max_new_tokens)
             if any(t in eos for t in out):
                 out = out[:min(out.index(t) for t in eos if t in out)]
@@ -98,7 +113,8 @@ def main(argv=None) -> int:
                 out.append(t)
                 if args.temperature > 0 and dsv4_rt is not None:
                     from ..server.engine import SamplingParams, sample_token
-                    lg = dsv4_rt.forward_logits([t])[0]
+                    lg = dsv4_rt.forward_logits([t])
+                    lg = lg[0] if lg.dim() > 1 else lg
                     t = sample_token(lg.float().cpu(), SamplingParams(max_tokens=1, temperature=args.temperature, top_p=args.top_p), gen)
                 else:
                     t = step(t)

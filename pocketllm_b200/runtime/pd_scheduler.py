@@ -1,4 +1,5 @@
-"""Prefill/decode scheduler for a single-stream engine.
+"""Prefill/decode scheduler: one request at a time for the single-stream engines, or (`next_batch`) one mixed batch per
+step for runtimes that take several requests together.
 
 Requests wait in two queues; a request whose prefill is done moves to the decode queue, and
 decode work always runs before a new prefill (a started generation is never starved by
@@ -44,6 +45,7 @@ class PDScheduler:
         self.max_pending, self.decode_slice = max_pending, decode_slice
         self._prefill: list[_Item] = []
         self._decode: list[_Item] = []
+        self._started: dict[Any, _Item] = {}      # next_batch: (hashable) requests whose prompt has been admitted
         self._seq = itertools.count()
         self._lock = threading.Condition()
         self.phase: str | None = None
@@ -70,7 +72,7 @@ class PDScheduler:
         self.prefill_done(request, priority)
 
     def finish(self, request: Any) -> None:
-        pass
+        self._started.pop(request, None)
 
     def pending(self) -> tuple[int, int]:
         with self._lock:
@@ -92,6 +94,46 @@ class PDScheduler:
             self.stats["max_wait_s"] = max(self.stats["max_wait_s"], time.perf_counter() - item.enqueued)
         self.apply_phase_resources(item.phase)
         return item.request, item.phase
+
+    def next_batch(self, max_requests: int, token_budget: int, tokens_left: Callable[[Any], int],
+                   admit: Callable[[Any], bool]) -> list[tuple[Any, str, int]]:
+        """The work of one mixed step as (request, phase, tokens): every waiting generation with one token, then prompts in
+        order with what is left of the budget (the last one may be cut). `tokens_left` = prompt tokens a request has yet to
+        run; `admit` says whether there is room to start a request (asked once, the first time it comes up; when it
+        declines, the prompts behind it wait too). Each request handed out is given back with `prefill_more`,
+        `prefill_done` / `requeue_decode` or `finish`."""
+        out: list[tuple[Any, str, int]] = []
+        with self._lock:
+            while self._decode and len(out) < max_requests:
+                out.append((heapq.heappop(self._decode).request, "decode", 1))
+                self.stats["decode_slices"] += 1
+            budget = token_budget - len(out)
+            while self._prefill and len(out) < max_requests and budget > 0:
+                item = self._prefill[0]
+                if item.request not in self._started:
+                    if not admit(item.request):
+                        break
+                    self._started[item.request] = item
+                    self.stats["prefills"] += 1
+                    self.stats["max_wait_s"] = max(self.stats["max_wait_s"], time.perf_counter() - item.enqueued)
+                heapq.heappop(self._prefill)
+                n = min(budget, tokens_left(item.request))
+                out.append((item.request, "prefill", n))
+                budget -= n
+        return out
+
+    def prefill_more(self, request: Any) -> None:
+        """A portion of the prompt has run and more is left: the request keeps its place."""
+        with self._lock:
+            heapq.heappush(self._prefill, self._started[request])
+
+    def drop(self, request: Any) -> None:
+        """Forget a request that waits in either queue (cancelled)."""
+        with self._lock:
+            self._started.pop(request, None)
+            for q in (self._prefill, self._decode):
+                q[:] = [i for i in q if i.request != request]
+                heapq.heapify(q)
 
     def apply_phase_resources(self, phase: str) -> None:
         if phase == self.phase:

@@ -128,6 +128,47 @@ class DSV4Backend:
             logits = rt.forward_logits([tok])[-1]
 
 
+class MixerBackend:
+    """Runtime that takes mixed batches (`runtime.mixer_runtime.MixerRuntime`). The serving engine drives `batch` directly, so
+    requests join and leave between steps; `generate` and `generate_batch` serve callers with requests in hand."""
+
+    def __init__(self, runtime, token_budget: int = 2048):
+        from ..runtime.batching import BatchEngine
+        self.rt = runtime
+        self.batch = BatchEngine(runtime, token_budget=token_budget)
+        self.max_batch_size = runtime.max_requests
+
+    def generate(self, prompt_ids: Sequence[int], p: SamplingParams) -> Iterator[int]:
+        rid = self.batch.submit(prompt_ids, p)
+        try:
+            while rid in self.batch.requests:
+                for r, tok, _ in self.batch.step():
+                    if r == rid:
+                        yield tok
+        finally:
+            self.batch.cancel(rid)
+
+    def generate_batch(self, prompts: Sequence[Sequence[int]], params: Sequence[SamplingParams]) -> list[list]:
+        return self.batch.run(prompts, params)
+
+
+class CharTokenizer:
+    """One token per character, for models without a tokenizer (tests, random weights)."""
+    eos_ids: tuple[int, ...] = ()
+
+    def __init__(self, vocab: int):
+        self.vocab = vocab
+
+    def encode_chat(self, messages, **_):
+        return [ord(c) % self.vocab for m in messages for c in dsv4._text(m.get("content"))] or [0]
+
+    def decode(self, ids):
+        return "".join(chr(int(i)) for i in ids)
+
+    def parse(self, text: str, thinking: bool) -> dict:
+        return {"role": "assistant", "content": text}
+
+
 class HFChatTokenizer:
     """`tokenizers.Tokenizer` + a chat renderer + a completion parser."""
 
@@ -157,13 +198,23 @@ class HFChatTokenizer:
 
 def build(kind: str, ckpt: str, max_context: int, qwen_dspark: str | None = None, tokenizer_path: str | None = None,
           layer_pipeline: bool = False, speculative: tuple[str, int] = ("off", 4)):
-    """(backend, tokenizer) for `--model qwen|gguf|dsv4`. Under torchrun every rank builds its shard (rank and world come
+    """(backend, tokenizer) for `--model qwen|gguf|dsv4|mixer`. Under torchrun every rank builds its shard (rank and world come
     from the environment). `tokenizer_path`: directory with tokenizer.json when it is not the checkpoint directory.
     `layer_pipeline` (dsv4, several ranks): contiguous layer ranges per rank instead of expert parallelism.
     `speculative` = (mode, draft length) of the typed configuration: `ngram` gives the Qwen backend a prompt-lookup drafter
     (greedy requests run as draft + verify rounds with the same tokens as plain decoding)."""
     import os
     rank, world, local = int(os.environ.get("RANK", "0")), int(os.environ.get("WORLD_SIZE", "1")), int(os.environ.get("LOCAL_RANK", "0"))
+    if kind == "mixer":
+        # Safetensors folder of a registered architecture that runs as mixed batches
+        from ..models import registry
+        if world > 1:
+            raise ValueError("mixer models run on one rank")
+        rt = registry.build_runtime(ckpt, max_context=max_context)
+        tok_file = Path(tokenizer_path if tokenizer_path and tokenizer_path != "chars" else ckpt) / "tokenizer.json"
+        if tokenizer_path == "chars" or not tok_file.exists():
+            return MixerBackend(rt), CharTokenizer(rt.vocab)
+        return MixerBackend(rt), build_tokenizer("hf", str(tok_file.parent))
     if kind == "dsv4":
         from tokenizers import Tokenizer
         from ..models import deepseek_v4_loader as loader

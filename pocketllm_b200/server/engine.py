@@ -3,7 +3,8 @@
 HTTP handler threads submit work and read their tokens from a per-request queue. A backend that declares
 `max_batch_size > 1` and implements `generate_batch` gets compatible non-streaming requests together: the worker
 waits a short window (`batch_wait_ms`) for more requests with the same sampling parameters and runs them as one call;
-every other request runs alone. Same role as the reference's `DeepSeekServingEngine` (src/server/engine.py:
+every other request runs alone. A backend with a `batch` engine (`runtime.batching.BatchEngine`) is driven step by step
+instead: every request joins the running batch when there is room and leaves it when it ends. Same role as the reference's `DeepSeekServingEngine` (src/server/engine.py:
 queue + one worker thread, `_collect_batch`, `_is_batch_compatible`).
 """
 from __future__ import annotations
@@ -89,7 +90,8 @@ class ServingEngine:
         self._q: "queue.Queue[_Job | None]" = queue.Queue(max_queue)
         self._held: list[_Job] = []          # taken off the queue while looking for batch partners, to run next
         self.stats = {"requests": 0, "tokens": 0, "errors": 0, "batches": 0, "batched_requests": 0}
-        self._thread = threading.Thread(target=self._loop, name="pocket-serving", daemon=True)
+        target = self._loop_continuous if getattr(backend, "batch", None) is not None else self._loop
+        self._thread = threading.Thread(target=target, name="pocket-serving", daemon=True)
         self._thread.start()
 
     def _collect_batch(self, first: _Job) -> list[_Job]:
@@ -158,6 +160,65 @@ class ServingEngine:
                 job.out.put(e)
             finally:
                 job.out.put(_DONE)
+
+    def _loop_continuous(self) -> None:
+        """Step loop over the backend's batch engine; requests are taken off the queue while the batch has room."""
+        eng = self.backend.batch
+        live: dict[int, _Job] = {}
+        first: set[int] = set()
+        closing = False
+        while True:
+            while not closing and len(live) < eng.max_batch:
+                try:
+                    job = self._q.get(block=not live)
+                except queue.Empty:
+                    break
+                if job is None:
+                    closing = True
+                    break
+                try:
+                    rid = eng.submit(job.prompt_ids, job.params)
+                except Exception as e:
+                    self.stats["errors"] += 1
+                    job.out.put(e)
+                    job.out.put(_DONE)
+                    continue
+                live[rid] = job
+                first.add(rid)
+            if not live:
+                if closing:
+                    return
+                continue
+            try:
+                events = eng.step()
+            except Exception as e:                       # the step is lost for everybody in it; the worker survives
+                eng.abort_all()
+                self.stats["errors"] += len(live)
+                for job in live.values():
+                    job.out.put(e)
+                    job.out.put(_DONE)
+                live.clear()
+                first.clear()
+                continue
+            self.stats["batches"] += 1
+            self.stats["batched_requests"] += len(live)
+            for rid, tok, finished in events:
+                job = live.get(rid)
+                if job is None:
+                    continue
+                if rid in first:
+                    job.out.put(("ttft", time.perf_counter() - job.submitted))
+                    first.discard(rid)
+                job.out.put(tok if isinstance(tok, TokenInfo) else int(tok))
+                self.stats["tokens"] += 1
+                if finished:
+                    self.stats["requests"] += 1
+                    job.out.put(_DONE)
+                    del live[rid]
+            for rid in [r for r, j in live.items() if j.cancelled.is_set()]:
+                eng.cancel(rid)
+                live.pop(rid).out.put(_DONE)
+                first.discard(rid)
 
     def stream(self, prompt_ids: Sequence[int], params: SamplingParams, batchable: bool = False) -> Iterator[object]:
         """Yields ("ttft", seconds) once, then token ids (`TokenInfo` objects when log-probabilities were asked for); raises what the backend raised. `batchable`: the caller does

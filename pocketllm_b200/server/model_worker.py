@@ -1,4 +1,4 @@
-"""Model worker of the native server: one of the Python model backends (DeepSeek-V4 runtime, GGUF runtimes, the Qwen
+"""Model worker of the native server: one of the Python model backends (DeepSeek-V4 runtime, GGUF runtimes, mixer decoders, the Qwen
 engine's Python binding) behind a JSON-lines protocol on stdin / stdout, so that `pocket_engine --serve --model-worker KIND`
 can serve every model family from the C++ HTTP / SSE front end while generation runs here on the GPU.
 
@@ -96,7 +96,7 @@ def serve(backend, kind: str, max_context: int, stdin=sys.stdin, stdout=sys.stdo
 
 def main(argv=None) -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", required=True, choices=["qwen", "gguf", "dsv4", "scripted"])
+    ap.add_argument("--model", required=True, choices=["qwen", "gguf", "dsv4", "mixer", "scripted"])
     ap.add_argument("--ckpt", default="")
     ap.add_argument("--max-context", type=int, default=4096)
     ap.add_argument("--tokenizer-path", default=None)

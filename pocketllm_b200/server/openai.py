@@ -379,7 +379,7 @@ def serve(app: OpenAIApp, host: str = "127.0.0.1", port: int = 8000) -> Threadin
 
 def detect_model_kind(ckpt: str, ckpt_format: str = "auto") -> str:
     """Backend for a checkpoint path: a GGUF file with the deepseek4 architecture or a DeepSeek-V4 Safetensors directory ->
-    `dsv4`, any other GGUF file -> `gguf`, a directory whose config names Gated DeltaNet fields -> `qwen`."""
+    `dsv4`, any other GGUF file -> `gguf`, a folder whose config.json names a registered architecture -> `mixer`, a directory whose config names Gated DeltaNet fields -> `qwen`."""
     from pathlib import Path
     path = Path(ckpt)
     fmt = ckpt_format
@@ -389,6 +389,9 @@ def detect_model_kind(ckpt: str, ckpt_format: str = "auto") -> str:
         from ..formats import gguf
         arch = gguf.GGUFFile(gguf.shard_paths(str(path))[0]).architecture()
         return "dsv4" if arch == "deepseek4" else "gguf"
+    from ..models import registry
+    if registry.folder_architecture(path):
+        return "mixer"
     cfg_file = path / "config.json"
     text = cfg_file.read_text() if cfg_file.exists() else "{}"
     return "qwen" if ("linear_num_value_heads" in text or "linear_num_key_heads" in text) else "dsv4"
@@ -403,7 +406,7 @@ def parse_server_args(argv=None, env=None):
     from ..config import Config
     env = os.environ if env is None else env
     ap = argparse.ArgumentParser()
-    ap.add_argument("--model", default=None, help="backend (qwen | gguf | dsv4; default: detected from the checkpoint) or, for any other "
+    ap.add_argument("--model", default=None, help="backend (qwen | gguf | dsv4 | mixer; default: detected from the checkpoint) or, for any other "
                                                   "value, the model id reported by /v1/models")
     ap.add_argument("--ckpt", "--ckpt-path", dest="ckpt", default=env.get("CKPT_PATH"))
     ap.add_argument("--ckpt-format", choices=["auto", "safetensors", "gguf"], default=env.get("CKPT_FORMAT", "auto"))
@@ -418,7 +421,7 @@ def parse_server_args(argv=None, env=None):
                     help="dsv4 under several ranks: legacy / baseline_4gpu = routed experts split over the ranks, layer_pp / layer_pp_4gpu = "
                          "contiguous layer ranges per rank (layer pipeline)")
     ap.add_argument("--pd-mode", choices=["off", "scheduler"], default="off",
-                    help="accepted for compatibility: requests run one at a time on the GPUs, so there is no CPU expert server to pause between phases")
+                    help="accepted for compatibility: models other than `mixer` run one request at a time on the GPUs, so there is no CPU expert server to pause between phases")
     ap.add_argument("--routed-experts-device", choices=["gpu", "cpu"], default="gpu")
     ap.add_argument("--qwen-dspark", default="", help="qwen: directory of an external DSpark block drafter; greedy requests run as speculative rounds")
     args = ap.parse_args(argv)
@@ -427,7 +430,7 @@ def parse_server_args(argv=None, env=None):
     if args.routed_experts_device == "cpu":
         ap.error("--routed-experts-device cpu: routed experts run on the GPUs here (experts beyond HBM are staged from pinned host memory)")
     cfg = Config.load(args.config, profile=args.serving_profile or None, env=env)
-    kinds = ("qwen", "gguf", "dsv4")
+    kinds = ("qwen", "gguf", "dsv4", "mixer")
     kind = args.model if args.model in kinds else detect_model_kind(args.ckpt, args.ckpt_format)
     name = args.model_name or (args.model if args.model and args.model not in kinds else None) or cfg.serving.model_name
     settings = {"kind": kind, "model_name": name, "host": args.host or cfg.serving.host, "port": args.port if args.port is not None else cfg.serving.port,
