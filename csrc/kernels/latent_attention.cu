@@ -7,7 +7,8 @@
 //   gather   cached rows of the positions a long portion can see -> contiguous rows (input of the key / value GEMM)
 //   absorb   q~ = W_uk^T q per head (few rows: scores are taken on the latent, keys are never expanded)
 //   rows     split-context attention of single rows over the cache, eight heads per block, online softmax in fp32
-//   out      merge of the splits and the sink, then W_uv
+//   merge    sum of the splits, with the sink in the denominator
+//   out      W_uv per head
 // Scores, weights and accumulators are fp32 in all of them; the cache and the weights are bf16 or (fp32 mode) fp32.
 #include "../common/pk_common.cuh"
 
@@ -283,55 +284,62 @@ __global__ void __launch_bounds__(32 * HB) latent_rows_kernel(const RowsParams p
 }
 
 struct OutParams {
-  const float* part_o;
-  const float* part_ml;
+  const float* part_o;    // merged: split 0
   int nsplit, H, K, V;
-  const float* sink;      // [H] or null
   const int* rows;
   int nrows;
   void* out;              // [rows of the step, ldo]
   int ldo;
 };
 
-// Merge of the splits and the sink for up to 8 rows of one head, then out[row, h * V + v] = W_uv[h, v] . o~ for 64 values.
+// o~[row, h, k] = sum over the splits, divided by the whole denominator (sink included). Written over split 0.
+__global__ void __launch_bounds__(128) latent_merge_kernel(float* part_o, const float* part_ml, int nsplit, int H, int K, const float* sink) {
+  pdl_trigger();
+  pdl_wait();
+  extern __shared__ float ws[];       // [nsplit]
+  const int r = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
+  const float* ml = part_ml + ((size_t)r * nsplit * H + h) * 2;
+  if (tid < 32) {
+    float mx = sink ? sink[h] : -INFINITY;
+    for (int s = lane; s < nsplit; s += 32) mx = fmaxf(mx, ml[(size_t)s * H * 2]);
+    mx = warp_max(mx);
+    float den = 0.f;
+    for (int s = lane; s < nsplit; s += 32) {
+      const float m = ml[(size_t)s * H * 2];
+      const float e = m == -INFINITY ? 0.f : expf(m - mx);
+      ws[s] = e;
+      den += e * ml[(size_t)s * H * 2 + 1];
+    }
+    den = warp_sum(den) + (sink ? expf(sink[h] - mx) : 0.f);
+    __syncwarp();
+    for (int s = lane; s < nsplit; s += 32) ws[s] /= den;
+  }
+  __syncthreads();
+  const int k = blockIdx.z * 128 + tid;
+  if (k >= K) return;
+  float* o = part_o + ((size_t)r * nsplit * H + h) * K + k;
+  float a = 0.f;
+  // an empty split holds zeros: every term is finite
+#pragma unroll 8
+  for (int s = 0; s < nsplit; ++s) a = fmaf(ws[s], o[(size_t)s * H * K], a);
+  *o = a;
+}
+
+// out[row, h * V + v] = W_uv[h, v] . o~[row, h] for up to 8 rows of one head and 16 values.
 template <typename WT, typename OutT>
 __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p, const WT* uv) {
   pdl_trigger();
   pdl_wait();
-  extern __shared__ float sm[];       // o~ [8][K], weights [8][nsplit]
-  float* os = sm;
-  float* ws = sm + 8 * p.K;
+  extern __shared__ float os[];       // o~ [8][K]
   const int h = blockIdx.x, r0 = blockIdx.y * 8, nr = min(8, p.nrows - r0), tid = threadIdx.x;
   const int warp = tid >> 5, lane = tid & 31;
-  if (warp < nr) {
-    float mx = p.sink ? p.sink[h] : -INFINITY;
-    const float* ml = p.part_ml + ((size_t)(r0 + warp) * p.nsplit * p.H + h) * 2;
-    for (int s = lane; s < p.nsplit; s += 32) mx = fmaxf(mx, ml[(size_t)s * p.H * 2]);
-    mx = warp_max(mx);
-    float den = 0.f;
-    for (int s = lane; s < p.nsplit; s += 32) {
-      const float m = ml[(size_t)s * p.H * 2];
-      const float e = m == -INFINITY ? 0.f : expf(m - mx);
-      ws[warp * p.nsplit + s] = e;
-      den += e * ml[(size_t)s * p.H * 2 + 1];
-    }
-    den = warp_sum(den) + (p.sink ? expf(p.sink[h] - mx) : 0.f);
-    __syncwarp();
-    for (int s = lane; s < p.nsplit; s += 32) ws[warp * p.nsplit + s] /= den;
-  }
-  __syncthreads();
   for (int i = tid; i < nr * p.K; i += 256) {
     const int r = i / p.K, k = i - r * p.K;
-    float a = 0.f;
-    for (int s = 0; s < p.nsplit; ++s) {
-      const float w = ws[r * p.nsplit + s];
-      if (w != 0.f) a = fmaf(w, p.part_o[(((size_t)(r0 + r) * p.nsplit + s) * p.H + h) * p.K + k], a);
-    }
-    os[r * p.K + k] = a;
+    os[i] = p.part_o[((size_t)(r0 + r) * p.nsplit * p.H + h) * p.K + k];
   }
   __syncthreads();
   OutT* out = reinterpret_cast<OutT*>(p.out);
-  for (int v = blockIdx.z * 64 + warp; v < min(p.V, (int)blockIdx.z * 64 + 64); v += 8) {
+  for (int v = blockIdx.z * 16 + warp; v < min(p.V, (int)blockIdx.z * 16 + 16); v += 8) {
     const WT* w = uv + ((size_t)h * p.V + v) * p.K;
     float acc[8];
 #pragma unroll
@@ -436,12 +444,14 @@ PK_API int pk_latent_rows(const float* qx, const int* rows, int nrows, const int
   return PK_ERR_UNSUPPORTED;
 }
 
-PK_API int pk_latent_out(const float* part_o, const float* part_ml, int nsplit, int H, int K, int V, const float* sink, const int* rows, int nrows,
+// Merge of the splits (in place), then W_uv. sink [H] or null.
+PK_API int pk_latent_out(float* part_o, const float* part_ml, int nsplit, int H, int K, int V, const float* sink, const int* rows, int nrows,
                          const void* uv, int f32, void* out, int ldo, cudaStream_t stream) {
   if (nrows < 1 || nsplit < 1 || H < 1 || K < 1 || V < 1 || ldo < H * V) return PK_ERR_BAD_ARG;
-  OutParams p{part_o, part_ml, nsplit, H, K, V, sink, rows, nrows, out, ldo};
-  const size_t smem = (size_t)8 * (K + nsplit) * sizeof(float);
-  const dim3 grid(H, (nrows + 7) / 8, (V + 63) / 64);
+  PK_LAUNCH_PDL(latent_merge_kernel, dim3(nrows, H, (K + 127) / 128), dim3(128), (size_t)nsplit * sizeof(float), stream, part_o, part_ml, nsplit, H, K, sink);
+  OutParams p{part_o, nsplit, H, K, V, rows, nrows, out, ldo};
+  const size_t smem = (size_t)8 * K * sizeof(float);
+  const dim3 grid(H, (nrows + 7) / 8, (V + 15) / 16);
   if (f32) {
     static PkDeviceOnce once;
     const int rc = max_smem(latent_out_kernel<float, float>, once, smem);

@@ -480,12 +480,24 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const Mixer mx, const C
   const size_t head = (size_t)sq.z * mx.H + h;
   float* state = is_n ? mx.N + head * D + d : mx.S + head * D * V + e;
   float s = sq.w > 0 ? *state : 0.f;
-  for (int c = c0; c < c0 + n; ++c) {
-    const size_t ch = (size_t)c * mx.H + h;
-    float* kv = is_n ? wk.NK + ch * D + d : wk.KV + ch * D * V + e;
-    const float add = *kv;
-    *kv = s;
-    s = fmaf(wk.dec[ch * D + d], s, add);
+  float* kv = is_n ? wk.NK + ((size_t)c0 * mx.H + h) * D + d : wk.KV + ((size_t)c0 * mx.H + h) * D * V + e;
+  const float* dec = wk.dec + ((size_t)c0 * mx.H + h) * D + d;
+  const size_t kv_step = (size_t)mx.H * D * (is_n ? 1 : V), dec_step = (size_t)mx.H * D;
+  constexpr int AHEAD = 8;      // chunks whose loads are in flight together: only the fma chain is serial
+  for (int c = 0; c < n; c += AHEAD) {
+    float add[AHEAD], dc[AHEAD];
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if (c + i < n) {
+        add[i] = kv[(size_t)(c + i) * kv_step];
+        dc[i] = dec[(size_t)(c + i) * dec_step];
+      }
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i)
+      if (c + i < n) {
+        kv[(size_t)(c + i) * kv_step] = s;
+        s = fmaf(dc[i], s, add[i]);
+      }
   }
   *state = s;
 }

@@ -26,86 +26,145 @@ struct NormParams {
   int ldo;
 };
 
-// PT = values per thread held in registers
-template <typename OutT, int PT>
-__global__ void __launch_bounds__(256) sandwich_norm_kernel(const NormParams p) {
+// A thread holds PT groups of VW adjacent values of its row (VW = 4 when width and strides allow 16-byte accesses).
+template <int VW>
+__device__ __forceinline__ void load_f32(const float* p, float (&v)[VW]) {
+  if (VW == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1 % VW] = x.y; v[2 % VW] = x.z; v[3 % VW] = x.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VW>
+__device__ __forceinline__ void store(float* p, const float (&v)[VW]) {
+  if (VW == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % VW], v[2 % VW], v[3 % VW]);
+  else *p = v[0];
+}
+template <int VW>
+__device__ __forceinline__ void store(bf16* p, const float (&v)[VW]) {
+  if (VW == 4) {
+    const bf162 a = __floats2bfloat162_rn(v[0], v[1 % VW]), b = __floats2bfloat162_rn(v[2 % VW], v[3 % VW]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16(v[0]);
+  }
+}
+
+template <typename OutT, int PT, int VW>
+__global__ void __launch_bounds__(1024) sandwich_norm_kernel(const NormParams p) {
   pdl_trigger();
-  pdl_wait();
   __shared__ float scratch[33];
   const int r = blockIdx.x, tid = threadIdx.x, nt = blockDim.x;
+  // the norm weights are not written by any kernel: fetched before the wait
+  float wb[PT][VW], wa[PT][VW];
+#pragma unroll
+  for (int i = 0; i < PT; ++i) {
+    const int c = (tid + i * nt) * VW;
+    if (c < p.width) {
+      if (p.w_post) load_f32<VW>(p.w_post + c, wb[i]);
+      if (p.w_pre) load_f32<VW>(p.w_pre + c, wa[i]);
+    }
+  }
+  pdl_wait();
   const int row = p.rows ? p.rows[r] : r;
   float* xr = p.x + (size_t)row * p.width;
-  float v[PT];
+  float v[PT][VW], u[PT][VW];
   if (p.tokens) {
     int t = p.tokens[row];
     t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
     const bf16* e = p.embed + (size_t)t * p.width;
 #pragma unroll
-    for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      v[i] = c < p.width ? __bfloat162float(e[c]) : 0.f;
-    }
+    for (int i = 0; i < PT; ++i)
+#pragma unroll
+      for (int j = 0; j < VW; ++j) {
+        const int c = (tid + i * nt) * VW + j;
+        v[i][j] = c < p.width ? __bfloat162float(e[c]) : 0.f;
+      }
   } else {
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      v[i] = c < p.width ? xr[c] : 0.f;
+      const int c = (tid + i * nt) * VW;
+#pragma unroll
+      for (int j = 0; j < VW; ++j) v[i][j] = 0.f;
+      if (c < p.width) load_f32<VW>(xr + c, v[i]);
     }
   }
   if (p.y) {
     const float* yr = p.y + (size_t)row * p.ldy;
-    float u[PT], ss = 0.f;
+    float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      u[i] = c < p.width ? yr[c] : 0.f;
-      ss = fmaf(u[i], u[i], ss);
+      const int c = (tid + i * nt) * VW;
+#pragma unroll
+      for (int j = 0; j < VW; ++j) u[i][j] = 0.f;
+      if (c < p.width) load_f32<VW>(yr + c, u[i]);
+#pragma unroll
+      for (int j = 0; j < VW; ++j) ss = fmaf(u[i][j], u[i][j], ss);
     }
     const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
 #pragma unroll
-    for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      if (c < p.width) v[i] += u[i] * rr * (p.bias + p.w_post[c]);
-    }
+    for (int i = 0; i < PT; ++i)
+      if ((tid + i * nt) * VW < p.width) {
+#pragma unroll
+        for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * rr * (p.bias + wb[i][j]);
+      }
   }
   if (p.rows == nullptr && (p.tokens || p.y)) {
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      if (c < p.width) xr[c] = v[i];
+      const int c = (tid + i * nt) * VW;
+      if (c < p.width) store<VW>(xr + c, v[i]);
     }
   }
   if (p.w_pre) {
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < PT; ++i) ss = fmaf(v[i], v[i], ss);
+    for (int i = 0; i < PT; ++i)
+#pragma unroll
+      for (int j = 0; j < VW; ++j) ss = fmaf(v[i][j], v[i][j], ss);
     const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
     OutT* o = reinterpret_cast<OutT*>(p.out) + (size_t)r * p.ldo;
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
-      const int c = tid + i * nt;
-      if (c < p.width) o[c] = (OutT)(v[i] * rr * (p.bias + p.w_pre[c]));
+      const int c = (tid + i * nt) * VW;
+      if (c < p.width) {
+        float w[VW];
+#pragma unroll
+        for (int j = 0; j < VW; ++j) w[j] = v[i][j] * rr * (p.bias + wa[i][j]);
+        store<VW>(o + c, w);
+      }
     }
     for (int c = p.width + tid; c < p.ldo; c += nt) o[c] = (OutT)0.f;
   }
 }
 
-template <typename OutT>
+template <typename OutT, int VW>
 int launch_norm(const NormParams& p, int M, cudaStream_t stream) {
-  const int nt = p.width >= 256 ? 256 : ((p.width + 31) / 32) * 32;
-  const int per = (p.width + nt - 1) / nt;
-#define PK_NORM_CASE(n)                                                                            \
-  if (per <= n) {                                                                                  \
-    PK_LAUNCH_PDL((sandwich_norm_kernel<OutT, n>), dim3(M), dim3(nt), (size_t)0, stream, p);       \
-    return PK_OK;                                                                                  \
+  const int groups = (p.width + VW - 1) / VW;
+  // one row: as many threads as help its latency; many rows: smaller blocks with a few groups per thread
+  const int cap = M <= 64 ? 1024 : 512;
+  const int nt = groups >= cap ? (groups > 8 * cap ? 1024 : cap) : ((groups + 31) / 32) * 32;
+  const int per = (groups + nt - 1) / nt;
+#define PK_NORM_CASE(n)                                                                                \
+  if (per <= n) {                                                                                      \
+    PK_LAUNCH_PDL((sandwich_norm_kernel<OutT, n, VW>), dim3(M), dim3(nt), (size_t)0, stream, p);       \
+    return PK_OK;                                                                                      \
   }
+  PK_NORM_CASE(1)
   PK_NORM_CASE(2)
+  PK_NORM_CASE(4)
   PK_NORM_CASE(8)
-  PK_NORM_CASE(16)
-  PK_NORM_CASE(32)
-  PK_NORM_CASE(64)
 #undef PK_NORM_CASE
   return PK_ERR_UNSUPPORTED;
+}
+
+template <typename OutT>
+int launch_any(const NormParams& p, int M, cudaStream_t stream) {
+  const bool v4 = (p.width & 3) == 0 && ((uintptr_t)p.x & 15) == 0 && (p.y == nullptr || ((p.ldy & 3) == 0 && ((uintptr_t)p.y & 15) == 0)) &&
+                  (p.w_post == nullptr || ((uintptr_t)p.w_post & 15) == 0) &&
+                  (p.w_pre == nullptr || (((uintptr_t)p.w_pre & 15) == 0 && (p.ldo & 3) == 0 && ((uintptr_t)p.out & 15) == 0));
+  return v4 ? launch_norm<OutT, 4>(p, M, stream) : launch_norm<OutT, 1>(p, M, stream);
 }
 
 // ---- per-sequence feedback of greedy decoding: next token and position stay on the device ----
@@ -125,7 +184,7 @@ __global__ void bump_kernel(int* step) { step[0] += 1; }
 }  // namespace
 
 // See the head of this file. tokens != null: x is filled from the embedding table; y != null: the normed sublayer output is
-// added first. rows != null: only the M listed rows are normed (x stays as it is). width up to 16384.
+// added first. rows != null: only the M listed rows are normed (x stays as it is). width up to 8192 (32768 when a multiple of 4).
 PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int vocab, const float* y, int ldy, const float* w_post,
                             const int* rows, int M, int width, const float* w_pre, int plus_one, float eps, void* out, int ldo,
                             int out_f32, cudaStream_t stream) {
@@ -134,7 +193,7 @@ PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int 
   if (tokens != nullptr && (embed == nullptr || vocab < 1)) return PK_ERR_BAD_ARG;
   if (w_pre != nullptr && (out == nullptr || ldo < width)) return PK_ERR_BAD_ARG;
   NormParams p{x, tokens, (const pk::bf16*)embed, vocab, y, ldy, w_post, rows, width, w_pre, plus_one ? 1.f : 0.f, eps, out, ldo};
-  return out_f32 ? launch_norm<float>(p, M, stream) : launch_norm<pk::bf16>(p, M, stream);
+  return out_f32 ? launch_any<float>(p, M, stream) : launch_any<pk::bf16>(p, M, stream);
 }
 
 // next [n] becomes the input token of every row, pos and the

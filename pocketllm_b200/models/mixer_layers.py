@@ -204,7 +204,7 @@ class LatentAttentionMixer:
         self.row = pad_to(K + R, 64)
         self.cache = torch.zeros(pages, mo.PAGE, self.row, dtype=dtype, device=device)
         span = min(self.window, context) if self.window else context
-        self.nsplit = max(1, min(64, (span + 127) // 128))
+        self.nsplit = max(1, min(64, (span + 31) // 32))
         # expanded keys [k | rotated part] and values as one matrix over a cached row; the rotated part passes through
         self.qk_panels, self.v_panels = pad_to(D + R, 64) // 64, (V + 63) // 64
         if self.v_panels > 1:
