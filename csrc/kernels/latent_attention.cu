@@ -50,18 +50,20 @@ struct PrepParams {
   int qf_ld;
 };
 
+// Block (row, group of eight heads), one warp per head; the first group also writes the cache row.
 template <typename CT>
-__global__ void __launch_bounds__(128) latent_prep_kernel(const PrepParams p) {
+__global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
   pdl_trigger();
-  pdl_wait();
   extern __shared__ float sm[];      // cos, sin [R / 2] each
   __shared__ float scratch[33];
   const int t = blockIdx.x, tid = threadIdx.x, half = p.R / 2;
+  const int warp = tid >> 5, lane = tid & 31;
+  pdl_wait();
   const float* pr = p.proj + (size_t)t * p.ld;
   const int pos = p.pos[t];
   float* cs = sm;
   float* sn = sm + half;
-  for (int i = tid; i < half; i += 128) {
+  for (int i = tid; i < half; i += 256) {
     double a = (double)pos * p.freq[i];
     a -= 6.283185307179586476925286766559 * rint(a * 0.15915494309189533576888376337251);
     float s, c;
@@ -69,49 +71,41 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const PrepParams p) {
     cs[i] = c * p.mag;
     sn[i] = s * p.mag;
   }
-  float ss = 0.f;
-  for (int i = tid; i < p.K; i += 128) {
-    const float v = pr[p.oc + i];
-    ss = fmaf(v, v, ss);
-  }
-  const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.K + p.eps);   // also orders cs / sn
-  CT* dst = reinterpret_cast<CT*>(p.c.cache) + cache_row(p.c, p.slot[t], pos);
-  for (int i = tid; i < p.c.row; i += 128) {
-    float v = 0.f;
-    if (i < p.K) v = pr[p.oc + i] * r * p.c_norm[i];
-    else if (i < p.K + p.R) {
-      const int j = i - p.K;
-      const float* kr = pr + p.oc + p.K;
-      v = j < half ? kr[j] * cs[j] - kr[j + half] * sn[j] : kr[j] * cs[j - half] + kr[j - half] * sn[j - half];
+  if (blockIdx.y == 0) {
+    float ss = 0.f;
+    for (int i = tid; i < p.K; i += 256) {
+      const float v = pr[p.oc + i];
+      ss = fmaf(v, v, ss);
     }
-    dst[i] = (CT)v;
-  }
-  const int QD = p.D + p.R;
-  if (p.qx) {
-    const int w = p.c.row - p.K;
-    for (int i = tid; i < p.H * w; i += 128) {
-      const int h = i / w, j = i - h * w;
+    const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.K + p.eps);   // also orders cs / sn
+    CT* dst = reinterpret_cast<CT*>(p.c.cache) + cache_row(p.c, p.slot[t], pos);
+    for (int i = tid; i < p.c.row; i += 256) {
       float v = 0.f;
-      if (j < p.R) {
-        const float* q = pr + p.oq + h * QD + p.D;
-        v = j < half ? q[j] * cs[j] - q[j + half] * sn[j] : q[j] * cs[j - half] + q[j - half] * sn[j - half];
+      if (i < p.K) v = pr[p.oc + i] * r * p.c_norm[i];
+      else if (i < p.K + p.R) {
+        const int j = i - p.K;
+        const float* kr = pr + p.oc + p.K;
+        v = j < half ? kr[j] * cs[j] - kr[j + half] * sn[j] : kr[j] * cs[j - half] + kr[j - half] * sn[j - half];
       }
-      p.qx[((size_t)t * p.H + h) * p.c.row + p.K + j] = v;
+      dst[i] = (CT)v;
     }
+  } else {
+    __syncthreads();
+  }
+  const int h = blockIdx.y * 8 + warp;
+  if (h >= p.H) return;
+  const float* q = pr + p.oq + h * (p.D + p.R);
+  const float* qr = q + p.D;
+  auto rotated = [&](int j) {
+    return j < half ? qr[j] * cs[j] - qr[j + half] * sn[j] : qr[j] * cs[j - half] + qr[j - half] * sn[j - half];
+  };
+  if (p.qx) {
+    float* dst = p.qx + ((size_t)t * p.H + h) * p.c.row + p.K;
+    for (int j = lane; j < p.c.row - p.K; j += 32) dst[j] = j < p.R ? rotated(j) : 0.f;
   }
   if (p.qf) {
-    for (int i = tid; i < p.H * p.qf_ld; i += 128) {
-      const int h = i / p.qf_ld, j = i - h * p.qf_ld;
-      const float* q = pr + p.oq + h * QD;
-      float v = 0.f;
-      if (j < p.D) v = q[j];
-      else if (j < QD) {
-        const int e = j - p.D;
-        q += p.D;
-        v = e < half ? q[e] * cs[e] - q[e + half] * sn[e] : q[e] * cs[e - half] + q[e - half] * sn[e - half];
-      }
-      p.qf[((size_t)t * p.H + h) * p.qf_ld + j] = __float2bfloat16(v);
-    }
+    bf16* dst = p.qf + ((size_t)t * p.H + h) * p.qf_ld;
+    for (int j = lane; j < p.qf_ld; j += 32) dst[j] = __float2bfloat16(j < p.D ? q[j] : j < p.D + p.R ? rotated(j - p.D) : 0.f);
   }
 }
 
@@ -396,8 +390,9 @@ PK_API int pk_latent_prep(const float* proj, int ld, int oq, int oc, int M, int 
   if (qf != nullptr && qf_ld < D + R) return PK_ERR_BAD_ARG;
   PrepParams p{proj, ld, oq, oc, H, D, R, K, c_norm, eps, freq, mag, pos, slot, Paged{cache, table, table_ld, row}, qx, (pk::bf16*)qf, qf_ld};
   const size_t smem = (size_t)(R + 2) * sizeof(float);
-  if (cache_f32) PK_LAUNCH_PDL(latent_prep_kernel<float>, dim3(M), dim3(128), smem, stream, p);
-  else PK_LAUNCH_PDL(latent_prep_kernel<pk::bf16>, dim3(M), dim3(128), smem, stream, p);
+  const dim3 grid(M, (qx != nullptr || qf != nullptr) ? (H + 7) / 8 : 1);
+  if (cache_f32) PK_LAUNCH_PDL(latent_prep_kernel<float>, grid, dim3(256), smem, stream, p);
+  else PK_LAUNCH_PDL(latent_prep_kernel<pk::bf16>, grid, dim3(256), smem, stream, p);
   return PK_OK;
 }
 

@@ -570,40 +570,48 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
 // ---------------------------------------------------------------------------------------
 // normalisation, output gate
 
-// One warp per (row, head). norm_w: [H * V] (per_head = 0) or [V] shared by the heads. last_slot[row] = slot whose portion
+// One block per (head, row). norm_w: [H * V] (per_head = 0) or [V] shared by the heads. last_slot[row] = slot whose portion
 // ends at this row, or -1: mLSTM's running maximum is stored there once every reader of the old one is done.
 template <int KIND, typename OutT>
 __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, int per_head, float eps,
-                                                        const int* last_slot, int rows, OutT* out, int ldo) {
+                                                        const int* last_slot, OutT* out, int ldo) {
   pdl_trigger();
   pdl_wait();
-  const int unit = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  __shared__ float scratch[33];
+  constexpr int KEEP = 4;       // values per thread that stay in registers between the two passes
+  const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
   const int H = mx.H, V = mx.V;
-  if (unit < rows * H) {
-    const int t = unit / H, h = unit - t * H;
-    const float* o = raw.o + (size_t)unit * V;
-    float inv = 1.f;
-    if (KIND == KIND_MLSTM) {
-      const float m = raw.m[unit];
-      inv = 1.f / (fmaxf(fabsf(raw.nq[unit]), expf(-m)) + 1e-6f);
-      if (lane == 0 && last_slot[t] >= 0) mx.Ms[(size_t)last_slot[t] * H + h] = m;
-    }
-    float ss = 0.f;
-    for (int v = lane; v < V; v += 32) {
-      const float x = o[v] * inv;
-      ss = fmaf(x, x, ss);
-    }
-    const float r = 1.f / sqrtf(warp_sum(ss) / (float)V + eps);
-    const float* gate = mx.proj + (size_t)t * mx.ld + mx.og + h * V;
-    OutT* dst = out + (size_t)t * ldo + h * V;
-    for (int v = lane; v < V; v += 32) {
-      const float z = gate[v];
-      const float s = 1.f / (1.f + expf(-z));
-      dst[v] = (OutT)(o[v] * inv * r * norm_w[per_head ? v : h * V + v] * (KIND == KIND_MLSTM ? s : z * s));
-    }
-    if (h == H - 1)
-      for (int v = H * V + lane; v < ldo; v += 32) out[(size_t)t * ldo + v] = (OutT)0.f;
+  const size_t unit = (size_t)t * H + h;
+  const float* o = raw.o + unit * V;
+  const float* gate = mx.proj + (size_t)t * mx.ld + mx.og + h * V;
+  float x[KEEP], z[KEEP], inv = 1.f, ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int v = tid + i * nt;
+    x[i] = v < V ? o[v] : 0.f;
+    z[i] = v < V ? gate[v] : 0.f;
   }
+  if (KIND == KIND_MLSTM) {
+    const float m = raw.m[unit];
+    inv = 1.f / (fmaxf(fabsf(raw.nq[unit]), expf(-m)) + 1e-6f);
+    if (tid == 0 && last_slot[t] >= 0) mx.Ms[(size_t)last_slot[t] * H + h] = m;
+  }
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) ss = fmaf(x[i] * inv, x[i] * inv, ss);
+  for (int v = tid + KEEP * nt; v < V; v += nt) ss = fmaf(o[v] * inv, o[v] * inv, ss);
+  const float r = inv / sqrtf(block_sum(ss, scratch) / (float)V + eps);
+  OutT* dst = out + (size_t)t * ldo + h * V;
+  const float* w = norm_w + (per_head ? 0 : h * V);
+  auto put = [&](int v, float xv, float zv) {
+    const float s = 1.f / (1.f + expf(-zv));
+    dst[v] = (OutT)(xv * r * w[v] * (KIND == KIND_MLSTM ? s : zv * s));
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if (tid + i * nt < V) put(tid + i * nt, x[i], z[i]);
+  for (int v = tid + KEEP * nt; v < V; v += nt) put(v, o[v], gate[v]);
+  if (h == H - 1)
+    for (int v = H * V + tid; v < ldo; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
 }
 
 template <int KIND>
@@ -742,13 +750,15 @@ PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head
   Mixer mx;
   Raw raw;
   if (!unpack(d, mx, raw) || norm_w == nullptr || last_slot == nullptr || rows < 1 || out == nullptr || ldo < mx.H * mx.V) return PK_ERR_BAD_ARG;
-  const dim3 grid((rows * mx.H + 7) / 8), block(256);
+  if (rows > 65535) return PK_ERR_BAD_ARG;
+  const int nt = (mx.V + 31) / 32 * 32;
+  const dim3 grid(mx.H, rows), block(nt < 256 ? nt : 256);
   if (d->kind == KIND_GLA) {
-    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, rows, (float*)out, ldo);
-    else PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, rows, (pk::bf16*)out, ldo);
+    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
+    else PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
   } else {
-    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, rows, (float*)out, ldo);
-    else PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, rows, (pk::bf16*)out, ldo);
+    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
+    else PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
   }
   return PK_OK;
 }

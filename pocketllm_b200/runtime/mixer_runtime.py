@@ -82,6 +82,7 @@ class _DecodeBatch:
         self.best_val, self.best = torch.zeros(n, device=device), torch.zeros(n, **i32)
         self.logits = None
         self.warm = False
+        self.nodes = self.feed_nodes = 0
         self.graph = None          # forward + logits
         self.feed_warm = False
         self.feed_graph = None     # forward + logits + greedy pick + feedback
@@ -100,7 +101,7 @@ class MixerRuntime:
         self._dec: dict[int, _DecodeBatch] = {}
         self._pinned = torch.zeros(8 * max_requests, dtype=torch.int32).pin_memory()
         self._copied = torch.cuda.Event()
-        self._single_pos = 0
+        self.launches = 0                          # kernels launched so far, graph nodes counted per replay
         self.launch_layers: list | None = None     # set to a list to collect the residual stream after every layer
 
     @property
@@ -146,7 +147,9 @@ class MixerRuntime:
         if all(len(e.tokens) == 1 for e in entries) and len(entries) <= mo.ROWS_MAX:
             logits = self._decode(entries)
         else:
+            n0 = mo.launches
             logits = self._mixed(entries)
+            self.launches += mo.launches - n0
         for e in entries:
             self.cache.advance(e.rid, len(e.tokens))
         return logits
@@ -243,17 +246,20 @@ class MixerRuntime:
         return self._forward(ctx, None, b.n)
 
     def _decode(self, entries: Sequence[StepEntry]) -> torch.Tensor:
-        b = self._batch(len(entries))
+        b, n0 = self._batch(len(entries)), mo.launches
         self._load_batch(b, [e.rid for e in entries], [int(e.tokens[0]) for e in entries])
         if not b.warm or not self.use_graphs or self.launch_layers is not None:
             b.logits, b.warm = self._decode_forward(b), True            # sizes every buffer of this batch size
+            self.launches += mo.launches - n0
         else:
             if b.graph is None:
                 torch.cuda.synchronize()
                 b.graph = torch.cuda.CUDAGraph()
                 with torch.cuda.graph(b.graph):
                     b.logits = self._decode_forward(b)
+                b.nodes = mo.launches - n0
             b.graph.replay()
+            self.launches += b.nodes
         want = [i for i, e in enumerate(entries) for _ in e.want]
         z = b.logits[:, :self.vocab]
         return z if want == list(range(b.n)) else z[want]
@@ -274,17 +280,22 @@ class MixerRuntime:
         b = self._batch(len(rids))
         self._load_batch(b, rids, tokens)
         b.step.zero_()
-        done = 0
+        done, n0 = 0, mo.launches
         if not b.feed_warm or not self.use_graphs:
             self._feed_step(b)
             b.feed_warm, done = True, 1
+            self.launches += mo.launches - n0
         if self.use_graphs and b.feed_graph is None and done < steps:
             torch.cuda.synchronize()
+            n0 = mo.launches
             b.feed_graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(b.feed_graph):
                 self._feed_step(b)
+            b.feed_nodes = mo.launches - n0
+        n0 = mo.launches
         for _ in range(done, steps):
             b.feed_graph.replay() if self.use_graphs else self._feed_step(b)
+        self.launches += (steps - done) * b.feed_nodes if self.use_graphs else mo.launches - n0
         out = b.hist[:, :steps].tolist()
         for r in rids:
             self.cache.advance(r, steps)

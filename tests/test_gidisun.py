@@ -241,3 +241,18 @@ def test_kernel_set_is_compiled_only_when_needed(tmp_path, monkeypatch):
     assert build.ensure_kernels("mixer") == lib            # no record of what the full library was built from
     build._write_stamp(full, [build.CSRC / s for s in build.KERNEL_SETS["mixer"]], build._headers_digest())
     assert build.ensure_kernels("mixer") == full
+
+
+def test_argument_kinds_match_the_launchers():
+    """The ctypes prototypes of `ops.mixer_ops` against the C signatures in the sources."""
+    import re
+
+    from pocketllm_b200 import build
+    from pocketllm_b200.ops import mixer_ops as mo
+    src = "\n".join((build.CSRC / s).read_text() for s in build.KERNEL_SETS["mixer"])
+    for name, kinds in mo._SIGNATURES.items():
+        m = re.search(r"PK_API int " + name + r"\(([^)]*)\)", src)
+        params = [p.strip() for p in m.group(1).split(",")]
+        assert params[-1] == "cudaStream_t stream"
+        got = "".join("p" if "*" in p else "f" if p.startswith("float") else "i" for p in params[:-1])
+        assert got == kinds, name
