@@ -143,7 +143,7 @@ __global__ void __launch_bounds__(512) latent_absorb_kernel(const float* proj, i
   for (int r = 0; r < 8; ++r) acc[r] = 0.f;
   if (k < K) {
     const WT* w = uk + (size_t)h * D * K + k;
-#pragma unroll 8
+#pragma unroll 16
     for (int d = grp; d < D; d += 4) {
       const float wv = to_f<WT>(w[(size_t)d * K]);
 #pragma unroll
@@ -194,7 +194,12 @@ __global__ void __launch_bounds__(32 * HB) latent_rows_kernel(const RowsParams p
   const int per = ((n + p.nsplit - 1) / p.nsplit + TK - 1) / TK * TK;
   const int s0 = first + sp * per, s1 = min(pos + 1, s0 + per);
   const int nh = min(HB, p.H - h0);
-  for (int i = tid; i < HB * row; i += 32 * HB) qs[i] = i < nh * row ? p.qx[((size_t)t * p.H + h0) * row + i] : 0.f;
+  {
+    const float4* src = reinterpret_cast<const float4*>(p.qx + ((size_t)t * p.H + h0) * row);
+#pragma unroll 5
+    for (int i = tid; i < HB * row / 4; i += 32 * HB)
+      reinterpret_cast<float4*>(qs)[i] = i < nh * row / 4 ? src[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
   float m = -INFINITY, l = 0.f;
   float acc[CP][2][HB];
 #pragma unroll
@@ -205,14 +210,24 @@ __global__ void __launch_bounds__(32 * HB) latent_rows_kernel(const RowsParams p
   for (int k0 = s0; k0 < s1; k0 += TK) {
     const int nk = min(TK, s1 - k0);
     __syncthreads();
-    for (int i = tid; i < TK * vec; i += 32 * HB) {
-      const int r = i / vec, v = i - r * vec;
-      uint4 x = make_uint4(0, 0, 0, 0);
-      if (r < nk) x = *reinterpret_cast<const uint4*>(reinterpret_cast<const CT*>(p.c.cache) + cache_row(p.c, slot, k0 + r) + v * VE);
-      *reinterpret_cast<uint4*>(ks + r * kld + v * VE) = x;
+    // four rows per warp; their addresses first, so that all loads of a column of lanes are in flight together
+    constexpr int RW = TK / HB;
+    const CT* src[RW];
+#pragma unroll
+    for (int j = 0; j < RW; ++j) {
+      const int r = warp + j * HB;
+      src[j] = reinterpret_cast<const CT*>(p.c.cache) + cache_row(p.c, slot, k0 + min(r, nk - 1));
+    }
+#pragma unroll 3
+    for (int v = lane; v < vec; v += 32) {
+      uint4 x[RW];
+#pragma unroll
+      for (int j = 0; j < RW; ++j) x[j] = *reinterpret_cast<const uint4*>(src[j] + v * VE);
+#pragma unroll
+      for (int j = 0; j < RW; ++j) *reinterpret_cast<uint4*>(ks + (warp + j * HB) * kld + v * VE) = x[j];
     }
     __syncthreads();
-    float s = 0.f;
+    float s4[4] = {0.f, 0.f, 0.f, 0.f};
     {
       const CT* kr = ks + lane * kld;
       const float* q = qs + warp * row;
@@ -221,10 +236,10 @@ __global__ void __launch_bounds__(32 * HB) latent_rows_kernel(const RowsParams p
         const uint4 raw = *reinterpret_cast<const uint4*>(kr + v);
         const CT* ke = reinterpret_cast<const CT*>(&raw);
 #pragma unroll
-        for (int e = 0; e < VE; ++e) s = fmaf(to_f<CT>(ke[e]), q[v + e], s);
+        for (int e = 0; e < VE; ++e) s4[e & 3] = fmaf(to_f<CT>(ke[e]), q[v + e], s4[e & 3]);
       }
     }
-    s = lane < nk ? s * p.scale : -INFINITY;
+    const float s = lane < nk ? ((s4[0] + s4[1]) + (s4[2] + s4[3])) * p.scale : -INFINITY;
     const float mn = fmaxf(m, warp_max(s));
     const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
     const float e = lane < nk ? expf(s - mn) : 0.f;
@@ -338,7 +353,7 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p, cons
     float acc[8];
 #pragma unroll
     for (int r = 0; r < 8; ++r) acc[r] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
     for (int k = lane; k < p.K; k += 32) {
       const float wv = to_f<WT>(w[k]);
 #pragma unroll

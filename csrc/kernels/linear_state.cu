@@ -467,39 +467,56 @@ __global__ void __launch_bounds__(256) chunk_kv_kernel(const Mixer mx, const Chu
   }
 }
 
-// Serial over the chunks of a sequence, one thread per state element: KV[c] <- state before chunk c, slot <- final state.
+// Serial over the chunks of a sequence, one thread per VW adjacent state elements: KV[c] <- state before chunk c, slot <-
+// final state.
+template <int VW>
 __global__ void __launch_bounds__(256) chunk_scan_kernel(const Mixer mx, const Chunks ck, const Work wk) {
   const int4 sq = ck.seqs[blockIdx.z];
   const int h = blockIdx.y, D = mx.D, V = mx.V;
-  const int e = blockIdx.x * 256 + threadIdx.x;      // element of [D, V], then of [D]
-  const int total = D * V + (wk.NK != nullptr ? D : 0);
-  if (e >= total) return;
-  const bool is_n = e >= D * V;
-  const int d = is_n ? e - D * V : e / V;
+  const int g = blockIdx.x * 256 + threadIdx.x;      // group of [D, V / VW], then element of [D]
+  const int groups = D * V / VW;
+  if (g >= groups + (wk.NK != nullptr ? D : 0)) return;
+  const bool is_n = g >= groups;
+  const int d = is_n ? g - groups : g * VW / V;
   const int c0 = ck.chunk0[blockIdx.z], n = (sq.y + CH - 1) / CH;
   const size_t head = (size_t)sq.z * mx.H + h;
-  float* state = is_n ? mx.N + head * D + d : mx.S + head * D * V + e;
-  float s = sq.w > 0 ? *state : 0.f;
-  float* kv = is_n ? wk.NK + ((size_t)c0 * mx.H + h) * D + d : wk.KV + ((size_t)c0 * mx.H + h) * D * V + e;
+  float* state = is_n ? mx.N + head * D + d : mx.S + head * D * V + (size_t)g * VW;
+  float* kv = is_n ? wk.NK + ((size_t)c0 * mx.H + h) * D + d : wk.KV + ((size_t)c0 * mx.H + h) * D * V + (size_t)g * VW;
   const float* dec = wk.dec + ((size_t)c0 * mx.H + h) * D + d;
   const size_t kv_step = (size_t)mx.H * D * (is_n ? 1 : V), dec_step = (size_t)mx.H * D;
+  auto load = [&](const float* p) {
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (VW == 4 && !is_n) v = *reinterpret_cast<const float4*>(p);
+    else v.x = *p;
+    return v;
+  };
+  auto store = [&](float* p, const float4& v) {
+    if (VW == 4 && !is_n) *reinterpret_cast<float4*>(p) = v;
+    else *p = v.x;
+  };
+  float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (sq.w > 0) s = load(state);
   constexpr int AHEAD = 8;      // chunks whose loads are in flight together: only the fma chain is serial
   for (int c = 0; c < n; c += AHEAD) {
-    float add[AHEAD], dc[AHEAD];
+    float4 add[AHEAD];
+    float dc[AHEAD];
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i)
       if (c + i < n) {
-        add[i] = kv[(size_t)(c + i) * kv_step];
+        add[i] = load(kv + (size_t)(c + i) * kv_step);
         dc[i] = dec[(size_t)(c + i) * dec_step];
       }
 #pragma unroll
     for (int i = 0; i < AHEAD; ++i)
       if (c + i < n) {
-        kv[(size_t)(c + i) * kv_step] = s;
-        s = fmaf(dc[i], s, add[i]);
+        store(kv + (size_t)(c + i) * kv_step, s);
+        s.x = fmaf(dc[i], s.x, add[i].x);
+        s.y = fmaf(dc[i], s.y, add[i].y);
+        s.z = fmaf(dc[i], s.z, add[i].z);
+        s.w = fmaf(dc[i], s.w, add[i].w);
       }
   }
-  *state = s;
+  store(state, s);
 }
 
 // o = q~ S_c + P V for one chunk, head and 64 value columns.
@@ -736,8 +753,11 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
   PK_CHECK_LAUNCH();
   chunk_kv_kernel<<<dim3(nchunks, H, dt * vt), 256, 0, stream>>>(mx, ck, wk, dt);
   PK_CHECK_LAUNCH();
-  const int elems = mx.D * mx.V + (d->kind == KIND_MLSTM ? mx.D : 0);
-  chunk_scan_kernel<<<dim3((elems + 255) / 256, H, nseq), 256, 0, stream>>>(mx, ck, wk);
+  const bool v4 = (mx.V & 3) == 0 && ((uintptr_t)mx.S & 15) == 0;
+  const int elems = mx.D * mx.V / (v4 ? 4 : 1) + (d->kind == KIND_MLSTM ? mx.D : 0);
+  const dim3 scan_grid((elems + 255) / 256, H, nseq);
+  if (v4) chunk_scan_kernel<4><<<scan_grid, 256, 0, stream>>>(mx, ck, wk);
+  else chunk_scan_kernel<1><<<scan_grid, 256, 0, stream>>>(mx, ck, wk);
   PK_CHECK_LAUNCH();
   chunk_out_kernel<<<dim3(nchunks, H, vt), 256, 0, stream>>>(mx, raw, ck, wk);
   PK_CHECK_LAUNCH();
