@@ -223,9 +223,10 @@ def kernels() -> None:
     for B, win in ((1, 1024), (8, 1024), (64, 640)):
         for k, (f, fl, nb) in _latent((32, 128, 64, 128, 512, win), B, 1500, True).items():
             show("latent rows: " + k, _roof(timed(f), fl, nb), B=B, window=win)
-    for r in bk.bench_dsv4_select_attend(64, 32768, 20):
-        if "sparse_attn" in r["op"]:
-            show("like kernel: sparse attention over 640 latent rows", r)
+    for M in (1, 8, 64):
+        for r in bk.bench_dsv4_select_attend(M, 32768, 20):
+            if "sparse_attn" in r["op"]:
+                show("like kernel: sparse attention over 640 latent rows", r)
     # few-row linears and norms
     for M in (1, 4, 8):
         for N, K, sw in ((28672, 4096, True), (4096, 14336, False), (12416, 4096, False)):
