@@ -32,7 +32,7 @@ constexpr int kEpiWarps = 8;
 constexpr int kThreads = 64 + kEpiWarps * 32;
 constexpr uint32_t kTmemCols = 512;       // two accumulators of 256 columns
 
-enum { EPI_BF16 = 0, EPI_SWIGLU = 1, EPI_RESID = 2, EPI_F32 = 3, EPI_PUSH = 4 };
+enum { EPI_BF16 = 0, EPI_SWIGLU = 1, EPI_RESID = 2, EPI_F32 = 3, EPI_PUSH = 4, EPI_RELU2 = 5 };
 
 struct Params {
   int M, N, K, epi;
@@ -54,6 +54,9 @@ struct Params {
   // computed and not stored)
   const int* seg;
   int n_groups;
+  // EPI_RELU2: bf16 max(acc * s, 0)^2, or max(acc, 0)^2 * s (scale_after), s = row_scale[row] (null: 1)
+  const float* row_scale;
+  int scale_after;
 };
 
 constexpr int kMaxGroups = 512;
@@ -404,6 +407,15 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
               }
             }
           } else {
+            if (p.epi == EPI_RELU2) {
+              const float s = p.row_scale ? __ldg(p.row_scale + m) : 1.f;
+              const float s0 = p.scale_after ? 1.f : s, s1 = p.scale_after ? s : 1.f;
+#pragma unroll
+              for (int i = 0; i < 32; ++i) {
+                const float a = fmaxf(__uint_as_float(r[i]) * s0, 0.f);
+                r[i] = __float_as_uint(a * a * s1);
+              }
+            }
             bf16* dst = p.C + (size_t)m * p.ldc + n;
             const bf16* rs = p.epi == EPI_RESID ? p.resid + (size_t)m * p.ldc + n : nullptr;
             if (n + 32 <= p.N) {
@@ -520,11 +532,12 @@ bool encode_bf16_2d(EncodeTiledFn encode, CUtensorMap* map, const void* base, ui
 // 1 (SwiGLU: every group's matrix holds N / 2 gate rows then N / 2 up rows) and 3 (fp32). One persistent launch walks
 // every (group, row tile, column block) that has rows; the tile list is derived from seg on the device, so the host
 // never reads the routing.
-PK_API int pk_gemm_bf16_grouped(const void* A, int lda, const void* W, const int* seg, int n_groups, int R, int N, int K, int epi, void* C, int ldc,
-                                uint32_t* status, int sm_count, cudaStream_t stream) {
+// Epilogue 5: squared ReLU with a factor per row, before (scale_after = 0) or after the activation.
+PK_API int pk_gemm_bf16_grouped_scaled(const void* A, int lda, const void* W, const int* seg, int n_groups, int R, int N, int K, int epi, void* C,
+                                       int ldc, const float* row_scale, int scale_after, uint32_t* status, int sm_count, cudaStream_t stream) {
   if (R < 1 || N < 1 || K < BK || (K % BK) != 0 || seg == nullptr || n_groups < 1 || n_groups > kMaxGroups) return PK_ERR_BAD_ARG;
   if (((uintptr_t)A & 15) != 0 || ((size_t)lda * 2) % 16 != 0 || ((uintptr_t)W & 15) != 0) return PK_ERR_BAD_ARG;
-  if (epi != EPI_BF16 && epi != EPI_SWIGLU && epi != EPI_F32) return PK_ERR_BAD_ARG;
+  if (epi != EPI_BF16 && epi != EPI_SWIGLU && epi != EPI_F32 && epi != EPI_RELU2) return PK_ERR_BAD_ARG;
   if (epi == EPI_SWIGLU && ((N & 1) != 0)) return PK_ERR_BAD_ARG;
   if (epi == EPI_SWIGLU && ((N >> 1) % 128) != 0) return PK_ERR_UNSUPPORTED;
   if (epi != EPI_SWIGLU && (N % 128) != 0) return PK_ERR_UNSUPPORTED;      // a column block must not reach into the next group's rows
@@ -547,6 +560,8 @@ PK_API int pk_gemm_bf16_grouped(const void* A, int lda, const void* W, const int
   p.status = status;
   p.seg = seg;
   p.n_groups = n_groups;
+  p.row_scale = row_scale;
+  p.scale_after = scale_after;
   const size_t smem = sizeof(Smem) + 1024;
   static PkDeviceOnce once;
   if (PkDeviceOnceGuard once_guard{once}; once_guard.needed()) {
@@ -559,6 +574,12 @@ PK_API int pk_gemm_bf16_grouped(const void* A, int lda, const void* W, const int
   gemm_bf16_kernel<<<sm_count > 0 ? sm_count : 148, kThreads, smem, stream>>>(tmap_a, tmap_w, p);
   PK_CHECK_LAUNCH();
   return PK_OK;
+}
+
+PK_API int pk_gemm_bf16_grouped(const void* A, int lda, const void* W, const int* seg, int n_groups, int R, int N, int K, int epi, void* C, int ldc,
+                                uint32_t* status, int sm_count, cudaStream_t stream) {
+  if (epi == EPI_RELU2) return PK_ERR_BAD_ARG;
+  return pk_gemm_bf16_grouped_scaled(A, lda, W, seg, n_groups, R, N, K, epi, C, ldc, nullptr, 0, status, sm_count, stream);
 }
 
 // A [M, K] bf16 (row stride lda elements), W [N, K] bf16 row-major, K a multiple of 64. Epilogues as in pk_gemm_umma;

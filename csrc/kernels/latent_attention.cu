@@ -10,7 +10,7 @@
 //   merge    sum of the splits, with the sink in the denominator
 //   out      W_uv per head
 // Scores, weights and accumulators are fp32 in all of them; the cache and the weights are bf16 or (fp32 mode) fp32.
-#include "../common/pk_common.cuh"
+#include "../common/pk_rotary.cuh"
 
 namespace {
 
@@ -64,10 +64,8 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
   float* cs = sm;
   float* sn = sm + half;
   for (int i = tid; i < half; i += 256) {
-    double a = (double)pos * p.freq[i];
-    a -= 6.283185307179586476925286766559 * rint(a * 0.15915494309189533576888376337251);
     float s, c;
-    sincosf((float)a, &s, &c);
+    rotary_sincos(p.freq[i], pos, s, c);
     cs[i] = c * p.mag;
     sn[i] = s * p.mag;
   }

@@ -1,8 +1,8 @@
-// Recurrent mixers with an outer-product state: gated linear attention (a decay per key channel) and the matrix memory of
-// xLSTM (scalar gates with a running maximum). Both are
+// Recurrent mixers with an outer-product state: gated linear attention (a decay per key channel), the matrix memory of
+// xLSTM (scalar gates with a running maximum) and retention (a constant decay per head, rotated queries and keys). All are
 //   S_t = diag(a_t) S_{t-1} + b_t k_t v_t^T,    o_t = S_t^T q_t          S: [key dim, value dim], fp32
 // with a_t a vector (GLA: a = sigmoid(z)^(1/tau), b = 1) or a scalar (mLSTM: a = exp(f + m_{t-1} - m_t), b = exp(i - m_t),
-// m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1).
+// m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1; retention: a = const, b = 1).
 // Everything here is fp32: gates, decays, states and products.
 //
 // State lives in slots [slot][head][key][value] so that requests of one batch keep theirs anywhere; a portion that starts
@@ -16,16 +16,17 @@
 //       scan    state before every chunk
 //       out     per (chunk, head, tile): q~ S_c + P V
 //     GLA's exponents are never split into exp(G_i) exp(-G_j) across a reference further away than the 16-token
-//     sub-chunk between them: every factor is at most 1, whatever the decay.
+//     sub-chunk between them: every factor is at most 1, whatever the decay. Retention takes the powers of its decays
+//     from a table.
 // A last kernel normalises every head's output (after mLSTM's division by max(|n.q|, exp(-m)) + 1e-6), applies the output
 // gate and writes the projection's input.
-#include "../common/pk_common.cuh"
+#include "../common/pk_rotary.cuh"
 
 namespace {
 
 using namespace pk;
 
-enum { KIND_GLA = 0, KIND_MLSTM = 1 };
+enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_RETENTION = 2 };
 constexpr int CH = 64;    // chunk
 constexpr int SB = 16;    // sub-chunk
 
@@ -48,6 +49,10 @@ struct Mixer {
   const float* a2b;    // [H * D]
   int rank;
   float inv_tau;
+  // retention
+  const double* freq;  // [rot / 2] angular frequencies of the rotated leading part of queries and keys
+  int rot;
+  const float* pw;     // [H, 65] powers 0 .. 64 of every head's decay
   // state
   float* S;            // [slots, H, D, V]
   float* N;            // [slots, H, D]      (mLSTM)
@@ -92,15 +97,38 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
     s[j] = live && d < D && sq.w > 0 ? Sp[(size_t)d * st] : 0.f;
   }
   float m_prev = KIND == KIND_MLSTM && sq.w > 0 ? mx.Ms[head] : 0.f;
+  const float decay = KIND == KIND_RETENTION ? mx.pw[h * (CH + 1) + 1] : 0.f;
   for (int t = 0; t < sq.y; ++t) {
     const float* pr = mx.proj + (size_t)(sq.x + t) * mx.ld;
-    for (int d = threadIdx.x; d < D; d += 32 * GR) {
-      qs[d] = pr[mx.oq + h * D + d] * mx.qscale;
-      ks[d] = pr[mx.ok + h * D + d];
-      if (KIND == KIND_GLA) {
-        float z = mx.a2b[h * D + d];
-        for (int r = 0; r < mx.rank; ++r) z = fmaf(mx.a2[(size_t)r * mx.H * D + h * D + d], pr[mx.oa + r], z);
-        as[d] = expf(log_sigmoid(z) * mx.inv_tau);
+    if (KIND == KIND_RETENTION) {
+      // one item per rotated pair, then one per channel that passes
+      const int half = mx.rot / 2;
+      const float* q = pr + mx.oq + h * D;
+      const float* k = pr + mx.ok + h * D;
+      for (int i = threadIdx.x; i < D - half; i += 32 * GR) {
+        if (i < half) {
+          float s, c, qu = q[i] * mx.qscale, qv = q[i + half] * mx.qscale, ku = k[i], kv = k[i + half];
+          rotary_sincos(mx.freq[i], sq.w + t, s, c);
+          rotate_pair(qu, qv, s, c);
+          rotate_pair(ku, kv, s, c);
+          qs[i] = qu;
+          qs[i + half] = qv;
+          ks[i] = ku;
+          ks[i + half] = kv;
+        } else {
+          qs[i + half] = q[i + half] * mx.qscale;
+          ks[i + half] = k[i + half];
+        }
+      }
+    } else {
+      for (int d = threadIdx.x; d < D; d += 32 * GR) {
+        qs[d] = pr[mx.oq + h * D + d] * mx.qscale;
+        ks[d] = pr[mx.ok + h * D + d];
+        if (KIND == KIND_GLA) {
+          float z = mx.a2b[h * D + d];
+          for (int r = 0; r < mx.rank; ++r) z = fmaf(mx.a2[(size_t)r * mx.H * D + h * D + d], pr[mx.oa + r], z);
+          as[d] = expf(log_sigmoid(z) * mx.inv_tau);
+        }
       }
     }
     if (KIND == KIND_MLSTM) {
@@ -117,9 +145,9 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
     float v = is_v ? pr[mx.ov + h * V + col] : (is_n ? 1.f : 0.f);
     __syncthreads();
     float part = 0.f;
-    if (KIND == KIND_MLSTM) {
-      const float a = s_sc[0];
-      v *= s_sc[1];
+    if (KIND != KIND_GLA) {
+      const float a = KIND == KIND_MLSTM ? s_sc[0] : decay;
+      if (KIND == KIND_MLSTM) v *= s_sc[1];
 #pragma unroll
       for (int j = 0; j < RPT; ++j) {
         const int d = g + j * GR;
@@ -323,6 +351,93 @@ __global__ void __launch_bounds__(256) mlstm_intra_kernel(const Mixer mx, const 
     for (int j = 0; j < 4; ++j) {
       const int s = tx * 4 + j;
       ov[j] = s <= r && r < len ? acc[i][j] * expf((float)(Fd[r] - Fd[s]) + (ig[s] - mi[r])) : 0.f;
+    }
+    *reinterpret_cast<float4*>(wk.P + (ch * CH + r) * CH + tx * 4) = out;
+  }
+}
+
+// Retention intra-chunk part. One block per (chunk, head). Channels are walked so that both halves of a rotated pair are
+// neighbours: c < rot is half (c & 1) of pair c / 2, the others follow unchanged.
+__global__ void __launch_bounds__(256) retention_intra_kernel(const Mixer mx, const Chunks ck, const Work wk) {
+  __shared__ float Qs[32][CH + 4], Ks[32][CH + 4];
+  __shared__ float pw[CH + 1];
+  const int c = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
+  const int4 cd = ck.chunks[c];
+  const int len = cd.y, D = mx.D, half = mx.rot / 2;
+  const int4 sq = ck.seqs[cd.z];
+  const int pos0 = sq.w + cd.x - sq.x;
+  const size_t ch = (size_t)c * mx.H + h;
+  if (tid <= CH) pw[tid] = mx.pw[h * (CH + 1) + tid];
+  __syncthreads();
+  const int tx = tid & 15, ty = tid >> 4;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int c0 = 0; c0 < D; c0 += 32) {
+    for (int i = tid; i < CH * 16; i += 256) {
+      const int r = i >> 4, x = (i & 15) * 2, cc = c0 + x;
+      const bool turn = cc < mx.rot;
+      const int d0 = turn ? cc >> 1 : cc, d1 = turn ? d0 + half : cc + 1;
+      float qu = 0.f, qv = 0.f, ku = 0.f, kv = 0.f;
+      if (cc < D && r < len) {
+        const float* pr = mx.proj + (size_t)(cd.x + r) * mx.ld + h * D;
+        qu = pr[mx.oq + d0] * mx.qscale;
+        ku = pr[mx.ok + d0];
+        if (d1 < D) {
+          qv = pr[mx.oq + d1] * mx.qscale;
+          kv = pr[mx.ok + d1];
+        }
+        if (turn) {
+          float s, co;
+          rotary_sincos(mx.freq[d0], pos0 + r, s, co);
+          rotate_pair(qu, qv, s, co);
+          rotate_pair(ku, kv, s, co);
+        }
+      }
+      if (cc < D) {
+        const float eq = r < len ? pw[r + 1] : 0.f, ek = r < len ? pw[len - 1 - r] : 0.f;
+        float* qt = wk.qt + (ch * CH + r) * D;
+        float* kt = wk.kt + (ch * CH + r) * D;
+        qt[d0] = qu * eq;
+        kt[d0] = ku * ek;
+        if (d1 < D) {
+          qt[d1] = qv * eq;
+          kt[d1] = kv * ek;
+        }
+        if (r == 0) {
+          wk.dec[ch * D + d0] = pw[len];
+          if (d1 < D) wk.dec[ch * D + d1] = pw[len];
+        }
+      }
+      Qs[x][r] = qu;
+      Qs[x + 1][r] = qv;
+      Ks[x][r] = ku;
+      Ks[x + 1][r] = kv;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int d = 0; d < 32; ++d) {
+      const float4 a = *reinterpret_cast<const float4*>(&Qs[d][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&Ks[d][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int r = ty * 4 + i;
+    float4 out;
+    float* ov = reinterpret_cast<float*>(&out);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int s = tx * 4 + j;
+      ov[j] = s <= r && r < len ? acc[i][j] * pw[r - s] : 0.f;
     }
     *reinterpret_cast<float4*>(wk.P + (ch * CH + r) * CH + tx * 4) = out;
   }
@@ -587,7 +702,7 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
 // ---------------------------------------------------------------------------------------
 // normalisation, output gate
 
-// One block per (head, row). norm_w: [H * V] (per_head = 0) or [V] shared by the heads. last_slot[row] = slot whose portion
+// One block per (head, row). norm_w: [H * V] (per_head = 0), [V] shared by the heads, or null (no weight). last_slot[row] = slot whose portion
 // ends at this row, or -1: mLSTM's running maximum is stored there once every reader of the old one is done.
 template <int KIND, typename OutT>
 __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, int per_head, float eps,
@@ -618,10 +733,10 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
   for (int v = tid + KEEP * nt; v < V; v += nt) ss = fmaf(o[v] * inv, o[v] * inv, ss);
   const float r = inv / sqrtf(block_sum(ss, scratch) / (float)V + eps);
   OutT* dst = out + (size_t)t * ldo + h * V;
-  const float* w = norm_w + (per_head ? 0 : h * V);
+  const float* w = norm_w ? norm_w + (per_head ? 0 : h * V) : nullptr;
   auto put = [&](int v, float xv, float zv) {
     const float s = 1.f / (1.f + expf(-zv));
-    dst[v] = (OutT)(xv * r * w[v] * (KIND == KIND_MLSTM ? s : zv * s));
+    dst[v] = (OutT)(xv * r * (w ? w[v] : 1.f) * (KIND == KIND_MLSTM ? s : zv * s));
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i)
@@ -692,7 +807,9 @@ struct PkStateMixer {
   float* o;
   float* nq;
   float* m;
-  int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank;
+  const double* freq;
+  const float* pw;
+  int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank, rot;
   float qscale, cap, inv_tau;
 };
 
@@ -700,9 +817,10 @@ static bool unpack(const PkStateMixer* d, Mixer& mx, Raw& raw) {
   if (d == nullptr || d->proj == nullptr || d->S == nullptr || d->o == nullptr || d->H < 1 || d->D < 1 || d->V < 1 || d->D > 512) return false;
   if (d->kind == KIND_MLSTM && (!d->bi || !d->bf || !d->N || !d->Ms || !d->nq || !d->m || !(d->cap > 0.f))) return false;
   if (d->kind == KIND_GLA && (!d->a2 || !d->a2b || d->rank < 1 || d->rank > 1024)) return false;
-  if (d->kind != KIND_GLA && d->kind != KIND_MLSTM) return false;
+  if (d->kind == KIND_RETENTION && (!d->pw || d->rot < 0 || (d->rot & 1) != 0 || d->rot > d->D || (d->rot > 0 && !d->freq))) return false;
+  if (d->kind != KIND_GLA && d->kind != KIND_MLSTM && d->kind != KIND_RETENTION) return false;
   mx = Mixer{d->proj, d->ld, d->oq, d->ok, d->ov, d->og, d->oi, d->of, d->oa, d->H, d->D, d->V, d->qscale, d->bi, d->bf,
-             d->cap, d->a2, d->a2b, d->rank, d->inv_tau, d->S, d->N, d->Ms};
+             d->cap, d->a2, d->a2b, d->rank, d->inv_tau, d->freq, d->rot, d->pw, d->S, d->N, d->Ms};
   raw = Raw{d->o, d->nq, d->m};
   return true;
 }
@@ -712,8 +830,11 @@ PK_API int pk_state_rows(const PkStateMixer* d, const void* seqs, int nseq, cuda
   Mixer mx;
   Raw raw;
   if (!unpack(d, mx, raw) || seqs == nullptr || nseq < 1) return PK_ERR_BAD_ARG;
-  return d->kind == KIND_GLA ? launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream)
-                             : launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
+  switch (d->kind) {
+    case KIND_GLA: return launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream);
+    case KIND_MLSTM: return launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
+    default: return launch_rows<KIND_RETENTION>(mx, raw, (const int4*)seqs, nseq, stream);
+  }
 }
 
 // Workspace floats of pk_state_chunks.
@@ -745,6 +866,8 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
     gla_gates_kernel<<<dim3(nchunks, CH / 8, z < 16 ? z : 16), 256, (size_t)8 * mx.rank * sizeof(float), stream>>>(mx, ck, wk);
     PK_CHECK_LAUNCH();
     gla_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
+  } else if (d->kind == KIND_RETENTION) {
+    retention_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
   } else {
     mlstm_gates_kernel<<<dim3(nseq, H), 256, 0, stream>>>(mx, raw, ck, wk);
     PK_CHECK_LAUNCH();
@@ -764,16 +887,16 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
   return PK_OK;
 }
 
-// Head norm, output gate and running-maximum write-back for all rows of a step.
+// Head norm, output gate (SiLU; mLSTM: sigmoid) and running-maximum write-back for all rows of a step. norm_w null: no weight.
 PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head, float eps, const int* last_slot, int rows, void* out,
                         int ldo, int out_f32, cudaStream_t stream) {
   Mixer mx;
   Raw raw;
-  if (!unpack(d, mx, raw) || norm_w == nullptr || last_slot == nullptr || rows < 1 || out == nullptr || ldo < mx.H * mx.V) return PK_ERR_BAD_ARG;
+  if (!unpack(d, mx, raw) || last_slot == nullptr || rows < 1 || out == nullptr || ldo < mx.H * mx.V) return PK_ERR_BAD_ARG;
   if (rows > 65535) return PK_ERR_BAD_ARG;
   const int nt = (mx.V + 31) / 32 * 32;
   const dim3 grid(mx.H, rows), block(nt < 256 ? nt : 256);
-  if (d->kind == KIND_GLA) {
+  if (d->kind != KIND_MLSTM) {
     if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
     else PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
   } else {

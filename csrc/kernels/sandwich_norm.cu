@@ -1,7 +1,9 @@
-// Residual and norm steps of decoders whose residual stream is kept in fp32 and whose sublayers are normed before and
-// after: one launch does everything between two projections,
-//   x   <- embedding row                    (first layer)    or
-//   x   <- x + rms(y) * (bias + w_post)     (y = the sublayer's output, fp32)
+// Residual and norm steps of decoders whose residual stream is kept in fp32: one launch does everything between two
+// projections,
+//   x   <- scale * embedding row            (first layer)    or
+//   x   <- x + rms(y) * (bias + w_post)     (y = the sublayer's output, fp32; no w_post: y as it is; y may be the sum of a
+//                                            few listed rows, the outputs of a token's experts)
+//   x   <- x + scale * embedding row        (again, before a further pass over the same layers)
 //   out <- rms(x) * (bias + w_pre)          (the next sublayer's input, bf16 or fp32, columns padded with zeros)
 // `bias` is 1 for weights stored around zero and 0 for plain weights. One block per row, the row stays in registers.
 #include "../common/pk_common.cuh"
@@ -12,11 +14,15 @@ using namespace pk;
 
 struct NormParams {
   float* x;              // [rows of the step, width] residual stream
-  const int* tokens;     // first layer: embedding ids (x is written)
+  const int* tokens;     // embedding ids, or null
   const bf16* embed;
   int vocab;
+  float embed_scale;
+  int embed_add;         // 0: x starts as the embedding row; 1: the row is added to x (after y)
   const float* y;        // [rows, ldy] or null
   int ldy;
+  const int* y_rows;     // [rows, y_top]: y of a row is the sum of these rows of `y` (null: the row of the same index)
+  int y_top;
   const float* w_post;
   const int* rows;       // output row r works on residual row rows[r] (null: r); x is not written then
   int width;
@@ -70,7 +76,7 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const NormParams p)
   const int row = p.rows ? p.rows[r] : r;
   float* xr = p.x + (size_t)row * p.width;
   float v[PT][VW], u[PT][VW];
-  if (p.tokens) {
+  auto add_embedding = [&]() {
     int t = p.tokens[row];
     t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
     const bf16* e = p.embed + (size_t)t * p.width;
@@ -79,37 +85,56 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const NormParams p)
 #pragma unroll
       for (int j = 0; j < VW; ++j) {
         const int c = (tid + i * nt) * VW + j;
-        v[i][j] = c < p.width ? __bfloat162float(e[c]) : 0.f;
+        if (c < p.width) v[i][j] = __fadd_rn(v[i][j], __fmul_rn(__bfloat162float(e[c]), p.embed_scale));
       }
-  } else {
+  };
+  const bool fresh = p.tokens && !p.embed_add;
 #pragma unroll
-    for (int i = 0; i < PT; ++i) {
-      const int c = (tid + i * nt) * VW;
+  for (int i = 0; i < PT; ++i) {
+    const int c = (tid + i * nt) * VW;
 #pragma unroll
-      for (int j = 0; j < VW; ++j) v[i][j] = 0.f;
-      if (c < p.width) load_f32<VW>(xr + c, v[i]);
-    }
+    for (int j = 0; j < VW; ++j) v[i][j] = 0.f;
+    if (!fresh && c < p.width) load_f32<VW>(xr + c, v[i]);
   }
+  if (fresh) add_embedding();
   if (p.y) {
-    const float* yr = p.y + (size_t)row * p.ldy;
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
       const int c = (tid + i * nt) * VW;
 #pragma unroll
       for (int j = 0; j < VW; ++j) u[i][j] = 0.f;
-      if (c < p.width) load_f32<VW>(yr + c, u[i]);
+      if (c < p.width) {
+        if (p.y_rows) {
+          for (int k = 0; k < p.y_top; ++k) {
+            float a[VW];
+            load_f32<VW>(p.y + (size_t)p.y_rows[(size_t)row * p.y_top + k] * p.ldy + c, a);
+#pragma unroll
+            for (int j = 0; j < VW; ++j) u[i][j] += a[j];
+          }
+        } else {
+          load_f32<VW>(p.y + (size_t)row * p.ldy + c, u[i]);
+        }
+      }
 #pragma unroll
       for (int j = 0; j < VW; ++j) ss = fmaf(u[i][j], u[i][j], ss);
     }
-    const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
+    if (p.w_post) {
+      const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
 #pragma unroll
-    for (int i = 0; i < PT; ++i)
-      if ((tid + i * nt) * VW < p.width) {
+      for (int i = 0; i < PT; ++i)
+        if ((tid + i * nt) * VW < p.width) {
 #pragma unroll
-        for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * rr * (p.bias + wb[i][j]);
-      }
+          for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * rr * (p.bias + wb[i][j]);
+        }
+    } else {
+#pragma unroll
+      for (int i = 0; i < PT; ++i)
+#pragma unroll
+        for (int j = 0; j < VW; ++j) v[i][j] += u[i][j];
+    }
   }
+  if (p.tokens && p.embed_add) add_embedding();
   if (p.rows == nullptr && (p.tokens || p.y)) {
 #pragma unroll
     for (int i = 0; i < PT; ++i) {
@@ -183,16 +208,18 @@ __global__ void bump_kernel(int* step) { step[0] += 1; }
 
 }  // namespace
 
-// See the head of this file. tokens != null: x is filled from the embedding table; y != null: the normed sublayer output is
-// added first. rows != null: only the M listed rows are normed (x stays as it is). width up to 8192 (32768 when a multiple of 4).
-PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int vocab, const float* y, int ldy, const float* w_post,
-                            const int* rows, int M, int width, const float* w_pre, int plus_one, float eps, void* out, int ldo,
-                            int out_f32, cudaStream_t stream) {
+// See the head of this file. tokens != null: x is filled from the embedding table (embed_add: the row is added); y != null: the
+// (normed) sublayer output is added first. rows != null: only the M listed rows are normed (x stays as it is). width up to
+// 8192 (32768 when a multiple of 4).
+PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int vocab, float embed_scale, int embed_add, const float* y, int ldy,
+                            const int* y_rows, int y_top, const float* w_post, const int* rows, int M, int width, const float* w_pre,
+                            int plus_one, float eps, void* out, int ldo, int out_f32, cudaStream_t stream) {
   if (M < 1 || width < 1 || x == nullptr) return PK_ERR_BAD_ARG;
-  if (y != nullptr && (w_post == nullptr || ldy < width)) return PK_ERR_BAD_ARG;
+  if (y != nullptr && (ldy < width || (y_rows != nullptr && y_top < 1))) return PK_ERR_BAD_ARG;
   if (tokens != nullptr && (embed == nullptr || vocab < 1)) return PK_ERR_BAD_ARG;
   if (w_pre != nullptr && (out == nullptr || ldo < width)) return PK_ERR_BAD_ARG;
-  NormParams p{x, tokens, (const pk::bf16*)embed, vocab, y, ldy, w_post, rows, width, w_pre, plus_one ? 1.f : 0.f, eps, out, ldo};
+  NormParams p{x, tokens, (const pk::bf16*)embed, vocab, embed_scale, embed_add, y, ldy, y_rows, y_top, w_post, rows, width, w_pre,
+               plus_one ? 1.f : 0.f, eps, out, ldo};
   return out_f32 ? launch_any<float>(p, M, stream) : launch_any<pk::bf16>(p, M, stream);
 }
 

@@ -7,14 +7,14 @@ The layers themselves are in `mixer_layers`, the step function in `runtime.mixer
 """
 from __future__ import annotations
 
-import json
 from dataclasses import dataclass
 from pathlib import Path
 
 import torch
 
-from ..formats import safetensors_io as st_io
+from . import mixer_checkpoint as mc
 from . import mixer_layers as ml
+from .mixer_checkpoint import load_tensors, save_checkpoint  # noqa: F401  (part of this module's interface)
 
 ARCH = "Gidisun"
 
@@ -32,9 +32,7 @@ class LayerConfig:
     def __post_init__(self) -> None:
         if self.type not in _MIXER_KEYS:
             raise ValueError(f"unknown mixer {self.type!r}; known: {sorted(_MIXER_KEYS)}")
-        missing = [k for k in _MIXER_KEYS[self.type] if k not in self.mixer]
-        if missing:
-            raise ValueError(f"{self.type} layer without {missing}")
+        mc.require_keys(f"{self.type} layer", self.mixer, _MIXER_KEYS[self.type])
         if self.mlp is not None and self.mlp.get("kind", "dense") != "dense":
             raise ValueError(f"unknown feed-forward {self.mlp.get('kind')!r}")
         if self.type == "latent_attention":
@@ -54,15 +52,13 @@ class GidisunConfig:
 
     @classmethod
     def from_dict(cls, d: dict) -> "GidisunConfig":
-        if d.get("architecture") != ARCH:
-            raise ValueError(f"architecture {d.get('architecture')!r} is not {ARCH}")
+        mc.check_architecture(d, ARCH)
         return cls(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]),
                    [LayerConfig(L["type"], L["mixer"], L.get("mlp")) for L in d["layers"]])
 
     @classmethod
     def load(cls, path: str | Path) -> "GidisunConfig":
-        p = Path(path)
-        return cls.from_dict(json.loads((p / "config.json" if p.is_dir() else p).read_text()))
+        return cls.from_dict(mc.read_config(path, ARCH))
 
     def to_dict(self) -> dict:
         return {"architecture": ARCH, "vocab": self.vocab, "width": self.width, "norm": {"eps": self.eps},
@@ -119,30 +115,11 @@ def random_tensors(c: GidisunConfig, seed: int = 0, decay_rank: int = 16, device
     return out
 
 
-def save_checkpoint(directory: str | Path, c: GidisunConfig, tensors: dict[str, torch.Tensor]) -> None:
-    d = Path(directory)
-    d.mkdir(parents=True, exist_ok=True)
-    (d / "config.json").write_text(json.dumps(c.to_dict()))
-    st_io.write_file(d / "model.safetensors", tensors)
-
-
-def load_tensors(path: str | Path) -> dict[str, torch.Tensor]:
-    src = st_io.SafetensorsModel(path)
-    return {n: src.get(n) for n in src.keys()}
-
-
 def build_model(c: GidisunConfig, tensors: dict[str, torch.Tensor], *, dtype: torch.dtype = torch.bfloat16, device: str = "cuda",
                 slots: int = 8, pages: int = 64) -> ml.MixerModel:
     """Weights in the kernels' layout, with room for `slots` requests and `pages` pages of their positions."""
-    if dtype not in (torch.bfloat16, torch.float32):
-        raise ValueError("dtype must be bfloat16 or float32")
-    plan = tensor_plan(c)
-    for name, shape in plan.items():
-        if name not in tensors:
-            raise KeyError(f"missing tensor {name}")
-        got = tuple(tensors[name].shape)
-        if got != shape and not (name.endswith(("mix.a1", "mix.a2")) and len(got) == 2):
-            raise ValueError(f"{name}: shape {got}, expected {shape}")
+    mc.check_dtype(dtype)
+    mc.check_tensors(tensor_plan(c), tensors, free=("mix.a1", "mix.a2"))
     f32 = lambda n: tensors[n].float().to(device)
     layers = []
     for i, L in enumerate(c.layers):
@@ -152,7 +129,7 @@ def build_model(c: GidisunConfig, tensors: dict[str, torch.Tensor], *, dtype: to
             mixer = ml.MIXERS[L.type](w, L.mixer, c.eps, dtype, device, pages, pages * ml.mo.PAGE)
         else:
             mixer = ml.MIXERS[L.type](w, L.mixer, c.eps, dtype, device, slots)
-        layer = ml.SandwichLayer(mixer, f32(p + "norm1"), f32(p + "norm1b"))
+        layer = ml.MixerLayer(mixer, f32(p + "norm1"), norm1b=f32(p + "norm1b"))
         if L.mlp is not None:
             layer.mlp = ml.SwiGLU({n: tensors[p + "mlp." + n] for n in ("gate", "up", "down")}, dtype, device)
             layer.norm2, layer.norm2b = f32(p + "norm2"), f32(p + "norm2b")
@@ -161,14 +138,6 @@ def build_model(c: GidisunConfig, tensors: dict[str, torch.Tensor], *, dtype: to
                          ml.FusedLinear([("head", tensors["head"])], dtype, device))
 
 
-def build_runtime(path, *, dtype: torch.dtype = torch.bfloat16, device: str = "cuda", max_requests: int = 8, max_tokens: int | None = None,
-                  max_context: int = 4096, **kw):
-    """Runtime over a checkpoint folder. `max_tokens`: positions that live requests hold at any time, all together (default:
-    `max_context` for every slot)."""
-    from ..runtime.mixer_runtime import MixerRuntime
-    c = GidisunConfig.load(path)
-    page = ml.mo.PAGE
-    per = (max_context + page - 1) // page
-    pages = max_requests * per if max_tokens is None else (max_tokens + page - 1) // page
-    model = build_model(c, load_tensors(path), dtype=dtype, device=device, slots=max_requests, pages=pages)
-    return MixerRuntime(model, max_requests=max_requests, pages=pages, device=device, **kw)
+def build_runtime(path, **kw):
+    """Runtime over a checkpoint folder (see `mixer_checkpoint.open_runtime`)."""
+    return mc.open_runtime(path, GidisunConfig.load, build_model, **kw)

@@ -8,8 +8,9 @@ scores and the residual stream in fp32) and float32 (everything, without reduced
 """
 from __future__ import annotations
 
+import copy
 import math
-from dataclasses import dataclass, field
+from dataclasses import dataclass, field, replace
 
 import torch
 
@@ -110,12 +111,23 @@ class RecurrentMixer:
                 raise ValueError(f"{n}: {w[n].shape[0]} rows, expected {r}")
         self.proj = FusedLinear([(n, w[n]) for n in ["q", "k", "v", "g"] + extra], dtype, device)
         self.out = FusedLinear([("o", w["o"])], dtype, device)
-        self.norm = _f32(w["norm"], device)
+        self.norm = _f32(w["norm"], device) if "norm" in w else None
         self.S = torch.zeros(slots, heads, dim, vdim, device=device)
         self.N = self.Ms = None
         a = self.proj.at
         self.keep: list[torch.Tensor] = []
         self.desc = dict(kind=kind, H=heads, D=dim, V=vdim, oq=a["q"], ok=a["k"], ov=a["v"], og=a["g"], qscale=dim ** -0.5, S=self.S.data_ptr())
+
+    def again(self):
+        """The same weights with states of their own (a further pass over the layer)."""
+        o = copy.copy(self)
+        o.desc = dict(self.desc)
+        for n in ("S", "N", "Ms"):
+            t = getattr(self, n)
+            if t is not None:
+                setattr(o, n, torch.zeros_like(t))
+                o.desc[n] = getattr(o, n).data_ptr()
+        return o
 
     def state_bytes(self) -> int:
         return sum(t.numel() * 4 for t in (self.S, self.N, self.Ms) if t is not None)
@@ -163,6 +175,20 @@ class GLAMixer(RecurrentMixer):
             raise ValueError(f"a2: shape {tuple(w['a2'].shape)}, expected {(self.H * self.D, rank)}")
         self.keep += [a2, a2b]
         self.desc.update(oa=self.proj.at["a1"], a2=a2.data_ptr(), a2b=a2b.data_ptr(), rank=rank, inv_tau=1.0 / float(m["tau"]))
+
+
+class RetentionMixer(RecurrentMixer):
+    """Linear attention with a constant decay per head and rotary positions; the head outputs are normed without a weight and
+    gated with SiLU."""
+
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, slots: int):
+        super().__init__(mo.KIND_RETENTION, w, [], m["heads"], m["dim"], m["vdim"], eps, dtype, device, slots)
+        rot = m.get("rot") or {"dims": 0, "base": 1.0}
+        freq = rotary_frequencies(rot["dims"], rot["base"])[0].to(device)
+        decay = torch.tensor([float(a) for a in m["decay"]], dtype=torch.float64)
+        powers = (decay[:, None] ** torch.arange(mo.CHUNK + 1, dtype=torch.float64)).float().to(device)
+        self.keep += [freq, powers]
+        self.desc.update(freq=freq.data_ptr() if rot["dims"] else None, rot=rot["dims"], pw=powers.data_ptr())
 
 
 def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> tuple[torch.Tensor, float]:
@@ -220,6 +246,11 @@ class LatentAttentionMixer:
             vs[:, :V, :K] = w["uv"].to(dtype).view(H, V, K)
             self.kv_w = kv.to(device)
 
+    def again(self):
+        o = copy.copy(self)
+        o.cache = torch.zeros_like(self.cache)
+        return o
+
     def cache_bytes(self) -> int:
         return self.cache.numel() * self.cache.element_size()
 
@@ -255,6 +286,85 @@ class LatentAttentionMixer:
         return self.out(ctx, mix, "y", torch.float32)
 
 
+class GroupedAttentionMixer:
+    """Grouped-query attention over pages of [keys | values]: causal, in a window or in chunks (`mask`), rotary positions on a
+    leading part of every query and key. With `diff` in its configuration a head has two softmax maps over the same values;
+    its output is a1 - lambda a2, normed without a weight and scaled by 1 - diff. Long portions in bf16 run the tensor-core
+    kernel on the pages, everything else the row kernel."""
+
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int, mask: str = "window"):
+        H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        diff = m.get("diff")
+        maps = 1 if diff is None else 2
+        if V > 512:
+            raise ValueError("attention takes value dims up to 512")
+        for n, r in (("q", H * maps * D), ("k", G * maps * D), ("v", G * V)):
+            if w[n].shape[0] != r:
+                raise ValueError(f"{n}: {w[n].shape[0]} rows, expected {r}")
+        self.H, self.G, self.D, self.V, self.maps, self.dtype = H, G, D, V, maps, dtype
+        self.proj = FusedLinear([("q", w["q"]), ("k", w["k"]), ("v", w["v"])], dtype, device)
+        self.out = FusedLinear([("o", w["o"])], dtype, device)
+        size = int((m.get("mask") or {}).get("size") or 0)
+        self.span = min(size, context) if size else context         # most positions a query sees
+        self.nsplit = max(1, min(64, (self.span + 31) // 32))
+        dp, vp = pad_to(D, 8), pad_to(V, 8)
+        self.row = G * (maps * dp + vp)
+        self.q_ld = pad_to(D, 64)
+        self.cache = torch.zeros(pages, mo.PAGE, self.row, dtype=dtype, device=device)
+        rot = m.get("rot") or {"dims": 0, "base": 1.0}
+        self.freq = rotary_frequencies(rot["dims"], rot["base"])[0].to(device)
+        a = self.proj.at
+        self.desc = dict(freq=self.freq.data_ptr() if rot["dims"] else None, oq=a["q"], ok=a["k"], ov=a["v"], H=H, G=G, maps=maps, D=D, V=V, R=rot["dims"],
+                         dp=dp, vp=vp, row=self.row, f32=int(dtype == torch.float32), window=size if mask == "window" else 0,
+                         chunk=size if mask == "chunk" else 0, q_ld=self.q_ld, scale=float(m["scale"]), eps=eps, post=1.0)
+        if maps == 2:
+            l = {n: w[n].double() for n in ("lq1", "lk1", "lq2", "lk2")}
+            lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + float(diff)
+            self.desc.update(lambda_=lam, head_norm=1, post=1.0 - float(diff))
+
+    def again(self):
+        o = copy.copy(self)
+        o.cache = torch.zeros_like(self.cache)
+        return o
+
+    def cache_bytes(self) -> int:
+        return self.cache.numel() * self.cache.element_size()
+
+    def describe(self, ctx: StepContext, p: torch.Tensor, out: torch.Tensor) -> mo.PagedAttention:
+        return mo.PagedAttention(proj=p.data_ptr(), ld=p.stride(0), pos=ctx.pos.data_ptr(), slot=ctx.slot.data_ptr(), cache=self.cache.data_ptr(),
+                                 table=ctx.table.data_ptr(), table_ld=ctx.table.stride(0), out=out.data_ptr(), ldo=out.stride(0),
+                                 status=ctx.status.data_ptr(), nsplit=1, **self.desc)
+
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+        T, ws, nq = ctx.T, ctx.ws, self.H * self.maps
+        p = self.proj(ctx, h, "proj", torch.float32)
+        mix = ws.rows("mix", T, self.out.K, self.dtype)
+        d = self.describe(ctx, p, mix)
+        form = mo.paged_prefill_form(self.maps, self.D, self.V) if ctx.n_long and self.dtype == torch.bfloat16 else -1
+        rows, nrows = (ctx.rows, ctx.n_rows) if form >= 0 or not ctx.n_long else (ctx.all_rows, T)
+        if nrows:
+            d.qx = ws.flat("qx", T * nq * self.D, torch.float32).data_ptr()
+        if form >= 0:
+            d.qf = ws.flat("qf", T * nq * self.q_ld, torch.bfloat16).data_ptr()
+        mo.paged_prep(d, T)
+        if form >= 0:
+            if form == 0:
+                d.part_o = ws.flat("raw_o", T * nq * self.V, torch.float32).data_ptr()
+            mo.paged_prefill(d, T, self.cache.shape[0], ctx.tiles, ctx.n_tiles, ctx.long)
+            if form == 0:
+                mo.paged_merge(d, None, T)         # rows of short portions are written again below
+        if nrows:
+            d.nsplit = self.nsplit if nrows <= 64 else 1
+            per = max(8, (64 << 20) // (d.nsplit * nq * self.V))
+            for a in range(0, nrows, per):
+                n = min(per, nrows - a)
+                d.part_o = ws.flat("part_o", n * d.nsplit * nq * self.V, torch.float32).data_ptr()
+                d.part_ml = ws.flat("part_ml", n * d.nsplit * nq * 2, torch.float32).data_ptr()
+                mo.paged_rows(d, rows[a:a + n], n)
+                mo.paged_merge(d, rows[a:a + n], n)
+        return self.out(ctx, mix, "y", torch.float32)
+
+
 class SwiGLU:
     """W_down (silu(W_gate h) * (W_up h)); the hidden size is padded to what the GEMM's epilogue takes."""
 
@@ -266,35 +376,78 @@ class SwiGLU:
         self.gate_up = gu.to(device)
         self.down = FusedLinear([("down", w["down"])], dtype, device, k_pad=self.ff)
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> tuple[torch.Tensor, None]:
         mid = ctx.ws.rows("mid", ctx.T, self.ff, self.dtype)
         mo.linear(h, self.gate_up, mid, ctx.status, swiglu=True)
-        return self.down(ctx, mid, "y", torch.float32)
+        return self.down(ctx, mid, "y", torch.float32), None
+
+
+class RoutedExperts:
+    """Routed experts W_down max(W_up x, 0)^2. Few rows (and fp32) stream the chosen experts' weights; many rows are grouped by
+    expert and multiplied on the tensor cores, and the sum over a token's experts is left to the norm that follows: `forward`
+    returns rows and, per token, which of them to add."""
+
+    def __init__(self, router_w: torch.Tensor, up: list[torch.Tensor], down: list[torch.Tensor], router: mo.Router, dtype, device):
+        E, (ff, K), W = router.experts, up[0].shape, down[0].shape[0]
+        self.route, self.W, self.dtype = router, W, dtype
+        self.router = FusedLinear([("router", router_w)], dtype, device)
+        self.ff, kp = pad_to(ff, 128), pad_to(K, 64)
+        self.up = torch.zeros(E, self.ff, kp, dtype=dtype, device=device)
+        self.down = torch.zeros(E, pad_to(W, 128), self.ff, dtype=dtype, device=device)
+        for e in range(E):
+            self.up[e, :ff, :K] = up[e].to(device=device, dtype=dtype)
+            self.down[e, :W, :ff] = down[e].to(device=device, dtype=dtype)
+
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor | None]:
+        T, ws, r = ctx.T, ctx.ws, self.route
+        R = T * r.top
+        z = self.router(ctx, h, "router", torch.float32)
+        ids = ws.flat("route_ids", R, torch.int32)
+        hidden = ws.rows("mid", R, self.ff, self.dtype)
+        if T <= mo.ROWS_MAX or self.dtype == torch.float32:
+            mo.expert_up_rows(r, z, h, self.up, ids, hidden)
+            y = ws.rows("y", T, self.down.shape[1], torch.float32)
+            mo.expert_down_rows(r, ids, hidden, self.down, self.W, y)
+            return y, None
+        place = ws.rows("route_place", T, r.top, torch.int32)
+        seg, scale = ws.flat("route_seg", r.experts + 1, torch.int32), ws.flat("route_scale", R, torch.float32)
+        x = ws.rows("route_x", R, self.up.shape[2], self.dtype)
+        mo.expert_group(r, z, h, ids, ws.flat("route_w", R, torch.float32), seg, place, scale, x)
+        mo.grouped_linear(x, self.up, seg, hidden, ctx.status, relu2=True, row_scale=scale, scale_after=r.on_output)
+        y = ws.rows("expert_y", R, self.down.shape[1], torch.float32)
+        mo.grouped_linear(hidden, self.down, seg, y, ctx.status)
+        return y, place
 
 
 @dataclass
-class SandwichLayer:
-    """A mixer and an optional feed-forward, each between two norms."""
+class MixerLayer:
+    """A mixer and an optional feed-forward, normed before and optionally (`norm1b`, `norm2b`) after."""
     mixer: object
     norm1: torch.Tensor
-    norm1b: torch.Tensor
-    mlp: SwiGLU | None = None
+    norm1b: torch.Tensor | None = None
+    mlp: object = None
     norm2: torch.Tensor | None = None
     norm2b: torch.Tensor | None = None
+    reinject: bool = False         # the embedding output is added to the residual stream before this layer
+
+    def again(self, reinject: bool) -> "MixerLayer":
+        """A further run of the layer: the same weights, a state or cache of its own."""
+        return replace(self, mixer=self.mixer.again(), reinject=reinject)
 
 
 @dataclass
 class MixerModel:
-    """What `runtime.mixer_runtime.MixerRuntime` runs: an embedding, layers, a final norm and an output matrix."""
+    """What `runtime.mixer_runtime.MixerRuntime` runs: an embedding, runs of layers, a final norm and an output matrix."""
     vocab: int
     width: int
     eps: float
     dtype: torch.dtype
     embed: torch.Tensor            # [vocab, width] bf16
-    layers: list[SandwichLayer]
-    final_norm: torch.Tensor
+    layers: list[MixerLayer]
+    final_norm: torch.Tensor       # a factor on the logits is part of it
     head: FusedLinear
     plus_one: bool = True          # norm weights are stored around zero
+    embed_scale: float = 1.0
 
     def windows(self) -> set[int]:
         return {L.mixer.window for L in self.layers if isinstance(L.mixer, LatentAttentionMixer)}

@@ -67,3 +67,8 @@ def _load() -> None:
     def _gidisun(path, **kw):
         from . import gidisun
         return gidisun.build_runtime(path, **kw)
+
+    @register("Pezarax", folder=True)
+    def _pezarax(path, **kw):
+        from . import pezarax
+        return pezarax.build_runtime(path, **kw)

@@ -1,20 +1,23 @@
-"""Bindings of the mixer-decoder kernels: sandwich norms on an fp32 residual stream, fp32 and few-row bf16 linears, recurrent
-outer-product states (gated linear attention, mLSTM), latent attention over a paged cache.
+"""Bindings of the mixer-decoder kernels: norms on an fp32 residual stream, fp32 and few-row bf16 linears, recurrent
+outer-product states (gated linear attention, mLSTM, retention), latent and grouped-query attention over a paged cache, routed
+experts.
 
 Every function launches on the current stream and writes into buffers its caller owns (so that a step can be captured in
 a CUDA graph); a non-zero status raises.
 """
 from __future__ import annotations
 
-import ctypes
 from ctypes import POINTER, Structure, byref, c_float, c_int, c_size_t, c_void_p
+from dataclasses import dataclass
 
 import torch
 
 from . import EPI_BF16, EPI_F32, EPI_SWIGLU, _check
 from . import lib as _lib
 
-KIND_GLA, KIND_MLSTM = 0, 1
+KIND_GLA, KIND_MLSTM, KIND_RETENTION = 0, 1, 2
+SCORES = {"sigmoid": 0, "softmax": 1}      # router scores
+EPI_RELU2 = 5       # grouped GEMM: squared ReLU with a factor per row
 PAGE = 64           # tokens per cache page
 CHUNK = 64          # tokens per chunk of the recurrent prefill form
 ROWS_MAX = 8        # widest portion (and batch) of the few-row kernels
@@ -22,9 +25,17 @@ ROWS_MAX = 8        # widest portion (and batch) of the few-row kernels
 
 class StateMixer(Structure):
     """`PkStateMixer`: columns of the fused projection, constants, state and raw outputs of one recurrent layer."""
-    _fields_ = [(n, c_void_p) for n in ("proj", "bi", "bf", "a2", "a2b", "S", "N", "Ms", "o", "nq", "m")] + \
-               [(n, c_int) for n in ("kind", "ld", "oq", "ok", "ov", "og", "oi", "of", "oa", "H", "D", "V", "rank")] + \
+    _fields_ = [(n, c_void_p) for n in ("proj", "bi", "bf", "a2", "a2b", "S", "N", "Ms", "o", "nq", "m", "freq", "pw")] + \
+               [(n, c_int) for n in ("kind", "ld", "oq", "ok", "ov", "og", "oi", "of", "oa", "H", "D", "V", "rank", "rot")] + \
                [(n, c_float) for n in ("qscale", "cap", "inv_tau")]
+
+
+class PagedAttention(Structure):
+    """`PkPagedAttention`: one grouped-query attention layer over one batch."""
+    _fields_ = [(n, c_void_p) for n in ("proj", "freq", "pos", "slot", "cache", "table", "qx", "qf", "part_o", "part_ml", "out", "status")] + \
+               [(n, c_int) for n in ("ld", "oq", "ok", "ov", "H", "G", "maps", "D", "V", "R", "dp", "vp", "row", "table_ld", "f32", "window", "chunk", "q_ld",
+                                     "ldo", "nsplit", "head_norm")] + \
+               [(n, c_float) for n in ("scale", "lambda_", "post", "eps")]
 
 
 _sms: dict[int, int] = {}
@@ -40,13 +51,16 @@ def sm_count() -> int:
 # argument kinds of the launchers, the stream excepted: p pointer, i int, f float
 _SIGNATURES = {
     "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
-    "pk_sandwich_norm": "pppipippiipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
+    "pk_sandwich_norm": "pppifipipippiipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
     "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii",
     "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipi",
     "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipi", "pk_latent_prefill": "pipipippiiiiifppip",
+    "pk_paged_prep": "pi", "pk_paged_rows": "ppi", "pk_paged_merge": "ppi", "pk_paged_prefill": "piipip",
+    "pk_expert_up_rows": "piiiiifipiipiiippii", "pk_expert_down_rows": "pipiipiiiipii", "pk_expert_group": "piiiiifipppppp" "iip",
+    "pk_gemm_bf16_grouped_scaled": "pippiiiiipipipi",
 }
 _bound: dict[tuple[int, str], object] = {}
-_KERNELS = {"pk_state_chunks": 5, "pk_latent_out": 2, "pk_argmax": 2, "pk_feed_tokens": 2}     # launches per call, where not 1
+_KERNELS = {"pk_state_chunks": 5, "pk_latent_out": 2, "pk_argmax": 2, "pk_feed_tokens": 2, "pk_expert_group": 3}     # launches per call, where not 1
 launches = 0        # kernels launched (or captured) by this process through `_call`
 
 
@@ -85,12 +99,15 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Te
 
 
 def sandwich_norm(x: torch.Tensor, *, eps: float, out: torch.Tensor | None = None, w_pre: torch.Tensor | None = None,
-                  tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, y: torch.Tensor | None = None,
-                  w_post: torch.Tensor | None = None, rows: torch.Tensor | None = None, count: int | None = None, plus_one: bool = True) -> None:
-    """One step of the residual stream x [rows, width] fp32 (see sandwich_norm.cu). `rows`/`count`: norm only these rows."""
+                  tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0, embed_add: bool = False,
+                  y: torch.Tensor | None = None, y_rows: torch.Tensor | None = None, w_post: torch.Tensor | None = None,
+                  rows: torch.Tensor | None = None, count: int | None = None, plus_one: bool = True) -> None:
+    """One step of the residual stream x [rows, width] fp32 (see sandwich_norm.cu). `rows`/`count`: norm only these rows; `y_rows`
+    [rows, n]: a row's y is the sum of these n rows of `y`; `embed_add`: the scaled embedding row is added instead of starting x."""
     M = (x.shape[0] if rows is None else rows.shape[0]) if count is None else count
-    _call("pk_sandwich_norm", x, tokens, embed, 0 if embed is None else embed.shape[0], y, 0 if y is None else y.stride(0), w_post, rows, M,
-          x.shape[1], w_pre, int(plus_one), eps, out, 0 if out is None else out.stride(0), int(out is not None and out.dtype == torch.float32))
+    _call("pk_sandwich_norm", x, tokens, embed, 0 if embed is None else embed.shape[0], embed_scale, int(embed_add), y, 0 if y is None else y.stride(0),
+          y_rows, 0 if y_rows is None else y_rows.shape[1], w_post, rows, M, x.shape[1], w_pre, int(plus_one), eps, out,
+          0 if out is None else out.stride(0), int(out is not None and out.dtype == torch.float32))
 
 
 def feed_tokens(nxt: torch.Tensor, tokens: torch.Tensor, pos: torch.Tensor, seqs: torch.Tensor, hist: torch.Tensor, step: torch.Tensor) -> None:
@@ -117,11 +134,13 @@ def state_chunk_workspace(d: StateMixer, nchunks: int) -> int:
 
 
 def state_chunks(d: StateMixer, seqs: torch.Tensor, nseq: int, chunks: torch.Tensor, chunk0: torch.Tensor, nchunks: int, ws: torch.Tensor) -> None:
+    global launches
     _call("pk_state_chunks", byref(d), seqs, nseq, chunks, chunk0, nchunks, ws)
+    launches -= int(d.kind == KIND_RETENTION)      # no gates
 
 
-def state_out(d: StateMixer, norm_w: torch.Tensor, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
-    """Head norm + output gate of `rows` rows; norm_w [H * V], or [V] when `per_head`."""
+def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
+    """Head norm + output gate of `rows` rows; norm_w [H * V], [V] when `per_head`, or None."""
     _call("pk_state_out", byref(d), norm_w, int(per_head), eps, last_slot, rows, out, out.stride(0), int(out.dtype == torch.float32))
 
 
@@ -157,3 +176,71 @@ def latent_prefill(q: torch.Tensor, nrows: int, kv: torch.Tensor, kv_rows: int, 
                    out: torch.Tensor, status: torch.Tensor) -> None:
     _call("pk_latent_prefill", q, nrows, kv, kv_rows, tiles, ntiles, seqs, gather, H, qk_panels, v_panels, V, window, scale, sink, out,
           out.stride(0), status)
+
+
+def paged_prep(a: PagedAttention, rows: int) -> None:
+    """Rotation, cache append and queries of all rows of a step."""
+    _call("pk_paged_prep", byref(a), rows)
+
+
+def paged_rows(a: PagedAttention, rows: torch.Tensor, nrows: int) -> None:
+    """Partial attention of the listed rows (splits into part_o / part_ml)."""
+    _call("pk_paged_rows", byref(a), rows, nrows)
+
+
+def paged_merge(a: PagedAttention, rows: torch.Tensor | None, nrows: int) -> None:
+    """Splits (or finished fp32 outputs) of the listed rows -> head outputs."""
+    _call("pk_paged_merge", byref(a), rows, nrows)
+
+
+def paged_prefill_form(maps: int, D: int, V: int) -> int:
+    """What the tensor-core kernel does with this shape: 1 finished outputs, 0 fp32 outputs for `paged_merge`, -1 nothing."""
+    fn = _lib.kernels().pk_paged_prefill_form
+    fn.restype, fn.argtypes = c_int, [c_int, c_int, c_int]
+    return int(fn(maps, D, V))
+
+
+def paged_prefill(a: PagedAttention, rows: int, pages: int, tiles: torch.Tensor, ntiles: int, seqs: torch.Tensor) -> None:
+    _call("pk_paged_prefill", byref(a), rows, pages, tiles, ntiles, seqs)
+
+
+@dataclass(frozen=True)
+class Router:
+    """How experts are chosen and weighted from router logits."""
+    experts: int
+    top: int
+    score: str = "sigmoid"
+    renorm: bool = False        # chosen weights divided by their sum
+    scale: float = 1.0
+    on_output: bool = False     # the weight multiplies an expert's output instead of its input
+
+    def args(self) -> tuple:
+        return self.experts, self.top, SCORES[self.score], int(self.renorm), self.scale
+
+
+def expert_up_rows(r: Router, logits: torch.Tensor, x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor) -> None:
+    """hidden [T * top, N] = squared ReLU of the chosen experts' up products; w [experts, N, K]; ids [T * top] out."""
+    E, N, K = w.shape
+    _call("pk_expert_up_rows", logits, logits.stride(0), *r.args(), int(r.on_output), x, x.stride(0), x.shape[0], w, N, K,
+          int(w.dtype == torch.float32), ids, hidden, hidden.stride(0), sm_count())
+
+
+def expert_down_rows(r: Router, ids: torch.Tensor, hidden: torch.Tensor, w: torch.Tensor, n: int, y: torch.Tensor) -> None:
+    """y [T, n] fp32 = sum over a token's experts of w[expert, :n] . hidden; w [experts, rows, K]."""
+    E, rows, K = w.shape
+    _call("pk_expert_down_rows", ids, r.top, hidden, hidden.stride(0), y.shape[0], w, n, rows, K, int(w.dtype == torch.float32), y, y.stride(0), sm_count())
+
+
+def expert_group(r: Router, logits: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, seg: torch.Tensor, place: torch.Tensor,
+                 row_scale: torch.Tensor, rows: torch.Tensor) -> None:
+    """Routes of the tokens grouped by expert, token rows gathered in that order (rows [T * top, K])."""
+    _call("pk_expert_group", logits, logits.stride(0), *r.args(), x.shape[0], ids, weights, seg, place, row_scale, x, x.stride(0), rows.shape[1], rows)
+
+
+def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, out: torch.Tensor, status: torch.Tensor, *, relu2: bool = False,
+                   row_scale: torch.Tensor | None = None, scale_after: bool = False) -> None:
+    """out rows of group g = x rows . w[g]^T on the tensor cores (x, w bf16; w [groups, N, K], N a multiple of 128, K of 64); fp32 out,
+    or bf16 squared ReLU with a factor per row."""
+    G, N, K = w.shape
+    _call("pk_gemm_bf16_grouped_scaled", x, x.stride(0), w, seg, G, x.shape[0], N, K, EPI_RELU2 if relu2 else EPI_F32, out, out.stride(0), row_scale,
+          int(scale_after), status, sm_count())

@@ -161,27 +161,31 @@ class MixerRuntime:
         x = ws.rows("x", T, m.width, torch.float32)
         h = ws.rows("h", T, hk, m.dtype)
         kw = dict(eps=m.eps, plus_one=m.plus_one)
+        emb = dict(tokens=ctx.tokens, embed=m.embed, embed_scale=m.embed_scale)
         first = m.layers[0].norm1 if m.layers else None
-        mo.sandwich_norm(x, tokens=ctx.tokens, embed=m.embed, w_pre=first, out=h, **kw)
-        y = w_post = None
+        mo.sandwich_norm(x, w_pre=first, out=h, **emb, **kw)
+        y: dict = {}                                                    # sublayer output that is still to be added to x
         for i, L in enumerate(m.layers):
             if i:
-                mo.sandwich_norm(x, y=y, w_post=w_post, w_pre=L.norm1, out=h, **kw)
                 if self.launch_layers is not None:
+                    mo.sandwich_norm(x, **y, **kw)
                     self.launch_layers.append(x.clone())
-            y, w_post = L.mixer.forward(ctx, h), L.norm1b
+                    y = {}
+                mo.sandwich_norm(x, w_pre=L.norm1, out=h, **y, **(dict(embed_add=True, **emb) if L.reinject else {}), **kw)
+            y = dict(y=L.mixer.forward(ctx, h), w_post=L.norm1b)
             if L.mlp is not None:
-                mo.sandwich_norm(x, y=y, w_post=w_post, w_pre=L.norm2, out=h, **kw)
-                y, w_post = L.mlp.forward(ctx, h), L.norm2b
-        if self.launch_layers is not None and y is not None:
-            mo.sandwich_norm(x, y=y, w_post=w_post, **kw)
+                mo.sandwich_norm(x, w_pre=L.norm2, out=h, **y, **kw)
+                out, rows = L.mlp.forward(ctx, h)
+                y = dict(y=out, y_rows=rows, w_post=L.norm2b)
+        if self.launch_layers is not None and y:
+            mo.sandwich_norm(x, **y, **kw)
             self.launch_layers.append(x.clone())
-            y = None
+            y = {}
         n = T if want is None else n_want
         if n == 0:
             return None
         hf = ws.rows("h_final", n, hk, m.dtype)
-        mo.sandwich_norm(x, y=y, w_post=w_post, rows=want, count=n, w_pre=m.final_norm, out=hf, **kw)
+        mo.sandwich_norm(x, rows=want, count=n, w_pre=m.final_norm, out=hf, **y, **kw)
         return m.head(ctx, hf, "logits", torch.float32)
 
     def _mixed(self, entries: Sequence[StepEntry]) -> torch.Tensor:
