@@ -70,10 +70,10 @@ def beacon_tensors(cfg: dict, seed=0) -> dict:
 
 
 class OracleRuntime:
-    """The oracle behind the interface of `MixerRuntime` (CPU, float64)."""
+    """An oracle behind the interface of `MixerRuntime` (CPU, float64)."""
 
-    def __init__(self, cfg: dict, weights: dict, max_requests=3, pages=12, page=16):
-        self.m, self.vocab, self.max_requests, self.max_tokens = mr.PlainModel(cfg, weights), cfg["vocab"], max_requests, pages * page
+    def __init__(self, cfg: dict, weights: dict, max_requests=3, pages=12, page=16, plain=mr.PlainModel):
+        self.m, self.vocab, self.max_requests, self.max_tokens = plain(cfg, weights), cfg["vocab"], max_requests, pages * page
         self.cache = RequestCache(max_requests, pages, page, device=None)
         self.st: dict = {}
         self.calls: list[list[int]] = []

@@ -9,45 +9,18 @@ import mixer_reference as mr
 import pytest
 import torch
 from gidisun_cases import BEACON, beacon_tensors, config, gla, latent, mlstm, tensors, tokens
+from mixer_checks import BF16, F32, check, feed, make_runtime, margin_prefix, traffic
 
 from pocketllm_b200.models import gidisun as gd
 from pocketllm_b200.server.engine import SamplingParams
 
 pytestmark = pytest.mark.gpu
 ROOT = Path(__file__).resolve().parent.parent
-TOL = {torch.float32: 1e-4, torch.bfloat16: 0.08}
-F32, BF16 = torch.float32, torch.bfloat16
 FULL = config([mlstm(ff=90), latent(ff=70), gla(), latent(heads=2, window=17, scaling=False), mlstm(heads=1, dim=9, vdim=40)], vocab=101, width=88)
 
 
-def runtime(cfg, t, dtype=F32, max_requests=4, pages=24, **kw):
-    from pocketllm_b200.runtime.mixer_runtime import MixerRuntime
-    model = gd.build_model(gd.GidisunConfig.from_dict(cfg), t, dtype=dtype, slots=max_requests, pages=pages)
-    return MixerRuntime(model, max_requests=max_requests, pages=pages, **kw)
-
-
-def feed(rt, rid, toks, cuts, end=True):
-    """Logits of all places of `toks`, run in portions of the given sizes (the last size repeats)."""
-    from pocketllm_b200.runtime.mixer_runtime import StepEntry
-    out, a, i = [], 0, 0
-    while a < len(toks):
-        n = min(cuts[min(i, len(cuts) - 1)], len(toks) - a)
-        out.append(rt.step([StepEntry(rid, toks[a:a + n], range(n))]).clone())
-        a, i = a + n, i + 1
-    rt.check_status()
-    if end:
-        rt.release(rid)
-    return torch.cat(out).double().cpu()
-
-
-def off(got, want):
-    """Per place: rms difference over the vocabulary relative to the logits' spread."""
-    return ((got - want).pow(2).mean(-1).sqrt() / want.std()).max().item()
-
-
-def check(got, want, dtype=F32, factor=1.0):
-    e = off(got, want)
-    assert e < TOL[dtype] * factor, e
+def runtime(cfg, t, dtype=F32, **kw):
+    return make_runtime(gd, gd.GidisunConfig, cfg, t, dtype, **kw)
 
 
 _memo: dict = {}
@@ -194,42 +167,13 @@ def test_portions(cuts, dtype):
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
 def test_unequal_requests_in_one_batch_and_reused_room(dtype):
-    """Twelve requests through three slots and few pages: portions beside single tokens, requests that rest for some steps,
-    pages and slots used again. Every place is compared with the request alone."""
-    from pocketllm_b200.runtime.mixer_runtime import StepEntry
+    """Twelve requests through three slots and few pages. Every place is compared with the request alone."""
     t = tensors(FULL, 8)
-    lens = [200, 1, 65, 64, 130, 2, 77, 9, 128, 33, 190, 17]
-    seqs = [tokens(n, FULL["vocab"], 20 + i) for i, n in enumerate(lens)]
-    rt = runtime(FULL, t, dtype, max_requests=3, pages=9)
-    g = torch.Generator().manual_seed(5)
-    at, got, live, nxt = {}, {i: [] for i in range(12)}, [], 0
-    while nxt < 12 or live:
-        while nxt < 12 and len(live) < 3 and sum(-(-lens[i] // 64) for i in live + [nxt]) <= 9:
-            live.append(nxt)
-            at[nxt] = 0
-            nxt += 1
-        entries = []
-        for i in live:
-            if len(live) > 1 and torch.rand(1, generator=g) < 0.2 and entries:
-                continue
-            n = [1, 1, 2, 5, 8, 9, 40, 64, 90][int(torch.randint(0, 9, (1,), generator=g))]
-            n = min(n, lens[i] - at[i])
-            entries.append(StepEntry(i, seqs[i][at[i]:at[i] + n], range(n)))
-        z = rt.step(entries).double().cpu()
-        a = 0
-        for e in entries:
-            n = len(e.tokens)
-            got[e.rid].append(z[a:a + n])
-            a += n
-            at[e.rid] += n
-            if at[e.rid] == lens[e.rid]:
-                rt.release(e.rid)
-                live.remove(e.rid)
-    rt.check_status()
-    assert rt.cache.free_pages == 9 and rt.cache.free_slots == 3
+    seqs = [tokens(n, FULL["vocab"], 20 + i) for i, n in enumerate([200, 1, 65, 64, 130, 2, 77, 9, 128, 33, 190, 17])]
+    got = traffic(runtime(FULL, t, dtype, max_requests=3, pages=9), seqs, 3, 9)
     m = mr.PlainModel(FULL, t)
-    for i in range(12):
-        check(torch.cat(got[i]), m.logits(seqs[i]), dtype)
+    for seq, z in zip(seqs, got):
+        check(z, m.logits(seq), dtype)
 
 
 def test_wanted_places_and_errors():
@@ -308,21 +252,6 @@ def test_long_decoding(dtype):
     want = oracle(FULL, t, seq, "long")
     rt = runtime(FULL, t, dtype)
     check(feed(rt, "a", seq, [20, 1]), want, dtype)
-
-
-def margin_prefix(m, prompt, n, eps):
-    """Greedy continuation of the oracle up to the first near-tie."""
-    st = m.new_state()
-    for x in prompt:
-        z = m.step(st, x)
-    out = []
-    for _ in range(n):
-        top = torch.topk(z, 2).values
-        if top[0] - top[1] < eps:
-            break
-        out.append(int(z.argmax()))
-        z = m.step(st, out[-1])
-    return out
 
 
 def test_greedy_generation_through_the_scheduler():
