@@ -279,79 +279,38 @@ def run_minimax(args) -> dict:
     return res if rank == 0 else {}
 
 
-def run_gidisun(args) -> dict:
-    """Prefill and decode throughput of the Gidisun design (mLSTM, GLA and windowed latent-attention layers with SwiGLU) at a
-    size that resembles a real model's layers, beside the closest existing model at equal size. One step = one request:
-    prefill of `--prompt-len` tokens, then `--decode-len` greedy tokens; a second figure decodes `--batch` requests together."""
+def run_mixer(args) -> dict:
+    """Prefill and decode throughput of a mixer decoder (Gidisun: mLSTM, GLA and windowed latent attention with SwiGLU; Pezarax:
+    retention and chunked differential attention with routed experts) at a size that resembles a real model's layers, beside
+    the closest other model at equal size. One step = one request: prefill of `--prompt-len` tokens, then `--decode-len` greedy
+    tokens; a second figure decodes `--batch` requests together."""
     import torch
-    from pocketllm_b200.runtime.mixer_runtime import StepEntry
     from pocketllm_b200.utils import bench_mixers as bm
     if args.gpus != 1:
-        raise SystemExit("--model gidisun runs on one GPU")
+        raise SystemExit(f"--model {args.model} runs on one GPU")
     torch.cuda.set_device(0)
-    B, n, d = args.batch, args.prompt_len, args.decode_len
-    rt, streamed = bm.build(args.size, B, n + d + 64)
+    B, n, d, k = args.batch, args.prompt_len, args.decode_len, args.steps
+    rt, streamed = bm.build(args.model, args.size, B, n + d + 64)
     g = torch.Generator().manual_seed(1234)
-    prompts = [torch.randint(0, bm.VOCAB, (n,), generator=g).tolist() for _ in range(args.warmup + args.steps)]
-    e0, e1, e2 = (torch.cuda.Event(enable_timing=True) for _ in range(3))
-
-    def request(prompt, rids):
-        """(first tokens, prefill ms, decode ms) of the same prompt for every id, decoded together."""
-        e0.record()
-        tok = [int(rt.step([StepEntry(r, prompt, (n - 1,))])[0].argmax()) for r in rids]
-        e1.record()
-        for a in range(0, d, rt.HIST):
-            k = min(rt.HIST, d - a)
-            out = rt.decode_greedy(rids, tok, k)
-            tok = [o[-1] for o in out]
-        e2.record()
-        torch.cuda.synchronize()
-        for r in rids:
-            rt.release(r)
-        return tok, e0.elapsed_time(e1), e1.elapsed_time(e2)
-
-    for i in range(args.warmup):
-        request(prompts[i], [0])
-        request(prompts[i], list(range(B)))
-    pre = dec = dec_b = 0.0
-    l0 = rt.launches
-    torch.cuda.synchronize()
-    t0 = time.perf_counter()
-    with ClockSampler(0) as clocks:
-        for i in range(args.steps):
-            toks, a, b = request(prompts[args.warmup + i], [0])
-            pre, dec = pre + a, dec + b
-        torch.cuda.synchronize()
-    wall_ms = (time.perf_counter() - t0) * 1e3
-    launches = rt.launches - l0
-    for i in range(args.steps):
-        dec_b += request(prompts[args.warmup + i], list(range(B)))[2]
-    # end to end through the step function: prompt ids from the host, every token read back as soon as its step ends
-    e_dec = 0.0
-    for i in range(args.steps):
-        tok = int(rt.step([StepEntry(0, prompts[args.warmup + i], (n - 1,))])[0].argmax())
-        torch.cuda.synchronize()
-        w0 = time.perf_counter()
-        for _ in range(d):
-            tok = int(rt.step([StepEntry(0, [tok], (0,))])[0].argmax())
-        e_dec += time.perf_counter() - w0
-        rt.release(0)
-    rt.check_status()
+    prompts = [torch.randint(0, bm.VOCAB, (n,), generator=g).tolist() for _ in range(args.warmup + k)]
+    clocks = ClockSampler(0)
+    r = bm.requests(rt, prompts, n, d, args.warmup, B, clocks)
+    layers, width = len(rt.model.layers), rt.model.width
     del rt
     torch.cuda.empty_cache()
-    like = bm.closest_model(args.size, n, d, args.steps)
-    value = args.steps * d / dec * 1e3
-    return {"metric": f"single-request decode tok/s (Gidisun, 8 layers of width {bm.SIZES[args.size][0]}, {n}-token prompt, {d} greedy steps)",
-            "value": round(value, 2), "unit": "tok/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
-            "ms_per_step": round((pre + dec) / args.steps, 3), "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
-            "data": "synthetic: uniform-random token prompts, random-init weights", "prefill_tok_s": round(args.steps * n / pre * 1e3, 1),
-            "decode_tok_s_batch": {"batch": B, "value": round(args.steps * d * B / dec_b * 1e3, 1)},
+    like = bm.closest_model(args.size, n, d, k) if args.model == "gidisun" else bm.closest_to_pezarax(args.size, prompts, n, d, args.warmup, B)
+    value = k * d / r["decode_ms"] * 1e3
+    return {"metric": f"single-request decode tok/s ({args.model.capitalize()}, {layers} layers of width {width}, {n}-token prompt, {d} greedy steps)",
+            "value": round(value, 2), "unit": "tok/s", "n_gpus": 1, "steps": k, "warmup": args.warmup,
+            "ms_per_step": round((r["prefill_ms"] + r["decode_ms"]) / k, 3), "higher_is_better": True, "scaling": "strong", "vs_baseline": None, "dtype": "bf16",
+            "data": "synthetic: uniform-random token prompts, random-init weights", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
+            "decode_tok_s_batch": {"batch": B, "value": round(k * d * B / r["batch_ms"] * 1e3, 1)},
             "decode_weight_gbs": round(streamed * value / 1e9, 1), "weight_gb": round(streamed / 1e9, 2), "closest_model": like,
-            "config": {"model": f"gidisun-{args.size}", "global_batch": 1, "seq_len": n, "decode_len": d, "parallelism": "tp1",
+            "config": {"model": f"{args.model}-{args.size}", "global_batch": 1, "seq_len": n, "decode_len": d, "parallelism": "tp1",
                        "l2": "weights larger than L2"},
             "clocks": clocks.summary(),
-            "e2e": {"value": round(args.steps * d / e_dec, 2), "unit": "tok/s", "h2d_bytes_per_step": n * 4 + d * 32, "d2h_bytes_per_step": (d + 1) * 8},
-            "gpu_launches": int(launches), "wall_ms": round(wall_ms, 1)}
+            "e2e": {"value": round(k * d / r["e2e_s"], 2), "unit": "tok/s", "h2d_bytes_per_step": n * 4 + d * 32, "d2h_bytes_per_step": (d + 1) * 8},
+            "gpu_launches": int(r["launches"]), "wall_ms": round(r["wall_ms"], 1)}
 
 
 # what the many-row GEMMs multiply, by the engine's prefill_gemm mode
@@ -373,9 +332,9 @@ def main() -> int:
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--decode-len", type=int, default=256)
     ap.add_argument("--prefill-chunk", type=int, default=512)
-    ap.add_argument("--model", default="qwen27b", choices=["qwen27b", "tiny", "minimax-m2", "gidisun"])
-    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="gidisun: width of the layers")
-    ap.add_argument("--batch", type=int, default=8, help="gidisun: requests decoded together for the second decode figure")
+    ap.add_argument("--model", default="qwen27b", choices=["qwen27b", "tiny", "minimax-m2", "gidisun", "pezarax"])
+    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="gidisun, pezarax: width of the layers")
+    ap.add_argument("--batch", type=int, default=8, help="gidisun, pezarax: requests decoded together for the second decode figure")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
@@ -384,8 +343,8 @@ def main() -> int:
         res = reference_arm.run(args)
     elif args.model == "minimax-m2":
         res = run_minimax(args)
-    elif args.model == "gidisun":
-        res = run_gidisun(args)
+    elif args.model in ("gidisun", "pezarax"):
+        res = run_mixer(args)
     else:
         res = run_ours(args)
     if res:

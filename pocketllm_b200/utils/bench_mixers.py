@@ -1,9 +1,10 @@
-"""Throughput of mixer decoders (Gidisun) at sizes that resemble a real model's layers, beside the closest existing model at
-equal size (the Qwen hybrid: DeltaNet + GQA, same width, feed-forward, depth and vocabulary), and the time of each new
-kernel beside the like kernel of the existing families.
+"""Throughput of mixer decoders at sizes that resemble a real model's layers, beside the closest other model at equal size
+(Gidisun: the Qwen hybrid, DeltaNet + GQA with the same width, feed-forward, depth and vocabulary; Pezarax: Gidisun with the
+same width, heads, depth and as many weights per token in its feed-forward), and the time of each design's kernels beside the
+like kernels of the other families.
 
-    python -m pocketllm_b200.utils.bench_mixers --kernels
-    python bench.py --model gidisun [--size 2k|4k]
+    python -m pocketllm_b200.utils.bench_mixers --kernels [gidisun|pezarax]
+    python bench.py --model gidisun|pezarax [--size 2k|4k]
 
 Random weights; every weight set is larger than L2. Device times by CUDA events.
 """
@@ -15,6 +16,7 @@ import json
 import torch
 
 from ..models import gidisun as gd
+from ..models import pezarax as pz
 
 VOCAB = 32000
 #            width  ff     mLSTM (heads, dim, vdim)  GLA              latent (heads, dim, rot, vdim, rank, window)
@@ -23,8 +25,26 @@ SIZES = {"2k": (2048, 6144, (8, 128, 256), (16, 128, 128), (16, 128, 64, 128, 51
 PATTERN = ("mlstm", "latent_attention", "gla", "gla", "mlstm", "latent_attention", "gla", "mlstm")
 
 
-def config(size: str) -> gd.GidisunConfig:
-    W, ff, m, g, a = SIZES[size]
+#                  width  retention (heads, dim, vdim)  attention (heads, kv heads, dim, vdim, chunk)  experts (number, top, ff)
+PEZARAX_SIZES = {"2k": (2048, (16, 128, 128), (16, 4, 64, 128, 1024), (32, 2, 1536)),
+                 "4k": (4096, (16, 128, 256), (32, 8, 64, 128, 1024), (32, 2, 3072))}
+PEZARAX_PATTERN = ("retention", "attention", "retention", "retention", "retention", "attention", "retention", "retention")
+
+
+def pezarax_config(size: str) -> pz.PezaraxConfig:
+    W, r, a, e = PEZARAX_SIZES[size]
+    decay = [1.0 - 2.0 ** (-5 - 8 * i / r[0]) for i in range(r[0])]
+    mix = {"retention": {"heads": r[0], "dim": r[1], "vdim": r[2], "decay": decay, "rot": {"base": 1e4, "dims": r[1]}},
+           "attention": {"heads": a[0], "kv_heads": a[1], "dim": a[2], "vdim": a[3], "scale": a[2] ** -0.5, "diff": 0.4, "mask": {"size": a[4]},
+                         "rot": {"base": 5e5, "dims": a[2]}}}
+    mlp = {"kind": "moe", "expert": {"ff": e[2]}, "router": {"experts": e[0], "top": e[1]}}
+    return pz.PezaraxConfig.from_dict({"architecture": pz.ARCH, "vocab": VOCAB, "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0}, "logit_scale": 0.5,
+                                       "layers": [{"type": t, "mixer": mix[t], "mlp": mlp} for t in PEZARAX_PATTERN]})
+
+
+def config(size: str, ff: int | None = None) -> gd.GidisunConfig:
+    W, dense_ff, m, g, a = SIZES[size]
+    ff = ff or dense_ff
     mix = {"mlstm": {"heads": m[0], "dim": m[1], "vdim": m[2], "gate_cap": 12.0},
            "gla": {"heads": g[0], "dim": g[1], "vdim": g[2], "tau": 14.0},
            "latent_attention": {"heads": a[0], "dim": a[1], "rot_dim": a[2], "vdim": a[3], "kv_rank": a[4], "scale": (a[1] + a[2]) ** -0.5,
@@ -34,13 +54,82 @@ def config(size: str) -> gd.GidisunConfig:
                                        "layers": [{"type": t, "mixer": mix[t], "mlp": {"kind": "dense", "ff": ff}} for t in PATTERN]})
 
 
-def build(size: str, batch: int, context: int):
+def build(design: str, size: str, batch: int, context: int, ff: int | None = None):
+    """(runtime with random weights, bytes of weights that one decoded token streams)."""
     from ..runtime.mixer_runtime import MixerRuntime
-    c = config(size)
-    t = {n: v.cpu() for n, v in gd.random_tensors(c, 0, device="cuda").items()}
+    mod, c = (gd, config(size, ff)) if design == "gidisun" else (pz, pezarax_config(size))
+    t = mod.random_tensors(c, 0, device="cuda")
     pages = batch * (-(-context // 64))
-    streamed = sum(v.numel() for n, v in t.items() if n != "embed") * 2
-    return MixerRuntime(gd.build_model(c, t, slots=batch, pages=pages), max_requests=batch, pages=pages), streamed
+    streamed = 0.0
+    for n, v in t.items():
+        share = 1.0
+        if ".mlp.e" in n:
+            L = c.layers[int(n[1:n.index(".")])]
+            share = L.top / L.experts
+        streamed += v.numel() * 2 * share if n != "embed" else 0.0
+    rt = MixerRuntime(mod.build_model(c, t, slots=batch, pages=pages), max_requests=batch, pages=pages)
+    return rt, streamed
+
+
+def requests(rt, prompts, n: int, d: int, warmup: int, batch: int, clocks=None) -> dict:
+    """Prefill and decode milliseconds of single requests, decode milliseconds of `batch` requests together, and end-to-end
+    decode seconds with every token read back: sums over the prompts behind the first `warmup`."""
+    import contextlib
+    import time
+
+    from ..runtime.mixer_runtime import StepEntry
+    e0, e1, e2 = (torch.cuda.Event(enable_timing=True) for _ in range(3))
+
+    def request(prompt, rids):
+        e0.record()
+        tok = [int(rt.step([StepEntry(r, prompt, (n - 1,))])[0].argmax()) for r in rids]
+        e1.record()
+        for a in range(0, d, rt.HIST):
+            out = rt.decode_greedy(rids, tok, min(rt.HIST, d - a))
+            tok = [o[-1] for o in out]
+        e2.record()
+        torch.cuda.synchronize()
+        for r in rids:
+            rt.release(r)
+        return e0.elapsed_time(e1), e1.elapsed_time(e2)
+
+    for p in prompts[:warmup]:
+        request(p, [0])
+        request(p, list(range(batch)))
+    r = dict(prefill_ms=0.0, decode_ms=0.0, batch_ms=0.0, e2e_s=0.0)
+    l0 = rt.launches
+    torch.cuda.synchronize()
+    t0 = time.perf_counter()
+    with clocks if clocks is not None else contextlib.nullcontext():
+        for p in prompts[warmup:]:
+            a, b = request(p, [0])
+            r["prefill_ms"] += a
+            r["decode_ms"] += b
+        torch.cuda.synchronize()
+    r.update(wall_ms=(time.perf_counter() - t0) * 1e3, launches=rt.launches - l0)
+    for p in prompts[warmup:]:
+        r["batch_ms"] += request(p, list(range(batch)))[1]
+    # end to end through the step function: prompt ids from the host, every token read back as soon as its step ends
+    for p in prompts[warmup:]:
+        tok = int(rt.step([StepEntry(0, p, (n - 1,))])[0].argmax())
+        torch.cuda.synchronize()
+        w0 = time.perf_counter()
+        for _ in range(d):
+            tok = int(rt.step([StepEntry(0, [tok], (0,))])[0].argmax())
+        r["e2e_s"] += time.perf_counter() - w0
+        rt.release(0)
+    rt.check_status()
+    return r
+
+
+def closest_to_pezarax(size: str, prompts, n: int, d: int, warmup: int, batch: int) -> dict:
+    """Gidisun with a SwiGLU of as many weights per token as the chosen experts have."""
+    _, _, _, (_, top, ff) = PEZARAX_SIZES[size]
+    rt, streamed = build("gidisun", size, batch, n + d + 64, ff=2 * top * ff // 3)
+    r, k = requests(rt, prompts, n, d, warmup, batch), len(prompts) - warmup
+    return {"model": "Gidisun (mLSTM, GLA, latent attention, SwiGLU; bf16 weights)", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
+            "decode_tok_s": round(k * d / r["decode_ms"] * 1e3, 1), "decode_tok_s_batch": round(k * d * batch / r["batch_ms"] * 1e3, 1),
+            "weight_gb_per_token": round(streamed / 1e9, 2), "decode_weight_gbs": round(streamed * k * d / r["decode_ms"] / 1e6, 1)}
 
 
 def closest_model(size: str, prompt: int, decode: int, reps: int) -> dict:
@@ -127,7 +216,9 @@ def _state(kind: str, dims, T: int, singles: bool):
     g = torch.Generator().manual_seed(0)
     r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
     w = {"q": r(H * D, W), "k": r(H * D, W), "v": r(H * V, W), "g": r(H * V, W), "o": r(W, H * V)}
-    if kind == "mlstm":
+    if kind == "retention":
+        m = ml.RetentionMixer(w, {"heads": H, "dim": D, "vdim": V, "decay": [0.99] * H, "rot": {"base": 1e4, "dims": D}}, 1e-5, torch.bfloat16, "cuda", b.slots)
+    elif kind == "mlstm":
         w.update({"i": r(H, W), "f": r(H, W), "i.b": torch.zeros(H), "f.b": torch.full((H,), 3.0), "norm": torch.ones(H * V)})
         m = ml.MLSTMMixer(w, {"heads": H, "dim": D, "vdim": V, "gate_cap": 12.0}, 1e-5, torch.bfloat16, "cuda", b.slots)
     else:
@@ -247,13 +338,145 @@ def kernels() -> None:
         show("like kernel: RMSNorm with residual add", _roof(timed(lambda: ops.rmsnorm(xb, w, parts=y[None], hidden_out=o)), 0, T * 4096 * 10.0), T=T)
 
 
+def _paged(dims, T: int, start: int, singles: bool):
+    """The attention of one differential layer after its input projection, without the output projection; returns
+    {kernel: (call, flops, bytes)}."""
+    from ..models import mixer_layers as ml
+    from ..ops import mixer_ops as mo
+    H, G, D, V, chunk = dims
+    W, nq = 1024, 2 * dims[0]
+    b = _Batch(T, start, start + T, singles=singles)
+    g = torch.Generator().manual_seed(0)
+    r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
+    m = ml.GroupedAttentionMixer({"q": r(nq * D, W), "k": r(2 * G * D, W), "v": r(G * V, W), "o": r(W, H * V), **{n: torch.zeros(D) for n in ("lq1", "lk1", "lq2", "lk2")}},
+                                 {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": D ** -0.5, "diff": 0.4, "mask": {"size": chunk} if chunk else None,
+                                  "rot": {"base": 1e4, "dims": D}}, 1e-5, torch.bfloat16, "cuda", b.pages, start + T, mask="chunk")
+    m.cache.normal_()
+    ctx, ws = b.ctx, b.ctx.ws
+    p = m.proj(ctx, torch.randn(T, m.proj.K, device="cuda").to(torch.bfloat16), "proj", torch.float32)
+    mix = ws.rows("mix", T, m.out.K, torch.bfloat16)
+    d = m.describe(ctx, p, mix)
+    see = lambda q: q + 1 - (q // chunk * chunk if chunk else 0)
+    span = T * see(start) if singles else sum(see(start + i) for i in range(T))
+    keep = (m, b, p, mix)
+    flops = 2.0 * span * nq * (D + V)
+    if singles:
+        d.nsplit = m.nsplit
+        po, pm = ws.flat("po", T * m.nsplit * nq * V, torch.float32), ws.flat("pm", T * m.nsplit * nq * 2, torch.float32)
+        qx = ws.flat("qx", T * nq * D, torch.float32)
+        d.qx, d.part_o, d.part_ml = qx.data_ptr(), po.data_ptr(), pm.data_ptr()
+        return {"prep": (lambda k=keep: mo.paged_prep(d, T), 0, 0), "rows": (lambda k=(po, pm, qx): mo.paged_rows(d, ctx.rows, T), flops, span * m.row * 2.0),
+                "merge": (lambda: mo.paged_merge(d, ctx.rows, T), 0, T * m.nsplit * nq * V * 4.0)}
+    qf = ws.flat("qf", T * nq * m.q_ld, torch.bfloat16)
+    d.qf = qf.data_ptr()
+    return {"prep": (lambda k=keep: mo.paged_prep(d, T), 0, T * (p.shape[1] * 4.0 + m.row * 2 + nq * m.q_ld * 2)),
+            "attention": (lambda k=qf: mo.paged_prefill(d, T, b.pages, ctx.tiles, ctx.n_tiles, ctx.long), flops, 0)}
+
+
+def _experts(W: int, E: int, top: int, ff: int, T: int, sets: int):
+    """Routed experts of `sets` layers (together larger than L2): {kernel: (call over all layers, flops, bytes)} per layer."""
+    from ..models import mixer_layers as ml
+    from ..ops import mixer_ops as mo
+    ctx = ml.StepContext(T, *[None] * 5, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
+    g = torch.Generator(device="cuda").manual_seed(0)
+    r = lambda *s: (torch.randn(*s, generator=g, device="cuda") * s[-1] ** -0.5).to(torch.bfloat16)
+    layers = [ml.RoutedExperts(r(E, W), [r(ff, W) for _ in range(E)], [r(W, ff) for _ in range(E)], mo.Router(E, top), torch.bfloat16, "cuda") for _ in range(sets)]
+    h = torch.randn(T, layers[0].up.shape[2], generator=g, device="cuda").to(torch.bfloat16)
+    R, ws = T * top, ctx.ws
+    z = [m.router(ctx, h, f"router{i}", torch.float32) for i, m in enumerate(layers)]
+    used = E * (1.0 - (1.0 - top / E) ** T)                            # experts that are expected to be used
+    flops, nbytes = 2.0 * R * W * ff, used * W * ff * 2.0
+    ids, hidden = ws.flat("ids", R, torch.int32), ws.rows("hid", R, layers[0].ff, torch.bfloat16)
+    keep = (layers, z)
+    out = {"whole layer with router": (lambda k=keep: [m.forward(ctx, h) for m in layers], 2 * flops, 2 * nbytes)}
+    if T <= mo.ROWS_MAX:
+        y = ws.rows("yy", T, layers[0].down.shape[1], torch.float32)
+        out["up rows (choice included)"] = (lambda: [mo.expert_up_rows(m.route, q, h, m.up, ids, hidden) for m, q in zip(layers, z)], flops, nbytes)
+        out["down rows"] = (lambda: [mo.expert_down_rows(m.route, ids, hidden, m.down, W, y) for m in layers], flops, nbytes)
+        return out
+    place, seg, sc = ws.rows("pl", T, top, torch.int32), ws.flat("sg", E + 1, torch.int32), ws.flat("sc", R, torch.float32)
+    x, y, rw = ws.rows("rx", R, h.shape[1], torch.bfloat16), ws.rows("yy", R, layers[0].down.shape[1], torch.float32), ws.flat("rw", R, torch.float32)
+    group = lambda m, q: mo.expert_group(m.route, q, h, ids, rw, seg, place, sc, x)
+    group(layers[0], z[0])
+    out["choice, grouping, gather"] = (lambda: [group(m, q) for m, q in zip(layers, z)], 0, T * W * 2.0 + R * W * 2.0)
+    group(layers[0], z[0])
+    out["up (grouped GEMM, squared ReLU)"] = (lambda: [mo.grouped_linear(x, m.up, seg, hidden, ctx.status, relu2=True, row_scale=sc) for m in layers], flops, nbytes)
+    out["down (grouped GEMM, fp32 out)"] = (lambda: [mo.grouped_linear(hidden, m.down, seg, y, ctx.status) for m in layers], flops, nbytes)
+    return out
+
+
+def pezarax_kernels() -> None:
+    from .. import ops
+    from ..ops import mixer_ops as mo
+    from . import bench_kernels as bk
+    show = lambda name, d, **kw: print(json.dumps({"kernel": name, **kw, **d}), flush=True)
+    dims = (16, 128, 256)
+    for T in (512, 2048):
+        for kind in ("retention", "gla"):
+            f, fl, _ = _state(kind, dims, T, False)
+            show(f"{kind} chunk form + head norm", _roof(timed(f), fl), T=T, dims=dims)
+        r = bk.bench_deltanet(T, 16, 32, 20)
+        show("like kernel: chunked DeltaNet", _roof(r["us"], 2.0 * T * 32 * (3 * 128 * 128 + 2.5 * 64 * 128 + 64 * 64 * 1.0)), T=T)
+    for B in (1, 8):
+        for kind in ("retention", "gla"):
+            f, _, nb = _state(kind, dims, B, True)
+            show(f"{kind} rows form + head norm", _roof(timed(f), 0, nb), B=B, dims=dims)
+    for dims in ((32, 8, 64, 128, 0), (32, 8, 64, 128, 1024), (32, 8, 128, 128, 0)):
+        for k, (f, fl, nb) in _paged(dims, 512, 8192 - 512, False).items():
+            show("differential prefill: " + k, _roof(timed(f), fl, nb), T=512, context=8192, dims=dims)
+    show("like kernel: GQA prefill", bk.bench_attention(512, 8192, 32, 8, 20))
+    for B, chunk in ((1, 1024), (8, 1024), (1, 0), (8, 0)):
+        start = 8191
+        for k, (f, fl, nb) in _paged((32, 8, 64, 128, chunk), B, start, True).items():
+            show("differential rows: " + k, _roof(timed(f), fl, nb), B=B, context=start + 1, chunk=chunk)
+    for B in (1, 8):
+        for ctx in (1024, 8192):
+            q = torch.randn(B, 32, 128, device="cuda").to(torch.bfloat16)
+            kc, vc = (torch.randn(8, ctx, 128, device="cuda").to(torch.bfloat16) for _ in range(2))
+            pos = torch.full((B,), ctx - 1, device="cuda", dtype=torch.int32)
+            ns = max(1, min(32, ctx // 64))
+            us = timed(lambda: ops.gqa_decode(q, kc, vc, pos, nsplit=ns))
+            show("like kernel: GQA decode rows", _roof(us, 4.0 * B * 32 * 128 * ctx, B * ctx * 8 * 256 * 2.0), B=B, context=ctx, nsplit=ns)
+    W, E, top, ff = 4096, 32, 2, 3072
+    for T in (1, 8, 64, 512, 2048):
+        sets = 2
+        for k, (f, fl, nb) in _experts(W, E, top, ff, T, sets).items():
+            us = timed(f, reps=8) / sets
+            show("experts: " + k, _roof(us, fl, nb), T=T)
+    for M in (1, 2, 8):
+        for N, K in ((ff * 2, W), (W, ff * 2)):
+            ws = [torch.randn(N, K, device="cuda").to(torch.bfloat16) for _ in range(max(2, -(-(300 << 20) // (N * K * 2))))]
+            x, y, s = torch.randn(M, K, device="cuda").to(torch.bfloat16), torch.empty(M, N, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+            us = timed(lambda: [mo.linear(x, w, y, s) for w in ws], reps=8) / len(ws)
+            show("like kernel: few-row linear", _roof(us, 0, N * K * 2.0), M=M, N=N, K=K)
+    from ctypes import c_int, c_void_p
+    for T in (64, 512, 2048):
+        R = T * top
+        seg = torch.linspace(0, R, E + 1, device="cuda").to(torch.int32)
+        a = torch.randn(R, W, device="cuda").to(torch.bfloat16)
+        w = torch.randn(E * 2 * ff // 2, W, device="cuda").to(torch.bfloat16)
+        c, s = torch.empty(R, ff // 2, device="cuda", dtype=torch.bfloat16), torch.zeros(1, dtype=torch.int32, device="cuda")
+        K = ops.lib.kernels()
+        ptr = lambda t: c_void_p(t.data_ptr())
+        call = lambda: K.pk_gemm_bf16_grouped(ptr(a), c_int(W), ptr(w), ptr(seg), c_int(E), c_int(R), c_int(ff), c_int(W), c_int(1), ptr(c), c_int(ff // 2), ptr(s),
+                                              c_int(mo.sm_count()), c_void_p(torch.cuda.current_stream().cuda_stream))
+        show("like kernel: grouped GEMM, SwiGLU", _roof(timed(call), 2.0 * R * W * ff, E * W * ff * 2.0), T=T)
+    for T in (1, 2048):
+        x, y, w = torch.randn(T, 4096, device="cuda"), torch.randn(2 * T, 4096, device="cuda"), torch.randn(4096, device="cuda")
+        place = torch.randperm(2 * T, device="cuda").to(torch.int32).view(T, 2)
+        o = torch.empty(T, 4096, device="cuda", dtype=torch.bfloat16)
+        show("residual add + norm", _roof(timed(lambda: mo.sandwich_norm(x, y=y, w_pre=w, out=o, eps=1e-5)), 0, T * 4096 * 14.0), T=T)
+        show("sum of two expert rows + residual add + norm", _roof(timed(lambda: mo.sandwich_norm(x, y=y, y_rows=place, w_pre=w, out=o, eps=1e-5)), 0, T * 4096 * 18.0), T=T)
+        show("like kernel: two norms + residual add", _roof(timed(lambda: mo.sandwich_norm(x, y=y, w_post=w, w_pre=w, out=o, eps=1e-5)), 0, T * 4096 * 14.0), T=T)
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernels", action="store_true")
+    ap.add_argument("--kernels", nargs="?", const="gidisun", choices=["gidisun", "pezarax"], help="time the design's kernels beside the like kernels")
     ap.add_argument("--size", default="2k", choices=sorted(SIZES))
     args = ap.parse_args()
     if args.kernels:
-        kernels()
+        {"gidisun": kernels, "pezarax": pezarax_kernels}[args.kernels]()
     else:
         print(json.dumps(closest_model(args.size, 512, 64, 3)))
     return 0
