@@ -35,50 +35,73 @@ __device__ __forceinline__ float to_f(T v) { return (float)v; }
 template <>
 __device__ __forceinline__ float to_f<bf16>(bf16 v) { return __bfloat162float(v); }
 
-// Block (row, share of the row's vectors), one warp per vector: H x maps queries, G x maps keys, G values.
-template <typename CT>
-__global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a, int per_block) {
+// Block (row, share of the row's vectors), up to NPW vectors per warp, dealt out in turn: H x maps queries, G x maps keys, G
+// values. The first pair of elements that a lane owns of every vector is on its way while the angles are computed.
+template <typename CT, int NPW>
+__global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a) {
   pdl_trigger();
   extern __shared__ float sm[];      // cos, sin [R / 2] each
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, half = a.R / 2;
+  const int nq = a.H * a.maps, nk = a.G * a.maps, total = nq + nk + a.G;
+  const int v0 = blockIdx.y * 8 + warp, step = gridDim.y * 8;
   pdl_wait();
   const float* pr = a.proj + (size_t)t * a.ld;
   const int pos = a.pos[t];
+  auto source = [&](int v) { return v < nq ? pr + a.oq + v * a.D : v < nq + nk ? pr + a.ok + (v - nq) * a.D : pr + a.ov + (v - nq - nk) * a.V; };
+  // pair i of a query or key: (i, i + half) while it turns, then single elements
+  float x0[NPW], y0[NPW];
+#pragma unroll
+  for (int j = 0; j < NPW; ++j) {
+    const int v = v0 + j * step;
+    x0[j] = y0[j] = 0.f;
+    if (v < nq + nk && lane < half) {
+      const float* src = source(v);
+      x0[j] = src[lane];
+      y0[j] = src[lane + half];
+    }
+  }
   float* cs = sm;
   float* sn = sm + half;
   for (int i = tid; i < half; i += 256) rotary_sincos(a.freq[i], pos, sn[i], cs[i]);
-  __syncthreads();
-  const int nq = a.H * a.maps, nk = a.G * a.maps, total = nq + nk + a.G;
   CT* crow = reinterpret_cast<CT*>(a.cache) + cache_row(a, a.slot[t], pos);
-  const int end = min(total, (int)(blockIdx.y + 1) * per_block);
-  for (int v = blockIdx.y * per_block + warp; v < end; v += 8) {
+  __syncthreads();
+#pragma unroll
+  for (int j = 0; j < NPW; ++j) {
+    const int v = v0 + j * step;
+    if (v >= total) break;
+    const float* src = source(v);
     if (v >= nq + nk) {
-      const int g = v - nq - nk;
-      const float* src = pr + a.ov + g * a.V;
-      CT* dst = crow + nk * a.dp + g * a.vp;
-      for (int i = lane; i < a.vp; i += 32) dst[i] = (CT)(i < a.V ? src[i] : 0.f);
+      CT* dst = crow + nk * a.dp + (v - nq - nk) * a.vp;
+      for (int i0 = lane; i0 < a.vp; i0 += 128) {
+        float x[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) x[k] = i0 + k * 32 < a.V ? src[i0 + k * 32] : 0.f;
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (i0 + k * 32 < a.vp) dst[i0 + k * 32] = (CT)x[k];
+      }
       continue;
     }
     const bool is_q = v < nq;
-    const float* src = is_q ? pr + a.oq + v * a.D : pr + a.ok + (v - nq) * a.D;
-    auto at = [&](int i) {
-      if (i >= a.D) return 0.f;
-      if (i >= a.R) return src[i];
-      return i < half ? src[i] * cs[i] - src[i + half] * sn[i] : src[i] * cs[i - half] + src[i - half] * sn[i - half];
+    CT* krow = is_q ? nullptr : crow + (v - nq) * a.dp;
+    float* qx = is_q && a.qx ? a.qx + ((size_t)t * nq + v) * a.D : nullptr;
+    bf16* qf = is_q && a.qf ? (bf16*)a.qf + ((size_t)t * nq + v) * a.q_ld : nullptr;
+    auto put = [&](int i, float x) {
+      if (krow) krow[i] = (CT)x;
+      if (qx) qx[i] = x;
+      if (qf) qf[i] = __float2bfloat16(x);
     };
-    if (!is_q) {
-      CT* dst = crow + (v - nq) * a.dp;
-      for (int i = lane; i < a.dp; i += 32) dst[i] = (CT)at(i);
-    } else {
-      if (a.qx) {
-        float* dst = a.qx + ((size_t)t * nq + v) * a.D;
-        for (int i = lane; i < a.D; i += 32) dst[i] = at(i);
-      }
-      if (a.qf) {
-        bf16* dst = (bf16*)a.qf + ((size_t)t * nq + v) * a.q_ld;
-        for (int i = lane; i < a.q_ld; i += 32) dst[i] = __float2bfloat16(at(i));
-      }
+    for (int i = lane; i < half; i += 32) {
+      float x = i == lane ? x0[j] : src[i], y = i == lane ? y0[j] : src[i + half];
+      rotate_pair(x, y, sn[i], cs[i]);
+      put(i, x);
+      put(i + half, y);
     }
+    for (int i = a.R + lane; i < a.D; i += 32) put(i, src[i]);
+    if (krow)
+      for (int i = a.D + lane; i < a.dp; i += 32) krow[i] = (CT)0.f;
+    if (qf)
+      for (int i = a.D + lane; i < a.q_ld; i += 32) qf[i] = __float2bfloat16(0.f);
   }
   if (a.row > nk * a.dp + a.G * a.vp && blockIdx.y == 0)
     for (int i = nk * a.dp + a.G * a.vp + tid; i < a.row; i += 256) crow[i] = (CT)0.f;
@@ -306,12 +329,16 @@ int launch_rows(const Attn& a, const int* rows, int nrows, cudaStream_t stream) 
 PK_API int pk_paged_prep(const PkPagedAttention* a, int M, cudaStream_t stream) {
   if (!shape_ok(a) || M < 1 || a->proj == nullptr || (a->R > 0 && a->freq == nullptr) || (a->qf != nullptr && a->q_ld < a->D)) return PK_ERR_BAD_ARG;
   const int total = a->H * a->maps + a->G * a->maps + a->G;
-  const int per = M <= 64 ? 8 : 32;
-  const dim3 grid(M, (total + per - 1) / per);
   const size_t smem = (size_t)(a->R + 2) * sizeof(float);
   if (smem > 48 * 1024) return PK_ERR_UNSUPPORTED;
-  if (a->f32) PK_LAUNCH_PDL(paged_prep_kernel<float>, grid, dim3(256), smem, stream, *a, per);
-  else PK_LAUNCH_PDL(paged_prep_kernel<pk::bf16>, grid, dim3(256), smem, stream, *a, per);
+  const dim3 few(M, (total + 7) / 8), many(M, (total + 31) / 32), block(256);
+  if (M <= 64) {
+    if (a->f32) PK_LAUNCH_PDL((paged_prep_kernel<float, 1>), few, block, smem, stream, *a);
+    else PK_LAUNCH_PDL((paged_prep_kernel<pk::bf16, 1>), few, block, smem, stream, *a);
+  } else {
+    if (a->f32) PK_LAUNCH_PDL((paged_prep_kernel<float, 4>), many, block, smem, stream, *a);
+    else PK_LAUNCH_PDL((paged_prep_kernel<pk::bf16, 4>), many, block, smem, stream, *a);
+  }
   return PK_OK;
 }
 

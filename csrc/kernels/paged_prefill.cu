@@ -3,12 +3,13 @@
 //
 // One CTA works one (head, tile of up to 128 query rows of one portion, slice of up to 128 value columns) and NMAP of the
 // head's maps. A step is one page, 64 positions; its keys and values arrive by TMA (no multicast) into two alternating
-// buffers, the address of a page being its row in the pool. Per step and map:
-//   S  = Q K^T      tcgen05.mma kind::f16, both operands K-major, fp32 S in TMEM
-//   P  = exp2(S-m)  four softmax warps, one query row per thread; fp32 weights, handed to the tensor cores as the sum of two
-//                   bf16 terms (16 significant bits)
-//   PV = P V        V as an MN-major operand; S of the next step is issued right behind it
-//   O  = O alpha + PV in fp32 registers
+// buffers each, the address of a page being its row in the pool. Per step and map:
+//   S  = Q K^T       tcgen05.mma kind::f16, both operands K-major, fp32 S in TMEM (two buffers: S of the next step is
+//                    computed while the softmax warps work on this one)
+//   P  = exp2(S-m)   four softmax warps, one query row per thread; fp32 weights, handed to the tensor cores as the sum of two
+//                    bf16 terms (16 significant bits)
+//   O += P V         V as an MN-major operand, O in TMEM. The reference m of a row only moves when its maximum has grown by
+//                    more than a factor of 2^8; its warp then rescales O in TMEM (weights up to 2^8 lose nothing in fp32)
 // With NMAP = 2 the maps share the loads of V, and while one map's warps are in their exponentials the other map's products
 // run; at the end the second map's warps hand lambda x their output through shared memory to the first map's, which take the
 // difference, norm it over the head and store it. Heads too wide for that run one map per CTA and leave fp32 outputs for the
@@ -39,7 +40,7 @@ struct Params {
 };
 
 struct Ctl {
-  uint64_t q_full, kv_full[2], kv_empty[2], s_full[2], p_ready[2], pv_full[2];
+  uint64_t q_full, k_full[2], k_empty[2], v_full[2], v_empty[2], s_full[2][2], p_ready[2], pv_full[2];
   uint32_t tmem_base;
   volatile uint32_t abort_flag;
 };
@@ -53,6 +54,14 @@ __device__ __forceinline__ uint64_t desc_mn_sw128(uint32_t smem_addr, uint32_t l
   d |= (uint64_t)1 << 46;
   d |= (uint64_t)2 << 61;
   return d;
+}
+
+constexpr float kSlack = 8.f;        // log2 of how far a row's maximum may run ahead of its reference
+
+__device__ __forceinline__ float exp2_approx(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 
 template <int VP, int NMAP>    // value columns of this CTA's slice: 64 or 128; maps worked together
@@ -70,9 +79,9 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   uint8_t* sv = sk + 2 * NMAP * qp * kKPanel;           // [2][NV]
   Ctl& ct = *reinterpret_cast<Ctl*>(sv + 2 * NV * kKPanel);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int vec0 = blockIdx.y * NMAP;                   // first query vector (head x maps + map)
+  const int vec0 = blockIdx.x * NMAP;                   // first query vector (head x maps + map)
   const int h = vec0 / a.maps, map0 = vec0 - h * a.maps, g = h / (a.H / a.G), vs = blockIdx.z;
-  const int4 tile = p.tiles[blockIdx.x];
+  const int4 tile = p.tiles[gridDim.y - 1 - blockIdx.y];     // the last tiles of a portion see most: they go first
   const int4 seq = p.seqs[tile.z];
   const int pos0 = seq.w + tile.x - seq.x;              // position of the tile's first row
   int first = 0;
@@ -84,9 +93,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   if (threadIdx.x == 0) {
     mbar_init(&ct.q_full, 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&ct.kv_full[i], 1);
-      mbar_init(&ct.kv_empty[i], 1);
-      mbar_init(&ct.s_full[i], 1);
+      mbar_init(&ct.k_full[i], 1);
+      mbar_init(&ct.k_empty[i], 1);
+      mbar_init(&ct.v_full[i], 1);
+      mbar_init(&ct.v_empty[i], 1);
+      mbar_init(&ct.s_full[i][0], 1);
+      mbar_init(&ct.s_full[i][1], 1);
       mbar_init(&ct.p_ready[i], 4);
       mbar_init(&ct.pv_full[i], 1);
     }
@@ -100,7 +112,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_s = ct.tmem_base, tmem_pv = ct.tmem_base + NMAP * 64;
+  const uint32_t tmem_s = ct.tmem_base, tmem_o = ct.tmem_base + NMAP * 128;      // S [NMAP][2 buffers] of 64 columns, O [NMAP] of VP
 
   if (warp == 1) {
     // ---------------- TMA producer ----------------
@@ -115,25 +127,31 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
         tma_load_2d(sq + i * kQPanel, &tmap_q, &ct.q_full, x, tile.x);
         tma_load_2d(sq + i * kQPanel + kQPanel / 2, &tmap_q, &ct.q_full, x, tile.x + kQ / 2);
       }
-      int issued = 0;
+      int k_issued = 0, v_issued = 0;
       int page = pages[0];
       for (int t = 0; t < n_tiles; ++t) {
         const int b = t & 1, y = page * kKV;
         if (t + 1 < n_tiles) page = pages[t + 1];
-        if (t >= 2 && !mbar_wait(&ct.kv_empty[b], ((t - 2) >> 1) & 1, &ct.abort_flag, p.a.status, 71)) break;
-        mbar_arrive_expect_tx(&ct.kv_full[b], (NMAP * qp + NV) * kKPanel);
+        if (t >= 2 && !mbar_wait(&ct.k_empty[b], ((t - 2) >> 1) & 1, &ct.abort_flag, a.status, 70)) break;
+        mbar_arrive_expect_tx(&ct.k_full[b], NMAP * qp * kKPanel);
         for (int i = 0; i < NMAP * qp; ++i)
-          tma_load_2d(sk + (b * NMAP * qp + i) * kKPanel, &tmap_c, &ct.kv_full[b], kx + (i / qp) * a.dp + (i % qp) * 64, y);
+          tma_load_2d(sk + (b * NMAP * qp + i) * kKPanel, &tmap_c, &ct.k_full[b], kx + (i / qp) * a.dp + (i % qp) * 64, y);
+        k_issued = t + 1;
+        if (t >= 2 && !mbar_wait(&ct.v_empty[b], ((t - 2) >> 1) & 1, &ct.abort_flag, a.status, 71)) break;
+        mbar_arrive_expect_tx(&ct.v_full[b], NV * kKPanel);
 #pragma unroll
-        for (int i = 0; i < NV; ++i) tma_load_2d(sv + (b * NV + i) * kKPanel, &tmap_c, &ct.kv_full[b], vx + i * 64, y);
-        issued = t + 1;
+        for (int i = 0; i < NV; ++i) tma_load_2d(sv + (b * NV + i) * kKPanel, &tmap_c, &ct.v_full[b], vx + i * 64, y);
+        v_issued = t + 1;
       }
       // every copy has landed before the CTA may exit, also when another warp gave up
       for (uint32_t i = 0; i < (1u << 20); ++i)
         if (mbar_try_wait(&ct.q_full, 0)) break;
-      for (int t = max(issued - 2, 0); t < issued; ++t)
+      for (int t = max(k_issued - 2, 0); t < k_issued; ++t)
         for (uint32_t i = 0; i < (1u << 20); ++i)
-          if (mbar_try_wait(&ct.kv_full[t & 1], (t >> 1) & 1)) break;
+          if (mbar_try_wait(&ct.k_full[t & 1], (t >> 1) & 1)) break;
+      for (int t = max(v_issued - 2, 0); t < v_issued; ++t)
+        for (uint32_t i = 0; i < (1u << 20); ++i)
+          if (mbar_try_wait(&ct.v_full[t & 1], (t >> 1) & 1)) break;
     }
     __syncwarp();
   } else if (warp == 0) {
@@ -141,23 +159,34 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc(1, 1, kQ, kKV);
       constexpr uint32_t idesc_pv = umma_idesc(1, 1, kQ, VP) | (1u << 16);   // V MN-major
-      auto issue_s = [&](int t, int m) {
-        const uint32_t qa = smem_u32(sq + m * qp * kQPanel), ka = smem_u32(sk + ((t & 1) * NMAP + m) * qp * kKPanel);
-        for (int j = 0; j < p.k_steps; ++j)
-          umma_f16(tmem_s + m * 64, smem_desc_k_sw128(qa + (j >> 2) * kQPanel + (j & 3) * 32),
-                   smem_desc_k_sw128(ka + (j >> 2) * kKPanel + (j & 3) * 32), idesc_s, j > 0 ? 1u : 0u);
-        umma_commit(&ct.s_full[m]);
+      // S of step t for every map; its buffers were read two steps ago
+      auto issue_s = [&](int t) {
+        const int b = t & 1;
+        for (int m = 0; m < NMAP; ++m) {
+          const uint32_t qa = smem_u32(sq + m * qp * kQPanel), ka = smem_u32(sk + (b * NMAP + m) * qp * kKPanel);
+          for (int j = 0; j < p.k_steps; ++j)
+            umma_f16(tmem_s + m * 128 + b * 64, smem_desc_k_sw128(qa + (j >> 2) * kQPanel + (j & 3) * 32),
+                     smem_desc_k_sw128(ka + (j >> 2) * kKPanel + (j & 3) * 32), idesc_s, j > 0 ? 1u : 0u);
+          umma_commit(&ct.s_full[m][b]);
+        }
+        if (t + 2 < n_tiles) umma_commit(&ct.k_empty[b]);
       };
-      bool ok = mbar_wait(&ct.q_full, 0, &ct.abort_flag, a.status, 72) && mbar_wait(&ct.kv_full[0], 0, &ct.abort_flag, a.status, 73);
+      bool ok = mbar_wait(&ct.q_full, 0, &ct.abort_flag, a.status, 72) && mbar_wait(&ct.k_full[0], 0, &ct.abort_flag, a.status, 73);
       if (ok) {
         tc_fence_after();
-        for (int m = 0; m < NMAP; ++m) issue_s(0, m);
+        issue_s(0);
       }
       for (int t = 0; t < n_tiles && ok; ++t) {
         const int b = t & 1;
-        if (t + 1 < n_tiles && !mbar_wait(&ct.kv_full[b ^ 1], ((t + 1) >> 1) & 1, &ct.abort_flag, a.status, 74)) break;
-        for (int m = 0; m < NMAP && ok; ++m) {
-          if (!mbar_wait(&ct.p_ready[m], t & 1, &ct.abort_flag, a.status, 75)) {
+        if (t + 1 < n_tiles) {
+          // p_ready of step t - 1 was waited for: the S buffers of step t + 1 are free
+          if (!mbar_wait(&ct.k_full[b ^ 1], ((t + 1) >> 1) & 1, &ct.abort_flag, a.status, 74)) break;
+          tc_fence_after();
+          issue_s(t + 1);
+        }
+        if (!mbar_wait(&ct.v_full[b], (t >> 1) & 1, &ct.abort_flag, a.status, 75)) break;
+        for (int m = 0; m < NMAP; ++m) {
+          if (!mbar_wait(&ct.p_ready[m], t & 1, &ct.abort_flag, a.status, 76)) {
             ok = false;
             break;
           }
@@ -165,12 +194,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           const uint32_t pa = smem_u32(sp + m * 2 * kQPanel), va = smem_u32(sv + b * NV * kKPanel);
 #pragma unroll
           for (int j = 0; j < 8; ++j)   // four k-steps of the leading bf16 term, then four of the remainder
-            umma_f16(tmem_pv + m * VP, smem_desc_k_sw128(pa + (j >> 2) * kQPanel + (j & 3) * 32), desc_mn_sw128(va + (j & 3) * 2048, kKPanel, 1024),
-                     idesc_pv, j > 0 ? 1u : 0u);
+            umma_f16(tmem_o + m * VP, smem_desc_k_sw128(pa + (j >> 2) * kQPanel + (j & 3) * 32), desc_mn_sw128(va + (j & 3) * 2048, kKPanel, 1024),
+                     idesc_pv, t > 0 || j > 0 ? 1u : 0u);
           umma_commit(&ct.pv_full[m]);
-          if (m == NMAP - 1 && t + 2 < n_tiles) umma_commit(&ct.kv_empty[b]);     // behind every product that reads step t's buffers
-          if (t + 1 < n_tiles) issue_s(t + 1, m);              // S of step t was read before p_ready
         }
+        if (ok && t + 2 < n_tiles) umma_commit(&ct.v_empty[b]);
       }
     }
     __syncwarp();
@@ -183,123 +211,164 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     if (a.window > 0) lo = max(lo, q_pos - a.window + 1);
     if (a.chunk > 0) lo = max(lo, q_pos / a.chunk * a.chunk);
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
-    const uint32_t ts = tmem_s + m * 64 + lane_off, tpv = tmem_pv + m * VP + lane_off;
-    float o[VP];
-#pragma unroll
-    for (int i = 0; i < VP; ++i) o[i] = 0.f;
-    float mx = -INFINITY, sum = 0.f;
+    const uint32_t ts = tmem_s + m * 128 + lane_off, to = tmem_o + m * VP + lane_off;
+    float ref = -INFINITY, sum = 0.f;      // the row's reference (log2 units) and the sum of its weights
     bool ok = true;
     uint8_t* prow = sp + m * 2 * kQPanel + r * 128;
     for (int t = 0; t < n_tiles; ++t) {
-      if (!mbar_wait(&ct.s_full[m], t & 1, &ct.abort_flag, a.status, 76)) {
+      if (!mbar_wait_warp(&ct.s_full[m][t & 1], (t >> 1) & 1, &ct.abort_flag, a.status, 77)) {
         ok = false;
         break;
       }
       tc_fence_after();
-      const int kv0 = first + t * kKV;
+      uint32_t s[2][32];
+      tmem_ld_32x32(ts + (t & 1) * 64, s[0]);
+      tmem_ld_32x32(ts + (t & 1) * 64 + 32, s[1]);
+      tmem_ld_wait();
       // visible columns of this row in this step: [c_lo, c_hi]
-      const int c_lo = lo - kv0, c_hi = q_pos - kv0;
-      float tmax = -INFINITY;
-#pragma unroll 1
-      for (int c = 0; c < 2; ++c) {
-        uint32_t s[32];
-        tmem_ld_32x32(ts + c * 32, s);
-        tmem_ld_wait();
+      const int c_lo = lo - (first + t * kKV), c_hi = q_pos - (first + t * kKV);
+      if (__any_sync(0xffffffffu, c_lo > 0 || c_hi < kKV - 1)) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-          if (c * 32 + i >= c_lo && c * 32 + i <= c_hi) tmax = fmaxf(tmax, __uint_as_float(s[i]));
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < c_lo || c * 32 + i > c_hi) s[c][i] = 0xff800000u;
       }
-      const float m_new = fmaxf(mx, tmax * p.scale_log2);
-      const float alpha = mx == -INFINITY ? 0.f : exp2f(mx - m_new);
-      const float mb = m_new == -INFINITY ? 0.f : m_new;
-      float tsum = 0.f;
+      float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int i = 0; i < 32; ++i) t4[i & 3] = fmaxf(t4[i & 3], __uint_as_float(s[c][i]));
+      const float top = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])) * p.scale_log2;
+      bool waited = t == 0;
+      if (ref == -INFINITY) ref = top;      // nothing was visible so far: sum and O are zero
+      const bool grow = top > ref + kSlack;
+      if (__any_sync(0xffffffffu, grow)) {
+        if (t > 0) {
+          if (!mbar_wait_warp(&ct.pv_full[m], (t - 1) & 1, &ct.abort_flag, a.status, 78)) {
+            ok = false;
+            break;
+          }
+          waited = true;
+          tc_fence_after();
+          const float alpha = grow ? exp2_approx(ref - top) : 1.f;
 #pragma unroll 1
-      for (int c = 0; c < 2; ++c) {
-        uint32_t s[32];
-        tmem_ld_32x32(ts + c * 32, s);
-        tmem_ld_wait();
+          for (int c = 0; c < VP / 32; ++c) {
+            uint32_t x[32];
+            tmem_ld_32x32(to + c * 32, x);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) x[i] = __float_as_uint(__uint_as_float(x[i]) * alpha);
+            tmem_st_32x32(to + c * 32, x);
+          }
+          tmem_st_wait();
+          sum *= alpha;
+        }
+        if (grow) ref = top;
+      }
+      const float mb = ref == -INFINITY ? 0.f : ref;
+      float u4[4] = {0.f, 0.f, 0.f, 0.f};
+      // weights as pairs: s[c][2e] <- leading terms, s[c][2e + 1] <- remainders
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
+#pragma unroll
+        for (int e = 0; e < 16; ++e) {
+          const float x = exp2_approx(fmaf(__uint_as_float(s[c][2 * e]), p.scale_log2, -mb));
+          const float y = exp2_approx(fmaf(__uint_as_float(s[c][2 * e + 1]), p.scale_log2, -mb));
+          u4[e & 3] += x + y;
+          const __nv_bfloat162 ph = __floats2bfloat162_rn(x, y);
+          const uint32_t hb = *reinterpret_cast<const uint32_t*>(&ph);
+          const __nv_bfloat162 pl = __floats2bfloat162_rn(x - __uint_as_float(hb << 16), y - __uint_as_float(hb & 0xffff0000u));
+          s[c][2 * e] = hb;
+          s[c][2 * e + 1] = *reinterpret_cast<const uint32_t*>(&pl);
+        }
+      sum += (u4[0] + u4[1]) + (u4[2] + u4[3]);
+      // the P buffers are free once the product of the step before is done
+      if (!waited && !mbar_wait_warp(&ct.pv_full[m], (t - 1) & 1, &ct.abort_flag, a.status, 79)) {
+        ok = false;
+        break;
+      }
+#pragma unroll
+      for (int c = 0; c < 2; ++c)
 #pragma unroll
         for (int gr = 0; gr < 4; ++gr) {
-          uint32_t hi[4], lw[4];
-#pragma unroll
-          for (int e = 0; e < 4; ++e) {
-            const int i = gr * 8 + e * 2, ci = c * 32 + i;
-            const float x = ci >= c_lo && ci <= c_hi ? exp2f(__uint_as_float(s[i]) * p.scale_log2 - mb) : 0.f;
-            const float y = ci + 1 >= c_lo && ci + 1 <= c_hi ? exp2f(__uint_as_float(s[i + 1]) * p.scale_log2 - mb) : 0.f;
-            tsum += x + y;
-            const __nv_bfloat162 ph = __floats2bfloat162_rn(x, y);
-            const __nv_bfloat162 pl = __floats2bfloat162_rn(x - __bfloat162float(ph.x), y - __bfloat162float(ph.y));
-            hi[e] = *reinterpret_cast<const uint32_t*>(&ph);
-            lw[e] = *reinterpret_cast<const uint32_t*>(&pl);
-          }
-          const int piece = (c * 4 + gr) ^ (r & 7);
-          *reinterpret_cast<uint4*>(prow + piece * 16) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-          *reinterpret_cast<uint4*>(prow + kQPanel + piece * 16) = make_uint4(lw[0], lw[1], lw[2], lw[3]);
+          const int piece = (c * 4 + gr) ^ (r & 7), e = gr * 8;
+          *reinterpret_cast<uint4*>(prow + piece * 16) = make_uint4(s[c][e], s[c][e + 2], s[c][e + 4], s[c][e + 6]);
+          *reinterpret_cast<uint4*>(prow + kQPanel + piece * 16) = make_uint4(s[c][e + 1], s[c][e + 3], s[c][e + 5], s[c][e + 7]);
         }
-      }
-      sum = sum * alpha + tsum;
-      mx = m_new;
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&ct.p_ready[m]);
-      if (!mbar_wait(&ct.pv_full[m], t & 1, &ct.abort_flag, a.status, 77)) {
-        ok = false;
-        break;
-      }
-      tc_fence_after();
-#pragma unroll
-      for (int c = 0; c < VP / 16; ++c) {
-        uint32_t pv[16];
-        tmem_ld_32x16(tpv + c * 16, pv);
-        tmem_ld_wait();
-#pragma unroll
-        for (int i = 0; i < 16; ++i) o[c * 16 + i] = fmaf(o[c * 16 + i], alpha, __uint_as_float(pv[i]));
-      }
-      tc_fence_before();
     }
+    if (ok && !mbar_wait_warp(&ct.pv_full[m], (n_tiles - 1) & 1, &ct.abort_flag, a.status, 69)) ok = false;
+    tc_fence_after();
     float inv = sum > 0.f ? 1.f / sum : 0.f;
     const bool row_ok = ok && r < tile.y;
     const int nv = min(VP, a.V - vs * 128);
+    float* xch = reinterpret_cast<float*>(sp);          // [VP][128 rows]
     if (NMAP == 2) {
-      // every product of this CTA is done (both groups waited for their last one): the P buffers are free
-      float* xch = reinterpret_cast<float*>(sp);          // [VP][128 rows]
+      // every product of this CTA is done once both groups have waited for their last one: the P buffers are free
       asm volatile("bar.sync 1, 256;" ::: "memory");
       if (m == 1) {
         inv *= a.lambda;
+#pragma unroll 1
+        for (int c = 0; c < VP / 32; ++c) {
+          uint32_t x[32];
+          tmem_ld_32x32(to + c * 32, x);
+          tmem_ld_wait();
 #pragma unroll
-        for (int i = 0; i < VP; ++i) xch[i * kQ + r] = o[i] * inv;
+          for (int i = 0; i < 32; ++i) xch[(c * 32 + i) * kQ + r] = __uint_as_float(x[i]) * inv;
+        }
       }
       asm volatile("bar.sync 1, 256;" ::: "memory");
-      if (m == 0) {
-#pragma unroll
-        for (int i = 0; i < VP; ++i) o[i] = fmaf(o[i], inv, -xch[i * kQ + r]);
-        inv = 1.f;
-      }
     }
-    if (m == 0 && row_ok) {
-      if (p.raw) {
-        float* dst = a.part_o + ((size_t)(tile.x + r) * a.H * a.maps + vec0) * a.V + vs * 128;
+    if (m == 0) {
+      // columns c * 32 .. of this row's output (all lanes of the warp take part)
+      auto output = [&](int c, float (&o)[32]) {
+        uint32_t x[32];
+        tmem_ld_32x32(to + c * 32, x);
+        tmem_ld_wait();
 #pragma unroll
-        for (int v = 0; v < VP; ++v)
-          if (v < nv) dst[v] = o[v] * inv;
-      } else {
-        if (a.head_norm) {
-          float ss = 0.f;
-#pragma unroll
-          for (int v = 0; v < VP; ++v)
-            if (v < nv) ss = fmaf(o[v] * inv, o[v] * inv, ss);
-          inv *= a.post / sqrtf(ss / (float)a.V + a.eps);
+        for (int i = 0; i < 32; ++i) {
+          o[i] = __uint_as_float(x[i]) * inv;
+          if (NMAP == 2) o[i] -= xch[(c * 32 + i) * kQ + r];
         }
-        bf16* dst = (bf16*)a.out + (size_t)(tile.x + r) * a.ldo + h * a.V + vs * 128;
+      };
+      float f = 1.f;
+      if (a.head_norm && !p.raw) {
+        float ss = 0.f;
+#pragma unroll 1
+        for (int c = 0; c < VP / 32; ++c) {
+          float o[32];
+          output(c, o);
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < nv) ss = fmaf(o[i], o[i], ss);
+        }
+        f = a.post / sqrtf(ss / (float)a.V + a.eps);
+      }
+#pragma unroll 1
+      for (int c = 0; c < VP / 32; ++c) {
+        float o[32];
+        output(c, o);
+        if (!row_ok) continue;
+        if (p.raw) {
+          float* dst = a.part_o + ((size_t)(tile.x + r) * a.H * a.maps + vec0) * a.V + vs * 128 + c * 32;
+#pragma unroll
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < nv) dst[i] = o[i];
+          continue;
+        }
+        bf16* dst = (bf16*)a.out + (size_t)(tile.x + r) * a.ldo + h * a.V + vs * 128 + c * 32;
         if ((a.V & 7) == 0) {
 #pragma unroll
-          for (int v = 0; v < VP / 8; ++v) {
-            if (v * 8 < nv) {
+          for (int v = 0; v < 4; ++v) {
+            if (c * 32 + v * 8 < nv) {
               uint32_t w[4];
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
-                const __nv_bfloat162 pr = __floats2bfloat162_rn(o[v * 8 + e * 2] * inv, o[v * 8 + e * 2 + 1] * inv);
+                const __nv_bfloat162 pr = __floats2bfloat162_rn(o[v * 8 + e * 2] * f, o[v * 8 + e * 2 + 1] * f);
                 w[e] = *reinterpret_cast<const uint32_t*>(&pr);
               }
               *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -307,12 +376,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           }
         } else {
 #pragma unroll
-          for (int v = 0; v < VP; ++v)
-            if (v < nv) dst[v] = __float2bfloat16(o[v] * inv);
+          for (int i = 0; i < 32; ++i)
+            if (c * 32 + i < nv) dst[i] = __float2bfloat16(o[i] * f);
         }
-        if (h == a.H - 1 && vs == 0)
-          for (int i = a.H * a.V; i < a.ldo; ++i) ((bf16*)a.out)[(size_t)(tile.x + r) * a.ldo + i] = __float2bfloat16(0.f);
       }
+      if (row_ok && !p.raw && h == a.H - 1 && vs == 0)
+        for (int i = a.H * a.V; i < a.ldo; ++i) ((bf16*)a.out)[(size_t)(tile.x + r) * a.ldo + i] = __float2bfloat16(0.f);
     }
   }
 
@@ -381,9 +450,10 @@ PK_API int pk_paged_prefill_form(int maps, int D, int V) {
 // Long portions (bf16): qf [rows, H x maps, q_ld] with q_ld a multiple of 64, cache of `pages` pages; tiles [ntiles] and seqs as in
 // Params.
 PK_API int pk_paged_prefill(const PkPagedAttention* a, int rows, int pages, const void* tiles, int ntiles, const void* seqs, cudaStream_t stream) {
-  if (a == nullptr || a->f32 || rows < 1 || pages < 1 || ntiles < 1 || tiles == nullptr || seqs == nullptr || a->qf == nullptr || a->cache == nullptr)
+  if (a == nullptr || a->f32 || rows < 1 || pages < 1 || ntiles < 1 || ntiles > 65535 || tiles == nullptr || seqs == nullptr || a->qf == nullptr || a->cache == nullptr)
     return PK_ERR_BAD_ARG;
   if (a->H < 1 || a->G < 1 || a->H % a->G != 0 || (a->maps != 1 && a->maps != 2) || a->D < 1 || a->V < 1 || a->V > 512 || a->V > a->vp) return PK_ERR_BAD_ARG;
+  if (!(a->scale > 0.f)) return PK_ERR_UNSUPPORTED;      // masked scores are -inf before the scale
   if ((a->dp & 7) != 0 || a->dp < a->D || (a->vp & 7) != 0 || (a->row & 7) != 0 || a->row < a->G * (a->maps * a->dp + a->vp) || (a->q_ld & 63) != 0 ||
       a->q_ld < a->D)
     return PK_ERR_BAD_ARG;
@@ -399,7 +469,7 @@ PK_API int pk_paged_prefill(const PkPagedAttention* a, int rows, int pages, cons
   Params p{*a, (const int4*)tiles, (const int4*)seqs, (a->D + 63) / 64, (a->D + 15) / 16, a->scale * 1.4426950408889634f, form == 0 ? 1 : 0};
   const int slices = (a->V + 127) / 128;
   const bool narrow = a->V <= 64;
-  if (form == 1 && a->maps == 2) return narrow ? launch<64, 2>(tq, tc, p, dim3(ntiles, a->H, 1), stream) : launch<128, 2>(tq, tc, p, dim3(ntiles, a->H, 1), stream);
-  const dim3 grid(ntiles, a->H * a->maps, slices);
+  if (form == 1 && a->maps == 2) return narrow ? launch<64, 2>(tq, tc, p, dim3(a->H, ntiles, 1), stream) : launch<128, 2>(tq, tc, p, dim3(a->H, ntiles, 1), stream);
+  const dim3 grid(a->H * a->maps, ntiles, slices);
   return narrow ? launch<64, 1>(tq, tc, p, grid, stream) : launch<128, 1>(tq, tc, p, grid, stream);
 }

@@ -22,9 +22,9 @@ struct Router {
   float scale;
 };
 
-// One warp. Lane j < top gets the j-th best expert and its weight (ties: the lower index first).
+// One warp, up to 32 PER experts. Lane j < top gets the j-th best expert and its weight (ties: the lower index first).
+template <int PER>
 __device__ __forceinline__ void select_experts(const Router& r, int token, int lane, int& expert, float& weight) {
-  constexpr int PER = kMaxExperts / 32;
   const float* z = r.z + (size_t)token * r.ldz;
   float v[PER];
 #pragma unroll
@@ -103,7 +103,8 @@ struct Vec<float> {
   }
 };
 
-// acc0 / acc1 += two weight rows . x over this warp's slice of K; U 16-byte pieces of each row in flight.
+// acc0 / acc1 += two weight rows . x over this warp's slice of K; U 16-byte pieces of each row in flight (few registers and
+// many warps stream faster than the reverse).
 template <typename T, int U>
 __device__ __forceinline__ void dot_rows(const T* w0, const T* w1, const T* x, int K, int slice, int slices, int lane, float& acc0, float& acc1) {
   constexpr int VN = Vec<T>::N;
@@ -171,7 +172,7 @@ struct RowsParams {
   int ldy;
 };
 
-template <typename T>
+template <typename T, int PER>
 __global__ void __launch_bounds__(32 * WARPS) expert_up_rows_kernel(const RowsParams p) {
   __shared__ float part[WARPS][2];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -180,7 +181,7 @@ __global__ void __launch_bounds__(32 * WARPS) expert_up_rows_kernel(const RowsPa
   const int route = blockIdx.x, t = route / p.r.top, j = route - t * p.r.top;
   int e;
   float s;
-  select_experts(p.r, t, lane, e, s);
+  select_experts<PER>(p.r, t, lane, e, s);
   e = __shfl_sync(0xffffffffu, e, j);
   s = __shfl_sync(0xffffffffu, s, j);
   if (blockIdx.y == 0 && threadIdx.x == 0) p.ids[route] = e;
@@ -190,7 +191,7 @@ __global__ void __launch_bounds__(32 * WARPS) expert_up_rows_kernel(const RowsPa
   float a0 = 0.f, a1 = 0.f;
   if (live) {
     const T* w = (const T*)p.w + (size_t)e * p.w_rows * p.K;
-    dot_rows<T, 4>(w + (size_t)n0 * p.K, w + (size_t)n1 * p.K, (const T*)p.x + (size_t)t * p.ldx, p.K, slice, p.slices, lane, a0, a1);
+    dot_rows<T, 2>(w + (size_t)n0 * p.K, w + (size_t)n1 * p.K, (const T*)p.x + (size_t)t * p.ldx, p.K, slice, p.slices, lane, a0, a1);
   }
   join_slices(part, warp, lane, slice, p.slices, a0, a1);
   if (live && slice == 0 && lane == 0) {
@@ -218,7 +219,7 @@ __global__ void __launch_bounds__(32 * WARPS) expert_down_rows_kernel(const Rows
     for (int j = 0; j < p.r.top; ++j) {
       const int route = t * p.r.top + j;
       const T* w = (const T*)p.w + (size_t)p.ids[route] * p.w_rows * p.K;
-      dot_rows<T, 4>(w + (size_t)n0 * p.K, w + (size_t)n1 * p.K, (const T*)p.x + (size_t)route * p.ldx, p.K, slice, p.slices, lane, a0, a1);
+      dot_rows<T, 2>(w + (size_t)n0 * p.K, w + (size_t)n1 * p.K, (const T*)p.x + (size_t)route * p.ldx, p.K, slice, p.slices, lane, a0, a1);
     }
   join_slices(part, warp, lane, slice, p.slices, a0, a1);
   if (live && slice == 0 && lane == 0) {
@@ -236,7 +237,7 @@ __global__ void __launch_bounds__(128) select_kernel(const Router r, int T, int*
   if (t >= T) return;
   int e;
   float w;
-  select_experts(r, t, lane, e, w);
+  select_experts<kMaxExperts / 32>(r, t, lane, e, w);
   if (lane < r.top) {
     ids[(size_t)t * r.top + lane] = e;
     weights[(size_t)t * r.top + lane] = w;
@@ -295,7 +296,7 @@ bool router_ok(const Router& r) {
 }
 
 int pick_slices(long long pairs, int K, int vec, int sm_count) {
-  const long long want = (long long)(sm_count > 0 ? sm_count : 148) * 16;
+  const long long want = (long long)(sm_count > 0 ? sm_count : 148) * 32;
   int s = 1;
   while (s < WARPS && pairs * s < want && K >= 64 * vec * s * 2) s *= 2;
   return s;
@@ -317,8 +318,10 @@ PK_API int pk_expert_up_rows(const float* logits, int ldz, int E, int top, int s
   p.slices = pick_slices((long long)pairs * T * top, K, f32 ? 4 : 8, sm_count);
   const dim3 grid(T * top, (pairs + WARPS / p.slices - 1) / (WARPS / p.slices));
   if (grid.y > 65535) return PK_ERR_UNSUPPORTED;
-  if (f32) PK_LAUNCH_PDL(expert_up_rows_kernel<float>, grid, dim3(32 * WARPS), (size_t)0, stream, p);
-  else PK_LAUNCH_PDL(expert_up_rows_kernel<pk::bf16>, grid, dim3(32 * WARPS), (size_t)0, stream, p);
+  const dim3 block(32 * WARPS);
+  if (f32) PK_LAUNCH_PDL((expert_up_rows_kernel<float, kMaxExperts / 32>), grid, block, (size_t)0, stream, p);
+  else if (E <= 64) PK_LAUNCH_PDL((expert_up_rows_kernel<pk::bf16, 2>), grid, block, (size_t)0, stream, p);
+  else PK_LAUNCH_PDL((expert_up_rows_kernel<pk::bf16, kMaxExperts / 32>), grid, block, (size_t)0, stream, p);
   return PK_OK;
 }
 

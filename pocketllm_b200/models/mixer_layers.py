@@ -310,6 +310,7 @@ class GroupedAttentionMixer:
         dp, vp = pad_to(D, 8), pad_to(V, 8)
         self.row = G * (maps * dp + vp)
         self.q_ld = pad_to(D, 64)
+        self.tensor_core = dtype == torch.bfloat16 and float(m["scale"]) > 0
         self.cache = torch.zeros(pages, mo.PAGE, self.row, dtype=dtype, device=device)
         rot = m.get("rot") or {"dims": 0, "base": 1.0}
         self.freq = rotary_frequencies(rot["dims"], rot["base"])[0].to(device)
@@ -340,7 +341,7 @@ class GroupedAttentionMixer:
         p = self.proj(ctx, h, "proj", torch.float32)
         mix = ws.rows("mix", T, self.out.K, self.dtype)
         d = self.describe(ctx, p, mix)
-        form = mo.paged_prefill_form(self.maps, self.D, self.V) if ctx.n_long and self.dtype == torch.bfloat16 else -1
+        form = mo.paged_prefill_form(self.maps, self.D, self.V) if ctx.n_long and self.tensor_core else -1
         rows, nrows = (ctx.rows, ctx.n_rows) if form >= 0 or not ctx.n_long else (ctx.all_rows, T)
         if nrows:
             d.qx = ws.flat("qx", T * nq * self.D, torch.float32).data_ptr()

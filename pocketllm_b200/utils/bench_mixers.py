@@ -340,7 +340,7 @@ def kernels() -> None:
 
 def _paged(dims, T: int, start: int, singles: bool):
     """The attention of one differential layer after its input projection, without the output projection; returns
-    {kernel: (call, flops, bytes)}."""
+    {kernel: (call, flops, bytes)}. The descriptor holds bare addresses: every call keeps the tensors behind them alive."""
     from ..models import mixer_layers as ml
     from ..ops import mixer_ops as mo
     H, G, D, V, chunk = dims
@@ -365,12 +365,12 @@ def _paged(dims, T: int, start: int, singles: bool):
         po, pm = ws.flat("po", T * m.nsplit * nq * V, torch.float32), ws.flat("pm", T * m.nsplit * nq * 2, torch.float32)
         qx = ws.flat("qx", T * nq * D, torch.float32)
         d.qx, d.part_o, d.part_ml = qx.data_ptr(), po.data_ptr(), pm.data_ptr()
-        return {"prep": (lambda k=keep: mo.paged_prep(d, T), 0, 0), "rows": (lambda k=(po, pm, qx): mo.paged_rows(d, ctx.rows, T), flops, span * m.row * 2.0),
-                "merge": (lambda: mo.paged_merge(d, ctx.rows, T), 0, T * m.nsplit * nq * V * 4.0)}
+        return {"prep": (lambda k=keep: mo.paged_prep(d, T), 0, 0), "rows": (lambda k=(keep, po, pm, qx): mo.paged_rows(d, ctx.rows, T), flops, span * m.row * 2.0),
+                "merge": (lambda k=(keep, po, pm): mo.paged_merge(d, ctx.rows, T), 0, T * m.nsplit * nq * V * 4.0)}
     qf = ws.flat("qf", T * nq * m.q_ld, torch.bfloat16)
     d.qf = qf.data_ptr()
     return {"prep": (lambda k=keep: mo.paged_prep(d, T), 0, T * (p.shape[1] * 4.0 + m.row * 2 + nq * m.q_ld * 2)),
-            "attention": (lambda k=qf: mo.paged_prefill(d, T, b.pages, ctx.tiles, ctx.n_tiles, ctx.long), flops, 0)}
+            "attention": (lambda k=(keep, qf): mo.paged_prefill(d, T, b.pages, ctx.tiles, ctx.n_tiles, ctx.long), flops, 0)}
 
 
 def _experts(W: int, E: int, top: int, ff: int, T: int, sets: int):
@@ -425,6 +425,8 @@ def pezarax_kernels() -> None:
         for k, (f, fl, nb) in _paged(dims, 512, 8192 - 512, False).items():
             show("differential prefill: " + k, _roof(timed(f), fl, nb), T=512, context=8192, dims=dims)
     show("like kernel: GQA prefill", bk.bench_attention(512, 8192, 32, 8, 20))
+    f, fl, nb = _latent((32, 128, 64, 128, 512, 1024), 512, 8192 - 512, False)["prep"]
+    show("like kernel: latent prep", _roof(timed(f), fl, nb), T=512)
     for B, chunk in ((1, 1024), (8, 1024), (1, 0), (8, 0)):
         start = 8191
         for k, (f, fl, nb) in _paged((32, 8, 64, 128, chunk), B, start, True).items():

@@ -160,6 +160,8 @@ ALONE = {
     "attention_values": config([attention(heads=2, kv=2, dim=60, rot=20, vdim=150, chunk=70)]),            # several value slices
     "attention_keys": config([attention(heads=2, kv=1, dim=150, rot=16, vdim=20, chunk=33, scale=0.08)]),  # one map per block
     "attention_wide_keys": config([attention(heads=2, kv=1, dim=260, rot=16, vdim=20, chunk=33, scale=0.06)]),   # beyond the tensor-core form
+    "attention_negative_scale": config([attention(scale=-0.2)]),
+    "attention_steep": config([attention(chunk=None, scale=4.0)]),                                         # maxima that grow along the row
     "attention_no_rot": config([attention(rot=0, diff=0.0)]),
     "experts": config([retention(mlp=moe(experts=6, top=3, ff=130))], width=65),
     "experts_one": config([retention(mlp=moe(experts=1, top=1, ff=20))]),
