@@ -17,6 +17,10 @@ struct PkPagedAttention {
   float* part_ml;         // [listed rows, nsplit, H x maps, 2] (null for the merge: part_o holds finished outputs, nsplit = 1)
   void* out;              // [rows, ldo], head h at h * V
   uint32_t* status;
+  const float* q_norm;    // [D] weight of the norm of every query before the rotation (null: none), k_norm: of every key
+  const float* k_norm;
+  const float* sink;      // [H x maps] score of a key without a value that every query sees (null: none)
+  float* v_first;         // [rows, G x V] values of another layer's same tokens (v_mix)
   int ld, oq, ok, ov;
   int H, G, maps, D, V, R;
   int dp, vp, row;        // widths in the cache (multiples of 8) and elements per cached position
@@ -24,6 +28,11 @@ struct PkPagedAttention {
   int window, chunk;      // visible positions of query i: all up to i; i - window < j (window > 0); i / chunk == j / chunk (chunk > 0)
   int q_ld, ldo, nsplit;
   int head_norm;          // outputs of a head are divided by their root mean square
+  int neighbours;         // rotated pairs are (2i, 2i + 1) instead of (i, i + R / 2)
+  int v_mix;              // 1: values are kept in v_first; 2: v <- (1 - mix) v + mix v_first
+  int gate;               // column of proj with one gate per head, sigmoid(gate) multiplies the head's output (-1: none)
+  int width;              // columns of out that belong to this layer: those behind H x V are set to zero
   float scale, lambda;    // maps == 2: output = first map - lambda x second map
-  float post, eps;        // factor behind the head norm; eps of it
+  float post, eps;        // factor on the outputs (behind the head norm); eps of the norms
+  float cap, mix;         // cap > 0: scores become cap tanh(score / cap)
 };

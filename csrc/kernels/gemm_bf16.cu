@@ -54,7 +54,8 @@ struct Params {
   // computed and not stored)
   const int* seg;
   int n_groups;
-  // EPI_RELU2: bf16 max(acc * s, 0)^2, or max(acc, 0)^2 * s (scale_after), s = row_scale[row] (null: 1)
+  // s = row_scale[row] (null: 1). EPI_RELU2: bf16 max(acc * s, 0)^2, or max(acc, 0)^2 * s (scale_after). EPI_SWIGLU:
+  // silu(gate * s) * up * s, or silu(gate) * up * s (scale_after)
   const float* row_scale;
   int scale_after;
 };
@@ -351,6 +352,14 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_consta
             add_parts(128 + c0, u);
           }
           if (!row_ok) continue;
+          if (p.row_scale) {
+            const float s = __ldg(p.row_scale + m);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+              u[i] = __float_as_uint(__uint_as_float(u[i]) * s);
+              if (!p.scale_after) g[i] = __float_as_uint(__uint_as_float(g[i]) * s);
+            }
+          }
           const int j0 = tn * 128 + c0;
           bf16* dst = p.C + (size_t)m * p.ldc + j0;
           if (j0 + 32 <= half_n) {
@@ -532,7 +541,7 @@ bool encode_bf16_2d(EncodeTiledFn encode, CUtensorMap* map, const void* base, ui
 // 1 (SwiGLU: every group's matrix holds N / 2 gate rows then N / 2 up rows) and 3 (fp32). One persistent launch walks
 // every (group, row tile, column block) that has rows; the tile list is derived from seg on the device, so the host
 // never reads the routing.
-// Epilogue 5: squared ReLU with a factor per row, before (scale_after = 0) or after the activation.
+// Epilogue 5: squared ReLU. Epilogues 1 and 5 take a factor per row, before (scale_after = 0) or after the activation.
 PK_API int pk_gemm_bf16_grouped_scaled(const void* A, int lda, const void* W, const int* seg, int n_groups, int R, int N, int K, int epi, void* C,
                                        int ldc, const float* row_scale, int scale_after, uint32_t* status, int sm_count, cudaStream_t stream) {
   if (R < 1 || N < 1 || K < BK || (K % BK) != 0 || seg == nullptr || n_groups < 1 || n_groups > kMaxGroups) return PK_ERR_BAD_ARG;

@@ -1,8 +1,12 @@
 // Recurrent mixers with an outer-product state: gated linear attention (a decay per key channel), the matrix memory of
-// xLSTM (scalar gates with a running maximum) and retention (a constant decay per head, rotated queries and keys). All are
+// xLSTM (scalar gates with a running maximum), retention (a constant decay per head, rotated queries and keys) and the
+// state-space recurrence of Mamba-2 (a scalar decay per token and head). All are
 //   S_t = diag(a_t) S_{t-1} + b_t k_t v_t^T,    o_t = S_t^T q_t          S: [key dim, value dim], fp32
 // with a_t a vector (GLA: a = sigmoid(z)^(1/tau), b = 1) or a scalar (mLSTM: a = exp(f + m_{t-1} - m_t), b = exp(i - m_t),
-// m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1; retention: a = const, b = 1).
+// m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1; retention: a = const, b = 1;
+// state space: k = B, q = C, v = x, a = exp(A dt), b = dt, dt = softplus(z + bias), B and C shared by a group of heads, and
+// o_t gets D x_t). The state-space inputs x, B and C pass a short causal convolution per channel and SiLU first; its last
+// inputs are part of a request's state, [slot][taps - 1][channel].
 // Everything here is fp32: gates, decays, states and products.
 //
 // State lives in slots [slot][head][key][value] so that requests of one batch keep theirs anywhere; a portion that starts
@@ -17,16 +21,17 @@
 //       out     per (chunk, head, tile): q~ S_c + P V
 //     GLA's exponents are never split into exp(G_i) exp(-G_j) across a reference further away than the 16-token
 //     sub-chunk between them: every factor is at most 1, whatever the decay. Retention takes the powers of its decays
-//     from a table.
+//     from a table. The state space needs q k^T only once per group and takes its factors exp(G_i - G_j) dt_j, dt_j
+//     exp(G_C - G_j) and exp(G_i) on the way into the products, where G is held as the sum of two floats.
 // A last kernel normalises every head's output (after mLSTM's division by max(|n.q|, exp(-m)) + 1e-6), applies the output
-// gate and writes the projection's input.
+// gate and writes the projection's input (state space: the gate comes first, the norm's parts need not be heads).
 #include "../common/pk_rotary.cuh"
 
 namespace {
 
 using namespace pk;
 
-enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_RETENTION = 2 };
+enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_RETENTION = 2, KIND_SSD = 3 };
 constexpr int CH = 64;    // chunk
 constexpr int SB = 16;    // sub-chunk
 
@@ -53,6 +58,15 @@ struct Mixer {
   const double* freq;  // [rot / 2] angular frequencies of the rotated leading part of queries and keys
   int rot;
   const float* pw;     // [H, 65] powers 0 .. 64 of every head's decay
+  // state space: x (H x V) | B (groups x D) | C (groups x D) are columns ov .. of proj, dt columns odt .., the gate columns og ..
+  const float* cw;     // [channels, taps] convolution, the last tap is the current token's
+  const float* cb;     // [channels]
+  const float* dtb;    // [H]
+  const float* A;      // [H] negative
+  const float* skip;   // [H]
+  float* Cs;           // [slots, taps - 1, channels] last inputs of the convolution
+  int groups, taps, odt;
+  __device__ __host__ int channels() const { return H * V + 2 * groups * D; }
   // state
   float* S;            // [slots, H, D, V]
   float* N;            // [slots, H, D]      (mLSTM)
@@ -65,6 +79,20 @@ struct Raw {
   float* nq;   // [rows, H]   n . q       (mLSTM)
   float* m;    // [rows, H]   running max (mLSTM)
 };
+
+// State space: input of the convolution `lag` tokens before the one at `row`, which is token `t` of its portion, at position pos.
+__device__ __forceinline__ float conv_input(const Mixer& mx, int slot, int row, int t, int pos, int lag, int ch) {
+  if (lag <= t) return mx.proj[(size_t)(row - lag) * mx.ld + mx.ov + ch];
+  if (lag > pos) return 0.f;
+  return mx.Cs[((size_t)slot * (mx.taps - 1) + mx.taps - 1 - (lag - t)) * mx.channels() + ch];
+}
+__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float conv_silu(const Mixer& mx, int slot, int row, int t, int pos, int ch) {
+  float y = mx.cb[ch];
+  for (int j = 0; j < mx.taps; ++j) y = fmaf(mx.cw[(size_t)ch * mx.taps + j], conv_input(mx, slot, row, t, pos, mx.taps - 1 - j, ch), y);
+  return silu_exact(y);
+}
+__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // ---------------------------------------------------------------------------------------
 // rows form
@@ -120,6 +148,18 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
           ks[i + half] = k[i + half];
         }
       }
+    } else if (KIND == KIND_SSD) {
+      const int b0 = mx.H * V + h / (mx.H / mx.groups) * D;
+      for (int i = threadIdx.x; i < 2 * D; i += 32 * GR) {
+        const bool is_q = i >= D;
+        const int d = is_q ? i - D : i;
+        (is_q ? qs : ks)[d] = conv_silu(mx, sq.z, sq.x + t, t, sq.w + t, b0 + (is_q ? mx.groups * D : 0) + d);
+      }
+      if (threadIdx.x == 0) {
+        const float dt = softplus(pr[mx.odt + h] + mx.dtb[h]);
+        s_sc[0] = expf(mx.A[h] * dt);
+        s_sc[1] = dt;
+      }
     } else {
       for (int d = threadIdx.x; d < D; d += 32 * GR) {
         qs[d] = pr[mx.oq + h * D + d] * mx.qscale;
@@ -142,12 +182,14 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       }
       m_prev = m;
     }
-    float v = is_v ? pr[mx.ov + h * V + col] : (is_n ? 1.f : 0.f);
+    float v = is_n ? 1.f : 0.f;
+    if (is_v) v = KIND == KIND_SSD ? conv_silu(mx, sq.z, sq.x + t, t, sq.w + t, h * V + col) : pr[mx.ov + h * V + col];
+    const float x = v;
     __syncthreads();
     float part = 0.f;
     if (KIND != KIND_GLA) {
-      const float a = KIND == KIND_MLSTM ? s_sc[0] : decay;
-      if (KIND == KIND_MLSTM) v *= s_sc[1];
+      const float a = KIND == KIND_RETENTION ? decay : s_sc[0];
+      if (KIND != KIND_RETENTION) v *= s_sc[1];
 #pragma unroll
       for (int j = 0; j < RPT; ++j) {
         const int d = g + j * GR;
@@ -172,6 +214,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       float o = 0.f;
 #pragma unroll
       for (int i = 0; i < GR; ++i) o += red[i * 33 + lane];
+      if (KIND == KIND_SSD) o = fmaf(mx.skip[h], x, o);
       if (is_n) raw.nq[(size_t)(sq.x + t) * mx.H + h] = o;
       else raw.o[((size_t)(sq.x + t) * mx.H + h) * V + col] = o;
     }
@@ -208,6 +251,10 @@ struct Work {
   float* P;      // [chunk, H, 64, 64]
   float* KV;     // [chunk, H, D, V]   k~^T V, then the state before the chunk
   float* NK;     // [chunk, H, D]      sum_j k~_j, then n before the chunk (mLSTM)
+  float* xbc;    // state space: [chunk * 64 + i, channels] x | B | C behind the convolution
+  float* dt;     // state space: [chunk, H, 64] step sizes
+  float2* G;     // state space: [chunk, H, 64] running log decay, high and low part
+  int dec_w;     // entries of dec per chunk and head: D, or 1 (one decay for all channels)
 };
 
 // GLA: log decay of every channel, z = a2 (a1 h) + bias. One block per (chunk, 8 rows of it), channels over the threads.
@@ -443,6 +490,110 @@ __global__ void __launch_bounds__(256) retention_intra_kernel(const Mixer mx, co
   }
 }
 
+// State space, what enters the recurrence: blocks (chunk, y) convolve 256 channels each; the blocks behind them take 8 heads
+// each, one warp per head: step sizes, running log decay over the chunk (summed in double precision), decay of the chunk.
+template <int TAPS>      // 0: any number
+__global__ void __launch_bounds__(256) ssd_inputs_kernel(const Mixer mx, const Chunks ck, const Work wk, int conv_blocks) {
+  const int c = blockIdx.x, tid = threadIdx.x;
+  const int4 cd = ck.chunks[c], sq = ck.seqs[cd.z];
+  const int t0 = cd.x - sq.x, pos0 = sq.w + t0;      // first token of the chunk
+  if ((int)blockIdx.y < conv_blocks) {
+    const int CD = mx.channels(), ch = blockIdx.y * 256 + tid;
+    if (ch >= CD) return;
+    float* out = wk.xbc + (size_t)c * CH * CD + ch;
+    if (TAPS == 0) {
+      for (int r = 0; r < cd.y; ++r) out[(size_t)r * CD] = conv_silu(mx, sq.z, cd.x + r, t0 + r, pos0 + r, ch);
+    } else {
+      constexpr int N = TAPS > 0 ? TAPS : 1, AHEAD = 8;
+      float w[N], win[N];
+#pragma unroll
+      for (int j = 0; j < N; ++j) w[j] = mx.cw[(size_t)ch * N + j];
+      const float b = mx.cb[ch];
+#pragma unroll
+      for (int j = 0; j + 1 < N; ++j) win[j + 1] = conv_input(mx, sq.z, cd.x, t0, pos0, N - 1 - j, ch);
+      const float* in = mx.proj + (size_t)cd.x * mx.ld + mx.ov + ch;
+      for (int r0 = 0; r0 < cd.y; r0 += AHEAD) {
+        float x[AHEAD];
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) x[i] = r0 + i < cd.y ? in[(size_t)(r0 + i) * mx.ld] : 0.f;
+#pragma unroll
+        for (int i = 0; i < AHEAD; ++i) {
+#pragma unroll
+          for (int j = 0; j + 1 < N; ++j) win[j] = win[j + 1];
+          win[N - 1] = x[i];
+          float y = b;
+#pragma unroll
+          for (int j = 0; j < N; ++j) y = fmaf(w[j], win[j], y);
+          if (r0 + i < cd.y) out[(size_t)(r0 + i) * CD] = silu_exact(y);
+        }
+      }
+    }
+    return;
+  }
+  const int h = (blockIdx.y - conv_blocks) * 8 + (tid >> 5), lane = tid & 31;
+  if (h >= mx.H) return;
+  const size_t ch = (size_t)c * mx.H + h;
+  float dt[2];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const int r = 2 * lane + i;
+    dt[i] = r < cd.y ? softplus(mx.proj[(size_t)(cd.x + r) * mx.ld + mx.odt + h] + mx.dtb[h]) : 0.f;
+  }
+  const double a = (double)mx.A[h], own = a * dt[0] + a * dt[1];
+  double run = own;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double v = __shfl_up_sync(0xffffffffu, run, o);
+    if (lane >= o) run += v;
+  }
+  const double g[2] = {run - a * dt[1], run};
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const float hi = (float)g[i];
+    wk.G[ch * CH + 2 * lane + i] = make_float2(hi, (float)(g[i] - (double)hi));
+    wk.dt[ch * CH + 2 * lane + i] = dt[i];
+  }
+  if (lane == 31) wk.dec[ch] = expf((float)run);      // tokens behind the chunk's last have dt = 0
+}
+
+// P_ij = C_i . B_j of a (chunk, group of heads).
+__global__ void __launch_bounds__(256) ssd_scores_kernel(const Mixer mx, const Chunks ck, const Work wk) {
+  __shared__ float Qs[32][CH + 4], Ks[32][CH + 4];
+  const int c = blockIdx.x, g = blockIdx.y, tid = threadIdx.x;
+  const int len = ck.chunks[c].y, D = mx.D, CD = mx.channels();
+  const float* kb = wk.xbc + (size_t)c * CH * CD + mx.H * mx.V + g * D;
+  const float* qb = kb + mx.groups * D;
+  const int tx = tid & 15, ty = tid >> 4;
+  float acc[4][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  for (int d0 = 0; d0 < D; d0 += 32) {
+    for (int i = tid; i < CH * 32; i += 256) {
+      const int r = i >> 5, d = i & 31;
+      const bool in = r < len && d0 + d < D;
+      Qs[d][r] = in ? qb[(size_t)r * CD + d0 + d] : 0.f;
+      Ks[d][r] = in ? kb[(size_t)r * CD + d0 + d] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int d = 0; d < 32; ++d) {
+      const float4 a = *reinterpret_cast<const float4*>(&Qs[d][ty * 4]);
+      const float4 b = *reinterpret_cast<const float4*>(&Ks[d][tx * 4]);
+      const float av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(av[i], bv[j], acc[i][j]);
+    }
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    *reinterpret_cast<float4*>(wk.P + (((size_t)c * mx.groups + g) * CH + ty * 4 + i) * CH + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+
 // GLA intra-chunk part. One block per (chunk, head); 32 channels at a time. Thread (ti, tj) owns the entries
 // (16 a + ti, 16 b + tj) for all sub-chunk pairs b <= a.
 __global__ void __launch_bounds__(256) gla_intra_kernel(const Mixer mx, const Chunks ck, const Work wk) {
@@ -536,6 +687,7 @@ __global__ void __launch_bounds__(256) gla_intra_kernel(const Mixer mx, const Ch
 }
 
 // KV = k~^T V for one chunk, head and 64 x 64 tile of the state; mLSTM's first value tile also sums k~ over the chunk.
+template <bool SSD>
 __global__ void __launch_bounds__(256) chunk_kv_kernel(const Mixer mx, const Chunks ck, const Work wk, int dtiles) {
   __shared__ float Ks[CH][64 + 4], Vs[CH][64 + 4];
   const int c = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
@@ -543,6 +695,23 @@ __global__ void __launch_bounds__(256) chunk_kv_kernel(const Mixer mx, const Chu
   const int4 cd = ck.chunks[c];
   const int D = mx.D, V = mx.V;
   const size_t ch = (size_t)c * mx.H + h;
+  if (SSD) {
+    __shared__ float w[CH];
+    const int CD = mx.channels();
+    if (tid < CH) {
+      const float2 g = wk.G[ch * CH + tid], e = wk.G[ch * CH + CH - 1];
+      w[tid] = tid < cd.y ? wk.dt[ch * CH + tid] * expf((e.x - g.x) + (e.y - g.y)) : 0.f;
+    }
+    __syncthreads();
+    const float* row = wk.xbc + (size_t)c * CH * CD;
+    const int b0 = mx.H * V + h / (mx.H / mx.groups) * D;
+    for (int i = tid; i < CH * 64; i += 256) {
+      const int r = i >> 6, x = i & 63;
+      const bool in = r < cd.y;
+      Ks[r][x] = in && d0 + x < D ? row[(size_t)r * CD + b0 + d0 + x] : 0.f;
+      Vs[r][x] = in && v0 + x < V ? row[(size_t)r * CD + h * V + v0 + x] * w[r] : 0.f;
+    }
+  } else
   for (int i = tid; i < CH * 64; i += 256) {
     const int r = i >> 6, x = i & 63;
     Ks[r][x] = d0 + x < D ? wk.kt[(ch * CH + r) * D + d0 + x] : 0.f;
@@ -597,8 +766,8 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const Mixer mx, const C
   const size_t head = (size_t)sq.z * mx.H + h;
   float* state = is_n ? mx.N + head * D + d : mx.S + head * D * V + (size_t)g * VW;
   float* kv = is_n ? wk.NK + ((size_t)c0 * mx.H + h) * D + d : wk.KV + ((size_t)c0 * mx.H + h) * D * V + (size_t)g * VW;
-  const float* dec = wk.dec + ((size_t)c0 * mx.H + h) * D + d;
-  const size_t kv_step = (size_t)mx.H * D * (is_n ? 1 : V), dec_step = (size_t)mx.H * D;
+  const float* dec = wk.dec + ((size_t)c0 * mx.H + h) * wk.dec_w + (wk.dec_w > 1 ? d : 0);
+  const size_t kv_step = (size_t)mx.H * D * (is_n ? 1 : V), dec_step = (size_t)mx.H * wk.dec_w;
   auto load = [&](const float* p) {
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (VW == 4 && !is_n) v = *reinterpret_cast<const float4*>(p);
@@ -635,6 +804,7 @@ __global__ void __launch_bounds__(256) chunk_scan_kernel(const Mixer mx, const C
 }
 
 // o = q~ S_c + P V for one chunk, head and 64 value columns.
+template <bool SSD>
 __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Raw raw, const Chunks ck, const Work wk) {
   __shared__ float As[32][CH + 4], Bs[32][64 + 4];
   const int c = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * 64, tid = threadIdx.x;
@@ -647,6 +817,22 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  // state space: rows of x and C, exp(G_i), running decays and steps of the chunk
+  __shared__ float eg[CH], dts[CH];
+  __shared__ float2 gs[CH];
+  const int CD = SSD ? mx.channels() : 0, group = SSD ? h / (mx.H / mx.groups) : 0;
+  const float* xrow = SSD ? wk.xbc + (size_t)c * CH * CD : nullptr;
+  const float* crow = SSD ? xrow + mx.H * V + (mx.groups + group) * D : nullptr;
+  const float* cb = SSD ? wk.P + ((size_t)c * mx.groups + group) * CH * CH : nullptr;
+  if (SSD) {
+    if (tid < CH) {
+      const float2 g = wk.G[ch * CH + tid];
+      gs[tid] = g;
+      eg[tid] = expf(g.x + g.y);
+      dts[tid] = wk.dt[ch * CH + tid];
+    }
+    __syncthreads();
+  }
   float nq = 0.f;     // mLSTM, value tile 0: thread tid < 64 owns row tid
   const bool want_n = wk.NK != nullptr && blockIdx.z == 0 && tid < CH;
   const int steps_d = (D + 31) / 32, steps = steps_d + CH / 32;
@@ -655,7 +841,16 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
     const int k0 = inter ? s * 32 : (s - steps_d) * 32;
     for (int i = tid; i < 32 * CH; i += 256) {
       const int r = i >> 5, x = i & 31;
-      if (inter) As[x][r] = k0 + x < D ? wk.qt[(ch * CH + r) * D + k0 + x] : 0.f;
+      if (SSD) {
+        float a = 0.f;
+        if (inter) {
+          if (r < cd.y && k0 + x < D) a = crow[(size_t)r * CD + k0 + x] * eg[r];
+        } else if (k0 + x <= r && r < cd.y) {
+          const float2 gi = gs[r], gj = gs[k0 + x];
+          a = cb[r * CH + k0 + x] * dts[k0 + x] * expf((gi.x - gj.x) + (gi.y - gj.y));
+        }
+        As[x][r] = a;
+      } else if (inter) As[x][r] = k0 + x < D ? wk.qt[(ch * CH + r) * D + k0 + x] : 0.f;
       else As[x][r] = wk.P[(ch * CH + r) * CH + k0 + x];
     }
     for (int i = tid; i < 32 * 64; i += 256) {
@@ -663,6 +858,7 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
       float b = 0.f;
       if (v0 + v < V) {
         if (inter) b = k0 + x < D ? wk.KV[(ch * D + k0 + x) * V + v0 + v] : 0.f;
+        else if (SSD) b = k0 + x < cd.y ? xrow[(size_t)(k0 + x) * CD + h * V + v0 + v] : 0.f;
         else b = k0 + x < cd.y ? mx.proj[(size_t)(cd.x + k0 + x) * mx.ld + mx.ov + h * V + v0 + v] : 0.f;
       }
       Bs[x][v] = b;
@@ -693,6 +889,7 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int v = v0 + tx * 4 + j;
+      if (SSD && v < V) acc[i][j] = fmaf(mx.skip[h], xrow[(size_t)r * CD + h * V + v], acc[i][j]);
       if (v < V) raw.o[((size_t)(cd.x + r) * mx.H + h) * V + v] = acc[i][j];
     }
   }
@@ -746,6 +943,50 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
     for (int v = H * V + tid; v < ldo; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
 }
 
+// State space: y silu(z), normed in `parts` equal parts of the heads' outputs laid end to end, times norm_w [H * V]. One block per
+// (part, row); columns from H * V up to `width` are set to zero. ahead[row]: tokens of the same portion before the row. The
+// block of a portion's last row keeps the convolution's last inputs.
+template <typename OutT>
+__global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, float eps, const int* last_slot, const int* ahead,
+                                                       const int* pos, OutT* out, int ldo, int width) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float scratch[33];
+  constexpr int KEEP = 4;
+  const int g = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
+  const int inner = mx.H * mx.V, n = inner / gridDim.x;
+  const float* o = raw.o + (size_t)t * inner + g * n;
+  const float* gate = mx.proj + (size_t)t * mx.ld + mx.og + g * n;
+  float x[KEEP], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int v = tid + i * nt;
+    x[i] = v < n ? o[v] * silu_exact(gate[v]) : 0.f;
+    ss = fmaf(x[i], x[i], ss);
+  }
+  for (int v = tid + KEEP * nt; v < n; v += nt) {
+    const float y = o[v] * silu_exact(gate[v]);
+    ss = fmaf(y, y, ss);
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  OutT* dst = out + (size_t)t * ldo + g * n;
+  const float* w = norm_w + g * n;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if (tid + i * nt < n) dst[tid + i * nt] = (OutT)(x[i] * r * w[tid + i * nt]);
+  for (int v = tid + KEEP * nt; v < n; v += nt) dst[v] = (OutT)(o[v] * silu_exact(gate[v]) * r * w[v]);
+  if (g == gridDim.x - 1)
+    for (int v = inner + tid; v < width; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
+  const int slot = last_slot[t];
+  if (slot >= 0 && mx.taps > 1) {
+    // entry i of the new line is `taps - 2 - i` tokens old; of the old line only later entries are read
+    const int CD = mx.channels(), before = ahead[t], p = pos[t];
+    for (int ch = g * nt + tid; ch < CD; ch += gridDim.x * nt)
+      for (int i = 0; i < mx.taps - 1; ++i)
+        mx.Cs[((size_t)slot * (mx.taps - 1) + i) * CD + ch] = conv_input(mx, slot, t, before, p, mx.taps - 2 - i, ch);
+  }
+}
+
 template <int KIND>
 int launch_rows(const Mixer& mx, const Raw& raw, const int4* seqs, int nseq, cudaStream_t stream) {
   const int cols = mx.V + (KIND == KIND_MLSTM ? 1 : 0);
@@ -783,10 +1024,18 @@ Work carve(float* ws, const Mixer& mx, int nchunks, int kind, size_t* total) {
     w.ig = take(c * CH * H);
     w.NK = take(c * H * D);
   }
-  w.qt = take(c * H * CH * D);
-  w.kt = take(c * H * CH * D);
-  w.dec = take(c * H * D);
-  w.P = take(c * H * CH * CH);
+  w.dec_w = kind == KIND_SSD ? 1 : mx.D;
+  w.dec = take(c * H * w.dec_w);
+  if (kind == KIND_SSD) {
+    w.xbc = take(c * CH * mx.channels());
+    w.dt = take(c * H * CH);
+    w.G = (float2*)take(c * H * CH * 2);
+    w.P = take(c * mx.groups * CH * CH);
+  } else {
+    w.qt = take(c * H * CH * D);
+    w.kt = take(c * H * CH * D);
+    w.P = take(c * H * CH * CH);
+  }
   w.KV = take(c * H * D * V);
   *total = off;
   return w;
@@ -809,7 +1058,13 @@ struct PkStateMixer {
   float* m;
   const double* freq;
   const float* pw;
-  int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank, rot;
+  const float* cw;
+  const float* cb;
+  const float* dtb;
+  const float* A;
+  const float* skip;
+  float* Cs;
+  int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank, rot, groups, taps, odt;
   float qscale, cap, inv_tau;
 };
 
@@ -818,9 +1073,13 @@ static bool unpack(const PkStateMixer* d, Mixer& mx, Raw& raw) {
   if (d->kind == KIND_MLSTM && (!d->bi || !d->bf || !d->N || !d->Ms || !d->nq || !d->m || !(d->cap > 0.f))) return false;
   if (d->kind == KIND_GLA && (!d->a2 || !d->a2b || d->rank < 1 || d->rank > 1024)) return false;
   if (d->kind == KIND_RETENTION && (!d->pw || d->rot < 0 || (d->rot & 1) != 0 || d->rot > d->D || (d->rot > 0 && !d->freq))) return false;
-  if (d->kind != KIND_GLA && d->kind != KIND_MLSTM && d->kind != KIND_RETENTION) return false;
+  if (d->kind == KIND_SSD && (!d->cw || !d->cb || !d->dtb || !d->A || !d->skip || d->groups < 1 || d->H % d->groups != 0 || d->taps < 1 ||
+                              (d->taps > 1 && !d->Cs)))
+    return false;
+  if (d->kind < KIND_GLA || d->kind > KIND_SSD) return false;
   mx = Mixer{d->proj, d->ld, d->oq, d->ok, d->ov, d->og, d->oi, d->of, d->oa, d->H, d->D, d->V, d->qscale, d->bi, d->bf,
-             d->cap, d->a2, d->a2b, d->rank, d->inv_tau, d->freq, d->rot, d->pw, d->S, d->N, d->Ms};
+             d->cap, d->a2, d->a2b, d->rank, d->inv_tau, d->freq, d->rot, d->pw, d->cw, d->cb, d->dtb, d->A, d->skip, d->Cs,
+             d->groups, d->taps, d->odt, d->S, d->N, d->Ms};
   raw = Raw{d->o, d->nq, d->m};
   return true;
 }
@@ -832,6 +1091,7 @@ PK_API int pk_state_rows(const PkStateMixer* d, const void* seqs, int nseq, cuda
   if (!unpack(d, mx, raw) || seqs == nullptr || nseq < 1) return PK_ERR_BAD_ARG;
   switch (d->kind) {
     case KIND_GLA: return launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream);
+    case KIND_SSD: return launch_rows<KIND_SSD>(mx, raw, (const int4*)seqs, nseq, stream);
     case KIND_MLSTM: return launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
     default: return launch_rows<KIND_RETENTION>(mx, raw, (const int4*)seqs, nseq, stream);
   }
@@ -843,6 +1103,7 @@ PK_API size_t pk_state_chunk_workspace(const PkStateMixer* d, int nchunks) {
   mx.H = d->H;
   mx.D = d->D;
   mx.V = d->V;
+  mx.groups = d->groups;
   size_t n = 0;
   carve(nullptr, mx, nchunks, d->kind, &n);
   return n;
@@ -866,6 +1127,15 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
     gla_gates_kernel<<<dim3(nchunks, CH / 8, z < 16 ? z : 16), 256, (size_t)8 * mx.rank * sizeof(float), stream>>>(mx, ck, wk);
     PK_CHECK_LAUNCH();
     gla_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
+  } else if (d->kind == KIND_SSD) {
+    const int cb = (mx.channels() + 255) / 256;
+    const dim3 grid(nchunks, cb + (H + 7) / 8);
+    if (mx.taps == 2) ssd_inputs_kernel<2><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);
+    else if (mx.taps == 3) ssd_inputs_kernel<3><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);
+    else if (mx.taps == 4) ssd_inputs_kernel<4><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);
+    else ssd_inputs_kernel<0><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);
+    PK_CHECK_LAUNCH();
+    ssd_scores_kernel<<<dim3(nchunks, mx.groups), 256, 0, stream>>>(mx, ck, wk);
   } else if (d->kind == KIND_RETENTION) {
     retention_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
   } else {
@@ -874,7 +1144,9 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
     mlstm_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, raw, ck, wk);
   }
   PK_CHECK_LAUNCH();
-  chunk_kv_kernel<<<dim3(nchunks, H, dt * vt), 256, 0, stream>>>(mx, ck, wk, dt);
+  const bool ssd = d->kind == KIND_SSD;
+  if (ssd) chunk_kv_kernel<true><<<dim3(nchunks, H, dt * vt), 256, 0, stream>>>(mx, ck, wk, dt);
+  else chunk_kv_kernel<false><<<dim3(nchunks, H, dt * vt), 256, 0, stream>>>(mx, ck, wk, dt);
   PK_CHECK_LAUNCH();
   const bool v4 = (mx.V & 3) == 0 && ((uintptr_t)mx.S & 15) == 0;
   const int elems = mx.D * mx.V / (v4 ? 4 : 1) + (d->kind == KIND_MLSTM ? mx.D : 0);
@@ -882,7 +1154,8 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
   if (v4) chunk_scan_kernel<4><<<scan_grid, 256, 0, stream>>>(mx, ck, wk);
   else chunk_scan_kernel<1><<<scan_grid, 256, 0, stream>>>(mx, ck, wk);
   PK_CHECK_LAUNCH();
-  chunk_out_kernel<<<dim3(nchunks, H, vt), 256, 0, stream>>>(mx, raw, ck, wk);
+  if (ssd) chunk_out_kernel<true><<<dim3(nchunks, H, vt), 256, 0, stream>>>(mx, raw, ck, wk);
+  else chunk_out_kernel<false><<<dim3(nchunks, H, vt), 256, 0, stream>>>(mx, raw, ck, wk);
   PK_CHECK_LAUNCH();
   return PK_OK;
 }
@@ -903,5 +1176,21 @@ PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head
     if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
     else PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
   }
+  return PK_OK;
+}
+
+// State space: gate, norm in `parts` parts, output rows [rows, ldo] of which `width` columns are this layer's; the last inputs of
+// the convolution are kept for every portion that ends (last_slot, ahead and pos per row).
+PK_API int pk_ssd_out(const PkStateMixer* d, const float* norm_w, int parts, float eps, const int* last_slot, const int* ahead, const int* pos, int rows,
+                      void* out, int ldo, int width, int out_f32, cudaStream_t stream) {
+  Mixer mx;
+  Raw raw;
+  if (!unpack(d, mx, raw) || d->kind != KIND_SSD || norm_w == nullptr || last_slot == nullptr || ahead == nullptr || pos == nullptr || rows < 1 ||
+      rows > 65535 || out == nullptr || parts < 1 || mx.H * mx.V % parts != 0 || width < mx.H * mx.V || ldo < width)
+    return PK_ERR_BAD_ARG;
+  const int n = mx.H * mx.V / parts, nt = (n + 31) / 32 * 32;
+  const dim3 grid(parts, rows), block(nt <= 256 ? nt : n > 2048 ? 1024 : 256);
+  if (out_f32) PK_LAUNCH_PDL(ssd_out_kernel<float>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, last_slot, ahead, pos, (float*)out, ldo, width);
+  else PK_LAUNCH_PDL(ssd_out_kernel<pk::bf16>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, last_slot, ahead, pos, (pk::bf16*)out, ldo, width);
   return PK_OK;
 }

@@ -1,8 +1,9 @@
-// Grouped-query attention over a paged cache, with the choices of its design as parameters: rotation of a leading part of
-// queries and keys, full causal / sliding-window / chunked visibility, one softmax map per head or two over the same values
-// whose difference a1 - lambda a2 is the head's output, an optional norm of every head's output.
+// Grouped-query attention over a paged cache, with the choices of its design as parameters: norms of queries and keys, rotation
+// of a leading part of them (pairs half a width apart, or neighbours), values mixed with those of an earlier layer, full causal /
+// sliding-window / chunked visibility, capped scores, a sink in the softmax, one softmax map per head or two over the same
+// values whose difference a1 - lambda a2 is the head's output, an optional norm of every head's output, a gate per head.
 //
-//   prep    per row: rotation, cache append, queries for the row kernel (fp32) and the tensor-core kernel (bf16)
+//   prep    per row: norm, rotation, cache append, queries for the row kernel (fp32) and the tensor-core kernel (bf16)
 //   rows    split-context attention of single rows: up to eight query vectors of one key head per block, fp32
 //   merge   sum of the splits, difference of the maps, head norm
 // Long portions of bf16 models run their attention in paged_prefill.cu.
@@ -48,7 +49,8 @@ __global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a) {
   const float* pr = a.proj + (size_t)t * a.ld;
   const int pos = a.pos[t];
   auto source = [&](int v) { return v < nq ? pr + a.oq + v * a.D : v < nq + nk ? pr + a.ok + (v - nq) * a.D : pr + a.ov + (v - nq - nk) * a.V; };
-  // pair i of a query or key: (i, i + half) while it turns, then single elements
+  // pair i of a query or key while it turns, then single elements
+  const int pa = a.neighbours ? 2 : 1, pb = a.neighbours ? 1 : half;      // pair i: (i * pa, i * pa + pb)
   float x0[NPW], y0[NPW];
 #pragma unroll
   for (int j = 0; j < NPW; ++j) {
@@ -56,8 +58,8 @@ __global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a) {
     x0[j] = y0[j] = 0.f;
     if (v < nq + nk && lane < half) {
       const float* src = source(v);
-      x0[j] = src[lane];
-      y0[j] = src[lane + half];
+      x0[j] = src[lane * pa];
+      y0[j] = src[lane * pa + pb];
     }
   }
   float* cs = sm;
@@ -72,10 +74,19 @@ __global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a) {
     const float* src = source(v);
     if (v >= nq + nk) {
       CT* dst = crow + nk * a.dp + (v - nq - nk) * a.vp;
+      float* vf = a.v_mix ? a.v_first + ((size_t)t * a.G + v - nq - nk) * a.V : nullptr;
       for (int i0 = lane; i0 < a.vp; i0 += 128) {
         float x[4];
 #pragma unroll
         for (int k = 0; k < 4; ++k) x[k] = i0 + k * 32 < a.V ? src[i0 + k * 32] : 0.f;
+        if (a.v_mix) {
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            if (i0 + k * 32 < a.V) {
+              if (a.v_mix == 1) vf[i0 + k * 32] = x[k];
+              else x[k] = (1.f - a.mix) * x[k] + a.mix * vf[i0 + k * 32];
+            }
+        }
 #pragma unroll
         for (int k = 0; k < 4; ++k)
           if (i0 + k * 32 < a.vp) dst[i0 + k * 32] = (CT)x[k];
@@ -86,18 +97,27 @@ __global__ void __launch_bounds__(256) paged_prep_kernel(const Attn a) {
     CT* krow = is_q ? nullptr : crow + (v - nq) * a.dp;
     float* qx = is_q && a.qx ? a.qx + ((size_t)t * nq + v) * a.D : nullptr;
     bf16* qf = is_q && a.qf ? (bf16*)a.qf + ((size_t)t * nq + v) * a.q_ld : nullptr;
+    const float* nw = is_q ? a.q_norm : a.k_norm;
+    float rn = 1.f;
+    if (nw) {
+      float ss = 0.f;
+      for (int i = lane; i < a.D; i += 32) ss = fmaf(src[i], src[i], ss);
+      rn = 1.f / sqrtf(warp_sum(ss) / (float)a.D + a.eps);
+    }
+    auto normed = [&](int i, float x) { return nw ? x * rn * nw[i] : x; };
     auto put = [&](int i, float x) {
       if (krow) krow[i] = (CT)x;
       if (qx) qx[i] = x;
       if (qf) qf[i] = __float2bfloat16(x);
     };
     for (int i = lane; i < half; i += 32) {
-      float x = i == lane ? x0[j] : src[i], y = i == lane ? y0[j] : src[i + half];
+      const int e = i * pa, o = e + pb;
+      float x = normed(e, i == lane ? x0[j] : src[e]), y = normed(o, i == lane ? y0[j] : src[o]);
       rotate_pair(x, y, sn[i], cs[i]);
-      put(i, x);
-      put(i + half, y);
+      put(e, x);
+      put(o, y);
     }
-    for (int i = a.R + lane; i < a.D; i += 32) put(i, src[i]);
+    for (int i = a.R + lane; i < a.D; i += 32) put(i, normed(i, src[i]));
     if (krow)
       for (int i = a.D + lane; i < a.dp; i += 32) krow[i] = (CT)0.f;
     if (qf)
@@ -175,7 +195,9 @@ __global__ void __launch_bounds__(32 * QB) paged_rows_kernel(const Attn a, const
         for (int e = 0; e < VE; ++e) s4[e & 3] = fmaf(to_f<CT>(ke[e]), q[v + e], s4[e & 3]);
       }
     }
-    const float s = lane < nk ? ((s4[0] + s4[1]) + (s4[2] + s4[3])) * a.scale : -INFINITY;
+    float s = ((s4[0] + s4[1]) + (s4[2] + s4[3])) * a.scale;
+    if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
+    if (lane >= nk) s = -INFINITY;
     const float mn = fmaxf(m, warp_max(s));
     const float alpha = m == -INFINITY ? 0.f : expf(m - mn);
     const float e = lane < nk ? expf(s - mn) : 0.f;
@@ -246,7 +268,8 @@ __global__ void __launch_bounds__(128) paged_merge_kernel(const Attn a, const in
     float* w = ws + warp * ns;
     if (a.part_ml) {
       const float* ml = a.part_ml + ((size_t)r * ns * nq + h * a.maps + warp) * 2;
-      float mx = -INFINITY;
+      const float sink = a.sink ? a.sink[h * a.maps + warp] : -INFINITY;
+      float mx = sink;
       for (int s = lane; s < ns; s += 32) mx = fmaxf(mx, ml[(size_t)s * nq * 2]);
       mx = warp_max(mx);
       float den = 0.f;
@@ -257,6 +280,7 @@ __global__ void __launch_bounds__(128) paged_merge_kernel(const Attn a, const in
         den += e * ml[(size_t)s * nq * 2 + 1];
       }
       den = warp_sum(den);
+      if (a.sink) den += expf(sink - mx);
       __syncwarp();
       for (int s = lane; s < ns; s += 32) w[s] /= den;
     } else if (lane == 0) {
@@ -284,21 +308,22 @@ __global__ void __launch_bounds__(128) paged_merge_kernel(const Attn a, const in
       ss = fmaf(o[i], o[i], ss);
     }
   }
-  const float f = a.head_norm ? a.post / sqrtf(block_sum(ss, scratch) / (float)a.V + a.eps) : 1.f;
   const int t = rows ? rows[r] : r;
+  float f = a.head_norm ? a.post / sqrtf(block_sum(ss, scratch) / (float)a.V + a.eps) : a.post;
+  if (a.gate >= 0) f /= 1.f + expf(-a.proj[(size_t)t * a.ld + a.gate + h]);
   OutT* dst = reinterpret_cast<OutT*>(a.out) + (size_t)t * a.ldo;
 #pragma unroll
   for (int i = 0; i < KEEP; ++i)
     if (tid + i * 128 < a.V) dst[h * a.V + tid + i * 128] = (OutT)(o[i] * f);
   if (h == a.H - 1)
-    for (int v = a.H * a.V + tid; v < a.ldo; v += 128) dst[v] = (OutT)0.f;
+    for (int v = a.H * a.V + tid; v < a.width; v += 128) dst[v] = (OutT)0.f;
 }
 
 bool shape_ok(const Attn* a) {
   return a != nullptr && a->H >= 1 && a->G >= 1 && a->H % a->G == 0 && (a->maps == 1 || a->maps == 2) && a->D >= 1 && a->V >= 1 && a->V <= 512 && a->R >= 0 &&
          (a->R & 1) == 0 && a->R <= a->D && a->dp >= a->D && (a->dp & 7) == 0 && a->vp >= a->V && (a->vp & 7) == 0 && (a->row & 7) == 0 &&
          a->row >= a->G * (a->maps * a->dp + a->vp) && a->cache != nullptr && a->table != nullptr && a->pos != nullptr && a->slot != nullptr &&
-         ((uintptr_t)a->cache & 15) == 0;
+         ((uintptr_t)a->cache & 15) == 0 && (a->v_mix == 0 || ((a->v_mix == 1 || a->v_mix == 2) && a->v_first != nullptr));
 }
 
 template <typename CT>
@@ -351,7 +376,7 @@ PK_API int pk_paged_rows(const PkPagedAttention* a, const int* rows, int nrows, 
 
 // Finished outputs of the listed rows (rows null: rows 0 .. nrows - 1).
 PK_API int pk_paged_merge(const PkPagedAttention* a, const int* rows, int nrows, cudaStream_t stream) {
-  if (!shape_ok(a) || nrows < 1 || a->part_o == nullptr || a->out == nullptr || a->ldo < a->H * a->V || a->nsplit < 1 || a->nsplit > 1024 ||
+  if (!shape_ok(a) || nrows < 1 || a->part_o == nullptr || a->out == nullptr || a->width < a->H * a->V || a->ldo < a->width || (a->gate >= 0 && a->proj == nullptr) || a->nsplit < 1 || a->nsplit > 1024 ||
       (a->part_ml == nullptr && a->nsplit != 1) || a->H > 65535)
     return PK_ERR_BAD_ARG;
   const size_t smem = (size_t)a->maps * a->nsplit * sizeof(float);

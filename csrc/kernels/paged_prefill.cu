@@ -1,5 +1,5 @@
 // Prefill attention of long portions on the 5th-generation tensor cores, straight from the paged cache (paged_attention.cu
-// describes the variants): grouped-query, causal, optional window or chunks, one or two softmax maps per head.
+// describes the variants): grouped-query, causal, optional window or chunks, capped scores, a sink, one or two softmax maps per head.
 //
 // One CTA works one (head, tile of up to 128 query rows of one portion, slice of up to 128 value columns) and NMAP of the
 // head's maps. A step is one page, 64 positions; its keys and values arrive by TMA (no multicast) into two alternating
@@ -36,6 +36,7 @@ struct Params {
   const int4* seqs;        // {first step row, tokens, slot, first position}
   int qk_panels, k_steps;  // key width in 64-element panels and in 16-element products
   float scale_log2;
+  float cap_in, cap_out;   // cap_in > 0: score x cap_in = 2 log2(e) score / cap; cap_out = cap log2(e)
   int raw;                 // outputs go to part_o [rows, H x maps, V]
 };
 
@@ -62,6 +63,13 @@ __device__ __forceinline__ float exp2_approx(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// y <- cap_out tanh(x / cap) from x cap_in, by tanh(u) = 1 - 2 / (exp(2 u) + 1): absolute error a few 2^-23 of the cap
+__device__ __forceinline__ float soft_cap_log2(float x, float cap_in, float cap_out) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(exp2_approx(x * cap_in) + 1.f));
+  return fmaf(-2.f * cap_out, r, cap_out);
 }
 
 template <int VP, int NMAP>    // value columns of this CTA's slice: 64 or 128; maps worked together
@@ -213,6 +221,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
     const uint32_t lane_off = (uint32_t)(q4 * 32) << 16;
     const uint32_t ts = tmem_s + m * 128 + lane_off, to = tmem_o + m * VP + lane_off;
     float ref = -INFINITY, sum = 0.f;      // the row's reference (log2 units) and the sum of its weights
+    if (a.sink) {                          // the sink is the first score of every row
+      ref = a.sink[vec0 + m] * 1.4426950408889634f;
+      sum = 1.f;
+    }
+    const float to_log2 = p.cap_in > 0.f ? 1.f : p.scale_log2;
     bool ok = true;
     uint8_t* prow = sp + m * 2 * kQPanel + r * 128;
     for (int t = 0; t < n_tiles; ++t) {
@@ -225,6 +238,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       tmem_ld_32x32(ts + (t & 1) * 64, s[0]);
       tmem_ld_32x32(ts + (t & 1) * 64 + 32, s[1]);
       tmem_ld_wait();
+      if (p.cap_in > 0.f) {
+#pragma unroll
+        for (int c = 0; c < 2; ++c)
+#pragma unroll
+          for (int i = 0; i < 32; ++i) s[c][i] = __float_as_uint(soft_cap_log2(__uint_as_float(s[c][i]), p.cap_in, p.cap_out));
+      }
       // visible columns of this row in this step: [c_lo, c_hi]
       const int c_lo = lo - (first + t * kKV), c_hi = q_pos - (first + t * kKV);
       if (__any_sync(0xffffffffu, c_lo > 0 || c_hi < kKV - 1)) {
@@ -239,11 +258,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       for (int c = 0; c < 2; ++c)
 #pragma unroll
         for (int i = 0; i < 32; ++i) t4[i & 3] = fmaxf(t4[i & 3], __uint_as_float(s[c][i]));
-      const float top = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])) * p.scale_log2;
+      const float top = fmaxf(fmaxf(t4[0], t4[1]), fmaxf(t4[2], t4[3])) * to_log2;
       bool waited = t == 0;
       if (ref == -INFINITY) ref = top;      // nothing was visible so far: sum and O are zero
       const bool grow = top > ref + kSlack;
       if (__any_sync(0xffffffffu, grow)) {
+        const float alpha = grow ? exp2_approx(ref - top) : 1.f;
         if (t > 0) {
           if (!mbar_wait_warp(&ct.pv_full[m], (t - 1) & 1, &ct.abort_flag, a.status, 78)) {
             ok = false;
@@ -251,7 +271,6 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           }
           waited = true;
           tc_fence_after();
-          const float alpha = grow ? exp2_approx(ref - top) : 1.f;
 #pragma unroll 1
           for (int c = 0; c < VP / 32; ++c) {
             uint32_t x[32];
@@ -262,8 +281,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
             tmem_st_32x32(to + c * 32, x);
           }
           tmem_st_wait();
-          sum *= alpha;
         }
+        sum *= alpha;
         if (grow) ref = top;
       }
       const float mb = ref == -INFINITY ? 0.f : ref;
@@ -273,8 +292,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
       for (int c = 0; c < 2; ++c)
 #pragma unroll
         for (int e = 0; e < 16; ++e) {
-          const float x = exp2_approx(fmaf(__uint_as_float(s[c][2 * e]), p.scale_log2, -mb));
-          const float y = exp2_approx(fmaf(__uint_as_float(s[c][2 * e + 1]), p.scale_log2, -mb));
+          const float x = exp2_approx(fmaf(__uint_as_float(s[c][2 * e]), to_log2, -mb));
+          const float y = exp2_approx(fmaf(__uint_as_float(s[c][2 * e + 1]), to_log2, -mb));
           u4[e & 3] += x + y;
           const __nv_bfloat162 ph = __floats2bfloat162_rn(x, y);
           const uint32_t hb = *reinterpret_cast<const uint32_t*>(&ph);
@@ -335,7 +354,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
           if (NMAP == 2) o[i] -= xch[(c * 32 + i) * kQ + r];
         }
       };
-      float f = 1.f;
+      float f = a.post;
       if (a.head_norm && !p.raw) {
         float ss = 0.f;
 #pragma unroll 1
@@ -348,6 +367,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
         }
         f = a.post / sqrtf(ss / (float)a.V + a.eps);
       }
+      if (a.gate >= 0 && !p.raw && row_ok) f /= 1.f + expf(-a.proj[(size_t)(tile.x + r) * a.ld + a.gate + h]);
 #pragma unroll 1
       for (int c = 0; c < VP / 32; ++c) {
         float o[32];
@@ -381,7 +401,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_co
         }
       }
       if (row_ok && !p.raw && h == a.H - 1 && vs == 0)
-        for (int i = a.H * a.V; i < a.ldo; ++i) ((bf16*)a.out)[(size_t)(tile.x + r) * a.ldo + i] = __float2bfloat16(0.f);
+        for (int i = a.H * a.V; i < a.width; ++i) ((bf16*)a.out)[(size_t)(tile.x + r) * a.ldo + i] = __float2bfloat16(0.f);
     }
   }
 
@@ -460,13 +480,16 @@ PK_API int pk_paged_prefill(const PkPagedAttention* a, int rows, int pages, cons
   if (((uintptr_t)a->qf & 15) != 0 || ((uintptr_t)a->cache & 15) != 0) return PK_ERR_BAD_ARG;
   const int form = pk_paged_prefill_form(a->maps, a->D, a->V);
   if (form < 0) return PK_ERR_UNSUPPORTED;
-  if (form == 0 ? a->part_o == nullptr : (a->out == nullptr || ((uintptr_t)a->out & 15) != 0 || (a->ldo & 7) != 0 || a->ldo < a->H * a->V)) return PK_ERR_BAD_ARG;
+  if (form == 0 ? a->part_o == nullptr : (a->out == nullptr || ((uintptr_t)a->out & 15) != 0 || (a->ldo & 7) != 0 || a->width < a->H * a->V || a->ldo < a->width ||
+                                    (a->gate >= 0 && a->proj == nullptr)))
+    return PK_ERR_BAD_ARG;
   EncodeTiledFn encode = encode_fn();
   if (encode == nullptr) return PK_ERR_UNSUPPORTED;
   CUtensorMap tq, tc;
   if (!encode_rows64(encode, &tq, a->qf, (uint64_t)a->H * a->maps * a->q_ld, (uint64_t)rows)) return PK_ERR_CUDA;
   if (!encode_rows64(encode, &tc, a->cache, (uint64_t)a->row, (uint64_t)pages * kKV)) return PK_ERR_CUDA;
-  Params p{*a, (const int4*)tiles, (const int4*)seqs, (a->D + 63) / 64, (a->D + 15) / 16, a->scale * 1.4426950408889634f, form == 0 ? 1 : 0};
+  Params p{*a, (const int4*)tiles, (const int4*)seqs, (a->D + 63) / 64, (a->D + 15) / 16, a->scale * 1.4426950408889634f,
+           a->cap > 0.f ? 2.f * 1.4426950408889634f * a->scale / a->cap : 0.f, a->cap * 1.4426950408889634f, form == 0 ? 1 : 0};
   const int slices = (a->V + 127) / 128;
   const bool narrow = a->V <= 64;
   if (form == 1 && a->maps == 2) return narrow ? launch<64, 2>(tq, tc, p, dim3(a->H, ntiles, 1), stream) : launch<128, 2>(tq, tc, p, dim3(a->H, ntiles, 1), stream);

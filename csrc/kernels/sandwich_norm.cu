@@ -2,7 +2,8 @@
 // projections,
 //   x   <- scale * embedding row            (first layer)    or
 //   x   <- x + rms(y) * (bias + w_post)     (y = the sublayer's output, fp32; no w_post: y as it is; y may be the sum of a
-//                                            few listed rows, the outputs of a token's experts)
+//                                            few listed rows, the outputs of a token's experts, and of another row times
+//                                            a factor; a constant may multiply the whole term)
 //   x   <- x + scale * embedding row        (again, before a further pass over the same layers)
 //   out <- rms(x) * (bias + w_pre)          (the next sublayer's input, bf16 or fp32, columns padded with zeros)
 // `bias` is 1 for weights stored around zero and 0 for plain weights. One block per row, the row stays in registers.
@@ -22,7 +23,11 @@ struct NormParams {
   const float* y;        // [rows, ldy] or null
   int ldy;
   const int* y_rows;     // [rows, y_top]: y of a row is the sum of these rows of `y` (null: the row of the same index)
-  int y_top;
+  int y_top;               // (a negative entry stands for no row)
+  float y_scale;           // factor on what is added
+  const void* skip;        // [rows, ld_skip] or null: y of a row gets skip_w[row] x this row
+  const float* skip_w;
+  int ld_skip, skip_f32;
   const float* w_post;
   const int* rows;       // output row r works on residual row rows[r] (null: r); x is not written then
   int width;
@@ -54,6 +59,19 @@ __device__ __forceinline__ void store(bf16* p, const float (&v)[VW]) {
     *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
   } else {
     *p = __float2bfloat16(v[0]);
+  }
+}
+
+template <int VW>
+__device__ __forceinline__ void load_any(const void* p, size_t at, bool f32, float (&v)[VW]) {
+  if (f32) {
+    load_f32<VW>((const float*)p + at, v);
+  } else if (VW == 4) {
+    const uint2 u = *reinterpret_cast<const uint2*>((const bf16*)p + at);
+    v[0] = __uint_as_float(u.x << 16); v[1 % VW] = __uint_as_float(u.x & 0xffff0000u);
+    v[2 % VW] = __uint_as_float(u.y << 16); v[3 % VW] = __uint_as_float(u.y & 0xffff0000u);
+  } else {
+    v[0] = __bfloat162float(((const bf16*)p)[at]);
   }
 }
 
@@ -108,12 +126,23 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const NormParams p)
         if (p.y_rows) {
           for (int k = 0; k < p.y_top; ++k) {
             float a[VW];
-            load_f32<VW>(p.y + (size_t)p.y_rows[(size_t)row * p.y_top + k] * p.ldy + c, a);
+            const int from = p.y_rows[(size_t)row * p.y_top + k];
+            if (from < 0) continue;
+            load_f32<VW>(p.y + (size_t)from * p.ldy + c, a);
 #pragma unroll
             for (int j = 0; j < VW; ++j) u[i][j] += a[j];
           }
         } else {
           load_f32<VW>(p.y + (size_t)row * p.ldy + c, u[i]);
+        }
+        if (p.skip) {      // may be the buffer of `out`: this thread alone reads and later writes these columns
+          const float f = p.skip_w[row];
+          float a[VW];
+          load_any<VW>(p.skip, (size_t)row * p.ld_skip + c, p.skip_f32, a);
+          if (f != 0.f) {
+#pragma unroll
+            for (int j = 0; j < VW; ++j) u[i][j] = fmaf(f, a[j], u[i][j]);
+          }
         }
       }
 #pragma unroll
@@ -125,13 +154,13 @@ __global__ void __launch_bounds__(1024) sandwich_norm_kernel(const NormParams p)
       for (int i = 0; i < PT; ++i)
         if ((tid + i * nt) * VW < p.width) {
 #pragma unroll
-          for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * rr * (p.bias + wb[i][j]);
+          for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * rr * (p.bias + wb[i][j]) * p.y_scale;
         }
     } else {
 #pragma unroll
       for (int i = 0; i < PT; ++i)
 #pragma unroll
-        for (int j = 0; j < VW; ++j) v[i][j] += u[i][j];
+        for (int j = 0; j < VW; ++j) v[i][j] += u[i][j] * p.y_scale;
     }
   }
   if (p.tokens && p.embed_add) add_embedding();
@@ -187,7 +216,7 @@ int launch_norm(const NormParams& p, int M, cudaStream_t stream) {
 template <typename OutT>
 int launch_any(const NormParams& p, int M, cudaStream_t stream) {
   const bool v4 = (p.width & 3) == 0 && ((uintptr_t)p.x & 15) == 0 && (p.y == nullptr || ((p.ldy & 3) == 0 && ((uintptr_t)p.y & 15) == 0)) &&
-                  (p.w_post == nullptr || ((uintptr_t)p.w_post & 15) == 0) &&
+                  (p.skip == nullptr || ((p.ld_skip & 3) == 0 && ((uintptr_t)p.skip & 15) == 0)) && (p.w_post == nullptr || ((uintptr_t)p.w_post & 15) == 0) &&
                   (p.w_pre == nullptr || (((uintptr_t)p.w_pre & 15) == 0 && (p.ldo & 3) == 0 && ((uintptr_t)p.out & 15) == 0));
   return v4 ? launch_norm<OutT, 4>(p, M, stream) : launch_norm<OutT, 1>(p, M, stream);
 }
@@ -209,16 +238,17 @@ __global__ void bump_kernel(int* step) { step[0] += 1; }
 }  // namespace
 
 // See the head of this file. tokens != null: x is filled from the embedding table (embed_add: the row is added); y != null: the
-// (normed) sublayer output is added first. rows != null: only the M listed rows are normed (x stays as it is). width up to
-// 8192 (32768 when a multiple of 4).
+// (normed) sublayer output x y_scale is added first, skip_w[row] x a row of `skip` being part of it. rows != null: only the M
+// listed rows are normed (x stays as it is). width up to 8192 (32768 when a multiple of 4).
 PK_API int pk_sandwich_norm(float* x, const int* tokens, const void* embed, int vocab, float embed_scale, int embed_add, const float* y, int ldy,
-                            const int* y_rows, int y_top, const float* w_post, const int* rows, int M, int width, const float* w_pre,
-                            int plus_one, float eps, void* out, int ldo, int out_f32, cudaStream_t stream) {
+                            const int* y_rows, int y_top, float y_scale, const void* skip, int ld_skip, int skip_f32, const float* skip_w,
+                            const float* w_post, const int* rows, int M, int width, const float* w_pre, int plus_one, float eps, void* out, int ldo, int out_f32, cudaStream_t stream) {
   if (M < 1 || width < 1 || x == nullptr) return PK_ERR_BAD_ARG;
   if (y != nullptr && (ldy < width || (y_rows != nullptr && y_top < 1))) return PK_ERR_BAD_ARG;
+  if (skip != nullptr && (y == nullptr || skip_w == nullptr || ld_skip < width)) return PK_ERR_BAD_ARG;
   if (tokens != nullptr && (embed == nullptr || vocab < 1)) return PK_ERR_BAD_ARG;
   if (w_pre != nullptr && (out == nullptr || ldo < width)) return PK_ERR_BAD_ARG;
-  NormParams p{x, tokens, (const pk::bf16*)embed, vocab, embed_scale, embed_add, y, ldy, y_rows, y_top, w_post, rows, width, w_pre,
+  NormParams p{x, tokens, (const pk::bf16*)embed, vocab, embed_scale, embed_add, y, ldy, y_rows, y_top, y_scale, skip, skip_w, ld_skip, skip_f32, w_post, rows, width, w_pre,
                plus_one ? 1.f : 0.f, eps, out, ldo};
   return out_f32 ? launch_any<float>(p, M, stream) : launch_any<pk::bf16>(p, M, stream);
 }

@@ -52,6 +52,7 @@ class StepContext:
     pos: torch.Tensor
     slot: torch.Tensor
     last_slot: torch.Tensor             # slot of the portion that ends at a row, else -1
+    ahead: torch.Tensor                 # tokens of the same portion before a row
     table: torch.Tensor                 # page table
     ws: Workspace
     status: torch.Tensor
@@ -191,14 +192,58 @@ class RetentionMixer(RecurrentMixer):
         self.desc.update(freq=freq.data_ptr() if rot["dims"] else None, rot=rot["dims"], pw=powers.data_ptr())
 
 
+class StateSpaceMixer:
+    """The state-space recurrence of Mamba-2: x, B and C through a short convolution, a scalar decay per token and head, gate before
+    a norm in equal parts. `scale` multiplies its output. Works on columns of a projection that its owner makes."""
+
+    def __init__(self, w: dict, m: dict, eps: float, device, slots: int, scale: float = 1.0):
+        H, V, N, G, taps = m["heads"], m["vdim"], m["state"], m["groups"], m["conv"]
+        self.H, self.V, self.N, self.parts, self.eps = H, V, N, m["norm_groups"], eps
+        if N > 512:
+            raise ValueError("state-space layers take states up to 512")
+        ch = H * V + 2 * G * N
+        for n, s in (("in", (2 * H * V + 2 * G * N + H, None)), ("conv", (ch, taps)), ("conv.b", (ch,)), ("dt_bias", (H,)), ("A_log", (H,)), ("D", (H,)),
+                     ("norm", (H * V,))):
+            if any(b is not None and a != b for a, b in zip(w[n].shape, s)):
+                raise ValueError(f"{n}: shape {tuple(w[n].shape)}, expected {s}")
+        f = lambda n: _f32(w[n], device)
+        self.const = {"cw": f("conv"), "cb": f("conv.b"), "dtb": f("dt_bias"), "A": -torch.exp(w["A_log"].double()).float().to(device), "skip": f("D")}
+        self.norm = f("norm") * scale
+        self.S = torch.zeros(slots, H, N, V, device=device)
+        self.line = torch.zeros(slots, max(taps - 1, 1), ch, device=device)
+        self.desc = dict(kind=mo.KIND_SSD, H=H, D=N, V=V, groups=G, taps=taps, qscale=1.0, S=self.S.data_ptr(), Cs=self.line.data_ptr(),
+                         **{n: t.data_ptr() for n, t in self.const.items()})
+
+    def at(self, first: int) -> None:
+        """The projection's columns z | x B C | dt start at `first`."""
+        inner = self.H * self.V
+        self.desc.update(og=first, ov=first + inner, odt=first + 2 * inner + 2 * self.desc["groups"] * self.N)
+
+    def state_bytes(self) -> int:
+        return (self.S.numel() + self.line.numel()) * 4
+
+    def run(self, ctx: StepContext, p: torch.Tensor, out: torch.Tensor) -> None:
+        ws = ctx.ws
+        o = ws.flat("raw_o", ctx.T * self.H * self.V, torch.float32)
+        d = mo.StateMixer(proj=p.data_ptr(), ld=p.stride(0), o=o.data_ptr(), **self.desc)
+        if ctx.n_short:
+            mo.state_rows(d, ctx.short, ctx.n_short)
+        if ctx.n_long:
+            scratch = ws.flat("state_chunks", mo.state_chunk_workspace(d, ctx.n_chunks), torch.float32)
+            mo.state_chunks(d, ctx.long, ctx.n_long, ctx.chunks, ctx.chunk0, ctx.n_chunks, scratch)
+        mo.ssd_out(d, self.norm, self.parts, self.eps, ctx.last_slot, ctx.ahead, ctx.pos, ctx.T, out)
+
+
 def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> tuple[torch.Tensor, float]:
-    """Angular frequency of every rotated pair (float64) and the factor on cos and sin. `scaling` = YaRN's {factor, original,
-    fast, slow}: pairs that turn fewer than `slow` times over the original context are slowed down by `factor`, those that
-    turn more than `fast` times keep their frequency, with a linear ramp over the pair index between."""
+    """Angular frequency of every rotated pair (float64) and the factor on cos and sin. `scaling` = {factor} slows every pair down
+    alike; YaRN's {factor, original, fast, slow}: pairs that turn fewer than `slow` times over the original context are slowed down
+    by `factor`, those that turn more than `fast` times keep their frequency, with a linear ramp over the pair index between."""
     i = torch.arange(dims // 2, dtype=torch.float64)
-    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
+    f = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / max(dims, 1))
     if not scaling:
         return f, 1.0
+    if "original" not in scaling:
+        return f / float(scaling["factor"]), 1.0
     turn = lambda t: dims * math.log(scaling["original"] / (t * 2.0 * math.pi)) / (2.0 * math.log(base))
     lo, hi = max(math.floor(turn(scaling["fast"])), 0), min(math.ceil(turn(scaling["slow"])), dims - 1)
     ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
@@ -286,24 +331,31 @@ class LatentAttentionMixer:
         return self.out(ctx, mix, "y", torch.float32)
 
 
-class GroupedAttentionMixer:
+class GroupedAttention:
     """Grouped-query attention over pages of [keys | values]: causal, in a window or in chunks (`mask`), rotary positions on a
-    leading part of every query and key. With `diff` in its configuration a head has two softmax maps over the same values;
-    its output is a1 - lambda a2, normed without a weight and scaled by 1 - diff. Long portions in bf16 run the tensor-core
-    kernel on the pages, everything else the row kernel."""
+    leading part of every query and key. Works on columns of a projection that its owner makes. Options of a design:
+      * `q.norm`, `k.norm` among the weights: norms of queries and keys before the rotation
+      * `neighbours`: rotated pairs are (2i, 2i + 1) instead of half a width apart
+      * `softcap` in the configuration: scores become cap tanh(score / cap)
+      * `sink`: score of a key without a value that every query sees
+      * `g` among the weights: a sigmoid gate per head on its output
+      * `v_mix` = "first" | "mix": the values are kept for later layers, or become (1 - vmix) v + vmix x (the kept ones)
+      * `diff` in the configuration: a head has two softmax maps over the same values, its output is a1 - lambda a2, normed without
+        a weight and scaled by 1 - diff
+      * `scale_out`: a factor on the outputs
+    Long portions in bf16 run the tensor-core kernel on the pages, everything else the row kernel."""
 
-    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int, mask: str = "window"):
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int, mask: str = "window", neighbours: bool = False,
+                 sink: float | None = None, v_mix: str | None = None, scale_out: float = 1.0):
         H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
         diff = m.get("diff")
         maps = 1 if diff is None else 2
         if V > 512:
             raise ValueError("attention takes value dims up to 512")
-        for n, r in (("q", H * maps * D), ("k", G * maps * D), ("v", G * V)):
-            if w[n].shape[0] != r:
+        for n, r in (("q", H * maps * D), ("k", G * maps * D), ("v", G * V), ("g", H), ("q.norm", D), ("k.norm", D)):
+            if n in w and w[n].shape[0] != r:
                 raise ValueError(f"{n}: {w[n].shape[0]} rows, expected {r}")
         self.H, self.G, self.D, self.V, self.maps, self.dtype = H, G, D, V, maps, dtype
-        self.proj = FusedLinear([("q", w["q"]), ("k", w["k"]), ("v", w["v"])], dtype, device)
-        self.out = FusedLinear([("o", w["o"])], dtype, device)
         size = int((m.get("mask") or {}).get("size") or 0)
         self.span = min(size, context) if size else context         # most positions a query sees
         self.nsplit = max(1, min(64, (self.span + 31) // 32))
@@ -313,34 +365,56 @@ class GroupedAttentionMixer:
         self.tensor_core = dtype == torch.bfloat16 and float(m["scale"]) > 0
         self.cache = torch.zeros(pages, mo.PAGE, self.row, dtype=dtype, device=device)
         rot = m.get("rot") or {"dims": 0, "base": 1.0}
-        self.freq = rotary_frequencies(rot["dims"], rot["base"])[0].to(device)
-        a = self.proj.at
-        self.desc = dict(freq=self.freq.data_ptr() if rot["dims"] else None, oq=a["q"], ok=a["k"], ov=a["v"], H=H, G=G, maps=maps, D=D, V=V, R=rot["dims"],
-                         dp=dp, vp=vp, row=self.row, f32=int(dtype == torch.float32), window=size if mask == "window" else 0,
-                         chunk=size if mask == "chunk" else 0, q_ld=self.q_ld, scale=float(m["scale"]), eps=eps, post=1.0)
+        freq, mag = rotary_frequencies(rot["dims"], rot["base"], rot.get("scaling"))
+        if mag != 1.0:
+            raise ValueError("grouped attention does not scale its rotations")
+        self.const = {"freq": freq.to(device)}                     # keeps what the descriptor points at
+        self.desc = dict(H=H, G=G, maps=maps, D=D, V=V, R=rot["dims"], dp=dp, vp=vp, row=self.row, f32=int(dtype == torch.float32),
+                         window=size if mask == "window" else 0, chunk=size if mask == "chunk" else 0, q_ld=self.q_ld, scale=float(m["scale"]), eps=eps,
+                         post=scale_out, neighbours=int(neighbours), gate=-1, cap=float(m.get("softcap") or 0.0), cache=self.cache.data_ptr())
+        for n, key in (("q.norm", "q_norm"), ("k.norm", "k_norm")):
+            if n in w:
+                self.const[key] = _f32(w[n], device)
+        if sink is not None:
+            self.const["sink"] = torch.full((H * maps,), float(sink), device=device)
+        self.desc.update({n: t.data_ptr() if t.numel() else None for n, t in self.const.items()})
+        if v_mix:
+            self.desc["v_mix"] = {"first": 1, "mix": 2}[v_mix]
+            if v_mix == "mix":
+                self.desc["mix"] = float(w["vmix"])
         if maps == 2:
             l = {n: w[n].double() for n in ("lq1", "lk1", "lq2", "lk2")}
             lam = float(torch.exp((l["lq1"] * l["lk1"]).sum()) - torch.exp((l["lq2"] * l["lk2"]).sum())) + float(diff)
-            self.desc.update(lambda_=lam, head_norm=1, post=1.0 - float(diff))
+            self.desc.update(lambda_=lam, head_norm=1, post=scale_out * (1.0 - float(diff)))
 
-    def again(self):
-        o = copy.copy(self)
-        o.cache = torch.zeros_like(self.cache)
-        return o
+    @staticmethod
+    def blocks(w: dict) -> list[tuple[str, torch.Tensor]]:
+        """Matrices of the projection."""
+        return [(n, w[n]) for n in ("q", "k", "v", "g") if n in w]
+
+    def at(self, columns: dict, prefix: str = "") -> None:
+        """Where the blocks of the projection start."""
+        self.desc.update({k: columns[prefix + n] for n, k in (("q", "oq"), ("k", "ok"), ("v", "ov"), ("g", "gate")) if prefix + n in columns})
+
+    def own_memory(self) -> None:
+        self.cache = torch.zeros_like(self.cache)
+        self.desc = dict(self.desc, cache=self.cache.data_ptr())
 
     def cache_bytes(self) -> int:
         return self.cache.numel() * self.cache.element_size()
 
     def describe(self, ctx: StepContext, p: torch.Tensor, out: torch.Tensor) -> mo.PagedAttention:
-        return mo.PagedAttention(proj=p.data_ptr(), ld=p.stride(0), pos=ctx.pos.data_ptr(), slot=ctx.slot.data_ptr(), cache=self.cache.data_ptr(),
-                                 table=ctx.table.data_ptr(), table_ld=ctx.table.stride(0), out=out.data_ptr(), ldo=out.stride(0),
-                                 status=ctx.status.data_ptr(), nsplit=1, **self.desc)
+        d = mo.PagedAttention(proj=p.data_ptr(), ld=p.stride(0), pos=ctx.pos.data_ptr(), slot=ctx.slot.data_ptr(), table=ctx.table.data_ptr(),
+                              table_ld=ctx.table.stride(0), out=out.data_ptr(), ldo=out.stride(0), width=out.shape[1], status=ctx.status.data_ptr(),
+                              nsplit=1, **self.desc)
+        if d.v_mix:
+            d.v_first = ctx.ws.flat("v_first", ctx.T * self.G * self.V, torch.float32).data_ptr()
+        return d
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+    def run(self, ctx: StepContext, p: torch.Tensor, out: torch.Tensor) -> None:
+        """Head outputs of all rows into `out` [rows, columns of this layer] (a view is fine)."""
         T, ws, nq = ctx.T, ctx.ws, self.H * self.maps
-        p = self.proj(ctx, h, "proj", torch.float32)
-        mix = ws.rows("mix", T, self.out.K, self.dtype)
-        d = self.describe(ctx, p, mix)
+        d = self.describe(ctx, p, out)
         form = mo.paged_prefill_form(self.maps, self.D, self.V) if ctx.n_long and self.tensor_core else -1
         rows, nrows = (ctx.rows, ctx.n_rows) if form >= 0 or not ctx.n_long else (ctx.all_rows, T)
         if nrows:
@@ -363,6 +437,55 @@ class GroupedAttentionMixer:
                 d.part_ml = ws.flat("part_ml", n * d.nsplit * nq * 2, torch.float32).data_ptr()
                 mo.paged_rows(d, rows[a:a + n], n)
                 mo.paged_merge(d, rows[a:a + n], n)
+
+
+class GroupedAttentionMixer(GroupedAttention):
+    """Grouped-query attention between a projection and an output matrix of its own."""
+
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int, **options):
+        super().__init__(w, m, eps, dtype, device, pages, context, **options)
+        self.proj = FusedLinear(self.blocks(w), dtype, device)
+        self.out = FusedLinear([("o", w["o"])], dtype, device)
+        self.at(self.proj.at)
+
+    def again(self):
+        o = copy.copy(self)
+        o.own_memory()
+        return o
+
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+        p = self.proj(ctx, h, "proj", torch.float32)
+        mix = ctx.ws.rows("mix", ctx.T, self.out.K, self.dtype)
+        self.run(ctx, p, mix)
+        return self.out(ctx, mix, "y", torch.float32)
+
+
+class ParallelMixer:
+    """Attention and a state-space recurrence side by side on the same input: one projection in front of both and one output matrix
+    behind both, their outputs laid end to end. What scales a side is part of its last factor (attention) or its norm's weight."""
+
+    def __init__(self, left: GroupedAttention, right: StateSpaceMixer, w_left: dict, w_right: dict, dtype, device):
+        self.left, self.right, self.dtype = left, right, dtype
+        self.proj = FusedLinear([("left." + n, t) for n, t in left.blocks(w_left)] + [("right", w_right["in"])], dtype, device)
+        left.at(self.proj.at, "left.")
+        right.at(self.proj.at["right"])
+        n = left.H * left.V
+        self.split = pad_to(n, 8)
+        o = torch.zeros(w_left["o"].shape[0], self.split + right.H * right.V, dtype=w_left["o"].dtype)
+        o[:, :n], o[:, self.split:] = w_left["o"], w_right["o"]
+        self.out = FusedLinear([("o", o)], dtype, device)
+
+    def cache_bytes(self) -> int:
+        return self.left.cache_bytes()
+
+    def state_bytes(self) -> int:
+        return self.right.state_bytes()
+
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+        p = self.proj(ctx, h, "proj", torch.float32)
+        mix = ctx.ws.rows("mix", ctx.T, self.out.K, self.dtype)
+        self.left.run(ctx, p, mix[:, :self.split])
+        self.right.run(ctx, p, mix[:, self.split:])
         return self.out(ctx, mix, "y", torch.float32)
 
 
@@ -377,47 +500,55 @@ class SwiGLU:
         self.gate_up = gu.to(device)
         self.down = FusedLinear([("down", w["down"])], dtype, device, k_pad=self.ff)
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> tuple[torch.Tensor, None]:
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> dict:
         mid = ctx.ws.rows("mid", ctx.T, self.ff, self.dtype)
         mo.linear(h, self.gate_up, mid, ctx.status, swiglu=True)
-        return self.down(ctx, mid, "y", torch.float32), None
+        return {"y": self.down(ctx, mid, "y", torch.float32)}
 
 
 class RoutedExperts:
-    """Routed experts W_down max(W_up x, 0)^2. Few rows (and fp32) stream the chosen experts' weights; many rows are grouped by
-    expert and multiplied on the tensor cores, and the sum over a token's experts is left to the norm that follows: `forward`
-    returns rows and, per token, which of them to add."""
+    """Routed experts W_down max(W_up x, 0)^2, or with `gate` matrices W_down (silu(W_gate x) * (W_up x)). Few rows (and fp32) stream
+    the chosen experts' weights; many rows are grouped by expert and multiplied on the tensor cores, and the sum over a token's
+    experts is left to the norm that follows, as is what experts that return their input add: `forward` returns what
+    `sandwich_norm` takes."""
 
-    def __init__(self, router_w: torch.Tensor, up: list[torch.Tensor], down: list[torch.Tensor], router: mo.Router, dtype, device):
+    def __init__(self, router_w: torch.Tensor, up: list[torch.Tensor], down: list[torch.Tensor], router: mo.Router, dtype, device,
+                 gate: list[torch.Tensor] | None = None, correction: torch.Tensor | None = None):
         E, (ff, K), W = router.experts, up[0].shape, down[0].shape[0]
-        self.route, self.W, self.dtype = router, W, dtype
+        self.route, self.W, self.dtype, self.gated = router, W, dtype, gate is not None
         self.router = FusedLinear([("router", router_w)], dtype, device)
+        self.correction = None if correction is None else _f32(correction, device)
         self.ff, kp = pad_to(ff, 128), pad_to(K, 64)
-        self.up = torch.zeros(E, self.ff, kp, dtype=dtype, device=device)
+        self.up = torch.zeros(E, self.ff * (2 if gate else 1), kp, dtype=dtype, device=device)
         self.down = torch.zeros(E, pad_to(W, 128), self.ff, dtype=dtype, device=device)
         for e in range(E):
-            self.up[e, :ff, :K] = up[e].to(device=device, dtype=dtype)
+            self.up[e, -self.ff:][:ff, :K] = up[e].to(device=device, dtype=dtype)
+            if gate:
+                self.up[e, :ff, :K] = gate[e].to(device=device, dtype=dtype)
             self.down[e, :W, :ff] = down[e].to(device=device, dtype=dtype)
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor | None]:
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> dict:
         T, ws, r = ctx.T, ctx.ws, self.route
         R = T * r.top
         z = self.router(ctx, h, "router", torch.float32)
         ids = ws.flat("route_ids", R, torch.int32)
         hidden = ws.rows("mid", R, self.ff, self.dtype)
+        skip_w = ws.flat("route_skip", T, torch.float32) if r.identity else None
+        skip = {"skip": h, "skip_w": skip_w} if r.identity else {}
+        kw = {"correction": self.correction, "skip_w": skip_w}
         if T <= mo.ROWS_MAX or self.dtype == torch.float32:
-            mo.expert_up_rows(r, z, h, self.up, ids, hidden)
+            mo.expert_up_rows(r, z, h, self.up, ids, hidden, gated=self.gated, **kw)
             y = ws.rows("y", T, self.down.shape[1], torch.float32)
             mo.expert_down_rows(r, ids, hidden, self.down, self.W, y)
-            return y, None
+            return {"y": y, **skip}
         place = ws.rows("route_place", T, r.top, torch.int32)
         seg, scale = ws.flat("route_seg", r.experts + 1, torch.int32), ws.flat("route_scale", R, torch.float32)
         x = ws.rows("route_x", R, self.up.shape[2], self.dtype)
-        mo.expert_group(r, z, h, ids, ws.flat("route_w", R, torch.float32), seg, place, scale, x)
-        mo.grouped_linear(x, self.up, seg, hidden, ctx.status, relu2=True, row_scale=scale, scale_after=r.on_output)
+        mo.expert_group(r, z, h, ids, ws.flat("route_w", R, torch.float32), seg, place, scale, x, **kw)
+        mo.grouped_linear(x, self.up, seg, hidden, ctx.status, relu2=not self.gated, swiglu=self.gated, row_scale=scale, scale_after=r.on_output)
         y = ws.rows("expert_y", R, self.down.shape[1], torch.float32)
         mo.grouped_linear(hidden, self.down, seg, y, ctx.status)
-        return y, place
+        return {"y": y, "y_rows": place, **skip}
 
 
 @dataclass
@@ -449,6 +580,7 @@ class MixerModel:
     head: FusedLinear
     plus_one: bool = True          # norm weights are stored around zero
     embed_scale: float = 1.0
+    residual_scale: float = 1.0    # factor on every sublayer's output
 
     def windows(self) -> set[int]:
         return {L.mixer.window for L in self.layers if isinstance(L.mixer, LatentAttentionMixer)}

@@ -72,3 +72,8 @@ def _load() -> None:
     def _pezarax(path, **kw):
         from . import pezarax
         return pezarax.build_runtime(path, **kw)
+
+    @register("Zemozen", folder=True)
+    def _zemozen(path, **kw):
+        from . import zemozen
+        return zemozen.build_runtime(path, **kw)

@@ -1,5 +1,5 @@
 """Bindings of the mixer-decoder kernels: norms on an fp32 residual stream, fp32 and few-row bf16 linears, recurrent
-outer-product states (gated linear attention, mLSTM, retention), latent and grouped-query attention over a paged cache, routed
+outer-product states (gated linear attention, mLSTM, retention, state space), latent and grouped-query attention over a paged cache, routed
 experts.
 
 Every function launches on the current stream and writes into buffers its caller owns (so that a step can be captured in
@@ -15,7 +15,7 @@ import torch
 from . import EPI_BF16, EPI_F32, EPI_SWIGLU, _check
 from . import lib as _lib
 
-KIND_GLA, KIND_MLSTM, KIND_RETENTION = 0, 1, 2
+KIND_GLA, KIND_MLSTM, KIND_RETENTION, KIND_SSD = 0, 1, 2, 3
 SCORES = {"sigmoid": 0, "softmax": 1}      # router scores
 EPI_RELU2 = 5       # grouped GEMM: squared ReLU with a factor per row
 PAGE = 64           # tokens per cache page
@@ -25,17 +25,19 @@ ROWS_MAX = 8        # widest portion (and batch) of the few-row kernels
 
 class StateMixer(Structure):
     """`PkStateMixer`: columns of the fused projection, constants, state and raw outputs of one recurrent layer."""
-    _fields_ = [(n, c_void_p) for n in ("proj", "bi", "bf", "a2", "a2b", "S", "N", "Ms", "o", "nq", "m", "freq", "pw")] + \
-               [(n, c_int) for n in ("kind", "ld", "oq", "ok", "ov", "og", "oi", "of", "oa", "H", "D", "V", "rank", "rot")] + \
+    _fields_ = [(n, c_void_p) for n in ("proj", "bi", "bf", "a2", "a2b", "S", "N", "Ms", "o", "nq", "m", "freq", "pw", "cw", "cb", "dtb", "A", "skip",
+                                        "Cs")] + \
+               [(n, c_int) for n in ("kind", "ld", "oq", "ok", "ov", "og", "oi", "of", "oa", "H", "D", "V", "rank", "rot", "groups", "taps", "odt")] + \
                [(n, c_float) for n in ("qscale", "cap", "inv_tau")]
 
 
 class PagedAttention(Structure):
     """`PkPagedAttention`: one grouped-query attention layer over one batch."""
-    _fields_ = [(n, c_void_p) for n in ("proj", "freq", "pos", "slot", "cache", "table", "qx", "qf", "part_o", "part_ml", "out", "status")] + \
+    _fields_ = [(n, c_void_p) for n in ("proj", "freq", "pos", "slot", "cache", "table", "qx", "qf", "part_o", "part_ml", "out", "status", "q_norm", "k_norm",
+                                        "sink", "v_first")] + \
                [(n, c_int) for n in ("ld", "oq", "ok", "ov", "H", "G", "maps", "D", "V", "R", "dp", "vp", "row", "table_ld", "f32", "window", "chunk", "q_ld",
-                                     "ldo", "nsplit", "head_norm")] + \
-               [(n, c_float) for n in ("scale", "lambda_", "post", "eps")]
+                                     "ldo", "nsplit", "head_norm", "neighbours", "v_mix", "gate", "width")] + \
+               [(n, c_float) for n in ("scale", "lambda_", "post", "eps", "cap", "mix")]
 
 
 _sms: dict[int, int] = {}
@@ -51,12 +53,12 @@ def sm_count() -> int:
 # argument kinds of the launchers, the stream excepted: p pointer, i int, f float
 _SIGNATURES = {
     "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
-    "pk_sandwich_norm": "pppifipipippiipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
-    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii",
+    "pk_sandwich_norm": "pppifipipifpiippp" "iipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
+    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii",
     "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipi",
     "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipi", "pk_latent_prefill": "pipipippiiiiifppip",
     "pk_paged_prep": "pi", "pk_paged_rows": "ppi", "pk_paged_merge": "ppi", "pk_paged_prefill": "piipip",
-    "pk_expert_up_rows": "piiiiifipiipiiippii", "pk_expert_down_rows": "pipiipiiiipii", "pk_expert_group": "piiiiifipppppp" "iip",
+    "pk_expert_up_rows": "piiiiifpipiipiipiiippii", "pk_expert_down_rows": "piipiipiiiipii", "pk_expert_group": "piiiiifpipipppppp" "iip",
     "pk_gemm_bf16_grouped_scaled": "pippiiiiipipipi",
 }
 _bound: dict[tuple[int, str], object] = {}
@@ -100,13 +102,16 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Te
 
 def sandwich_norm(x: torch.Tensor, *, eps: float, out: torch.Tensor | None = None, w_pre: torch.Tensor | None = None,
                   tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0, embed_add: bool = False,
-                  y: torch.Tensor | None = None, y_rows: torch.Tensor | None = None, w_post: torch.Tensor | None = None,
-                  rows: torch.Tensor | None = None, count: int | None = None, plus_one: bool = True) -> None:
+                  y: torch.Tensor | None = None, y_rows: torch.Tensor | None = None, y_scale: float = 1.0, skip: torch.Tensor | None = None,
+                  skip_w: torch.Tensor | None = None, w_post: torch.Tensor | None = None, rows: torch.Tensor | None = None, count: int | None = None,
+                  plus_one: bool = True) -> None:
     """One step of the residual stream x [rows, width] fp32 (see sandwich_norm.cu). `rows`/`count`: norm only these rows; `y_rows`
-    [rows, n]: a row's y is the sum of these n rows of `y`; `embed_add`: the scaled embedding row is added instead of starting x."""
+    [rows, n]: a row's y is the sum of these n rows of `y` (negative: none); `skip_w` [rows] x the row of `skip` is part of y; y is
+    multiplied by `y_scale`; `embed_add`: the scaled embedding row is added instead of starting x."""
     M = (x.shape[0] if rows is None else rows.shape[0]) if count is None else count
     _call("pk_sandwich_norm", x, tokens, embed, 0 if embed is None else embed.shape[0], embed_scale, int(embed_add), y, 0 if y is None else y.stride(0),
-          y_rows, 0 if y_rows is None else y_rows.shape[1], w_post, rows, M, x.shape[1], w_pre, int(plus_one), eps, out,
+          y_rows, 0 if y_rows is None else y_rows.shape[1], y_scale, skip, 0 if skip is None else skip.stride(0),
+          int(skip is not None and skip.dtype == torch.float32), skip_w, w_post, rows, M, x.shape[1], w_pre, int(plus_one), eps, out,
           0 if out is None else out.stride(0), int(out is not None and out.dtype == torch.float32))
 
 
@@ -142,6 +147,12 @@ def state_chunks(d: StateMixer, seqs: torch.Tensor, nseq: int, chunks: torch.Ten
 def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
     """Head norm + output gate of `rows` rows; norm_w [H * V], [V] when `per_head`, or None."""
     _call("pk_state_out", byref(d), norm_w, int(per_head), eps, last_slot, rows, out, out.stride(0), int(out.dtype == torch.float32))
+
+
+def ssd_out(d: StateMixer, norm_w: torch.Tensor, parts: int, eps: float, last_slot: torch.Tensor, ahead: torch.Tensor, pos: torch.Tensor, rows: int,
+            out: torch.Tensor) -> None:
+    """Gate and norm of a state-space layer, the line of its convolution; `out` [rows, columns of this layer] (a view is fine)."""
+    _call("pk_ssd_out", byref(d), norm_w, parts, eps, last_slot, ahead, pos, rows, out, out.stride(0), out.shape[1], int(out.dtype == torch.float32))
 
 
 def latent_prep(proj: torch.Tensor, oq: int, oc: int, H: int, D: int, R: int, K: int, c_norm: torch.Tensor, eps: float, freq: torch.Tensor,
@@ -213,34 +224,43 @@ class Router:
     renorm: bool = False        # chosen weights divided by their sum
     scale: float = 1.0
     on_output: bool = False     # the weight multiplies an expert's output instead of its input
+    identity: int = 0           # experts behind the others that return their input
 
-    def args(self) -> tuple:
-        return self.experts, self.top, SCORES[self.score], int(self.renorm), self.scale
+    @property
+    def outputs(self) -> int:
+        return self.experts + self.identity
+
+    def args(self, correction: torch.Tensor | None, skip_w: torch.Tensor | None) -> tuple:
+        return self.outputs, self.top, SCORES[self.score], int(self.renorm), self.scale, correction, self.identity, skip_w
 
 
-def expert_up_rows(r: Router, logits: torch.Tensor, x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor) -> None:
-    """hidden [T * top, N] = squared ReLU of the chosen experts' up products; w [experts, N, K]; ids [T * top] out."""
+def expert_up_rows(r: Router, logits: torch.Tensor, x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor, *, gated: bool = False,
+                   correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None) -> None:
+    """hidden [T * top, N] = squared ReLU of the chosen experts' up products, w [experts, N, K]; `gated`: silu(gate) * up, w [experts, N
+    gate rows and N up rows, K]. ids [T * top] out; `correction` [outputs] counts for the choice; skip_w [T] out (identities)."""
     E, N, K = w.shape
-    _call("pk_expert_up_rows", logits, logits.stride(0), *r.args(), int(r.on_output), x, x.stride(0), x.shape[0], w, N, K,
-          int(w.dtype == torch.float32), ids, hidden, hidden.stride(0), sm_count())
+    _call("pk_expert_up_rows", logits, logits.stride(0), *r.args(correction, skip_w), int(r.on_output), int(gated), x, x.stride(0), x.shape[0], w,
+          N // 2 if gated else N, K, int(w.dtype == torch.float32), ids, hidden, hidden.stride(0), sm_count())
 
 
 def expert_down_rows(r: Router, ids: torch.Tensor, hidden: torch.Tensor, w: torch.Tensor, n: int, y: torch.Tensor) -> None:
     """y [T, n] fp32 = sum over a token's experts of w[expert, :n] . hidden; w [experts, rows, K]."""
     E, rows, K = w.shape
-    _call("pk_expert_down_rows", ids, r.top, hidden, hidden.stride(0), y.shape[0], w, n, rows, K, int(w.dtype == torch.float32), y, y.stride(0), sm_count())
+    _call("pk_expert_down_rows", ids, r.top, r.experts, hidden, hidden.stride(0), y.shape[0], w, n, rows, K, int(w.dtype == torch.float32), y, y.stride(0),
+          sm_count())
 
 
 def expert_group(r: Router, logits: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, seg: torch.Tensor, place: torch.Tensor,
-                 row_scale: torch.Tensor, rows: torch.Tensor) -> None:
+                 row_scale: torch.Tensor, rows: torch.Tensor, *, correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None) -> None:
     """Routes of the tokens grouped by expert, token rows gathered in that order (rows [T * top, K])."""
-    _call("pk_expert_group", logits, logits.stride(0), *r.args(), x.shape[0], ids, weights, seg, place, row_scale, x, x.stride(0), rows.shape[1], rows)
+    _call("pk_expert_group", logits, logits.stride(0), *r.args(correction, skip_w), x.shape[0], ids, weights, seg, place, row_scale, x, x.stride(0),
+          rows.shape[1], rows)
 
 
 def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg: torch.Tensor, out: torch.Tensor, status: torch.Tensor, *, relu2: bool = False,
-                   row_scale: torch.Tensor | None = None, scale_after: bool = False) -> None:
+                   swiglu: bool = False, row_scale: torch.Tensor | None = None, scale_after: bool = False) -> None:
     """out rows of group g = x rows . w[g]^T on the tensor cores (x, w bf16; w [groups, N, K], N a multiple of 128, K of 64); fp32 out,
-    or bf16 squared ReLU with a factor per row."""
+    or bf16 squared ReLU, or SwiGLU (N / 2 gate rows, then N / 2 up rows) with a factor per row."""
     G, N, K = w.shape
-    _call("pk_gemm_bf16_grouped_scaled", x, x.stride(0), w, seg, G, x.shape[0], N, K, EPI_RELU2 if relu2 else EPI_F32, out, out.stride(0), row_scale,
+    _call("pk_gemm_bf16_grouped_scaled", x, x.stride(0), w, seg, G, x.shape[0], N, K, EPI_RELU2 if relu2 else EPI_SWIGLU if swiglu else EPI_F32, out, out.stride(0), row_scale,
           int(scale_after), status, sm_count())

@@ -199,7 +199,7 @@ class _Batch:
         slots, pages = (T if singles else 1), -(-context // 64)
         table = dev(range(slots * pages)).view(slots, pages)
         self.pages, self.slots = slots * pages, slots
-        self.ctx = StepContext(T, dev([0] * T), dev(p["pos"]), dev(p["slot"]), dev(p["last"]), table, Workspace("cuda"),
+        self.ctx = StepContext(T, dev([0] * T), dev(p["pos"]), dev(p["slot"]), dev(p["last"]), dev(p["ahead"]), table, Workspace("cuda"),
                                torch.zeros(1, dtype=torch.int32, device="cuda"), short=dev(p["short"]), n_short=len(p["short"]), rows=dev(p["rows"]),
                                n_rows=len(p["rows"]), all_rows=dev(range(T)), long=dev(p["long"]), n_long=len(p["long"]), chunks=dev(p["chunks"]),
                                chunk0=dev(p["chunk0"]), n_chunks=len(p["chunks"]), tiles=dev(p["tiles"]), n_tiles=len(p["tiles"]),
@@ -377,7 +377,7 @@ def _experts(W: int, E: int, top: int, ff: int, T: int, sets: int):
     """Routed experts of `sets` layers (together larger than L2): {kernel: (call over all layers, flops, bytes)} per layer."""
     from ..models import mixer_layers as ml
     from ..ops import mixer_ops as mo
-    ctx = ml.StepContext(T, *[None] * 5, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
+    ctx = ml.StepContext(T, *[None] * 6, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
     g = torch.Generator(device="cuda").manual_seed(0)
     r = lambda *s: (torch.randn(*s, generator=g, device="cuda") * s[-1] ** -0.5).to(torch.bfloat16)
     layers = [ml.RoutedExperts(r(E, W), [r(ff, W) for _ in range(E)], [r(W, ff) for _ in range(E)], mo.Router(E, top), torch.bfloat16, "cuda") for _ in range(sets)]

@@ -92,10 +92,11 @@ def test_routed_experts(T, E, top, W, ff, kw, dtype):
     z[:, E:] = 50.0                                                   # padding columns are nobody's experts
     zc = z.cuda()
     m.router = lambda ctx, h, name, dt: zc
-    ctx = ml.StepContext(T, *[None] * 5, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
+    ctx = ml.StepContext(T, *[None] * 6, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
     h = torch.zeros(T, m.up.shape[2], device="cuda", dtype=dtype)
     h[:, :W] = x.to(dtype)
-    y, rows = m.forward(ctx, h)
+    out = m.forward(ctx, h)
+    y, rows = out["y"], out.get("y_rows")
     got = (y if rows is None else y[rows.long()].sum(1))[:, :W].double().cpu()
     want = plain_experts(z[:, :E].double(), x.double(), up.to(dtype).double(), down.to(dtype).double(), top, **kw)
     assert ((got - want).norm() / want.norm()).item() < (1e-5 if dtype == F32 else 8e-3)
