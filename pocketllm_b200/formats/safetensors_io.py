@@ -49,7 +49,7 @@ def write_file(path: str | os.PathLike, tensors: Mapping[str, torch.Tensor], met
         f.write(blob)
         for name in order:
             t = tensors[name].detach().contiguous().cpu()
-            f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() else b"")
+            f.write(t.reshape(-1).view(torch.uint8).numpy().tobytes() if t.numel() else b"")
 
 
 def write_sharded(directory: str | os.PathLike, tensors: Mapping[str, torch.Tensor], max_shard_bytes: int = 4 << 30,

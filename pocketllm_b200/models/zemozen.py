@@ -160,7 +160,7 @@ def random_tensors(c: ZemozenConfig, seed: int = 0, device: str = "cpu", gain: f
     out = {}
     for name, shape in tensor_plan(c).items():
         base = name.rsplit(".", 1)[-1]
-        z = torch.randn(*shape, generator=g, device=device)
+        z = torch.randn(shape, generator=g, device=device)
         if base == "vmix":
             t = 0.4 + 0.1 * z
         elif base == "A_log":
