@@ -1,10 +1,10 @@
 """Throughput of mixer decoders at sizes that resemble a real model's layers, beside the closest other model at equal size
 (Gidisun: the Qwen hybrid, DeltaNet + GQA with the same width, feed-forward, depth and vocabulary; Pezarax: Gidisun with the
-same width, heads, depth and as many weights per token in its feed-forward), and the time of each design's kernels beside the
-like kernels of the other families.
+same width, heads, depth and as many weights per token in its feed-forward; Zemozen: Pezarax with the same width, depth, number
+of experts and weights per expert), and the time of each design's kernels beside the like kernels of the other families.
 
-    python -m pocketllm_b200.utils.bench_mixers --kernels [gidisun|pezarax]
-    python bench.py --model gidisun|pezarax [--size 2k|4k]
+    python -m pocketllm_b200.utils.bench_mixers --kernels [gidisun|pezarax|zemozen]
+    python bench.py --model gidisun|pezarax|zemozen [--size 2k|4k]
 
 Random weights; every weight set is larger than L2. Device times by CUDA events.
 """
@@ -17,6 +17,7 @@ import torch
 
 from ..models import gidisun as gd
 from ..models import pezarax as pz
+from ..models import zemozen as zm
 
 VOCAB = 32000
 #            width  ff     mLSTM (heads, dim, vdim)  GLA              latent (heads, dim, rot, vdim, rank, window)
@@ -42,6 +43,23 @@ def pezarax_config(size: str) -> pz.PezaraxConfig:
                                        "layers": [{"type": t, "mixer": mix[t], "mlp": mlp} for t in PEZARAX_PATTERN]})
 
 
+#                  width  both attentions (heads, kv heads, dim, vdim, window)  state space (heads, vdim, state, groups)  experts (number, identities, top, ff)
+ZEMOZEN_SIZES = {"2k": (2048, (16, 4, 128, 128, 1024), (32, 64, 128, 4), (32, 4, 2, 1024)),
+                 "4k": (4096, (32, 8, 128, 128, 1024), (64, 64, 128, 8), (32, 4, 2, 2048))}
+ZEMOZEN_PATTERN = ("parallel", "parallel", "attention", "parallel", "parallel", "parallel", "attention", "parallel")
+
+
+def zemozen_config(size: str) -> zm.ZemozenConfig:
+    W, a, s, e = ZEMOZEN_SIZES[size]
+    att = {"heads": a[0], "kv_heads": a[1], "dim": a[2], "vdim": a[3], "scale": a[2] ** -0.5, "mask": {"size": a[4]}, "rot": {"base": 5e5, "dims": a[2]}}
+    mix = {"attention": att | {"v_mix": True, "rot": att["rot"] | {"scaling": {"factor": 8.0}}},
+           "parallel": {"left": att | {"softcap": 30.0}, "left_scale": 0.8, "right_scale": 0.9,
+                        "right": {"heads": s[0], "vdim": s[1], "state": s[2], "groups": s[3], "conv": 4, "norm_groups": s[3]}}}
+    mlp = {"kind": "moe", "expert": {"ff": e[3]}, "router": {"experts": e[0], "identity": e[1], "top": e[2]}}
+    return zm.ZemozenConfig.from_dict({"architecture": zm.ARCH, "vocab": VOCAB, "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": 8.0},
+                                       "residual_mult": 0.7, "layers": [{"type": t, "mixer": mix[t], "mlp": mlp} for t in ZEMOZEN_PATTERN]})
+
+
 def config(size: str, ff: int | None = None) -> gd.GidisunConfig:
     W, dense_ff, m, g, a = SIZES[size]
     ff = ff or dense_ff
@@ -57,7 +75,7 @@ def config(size: str, ff: int | None = None) -> gd.GidisunConfig:
 def build(design: str, size: str, batch: int, context: int, ff: int | None = None):
     """(runtime with random weights, bytes of weights that one decoded token streams)."""
     from ..runtime.mixer_runtime import MixerRuntime
-    mod, c = (gd, config(size, ff)) if design == "gidisun" else (pz, pezarax_config(size))
+    mod, c = {"gidisun": lambda: (gd, config(size, ff)), "pezarax": lambda: (pz, pezarax_config(size)), "zemozen": lambda: (zm, zemozen_config(size))}[design]()
     t = mod.random_tensors(c, 0, device="cuda")
     pages = batch * (-(-context // 64))
     streamed = 0.0
@@ -65,7 +83,7 @@ def build(design: str, size: str, batch: int, context: int, ff: int | None = Non
         share = 1.0
         if ".mlp.e" in n:
             L = c.layers[int(n[1:n.index(".")])]
-            share = L.top / L.experts
+            share = L.top / (L.experts + getattr(L, "identity", 0))
         streamed += v.numel() * 2 * share if n != "embed" else 0.0
     rt = MixerRuntime(mod.build_model(c, t, slots=batch, pages=pages), max_requests=batch, pages=pages)
     return rt, streamed
@@ -128,6 +146,15 @@ def closest_to_pezarax(size: str, prompts, n: int, d: int, warmup: int, batch: i
     rt, streamed = build("gidisun", size, batch, n + d + 64, ff=2 * top * ff // 3)
     r, k = requests(rt, prompts, n, d, warmup, batch), len(prompts) - warmup
     return {"model": "Gidisun (mLSTM, GLA, latent attention, SwiGLU; bf16 weights)", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
+            "decode_tok_s": round(k * d / r["decode_ms"] * 1e3, 1), "decode_tok_s_batch": round(k * d * batch / r["batch_ms"] * 1e3, 1),
+            "weight_gb_per_token": round(streamed / 1e9, 2), "decode_weight_gbs": round(streamed * k * d / r["decode_ms"] / 1e6, 1)}
+
+
+def closest_to_zemozen(size: str, prompts, n: int, d: int, warmup: int, batch: int) -> dict:
+    """Pezarax with as many experts of as many weights."""
+    rt, streamed = build("pezarax", size, batch, n + d + 64)
+    r, k = requests(rt, prompts, n, d, warmup, batch), len(prompts) - warmup
+    return {"model": "Pezarax (retention, differential attention, routed experts; bf16 weights)", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
             "decode_tok_s": round(k * d / r["decode_ms"] * 1e3, 1), "decode_tok_s_batch": round(k * d * batch / r["batch_ms"] * 1e3, 1),
             "weight_gb_per_token": round(streamed / 1e9, 2), "decode_weight_gbs": round(streamed * k * d / r["decode_ms"] / 1e6, 1)}
 
@@ -240,6 +267,30 @@ def _state(kind: str, dims, T: int, singles: bool):
     call.keep = (m, b, p)
     flops = 2.0 * T * H * (2 * D * V + 64 * D + 64 * V)
     return call, flops, T * H * D * V * 8.0 if singles else 0.0
+
+
+def _state_space(dims, T: int, singles: bool):
+    """The state-space recurrence of one layer with its convolution, gate and norm: (call, flops, bytes of states)."""
+    from ..models import mixer_layers as ml
+    from ..ops import mixer_ops as mo
+    H, V, N, G = dims
+    W, inner = 1024, dims[0] * dims[1]
+    ch = inner + 2 * G * N
+    b = _Batch(T, 4096, 64, singles=singles)
+    g = torch.Generator().manual_seed(0)
+    r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
+    w = {"in": r(2 * inner + 2 * G * N + H, W), "conv": r(ch, 4), "conv.b": torch.zeros(ch), "dt_bias": torch.full((H,), -3.0), "A_log": torch.zeros(H),
+         "D": torch.ones(H), "norm": torch.ones(inner)}
+    m = ml.StateSpaceMixer(w, {"heads": H, "vdim": V, "state": N, "groups": G, "conv": 4, "norm_groups": G}, 1e-5, "cuda", b.slots)
+    m.at(0)
+    p = ml.FusedLinear([("in", w["in"])], torch.bfloat16, "cuda")(b.ctx, torch.randn(T, W, device="cuda").to(torch.bfloat16), "proj", torch.float32)
+    mix = b.ctx.ws.rows("mix", T, inner, torch.bfloat16)
+
+    def call():
+        m.run(b.ctx, p, mix)
+    call.keep = (m, b, p, mix)
+    flops = 2.0 * T * (H * (2 * N * V + 32 * V) + G * 64 * N)       # states twice, weights of a chunk's earlier tokens (half of 64), products of a group
+    return call, flops, T * H * N * V * 8.0 if singles else 0.0
 
 
 def _latent(dims, T: int, start: int, singles: bool):
@@ -358,6 +409,34 @@ def _paged(dims, T: int, start: int, singles: bool):
     d = m.describe(ctx, p, mix)
     see = lambda q: q + 1 - (q // chunk * chunk if chunk else 0)
     span = T * see(start) if singles else sum(see(start + i) for i in range(T))
+    return _paged_calls(m, b, p, mix, d, T, span, singles)
+
+
+def _windowed(dims, T: int, start: int, singles: bool, parallel: bool):
+    """The same for one of Zemozen's attentions: mixed values and a gate per head, or capped scores and a sink."""
+    from ..models import mixer_layers as ml
+    H, G, D, V, window = dims
+    W = 1024
+    b = _Batch(T, start, start + T, singles=singles)
+    g = torch.Generator().manual_seed(0)
+    r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
+    w = {"q": r(H * D, W), "k": r(G * D, W), "v": r(G * V, W), "o": r(W, H * V), "q.norm": torch.ones(D), "k.norm": torch.ones(D)}
+    c = {"heads": H, "kv_heads": G, "dim": D, "vdim": V, "scale": D ** -0.5, "mask": {"size": window} if window else None, "rot": {"base": 1e4, "dims": D}}
+    if parallel:
+        m = ml.GroupedAttentionMixer(w, c | {"softcap": 30.0}, 1e-5, torch.bfloat16, "cuda", b.pages, start + T, neighbours=True, sink=0.0)
+    else:
+        w.update(g=r(H, W), vmix=torch.tensor(0.4))
+        m = ml.GroupedAttentionMixer(w, c, 1e-5, torch.bfloat16, "cuda", b.pages, start + T, v_mix="mix")
+    m.cache.normal_()
+    p = m.proj(b.ctx, torch.randn(T, m.proj.K, device="cuda").to(torch.bfloat16), "proj", torch.float32)
+    mix = b.ctx.ws.rows("mix", T, m.out.K, torch.bfloat16)
+    see = lambda q: min(q + 1, window or 1 << 30)
+    return _paged_calls(m, b, p, mix, m.describe(b.ctx, p, mix), T, T * see(start) if singles else sum(see(start + i) for i in range(T)), singles)
+
+
+def _paged_calls(m, b, p, mix, d, T: int, span: int, singles: bool) -> dict:
+    from ..ops import mixer_ops as mo
+    ctx, ws, nq, D, V = b.ctx, b.ctx.ws, m.H * m.maps, m.D, m.V
     keep = (m, b, p, mix)
     flops = 2.0 * span * nq * (D + V)
     if singles:
@@ -373,34 +452,49 @@ def _paged(dims, T: int, start: int, singles: bool):
             "attention": (lambda k=(keep, qf): mo.paged_prefill(d, T, b.pages, ctx.tiles, ctx.n_tiles, ctx.long), flops, 0)}
 
 
-def _experts(W: int, E: int, top: int, ff: int, T: int, sets: int):
-    """Routed experts of `sets` layers (together larger than L2): {kernel: (call over all layers, flops, bytes)} per layer."""
+def _experts(W: int, E: int, top: int, ff: int, T: int, sets: int, identity: int | None = None):
+    """Routed experts of `sets` layers (together larger than L2): {kernel: (call over all layers, flops, bytes)} per layer.
+    `identity`: gated experts, behind them as many identities."""
     from ..models import mixer_layers as ml
     from ..ops import mixer_ops as mo
     ctx = ml.StepContext(T, *[None] * 6, ml.Workspace("cuda"), torch.zeros(1, dtype=torch.int32, device="cuda"))
     g = torch.Generator(device="cuda").manual_seed(0)
     r = lambda *s: (torch.randn(*s, generator=g, device="cuda") * s[-1] ** -0.5).to(torch.bfloat16)
-    layers = [ml.RoutedExperts(r(E, W), [r(ff, W) for _ in range(E)], [r(W, ff) for _ in range(E)], mo.Router(E, top), torch.bfloat16, "cuda") for _ in range(sets)]
+    gated = identity is not None
+    rows = lambda: [r(ff, W) for _ in range(E)]
+    if gated:
+        router = mo.Router(E, top, score="softmax", renorm=True, on_output=True, identity=identity)
+        new = lambda: ml.RoutedExperts(r(router.outputs, W), rows(), [r(W, ff) for _ in range(E)], router, torch.bfloat16, "cuda", gate=rows(),
+                                       correction=torch.zeros(router.outputs))
+    else:
+        new = lambda: ml.RoutedExperts(r(E, W), rows(), [r(W, ff) for _ in range(E)], mo.Router(E, top), torch.bfloat16, "cuda")
+    layers = [new() for _ in range(sets)]
     h = torch.randn(T, layers[0].up.shape[2], generator=g, device="cuda").to(torch.bfloat16)
     R, ws = T * top, ctx.ws
     z = [m.router(ctx, h, f"router{i}", torch.float32) for i, m in enumerate(layers)]
-    used = E * (1.0 - (1.0 - top / E) ** T)                            # experts that are expected to be used
-    flops, nbytes = 2.0 * R * W * ff, used * W * ff * 2.0
+    n = E + (identity or 0)
+    used = E * (1.0 - (1.0 - top / n) ** T)                            # experts that are expected to be used
+    flops, nbytes = 2.0 * R * E / n * W * ff, used * W * ff * 2.0      # of the down product
+    up = 2 if gated else 1
+    kw = lambda m: {"correction": m.correction, "skip_w": ws.flat("skip", T, torch.float32)} if gated else {}
     ids, hidden = ws.flat("ids", R, torch.int32), ws.rows("hid", R, layers[0].ff, torch.bfloat16)
     keep = (layers, z)
-    out = {"whole layer with router": (lambda k=keep: [m.forward(ctx, h) for m in layers], 2 * flops, 2 * nbytes)}
+    out = {"whole layer with router": (lambda k=keep: [m.forward(ctx, h) for m in layers], (up + 1) * flops, (up + 1) * nbytes)}
     if T <= mo.ROWS_MAX:
         y = ws.rows("yy", T, layers[0].down.shape[1], torch.float32)
-        out["up rows (choice included)"] = (lambda: [mo.expert_up_rows(m.route, q, h, m.up, ids, hidden) for m, q in zip(layers, z)], flops, nbytes)
+        out["up rows (choice included)"] = (lambda: [mo.expert_up_rows(m.route, q, h, m.up, ids, hidden, gated=gated, **kw(m)) for m, q in zip(layers, z)],
+                                           up * flops, up * nbytes)
         out["down rows"] = (lambda: [mo.expert_down_rows(m.route, ids, hidden, m.down, W, y) for m in layers], flops, nbytes)
         return out
     place, seg, sc = ws.rows("pl", T, top, torch.int32), ws.flat("sg", E + 1, torch.int32), ws.flat("sc", R, torch.float32)
     x, y, rw = ws.rows("rx", R, h.shape[1], torch.bfloat16), ws.rows("yy", R, layers[0].down.shape[1], torch.float32), ws.flat("rw", R, torch.float32)
-    group = lambda m, q: mo.expert_group(m.route, q, h, ids, rw, seg, place, sc, x)
+    group = lambda m, q: mo.expert_group(m.route, q, h, ids, rw, seg, place, sc, x, **kw(m))
     group(layers[0], z[0])
     out["choice, grouping, gather"] = (lambda: [group(m, q) for m, q in zip(layers, z)], 0, T * W * 2.0 + R * W * 2.0)
     group(layers[0], z[0])
-    out["up (grouped GEMM, squared ReLU)"] = (lambda: [mo.grouped_linear(x, m.up, seg, hidden, ctx.status, relu2=True, row_scale=sc) for m in layers], flops, nbytes)
+    out["up (grouped GEMM, SwiGLU)" if gated else "up (grouped GEMM, squared ReLU)"] = (
+        lambda: [mo.grouped_linear(x, m.up, seg, hidden, ctx.status, relu2=not gated, swiglu=gated, row_scale=sc, scale_after=gated) for m in layers],
+        up * flops, up * nbytes)
     out["down (grouped GEMM, fp32 out)"] = (lambda: [mo.grouped_linear(hidden, m.down, seg, y, ctx.status) for m in layers], flops, nbytes)
     return out
 
@@ -472,13 +566,57 @@ def pezarax_kernels() -> None:
         show("like kernel: two norms + residual add", _roof(timed(lambda: mo.sandwich_norm(x, y=y, w_post=w, w_pre=w, out=o, eps=1e-5)), 0, T * 4096 * 14.0), T=T)
 
 
+def zemozen_kernels() -> None:
+    """The new kernels and variants, each followed by the like kernel of Pezarax in the same run."""
+    from ..ops import mixer_ops as mo
+    show = lambda name, d, **kw: print(json.dumps({"kernel": name, **kw, **d}), flush=True)
+    space, ret = (64, 64, 128, 8), (16, 128, 256)
+    for T in (512, 2048):
+        f, fl, _ = _state_space(space, T, False)
+        show("state space chunk form (convolution, gate, norm included)", _roof(timed(f), fl), T=T, dims=space)
+        f, fl, _ = _state("retention", ret, T, False)
+        show("like kernel: retention chunk form + head norm", _roof(timed(f), fl), T=T, dims=ret)
+    for B in (1, 8):
+        f, _, nb = _state_space(space, B, True)
+        show("state space rows form (convolution, gate, norm included)", _roof(timed(f), 0, nb), B=B, dims=space)
+        f, _, nb = _state("retention", ret, B, True)
+        show("like kernel: retention rows form + head norm", _roof(timed(f), 0, nb), B=B, dims=ret)
+    for T in (512, 2048):
+        for window in (0, 1024):
+            for par in (False, True):
+                for k, (f, fl, nb) in _windowed((32, 8, 128, 128, window), T, 8192 - T, False, par).items():
+                    show(("capped" if par else "gated") + " prefill: " + k, _roof(timed(f), fl, nb), T=T, context=8192, window=window)
+            for k, (f, fl, nb) in _paged((32, 8, 64, 128, window), T, 8192 - T, False).items():
+                show("like kernel: differential prefill: " + k, _roof(timed(f), fl, nb), T=T, context=8192, chunk=window)
+    for B in (1, 8):
+        for window in (1024, 0):
+            for par in (False, True):
+                for k, (f, fl, nb) in _windowed((32, 8, 128, 128, window), B, 8191, True, par).items():
+                    show(("capped" if par else "gated") + " rows: " + k, _roof(timed(f), fl, nb), B=B, context=8192, window=window)
+            for k, (f, fl, nb) in _paged((32, 8, 64, 128, window), B, 8191, True).items():
+                show("like kernel: differential rows: " + k, _roof(timed(f), fl, nb), B=B, context=8192, chunk=window)
+    W, E, top = 4096, 32, 2
+    for T in (1, 8, 64, 512, 2048):
+        for name, ff, ident in (("gated experts: ", 2048, 4), ("like kernel: experts: ", 3072, None)):
+            for k, (f, fl, nb) in _experts(W, E, top, ff, T, 2, ident).items():
+                show(name + k, _roof(timed(f, reps=8) / 2, fl, nb), T=T)
+    for T in (1, 2048):
+        x, y, w = torch.randn(T, 4096, device="cuda"), torch.randn(2 * T, 4096, device="cuda"), torch.randn(4096, device="cuda")
+        place = torch.randperm(2 * T, device="cuda").to(torch.int32).view(T, 2)
+        o, sw = torch.empty(T, 4096, device="cuda", dtype=torch.bfloat16), torch.rand(T, device="cuda")
+        f = lambda: mo.sandwich_norm(x, y=y, y_rows=place, y_scale=0.7, skip=o, skip_w=sw, w_pre=w, out=o, eps=1e-5)
+        show("expert rows + identity + residual add + norm", _roof(timed(f), 0, T * 4096 * 20.0), T=T)
+        show("like kernel: sum of two expert rows + residual add + norm", _roof(timed(lambda: mo.sandwich_norm(x, y=y, y_rows=place, w_pre=w, out=o, eps=1e-5)), 0,
+                                                                               T * 4096 * 18.0), T=T)
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernels", nargs="?", const="gidisun", choices=["gidisun", "pezarax"], help="time the design's kernels beside the like kernels")
+    ap.add_argument("--kernels", nargs="?", const="gidisun", choices=["gidisun", "pezarax", "zemozen"], help="time the design's kernels beside the like kernels")
     ap.add_argument("--size", default="2k", choices=sorted(SIZES))
     args = ap.parse_args()
     if args.kernels:
-        {"gidisun": kernels, "pezarax": pezarax_kernels}[args.kernels]()
+        {"gidisun": kernels, "pezarax": pezarax_kernels, "zemozen": zemozen_kernels}[args.kernels]()
     else:
         print(json.dumps(closest_model(args.size, 512, 64, 3)))
     return 0
