@@ -6,7 +6,7 @@
 // m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1; retention: a = const, b = 1;
 // state space: k = B, q = C, v = x, a = exp(A dt), b = dt, dt = softplus(z + bias), B and C shared by a group of heads, and
 // o_t gets D x_t). The state-space inputs x, B and C pass a short causal convolution per channel and SiLU first; its last
-// inputs are part of a request's state, [slot][taps - 1][channel].
+// inputs are part of a request's state, a ring [slot][position modulo (taps - 1)][channel].
 // Everything here is fp32: gates, decays, states and products.
 //
 // State lives in slots [slot][head][key][value] so that requests of one batch keep theirs anywhere; a portion that starts
@@ -64,7 +64,7 @@ struct Mixer {
   const float* dtb;    // [H]
   const float* A;      // [H] negative
   const float* skip;   // [H]
-  float* Cs;           // [slots, taps - 1, channels] last inputs of the convolution
+  float* Cs;           // [slots, taps - 1, channels] last inputs of the convolution, by position modulo (taps - 1)
   int groups, taps, odt;
   __device__ __host__ int channels() const { return H * V + 2 * groups * D; }
   // state
@@ -82,14 +82,25 @@ struct Raw {
 
 // State space: input of the convolution `lag` tokens before the one at `row`, which is token `t` of its portion, at position pos.
 __device__ __forceinline__ float conv_input(const Mixer& mx, int slot, int row, int t, int pos, int lag, int ch) {
-  if (lag <= t) return mx.proj[(size_t)(row - lag) * mx.ld + mx.ov + ch];
   if (lag > pos) return 0.f;
-  return mx.Cs[((size_t)slot * (mx.taps - 1) + mx.taps - 1 - (lag - t)) * mx.channels() + ch];
+  const float* ring = mx.Cs + ((size_t)slot * (mx.taps - 1) + (pos - lag) % max(mx.taps - 1, 1)) * mx.channels() + ch;
+  return *(lag <= t ? mx.proj + (size_t)(row - lag) * mx.ld + mx.ov + ch : ring);
 }
 __device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
+// Convolution and SiLU of one channel; TAPS 0: any number of taps.
+template <int TAPS>
 __device__ __forceinline__ float conv_silu(const Mixer& mx, int slot, int row, int t, int pos, int ch) {
   float y = mx.cb[ch];
-  for (int j = 0; j < mx.taps; ++j) y = fmaf(mx.cw[(size_t)ch * mx.taps + j], conv_input(mx, slot, row, t, pos, mx.taps - 1 - j, ch), y);
+  if (TAPS > 0) {
+    constexpr int N = TAPS > 0 ? TAPS : 1;
+    float x[N];
+#pragma unroll
+    for (int j = 0; j < N; ++j) x[j] = conv_input(mx, slot, row, t, pos, N - 1 - j, ch);
+#pragma unroll
+    for (int j = 0; j < N; ++j) y = fmaf(mx.cw[(size_t)ch * N + j], x[j], y);
+  } else {
+    for (int j = 0; j < mx.taps; ++j) y = fmaf(mx.cw[(size_t)ch * mx.taps + j], conv_input(mx, slot, row, t, pos, mx.taps - 1 - j, ch), y);
+  }
   return silu_exact(y);
 }
 __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
@@ -99,7 +110,7 @@ __device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1
 
 constexpr int GR = 8;   // row groups (warps) of a block
 
-template <int KIND, int RPT>
+template <int KIND, int RPT, int TAPS>      // TAPS: of the state space's convolution (0: any number)
 __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, const Raw raw, const int4* seqs) {
   pdl_trigger();
   pdl_wait();
@@ -153,7 +164,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       for (int i = threadIdx.x; i < 2 * D; i += 32 * GR) {
         const bool is_q = i >= D;
         const int d = is_q ? i - D : i;
-        (is_q ? qs : ks)[d] = conv_silu(mx, sq.z, sq.x + t, t, sq.w + t, b0 + (is_q ? mx.groups * D : 0) + d);
+        (is_q ? qs : ks)[d] = conv_silu<TAPS>(mx, sq.z, sq.x + t, t, sq.w + t, b0 + (is_q ? mx.groups * D : 0) + d);
       }
       if (threadIdx.x == 0) {
         const float dt = softplus(pr[mx.odt + h] + mx.dtb[h]);
@@ -183,7 +194,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       m_prev = m;
     }
     float v = is_n ? 1.f : 0.f;
-    if (is_v) v = KIND == KIND_SSD ? conv_silu(mx, sq.z, sq.x + t, t, sq.w + t, h * V + col) : pr[mx.ov + h * V + col];
+    if (is_v) v = KIND == KIND_SSD ? conv_silu<TAPS>(mx, sq.z, sq.x + t, t, sq.w + t, h * V + col) : pr[mx.ov + h * V + col];
     const float x = v;
     __syncthreads();
     float part = 0.f;
@@ -502,7 +513,7 @@ __global__ void __launch_bounds__(256) ssd_inputs_kernel(const Mixer mx, const C
     if (ch >= CD) return;
     float* out = wk.xbc + (size_t)c * CH * CD + ch;
     if (TAPS == 0) {
-      for (int r = 0; r < cd.y; ++r) out[(size_t)r * CD] = conv_silu(mx, sq.z, cd.x + r, t0 + r, pos0 + r, ch);
+      for (int r = 0; r < cd.y; ++r) out[(size_t)r * CD] = conv_silu<0>(mx, sq.z, cd.x + r, t0 + r, pos0 + r, ch);
     } else {
       constexpr int N = TAPS > 0 ? TAPS : 1, AHEAD = 8;
       float w[N], win[N];
@@ -944,10 +955,10 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
 }
 
 // State space: y silu(z), normed in `parts` equal parts of the heads' outputs laid end to end, times norm_w [H * V]. One block per
-// (part, row); columns from H * V up to `width` are set to zero. ahead[row]: tokens of the same portion before the row. The
-// block of a portion's last row keeps the convolution's last inputs.
+// (part, row); columns from H * V up to `width` are set to zero. behind[row]: tokens of the same portion after the row; the
+// last rows of a portion leave their inputs in the convolution's ring.
 template <typename OutT>
-__global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, float eps, const int* last_slot, const int* ahead,
+__global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, float eps, const int* slots, const int* behind,
                                                        const int* pos, OutT* out, int ldo, int width) {
   pdl_trigger();
   pdl_wait();
@@ -955,6 +966,19 @@ __global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw
   constexpr int KEEP = 4;
   const int g = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
   const int inner = mx.H * mx.V, n = inner / gridDim.x;
+  if (behind[t] < mx.taps - 1) {
+    const int CD = mx.channels(), step = gridDim.x * nt;
+    const float* src = mx.proj + (size_t)t * mx.ld + mx.ov;
+    float* ring = mx.Cs + ((size_t)slots[t] * (mx.taps - 1) + pos[t] % (mx.taps - 1)) * CD;
+    for (int ch = g * nt + tid; ch < CD; ch += 4 * step) {
+      float in[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) in[i] = ch + i * step < CD ? src[ch + i * step] : 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (ch + i * step < CD) ring[ch + i * step] = in[i];
+    }
+  }
   const float* o = raw.o + (size_t)t * inner + g * n;
   const float* gate = mx.proj + (size_t)t * mx.ld + mx.og + g * n;
   float x[KEEP], ss = 0.f;
@@ -977,17 +1001,9 @@ __global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw
   for (int v = tid + KEEP * nt; v < n; v += nt) dst[v] = (OutT)(o[v] * silu_exact(gate[v]) * r * w[v]);
   if (g == gridDim.x - 1)
     for (int v = inner + tid; v < width; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
-  const int slot = last_slot[t];
-  if (slot >= 0 && mx.taps > 1) {
-    // entry i of the new line is `taps - 2 - i` tokens old; of the old line only later entries are read
-    const int CD = mx.channels(), before = ahead[t], p = pos[t];
-    for (int ch = g * nt + tid; ch < CD; ch += gridDim.x * nt)
-      for (int i = 0; i < mx.taps - 1; ++i)
-        mx.Cs[((size_t)slot * (mx.taps - 1) + i) * CD + ch] = conv_input(mx, slot, t, before, p, mx.taps - 2 - i, ch);
-  }
 }
 
-template <int KIND>
+template <int KIND, int TAPS = 0>
 int launch_rows(const Mixer& mx, const Raw& raw, const int4* seqs, int nseq, cudaStream_t stream) {
   const int cols = mx.V + (KIND == KIND_MLSTM ? 1 : 0);
   const dim3 grid((cols + 31) / 32, mx.H, nseq);
@@ -995,7 +1011,7 @@ int launch_rows(const Mixer& mx, const Raw& raw, const int4* seqs, int nseq, cud
   const int rpt = (mx.D + GR - 1) / GR;
 #define PK_ROWS_CASE(n)                                                                             \
   if (rpt <= n) {                                                                                   \
-    PK_LAUNCH_PDL((state_rows_kernel<KIND, n>), grid, dim3(32 * GR), smem, stream, mx, raw, seqs);  \
+    PK_LAUNCH_PDL((state_rows_kernel<KIND, n, TAPS>), grid, dim3(32 * GR), smem, stream, mx, raw, seqs);  \
     return PK_OK;                                                                                   \
   }
   PK_ROWS_CASE(4)
@@ -1091,7 +1107,10 @@ PK_API int pk_state_rows(const PkStateMixer* d, const void* seqs, int nseq, cuda
   if (!unpack(d, mx, raw) || seqs == nullptr || nseq < 1) return PK_ERR_BAD_ARG;
   switch (d->kind) {
     case KIND_GLA: return launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream);
-    case KIND_SSD: return launch_rows<KIND_SSD>(mx, raw, (const int4*)seqs, nseq, stream);
+    case KIND_SSD:
+      if (mx.taps == 4) return launch_rows<KIND_SSD, 4>(mx, raw, (const int4*)seqs, nseq, stream);
+      if (mx.taps == 3) return launch_rows<KIND_SSD, 3>(mx, raw, (const int4*)seqs, nseq, stream);
+      return launch_rows<KIND_SSD>(mx, raw, (const int4*)seqs, nseq, stream);
     case KIND_MLSTM: return launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
     default: return launch_rows<KIND_RETENTION>(mx, raw, (const int4*)seqs, nseq, stream);
   }
@@ -1180,17 +1199,17 @@ PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head
 }
 
 // State space: gate, norm in `parts` parts, output rows [rows, ldo] of which `width` columns are this layer's; the last inputs of
-// the convolution are kept for every portion that ends (last_slot, ahead and pos per row).
-PK_API int pk_ssd_out(const PkStateMixer* d, const float* norm_w, int parts, float eps, const int* last_slot, const int* ahead, const int* pos, int rows,
+// every portion go into the convolution's ring (slots, behind and pos per row).
+PK_API int pk_ssd_out(const PkStateMixer* d, const float* norm_w, int parts, float eps, const int* slots, const int* behind, const int* pos, int rows,
                       void* out, int ldo, int width, int out_f32, cudaStream_t stream) {
   Mixer mx;
   Raw raw;
-  if (!unpack(d, mx, raw) || d->kind != KIND_SSD || norm_w == nullptr || last_slot == nullptr || ahead == nullptr || pos == nullptr || rows < 1 ||
+  if (!unpack(d, mx, raw) || d->kind != KIND_SSD || norm_w == nullptr || slots == nullptr || behind == nullptr || pos == nullptr || rows < 1 ||
       rows > 65535 || out == nullptr || parts < 1 || mx.H * mx.V % parts != 0 || width < mx.H * mx.V || ldo < width)
     return PK_ERR_BAD_ARG;
   const int n = mx.H * mx.V / parts, nt = (n + 31) / 32 * 32;
   const dim3 grid(parts, rows), block(nt <= 256 ? nt : n > 2048 ? 1024 : 256);
-  if (out_f32) PK_LAUNCH_PDL(ssd_out_kernel<float>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, last_slot, ahead, pos, (float*)out, ldo, width);
-  else PK_LAUNCH_PDL(ssd_out_kernel<pk::bf16>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, last_slot, ahead, pos, (pk::bf16*)out, ldo, width);
+  if (out_f32) PK_LAUNCH_PDL(ssd_out_kernel<float>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, slots, behind, pos, (float*)out, ldo, width);
+  else PK_LAUNCH_PDL(ssd_out_kernel<pk::bf16>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, slots, behind, pos, (pk::bf16*)out, ldo, width);
   return PK_OK;
 }

@@ -52,7 +52,7 @@ class StepContext:
     pos: torch.Tensor
     slot: torch.Tensor
     last_slot: torch.Tensor             # slot of the portion that ends at a row, else -1
-    ahead: torch.Tensor                 # tokens of the same portion before a row
+    behind: torch.Tensor                 # tokens of the same portion after a row
     table: torch.Tensor                 # page table
     ws: Workspace
     status: torch.Tensor
@@ -210,8 +210,8 @@ class StateSpaceMixer:
         self.const = {"cw": f("conv"), "cb": f("conv.b"), "dtb": f("dt_bias"), "A": -torch.exp(w["A_log"].double()).float().to(device), "skip": f("D")}
         self.norm = f("norm") * scale
         self.S = torch.zeros(slots, H, N, V, device=device)
-        self.line = torch.zeros(slots, max(taps - 1, 1), ch, device=device)
-        self.desc = dict(kind=mo.KIND_SSD, H=H, D=N, V=V, groups=G, taps=taps, qscale=1.0, S=self.S.data_ptr(), Cs=self.line.data_ptr(),
+        self.ring = torch.zeros(slots, max(taps - 1, 1), ch, device=device)
+        self.desc = dict(kind=mo.KIND_SSD, H=H, D=N, V=V, groups=G, taps=taps, qscale=1.0, S=self.S.data_ptr(), Cs=self.ring.data_ptr(),
                          **{n: t.data_ptr() for n, t in self.const.items()})
 
     def at(self, first: int) -> None:
@@ -220,7 +220,7 @@ class StateSpaceMixer:
         self.desc.update(og=first, ov=first + inner, odt=first + 2 * inner + 2 * self.desc["groups"] * self.N)
 
     def state_bytes(self) -> int:
-        return (self.S.numel() + self.line.numel()) * 4
+        return (self.S.numel() + self.ring.numel()) * 4
 
     def run(self, ctx: StepContext, p: torch.Tensor, out: torch.Tensor) -> None:
         ws = ctx.ws
@@ -231,7 +231,7 @@ class StateSpaceMixer:
         if ctx.n_long:
             scratch = ws.flat("state_chunks", mo.state_chunk_workspace(d, ctx.n_chunks), torch.float32)
             mo.state_chunks(d, ctx.long, ctx.n_long, ctx.chunks, ctx.chunk0, ctx.n_chunks, scratch)
-        mo.ssd_out(d, self.norm, self.parts, self.eps, ctx.last_slot, ctx.ahead, ctx.pos, ctx.T, out)
+        mo.ssd_out(d, self.norm, self.parts, self.eps, ctx.slot, ctx.behind, ctx.pos, ctx.T, out)
 
 
 def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> tuple[torch.Tensor, float]:

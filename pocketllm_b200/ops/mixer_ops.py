@@ -149,10 +149,10 @@ def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: f
     _call("pk_state_out", byref(d), norm_w, int(per_head), eps, last_slot, rows, out, out.stride(0), int(out.dtype == torch.float32))
 
 
-def ssd_out(d: StateMixer, norm_w: torch.Tensor, parts: int, eps: float, last_slot: torch.Tensor, ahead: torch.Tensor, pos: torch.Tensor, rows: int,
+def ssd_out(d: StateMixer, norm_w: torch.Tensor, parts: int, eps: float, slots: torch.Tensor, behind: torch.Tensor, pos: torch.Tensor, rows: int,
             out: torch.Tensor) -> None:
-    """Gate and norm of a state-space layer, the line of its convolution; `out` [rows, columns of this layer] (a view is fine)."""
-    _call("pk_ssd_out", byref(d), norm_w, parts, eps, last_slot, ahead, pos, rows, out, out.stride(0), out.shape[1], int(out.dtype == torch.float32))
+    """Gate and norm of a state-space layer, the ring of its convolution; `out` [rows, columns of this layer] (a view is fine)."""
+    _call("pk_ssd_out", byref(d), norm_w, parts, eps, slots, behind, pos, rows, out, out.stride(0), out.shape[1], int(out.dtype == torch.float32))
 
 
 def latent_prep(proj: torch.Tensor, oq: int, oc: int, H: int, D: int, R: int, K: int, c_norm: torch.Tensor, eps: float, freq: torch.Tensor,

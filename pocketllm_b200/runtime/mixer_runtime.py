@@ -34,9 +34,9 @@ class StepEntry:
 def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence[int], windows: Sequence[int], rows_max: int = mo.ROWS_MAX,
                   chunk: int = mo.CHUNK, tile: int = 128) -> dict:
     """Index arrays (numpy int32) of a batch: per row its position, slot, (for a portion's last row) the slot again and how many
-    tokens of its portion come before it, and the work lists of short and long portions. Pure host logic."""
+    tokens of its portion come after it, and the work lists of short and long portions. Pure host logic."""
     T = int(sum(lengths))
-    pos, slot, last, ahead = np.empty(T, np.int32), np.empty(T, np.int32), np.full(T, -1, np.int32), np.empty(T, np.int32)
+    pos, slot, last, behind = np.empty(T, np.int32), np.empty(T, np.int32), np.full(T, -1, np.int32), np.empty(T, np.int32)
     short, rows, long, chunks, chunk0, tiles = [], [], [], [], [], []
     gather = {w: [] for w in windows}
     total = {w: 0 for w in windows}
@@ -46,7 +46,7 @@ def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence
         pos[r0:r0 + n] = np.arange(p0, p0 + n)
         slot[r0:r0 + n] = s
         last[r0 + n - 1] = s
-        ahead[r0:r0 + n] = np.arange(n)
+        behind[r0:r0 + n] = np.arange(n - 1, -1, -1)
         seq = (r0, n, s, p0)
         if n <= rows_max:
             short.append(seq)
@@ -63,7 +63,7 @@ def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence
                 total[w] += p0 + n - first
                 longest[w] = max(longest[w], p0 + n - first)
         r0 += n
-    return {"T": T, "pos": pos, "slot": slot, "last": last, "ahead": ahead, "short": short, "rows": rows, "long": long, "chunks": chunks, "chunk0": chunk0,
+    return {"T": T, "pos": pos, "slot": slot, "last": last, "behind": behind, "short": short, "rows": rows, "long": long, "chunks": chunks, "chunk0": chunk0,
             "tiles": tiles, "gather": gather, "total": total, "longest": longest}
 
 
@@ -76,7 +76,7 @@ class _DecodeBatch:
         self.packed = torch.zeros(n * 8, **i32)              # seqs (4 n) | tokens | pos | slot | last: one copy per step
         self.seqs = self.packed[:4 * n].view(n, 4)
         self.tokens, self.pos, self.slot, self.last = (self.packed[(4 + k) * n:(5 + k) * n] for k in range(4))
-        self.rows, self.ahead = torch.arange(n, **i32), torch.zeros(n, **i32)
+        self.rows, self.behind = torch.arange(n, **i32), torch.zeros(n, **i32)
         self.hist = torch.zeros(n, hist, **i32)
         self.step = torch.zeros(1, **i32)
         self.cand_val, self.cand_idx = torch.zeros(n, 64, device=device), torch.zeros(n, 64, **i32)
@@ -209,7 +209,7 @@ class MixerRuntime:
             off += len(a) + pad
 
         put("tokens", np.concatenate([np.asarray(e.tokens, np.int32) for e in entries]))
-        for n in ("pos", "slot", "last", "ahead", "short", "rows", "long", "chunks", "chunk0", "tiles"):
+        for n in ("pos", "slot", "last", "behind", "short", "rows", "long", "chunks", "chunk0", "tiles"):
             put(n, p[n])
         put("all", np.arange(T))
         put("want", want)
@@ -217,7 +217,7 @@ class MixerRuntime:
             put(f"gather{w}", p["gather"][w])
         dev = torch.from_numpy(np.concatenate(arrays)).to(self.device)
         at = lambda n: dev[parts[n][0]:parts[n][0] + parts[n][1]]
-        ctx = StepContext(T, at("tokens"), at("pos"), at("slot"), at("last"), at("ahead"), self.cache.device_table, self.ws, self.status,
+        ctx = StepContext(T, at("tokens"), at("pos"), at("slot"), at("last"), at("behind"), self.cache.device_table, self.ws, self.status,
                           short=at("short"), n_short=len(p["short"]), rows=at("rows"), n_rows=len(p["rows"]), all_rows=at("all"),
                           long=at("long"), n_long=len(p["long"]), chunks=at("chunks"), chunk0=at("chunk0"), n_chunks=len(p["chunks"]),
                           tiles=at("tiles"), n_tiles=len(p["tiles"]),
@@ -246,7 +246,7 @@ class MixerRuntime:
         self._copied.record()
 
     def _decode_forward(self, b: _DecodeBatch) -> torch.Tensor:
-        ctx = StepContext(b.n, b.tokens, b.pos, b.slot, b.last, b.ahead, self.cache.device_table, self.dec_ws, self.status, short=b.seqs, n_short=b.n,
+        ctx = StepContext(b.n, b.tokens, b.pos, b.slot, b.last, b.behind, self.cache.device_table, self.dec_ws, self.status, short=b.seqs, n_short=b.n,
                           rows=b.rows, n_rows=b.n, all_rows=b.rows)
         return self._forward(ctx, None, b.n)
 

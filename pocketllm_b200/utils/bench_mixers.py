@@ -226,7 +226,7 @@ class _Batch:
         slots, pages = (T if singles else 1), -(-context // 64)
         table = dev(range(slots * pages)).view(slots, pages)
         self.pages, self.slots = slots * pages, slots
-        self.ctx = StepContext(T, dev([0] * T), dev(p["pos"]), dev(p["slot"]), dev(p["last"]), dev(p["ahead"]), table, Workspace("cuda"),
+        self.ctx = StepContext(T, dev([0] * T), dev(p["pos"]), dev(p["slot"]), dev(p["last"]), dev(p["behind"]), table, Workspace("cuda"),
                                torch.zeros(1, dtype=torch.int32, device="cuda"), short=dev(p["short"]), n_short=len(p["short"]), rows=dev(p["rows"]),
                                n_rows=len(p["rows"]), all_rows=dev(range(T)), long=dev(p["long"]), n_long=len(p["long"]), chunks=dev(p["chunks"]),
                                chunk0=dev(p["chunk0"]), n_chunks=len(p["chunks"]), tiles=dev(p["tiles"]), n_tiles=len(p["tiles"]),

@@ -85,7 +85,7 @@ def test_layers_of_the_model():
     a = p.proj.at
     assert (left.desc["oq"], left.desc["ok"], left.desc["ov"]) == (0, 4 * 40, 5 * 40) and a["right"] == 5 * 40 + 130
     assert (right.desc["og"], right.desc["ov"], right.desc["odt"]) == (a["right"], a["right"] + 132, a["right"] + 2 * 132 + 140)
-    assert right.S.shape == (3, 4, 70, 33) and right.line.shape == (3, 2, 132 + 140) and left.cache.shape == (5, 64, 40 + 136)
+    assert right.S.shape == (3, 4, 70, 33) and right.ring.shape == (3, 2, 132 + 140) and left.cache.shape == (5, 64, 40 + 136)
     assert p.split == 520 and torch.equal(p.out.w[:88, 520:520 + 132], t["l3.mix.right.o"]) and (p.out.w[:, 652:] == 0).all()
     assert torch.allclose(right.norm, t["l3.mix.right.norm"].float() * 0.4)
     assert m.layers[1].mixer.desc["gate"] == m.layers[1].mixer.proj.at["g"] and m.layers[1].mixer.desc["neighbours"] == 0
@@ -99,9 +99,9 @@ def test_slowed_down_rotations():
     assert mag == 1.0 and f.tolist() == pytest.approx([100.0 ** (-i / 4) / 5 for i in range(4)])
 
 
-def test_portions_know_the_tokens_before_a_row():
+def test_portions_know_the_tokens_after_a_row():
     p = plan_portions([3, 1, 10], [5, 0, 64], [0, 2, 1], windows=[])
-    assert p["ahead"].tolist() == [0, 1, 2, 0] + list(range(10))
+    assert p["behind"].tolist() == [2, 1, 0, 0] + list(range(9, -1, -1))
 
 
 @pytest.mark.parametrize("fault", ["window", "window_parallel", "sink", "cap", "pairs", "head_norm", "v_mix", "gate", "skip", "groups", "residual",
