@@ -26,6 +26,7 @@
 // A last kernel normalises every head's output (after mLSTM's division by max(|n.q|, exp(-m)) + 1e-6), applies the output
 // gate and writes the projection's input (state space: the gate comes first, the norm's parts need not be heads).
 #include "../common/pk_rotary.cuh"
+#include "../common/pk_state.cuh"
 
 namespace {
 
@@ -66,7 +67,6 @@ struct Mixer {
   const float* skip;   // [H]
   float* Cs;           // [slots, taps - 1, channels] last inputs of the convolution, by position modulo (taps - 1)
   int groups, taps, odt;
-  __device__ __host__ int channels() const { return H * V + 2 * groups * D; }
   // state
   float* S;            // [slots, H, D, V]
   float* N;            // [slots, H, D]      (mLSTM)
@@ -79,31 +79,6 @@ struct Raw {
   float* nq;   // [rows, H]   n . q       (mLSTM)
   float* m;    // [rows, H]   running max (mLSTM)
 };
-
-// State space: input of the convolution `lag` tokens before the one at `row`, which is token `t` of its portion, at position pos.
-__device__ __forceinline__ float conv_input(const Mixer& mx, int slot, int row, int t, int pos, int lag, int ch) {
-  if (lag > pos) return 0.f;
-  const float* ring = mx.Cs + ((size_t)slot * (mx.taps - 1) + (pos - lag) % max(mx.taps - 1, 1)) * mx.channels() + ch;
-  return *(lag <= t ? mx.proj + (size_t)(row - lag) * mx.ld + mx.ov + ch : ring);
-}
-__device__ __forceinline__ float silu_exact(float z) { return z / (1.f + expf(-z)); }
-// Convolution and SiLU of one channel; TAPS 0: any number of taps.
-template <int TAPS>
-__device__ __forceinline__ float conv_silu(const Mixer& mx, int slot, int row, int t, int pos, int ch) {
-  float y = mx.cb[ch];
-  if (TAPS > 0) {
-    constexpr int N = TAPS > 0 ? TAPS : 1;
-    float x[N];
-#pragma unroll
-    for (int j = 0; j < N; ++j) x[j] = conv_input(mx, slot, row, t, pos, N - 1 - j, ch);
-#pragma unroll
-    for (int j = 0; j < N; ++j) y = fmaf(mx.cw[(size_t)ch * N + j], x[j], y);
-  } else {
-    for (int j = 0; j < mx.taps; ++j) y = fmaf(mx.cw[(size_t)ch * mx.taps + j], conv_input(mx, slot, row, t, pos, mx.taps - 1 - j, ch), y);
-  }
-  return silu_exact(y);
-}
-__device__ __forceinline__ float softplus(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // ---------------------------------------------------------------------------------------
 // rows form
@@ -509,69 +484,25 @@ __global__ void __launch_bounds__(256) ssd_inputs_kernel(const Mixer mx, const C
   const int4 cd = ck.chunks[c], sq = ck.seqs[cd.z];
   const int t0 = cd.x - sq.x, pos0 = sq.w + t0;      // first token of the chunk
   if ((int)blockIdx.y < conv_blocks) {
-    const int CD = mx.channels(), ch = blockIdx.y * 256 + tid;
+    const int CD = ssd_channels(mx), ch = blockIdx.y * 256 + tid;
     if (ch >= CD) return;
     float* out = wk.xbc + (size_t)c * CH * CD + ch;
-    if (TAPS == 0) {
-      for (int r = 0; r < cd.y; ++r) out[(size_t)r * CD] = conv_silu<0>(mx, sq.z, cd.x + r, t0 + r, pos0 + r, ch);
-    } else {
-      constexpr int N = TAPS > 0 ? TAPS : 1, AHEAD = 8;
-      float w[N], win[N];
-#pragma unroll
-      for (int j = 0; j < N; ++j) w[j] = mx.cw[(size_t)ch * N + j];
-      const float b = mx.cb[ch];
-#pragma unroll
-      for (int j = 0; j + 1 < N; ++j) win[j + 1] = conv_input(mx, sq.z, cd.x, t0, pos0, N - 1 - j, ch);
-      const float* in = mx.proj + (size_t)cd.x * mx.ld + mx.ov + ch;
-      for (int r0 = 0; r0 < cd.y; r0 += AHEAD) {
-        float x[AHEAD];
-#pragma unroll
-        for (int i = 0; i < AHEAD; ++i) x[i] = r0 + i < cd.y ? in[(size_t)(r0 + i) * mx.ld] : 0.f;
-#pragma unroll
-        for (int i = 0; i < AHEAD; ++i) {
-#pragma unroll
-          for (int j = 0; j + 1 < N; ++j) win[j] = win[j + 1];
-          win[N - 1] = x[i];
-          float y = b;
-#pragma unroll
-          for (int j = 0; j < N; ++j) y = fmaf(w[j], win[j], y);
-          if (r0 + i < cd.y) out[(size_t)(r0 + i) * CD] = silu_exact(y);
-        }
-      }
-    }
+    conv_silu_rows<TAPS>(mx, sq.z, cd.x, t0, pos0, cd.y, ch, [&](int r, float y) { out[(size_t)r * CD] = y; });
     return;
   }
   const int h = (blockIdx.y - conv_blocks) * 8 + (tid >> 5), lane = tid & 31;
   if (h >= mx.H) return;
   const size_t ch = (size_t)c * mx.H + h;
-  float dt[2];
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const int r = 2 * lane + i;
-    dt[i] = r < cd.y ? softplus(mx.proj[(size_t)(cd.x + r) * mx.ld + mx.odt + h] + mx.dtb[h]) : 0.f;
-  }
-  const double a = (double)mx.A[h], own = a * dt[0] + a * dt[1];
-  double run = own;
-#pragma unroll
-  for (int o = 1; o < 32; o <<= 1) {
-    const double v = __shfl_up_sync(0xffffffffu, run, o);
-    if (lane >= o) run += v;
-  }
-  const double g[2] = {run - a * dt[1], run};
-#pragma unroll
-  for (int i = 0; i < 2; ++i) {
-    const float hi = (float)g[i];
-    wk.G[ch * CH + 2 * lane + i] = make_float2(hi, (float)(g[i] - (double)hi));
-    wk.dt[ch * CH + 2 * lane + i] = dt[i];
-  }
-  if (lane == 31) wk.dec[ch] = expf((float)run);      // tokens behind the chunk's last have dt = 0
+  float total;
+  ssd_decays<CH / 32>(mx, cd.x, cd.y, h, lane, wk.dt + ch * CH, wk.G + ch * CH, &total);
+  if (lane == 31) wk.dec[ch] = expf(total);
 }
 
 // P_ij = C_i . B_j of a (chunk, group of heads).
 __global__ void __launch_bounds__(256) ssd_scores_kernel(const Mixer mx, const Chunks ck, const Work wk) {
   __shared__ float Qs[32][CH + 4], Ks[32][CH + 4];
   const int c = blockIdx.x, g = blockIdx.y, tid = threadIdx.x;
-  const int len = ck.chunks[c].y, D = mx.D, CD = mx.channels();
+  const int len = ck.chunks[c].y, D = mx.D, CD = ssd_channels(mx);
   const float* kb = wk.xbc + (size_t)c * CH * CD + mx.H * mx.V + g * D;
   const float* qb = kb + mx.groups * D;
   const int tx = tid & 15, ty = tid >> 4;
@@ -708,7 +639,7 @@ __global__ void __launch_bounds__(256) chunk_kv_kernel(const Mixer mx, const Chu
   const size_t ch = (size_t)c * mx.H + h;
   if (SSD) {
     __shared__ float w[CH];
-    const int CD = mx.channels();
+    const int CD = ssd_channels(mx);
     if (tid < CH) {
       const float2 g = wk.G[ch * CH + tid], e = wk.G[ch * CH + CH - 1];
       w[tid] = tid < cd.y ? wk.dt[ch * CH + tid] * expf((e.x - g.x) + (e.y - g.y)) : 0.f;
@@ -831,7 +762,7 @@ __global__ void __launch_bounds__(256) chunk_out_kernel(const Mixer mx, const Ra
   // state space: rows of x and C, exp(G_i), running decays and steps of the chunk
   __shared__ float eg[CH], dts[CH];
   __shared__ float2 gs[CH];
-  const int CD = SSD ? mx.channels() : 0, group = SSD ? h / (mx.H / mx.groups) : 0;
+  const int CD = SSD ? ssd_channels(mx) : 0, group = SSD ? h / (mx.H / mx.groups) : 0;
   const float* xrow = SSD ? wk.xbc + (size_t)c * CH * CD : nullptr;
   const float* crow = SSD ? xrow + mx.H * V + (mx.groups + group) * D : nullptr;
   const float* cb = SSD ? wk.P + ((size_t)c * mx.groups + group) * CH * CH : nullptr;
@@ -967,7 +898,7 @@ __global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw
   const int g = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
   const int inner = mx.H * mx.V, n = inner / gridDim.x;
   if (behind[t] < mx.taps - 1) {
-    const int CD = mx.channels(), step = gridDim.x * nt;
+    const int CD = ssd_channels(mx), step = gridDim.x * nt;
     const float* src = mx.proj + (size_t)t * mx.ld + mx.ov;
     float* ring = mx.Cs + ((size_t)slots[t] * (mx.taps - 1) + pos[t] % (mx.taps - 1)) * CD;
     for (int ch = g * nt + tid; ch < CD; ch += 4 * step) {
@@ -1043,7 +974,7 @@ Work carve(float* ws, const Mixer& mx, int nchunks, int kind, size_t* total) {
   w.dec_w = kind == KIND_SSD ? 1 : mx.D;
   w.dec = take(c * H * w.dec_w);
   if (kind == KIND_SSD) {
-    w.xbc = take(c * CH * mx.channels());
+    w.xbc = take(c * CH * ssd_channels(mx));
     w.dt = take(c * H * CH);
     w.G = (float2*)take(c * H * CH * 2);
     w.P = take(c * mx.groups * CH * CH);
@@ -1058,31 +989,6 @@ Work carve(float* ws, const Mixer& mx, int nchunks, int kind, size_t* total) {
 }
 
 }  // namespace
-
-// Plain mirror of `Mixer` / `Raw` for callers (all pointers device pointers).
-struct PkStateMixer {
-  const float* proj;
-  const float* bi;
-  const float* bf;
-  const float* a2;
-  const float* a2b;
-  float* S;
-  float* N;
-  float* Ms;
-  float* o;
-  float* nq;
-  float* m;
-  const double* freq;
-  const float* pw;
-  const float* cw;
-  const float* cb;
-  const float* dtb;
-  const float* A;
-  const float* skip;
-  float* Cs;
-  int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank, rot, groups, taps, odt;
-  float qscale, cap, inv_tau;
-};
 
 static bool unpack(const PkStateMixer* d, Mixer& mx, Raw& raw) {
   if (d == nullptr || d->proj == nullptr || d->S == nullptr || d->o == nullptr || d->H < 1 || d->D < 1 || d->V < 1 || d->D > 512) return false;
@@ -1147,7 +1053,7 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
     PK_CHECK_LAUNCH();
     gla_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
   } else if (d->kind == KIND_SSD) {
-    const int cb = (mx.channels() + 255) / 256;
+    const int cb = (ssd_channels(mx) + 255) / 256;
     const dim3 grid(nchunks, cb + (H + 7) / 8);
     if (mx.taps == 2) ssd_inputs_kernel<2><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);
     else if (mx.taps == 3) ssd_inputs_kernel<3><<<grid, 256, 0, stream>>>(mx, ck, wk, cb);

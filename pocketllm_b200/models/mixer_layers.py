@@ -68,6 +68,7 @@ class StepContext:
     n_chunks: int = 0
     tiles: torch.Tensor | None = None   # {first row, rows, sequence, 0}: up to 128 query rows of a long portion
     n_tiles: int = 0
+    tile0: torch.Tensor | None = None   # first tile of every long portion
     gather: dict = field(default_factory=dict)   # window -> ({first key row, its position} per long sequence, key rows, longest)
 
 
@@ -194,11 +195,12 @@ class RetentionMixer(RecurrentMixer):
 
 class StateSpaceMixer:
     """The state-space recurrence of Mamba-2: x, B and C through a short convolution, a scalar decay per token and head, gate before
-    a norm in equal parts. `scale` multiplies its output. Works on columns of a projection that its owner makes."""
+    a norm in equal parts. `scale` multiplies its output. Works on columns of a projection that its owner makes. Long portions in
+    bf16 run on the tensor cores where the shape fits them."""
 
-    def __init__(self, w: dict, m: dict, eps: float, device, slots: int, scale: float = 1.0):
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, slots: int, scale: float = 1.0):
         H, V, N, G, taps = m["heads"], m["vdim"], m["state"], m["groups"], m["conv"]
-        self.H, self.V, self.N, self.parts, self.eps = H, V, N, m["norm_groups"], eps
+        self.H, self.V, self.N, self.parts, self.eps, self.dtype = H, V, N, m["norm_groups"], eps, dtype
         if N > 512:
             raise ValueError("state-space layers take states up to 512")
         ch = H * V + 2 * G * N
@@ -229,8 +231,12 @@ class StateSpaceMixer:
         if ctx.n_short:
             mo.state_rows(d, ctx.short, ctx.n_short)
         if ctx.n_long:
-            scratch = ws.flat("state_chunks", mo.state_chunk_workspace(d, ctx.n_chunks), torch.float32)
-            mo.state_chunks(d, ctx.long, ctx.n_long, ctx.chunks, ctx.chunk0, ctx.n_chunks, scratch)
+            n = mo.ssd_tile_workspace(d, ctx.n_tiles) if self.dtype == torch.bfloat16 else 0
+            if n:
+                mo.ssd_tiles(d, ctx.long, ctx.n_long, ctx.tiles, ctx.tile0, ctx.n_tiles, ws.flat("state_chunks", n, torch.float32), ctx.status)
+            else:
+                scratch = ws.flat("state_chunks", mo.state_chunk_workspace(d, ctx.n_chunks), torch.float32)
+                mo.state_chunks(d, ctx.long, ctx.n_long, ctx.chunks, ctx.chunk0, ctx.n_chunks, scratch)
         mo.ssd_out(d, self.norm, self.parts, self.eps, ctx.slot, ctx.behind, ctx.pos, ctx.T, out)
 
 

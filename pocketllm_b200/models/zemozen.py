@@ -200,7 +200,7 @@ def build_model(c: ZemozenConfig, tensors: dict[str, torch.Tensor], *, dtype: to
         else:
             wl, wr = sub(p + "mix.left."), sub(p + "mix.right.")
             left = ml.GroupedAttention(wl, m["left"], c.eps, dtype, device, pages, context, neighbours=True, sink=0.0, scale_out=float(m["left_scale"]))
-            right = ml.StateSpaceMixer(wr, m["right"], c.eps, device, slots, scale=float(m["right_scale"]))
+            right = ml.StateSpaceMixer(wr, m["right"], c.eps, dtype, device, slots, scale=float(m["right_scale"]))
             mixer = ml.ParallelMixer(left, right, wl, wr, dtype, device)
         layer = ml.MixerLayer(mixer, f32(p + "norm1"))
         if L.mlp is not None:

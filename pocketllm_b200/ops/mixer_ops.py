@@ -54,7 +54,7 @@ def sm_count() -> int:
 _SIGNATURES = {
     "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
     "pk_sandwich_norm": "pppifipipifpiippp" "iipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
-    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii",
+    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii", "pk_ssd_tiles": "ppippipp",
     "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipi",
     "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipi", "pk_latent_prefill": "pipipippiiiiifppip",
     "pk_paged_prep": "pi", "pk_paged_rows": "ppi", "pk_paged_merge": "ppi", "pk_paged_prefill": "piipip",
@@ -62,7 +62,7 @@ _SIGNATURES = {
     "pk_gemm_bf16_grouped_scaled": "pippiiiiipipipi",
 }
 _bound: dict[tuple[int, str], object] = {}
-_KERNELS = {"pk_state_chunks": 5, "pk_latent_out": 2, "pk_argmax": 2, "pk_feed_tokens": 2, "pk_expert_group": 3}     # launches per call, where not 1
+_KERNELS = {"pk_state_chunks": 5, "pk_ssd_tiles": 4, "pk_latent_out": 2, "pk_argmax": 2, "pk_feed_tokens": 2, "pk_expert_group": 3}     # launches per call, where not 1
 launches = 0        # kernels launched (or captured) by this process through `_call`
 
 
@@ -147,6 +147,19 @@ def state_chunks(d: StateMixer, seqs: torch.Tensor, nseq: int, chunks: torch.Ten
 def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
     """Head norm + output gate of `rows` rows; norm_w [H * V], [V] when `per_head`, or None."""
     _call("pk_state_out", byref(d), norm_w, int(per_head), eps, last_slot, rows, out, out.stride(0), int(out.dtype == torch.float32))
+
+
+def ssd_tile_workspace(d: StateMixer, ntiles: int) -> int:
+    """Workspace floats of `ssd_tiles`; 0: the shape does not fit it."""
+    fn = _lib.kernels().pk_ssd_tile_workspace
+    fn.restype, fn.argtypes = c_size_t, [POINTER(StateMixer), c_int]
+    return int(fn(byref(d), ntiles))
+
+
+def ssd_tiles(d: StateMixer, seqs: torch.Tensor, nseq: int, tiles: torch.Tensor, tile0: torch.Tensor, ntiles: int, ws: torch.Tensor,
+              status: torch.Tensor) -> None:
+    """Recurrence of long portions on the tensor cores, in tiles of 128 tokens."""
+    _call("pk_ssd_tiles", byref(d), seqs, nseq, tiles, tile0, ntiles, ws, status)
 
 
 def ssd_out(d: StateMixer, norm_w: torch.Tensor, parts: int, eps: float, slots: torch.Tensor, behind: torch.Tensor, pos: torch.Tensor, rows: int,

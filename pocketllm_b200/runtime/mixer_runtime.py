@@ -37,7 +37,7 @@ def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence
     tokens of its portion come after it, and the work lists of short and long portions. Pure host logic."""
     T = int(sum(lengths))
     pos, slot, last, behind = np.empty(T, np.int32), np.empty(T, np.int32), np.full(T, -1, np.int32), np.empty(T, np.int32)
-    short, rows, long, chunks, chunk0, tiles = [], [], [], [], [], []
+    short, rows, long, chunks, chunk0, tiles, tile0 = [], [], [], [], [], [], []
     gather = {w: [] for w in windows}
     total = {w: 0 for w in windows}
     longest = {w: 0 for w in windows}
@@ -55,6 +55,7 @@ def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence
             i = len(long)
             long.append(seq)
             chunk0.append(len(chunks))
+            tile0.append(len(tiles))
             chunks += [(r0 + a, min(chunk, n - a), i, a // chunk) for a in range(0, n, chunk)]
             tiles += [(r0 + a, min(tile, n - a), i, 0) for a in range(0, n, tile)]
             for w in gather:
@@ -64,7 +65,7 @@ def plan_portions(lengths: Sequence[int], starts: Sequence[int], slots: Sequence
                 longest[w] = max(longest[w], p0 + n - first)
         r0 += n
     return {"T": T, "pos": pos, "slot": slot, "last": last, "behind": behind, "short": short, "rows": rows, "long": long, "chunks": chunks, "chunk0": chunk0,
-            "tiles": tiles, "gather": gather, "total": total, "longest": longest}
+            "tiles": tiles, "tile0": tile0, "gather": gather, "total": total, "longest": longest}
 
 
 class _DecodeBatch:
@@ -209,7 +210,7 @@ class MixerRuntime:
             off += len(a) + pad
 
         put("tokens", np.concatenate([np.asarray(e.tokens, np.int32) for e in entries]))
-        for n in ("pos", "slot", "last", "behind", "short", "rows", "long", "chunks", "chunk0", "tiles"):
+        for n in ("pos", "slot", "last", "behind", "short", "rows", "long", "chunks", "chunk0", "tiles", "tile0"):
             put(n, p[n])
         put("all", np.arange(T))
         put("want", want)
@@ -220,7 +221,7 @@ class MixerRuntime:
         ctx = StepContext(T, at("tokens"), at("pos"), at("slot"), at("last"), at("behind"), self.cache.device_table, self.ws, self.status,
                           short=at("short"), n_short=len(p["short"]), rows=at("rows"), n_rows=len(p["rows"]), all_rows=at("all"),
                           long=at("long"), n_long=len(p["long"]), chunks=at("chunks"), chunk0=at("chunk0"), n_chunks=len(p["chunks"]),
-                          tiles=at("tiles"), n_tiles=len(p["tiles"]),
+                          tiles=at("tiles"), n_tiles=len(p["tiles"]), tile0=at("tile0"),
                           gather={w: (at(f"gather{w}"), p["total"][w], p["longest"][w]) for w in self._windows})
         self.ws.trim()
         logits = self._forward(ctx, at("want"), len(want))

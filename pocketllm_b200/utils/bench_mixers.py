@@ -229,7 +229,7 @@ class _Batch:
         self.ctx = StepContext(T, dev([0] * T), dev(p["pos"]), dev(p["slot"]), dev(p["last"]), dev(p["behind"]), table, Workspace("cuda"),
                                torch.zeros(1, dtype=torch.int32, device="cuda"), short=dev(p["short"]), n_short=len(p["short"]), rows=dev(p["rows"]),
                                n_rows=len(p["rows"]), all_rows=dev(range(T)), long=dev(p["long"]), n_long=len(p["long"]), chunks=dev(p["chunks"]),
-                               chunk0=dev(p["chunk0"]), n_chunks=len(p["chunks"]), tiles=dev(p["tiles"]), n_tiles=len(p["tiles"]),
+                               chunk0=dev(p["chunk0"]), n_chunks=len(p["chunks"]), tiles=dev(p["tiles"]), n_tiles=len(p["tiles"]), tile0=dev(p["tile0"]),
                                gather={w: (dev(p["gather"][w]), p["total"][w], p["longest"][w]) for w in windows})
 
 
@@ -269,7 +269,7 @@ def _state(kind: str, dims, T: int, singles: bool):
     return call, flops, T * H * D * V * 8.0 if singles else 0.0
 
 
-def _state_space(dims, T: int, singles: bool):
+def _state_space(dims, T: int, singles: bool, dtype=torch.bfloat16):
     """The state-space recurrence of one layer with its convolution, gate and norm: (call, flops, bytes of states)."""
     from ..models import mixer_layers as ml
     from ..ops import mixer_ops as mo
@@ -281,10 +281,10 @@ def _state_space(dims, T: int, singles: bool):
     r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
     w = {"in": r(2 * inner + 2 * G * N + H, W), "conv": r(ch, 4), "conv.b": torch.zeros(ch), "dt_bias": torch.full((H,), -3.0), "A_log": torch.zeros(H),
          "D": torch.ones(H), "norm": torch.ones(inner)}
-    m = ml.StateSpaceMixer(w, {"heads": H, "vdim": V, "state": N, "groups": G, "conv": 4, "norm_groups": G}, 1e-5, "cuda", b.slots)
+    m = ml.StateSpaceMixer(w, {"heads": H, "vdim": V, "state": N, "groups": G, "conv": 4, "norm_groups": G}, 1e-5, dtype, "cuda", b.slots)
     m.at(0)
     p = ml.FusedLinear([("in", w["in"])], torch.bfloat16, "cuda")(b.ctx, torch.randn(T, W, device="cuda").to(torch.bfloat16), "proj", torch.float32)
-    mix = b.ctx.ws.rows("mix", T, inner, torch.bfloat16)
+    mix = b.ctx.ws.rows("mix", T, inner, dtype)
 
     def call():
         m.run(b.ctx, p, mix)
@@ -572,8 +572,10 @@ def zemozen_kernels() -> None:
     show = lambda name, d, **kw: print(json.dumps({"kernel": name, **kw, **d}), flush=True)
     space, ret = (64, 64, 128, 8), (16, 128, 256)
     for T in (512, 2048):
-        f, fl, _ = _state_space(space, T, False)
-        show("state space chunk form (convolution, gate, norm included)", _roof(timed(f), fl), T=T, dims=space)
+        for dt in (torch.bfloat16, torch.float32):
+            f, fl, _ = _state_space(space, T, False, dt)
+            show("state space prefill, " + ("tensor cores" if dt == torch.bfloat16 else "fp32") + " (convolution, gate, norm included)", _roof(timed(f), fl), T=T,
+                 dims=space)
         f, fl, _ = _state("retention", ret, T, False)
         show("like kernel: retention chunk form + head norm", _roof(timed(f), fl), T=T, dims=ret)
     for B in (1, 8):

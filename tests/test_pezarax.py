@@ -166,7 +166,7 @@ def test_descriptor_mirrors_the_header():
 
     from pocketllm_b200 import build
     from pocketllm_b200.ops import mixer_ops as mo
-    for cls, file, name in ((mo.PagedAttention, "common/pk_paged.h", "PkPagedAttention"), (mo.StateMixer, "kernels/linear_state.cu", "PkStateMixer")):
+    for cls, file, name in ((mo.PagedAttention, "common/pk_paged.h", "PkPagedAttention"), (mo.StateMixer, "common/pk_state.cuh", "PkStateMixer")):
         body = re.search(r"struct " + name + r" \{(.*?)\};", (build.CSRC / file).read_text(), re.S).group(1)
         body = re.sub(r"//[^\n]*", "", body)
         want = []

@@ -102,6 +102,8 @@ def test_slowed_down_rotations():
 def test_portions_know_the_tokens_after_a_row():
     p = plan_portions([3, 1, 10], [5, 0, 64], [0, 2, 1], windows=[])
     assert p["behind"].tolist() == [2, 1, 0, 0] + list(range(9, -1, -1))
+    p = plan_portions([300, 2, 128, 129], [0, 5, 64, 1], [0, 2, 1, 3], windows=[])
+    assert p["tile0"] == [0, 3, 4] and [t[:3] for t in p["tiles"]] == [(0, 128, 0), (128, 128, 0), (256, 44, 0), (302, 128, 1), (430, 128, 2), (558, 1, 2)]
 
 
 @pytest.mark.parametrize("fault", ["window", "window_parallel", "sink", "cap", "pairs", "head_norm", "v_mix", "gate", "skip", "groups", "residual",
