@@ -1,4 +1,4 @@
-// Descriptor of recurrent mixers with an outer-product state (linear_state.cu, ssd_prefill.cu), plain data mirrored by the Python
+// Descriptor of recurrent mixers with an outer-product state (linear_state.cu, ssd.cu), plain data mirrored by the Python
 // bindings; inputs of the state-space recurrence.
 #pragma once
 #include "pk_common.cuh"

@@ -24,7 +24,7 @@
 //     from a table. The state space needs q k^T only once per group and takes its factors exp(G_i - G_j) dt_j, dt_j
 //     exp(G_C - G_j) and exp(G_i) on the way into the products, where G is held as the sum of two floats.
 // A last kernel normalises every head's output (after mLSTM's division by max(|n.q|, exp(-m)) + 1e-6), applies the output
-// gate and writes the projection's input (state space: the gate comes first, the norm's parts need not be heads).
+// gate and writes the projection's input. Of the state space only the fp32 chunk form is here, its other kernels are in ssd.cu.
 #include "../common/pk_rotary.cuh"
 #include "../common/pk_state.cuh"
 
@@ -85,7 +85,7 @@ struct Raw {
 
 constexpr int GR = 8;   // row groups (warps) of a block
 
-template <int KIND, int RPT, int TAPS>      // TAPS: of the state space's convolution (0: any number)
+template <int KIND, int RPT>
 __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, const Raw raw, const int4* seqs) {
   pdl_trigger();
   pdl_wait();
@@ -134,18 +134,6 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
           ks[i + half] = k[i + half];
         }
       }
-    } else if (KIND == KIND_SSD) {
-      const int b0 = mx.H * V + h / (mx.H / mx.groups) * D;
-      for (int i = threadIdx.x; i < 2 * D; i += 32 * GR) {
-        const bool is_q = i >= D;
-        const int d = is_q ? i - D : i;
-        (is_q ? qs : ks)[d] = conv_silu<TAPS>(mx, sq.z, sq.x + t, t, sq.w + t, b0 + (is_q ? mx.groups * D : 0) + d);
-      }
-      if (threadIdx.x == 0) {
-        const float dt = softplus(pr[mx.odt + h] + mx.dtb[h]);
-        s_sc[0] = expf(mx.A[h] * dt);
-        s_sc[1] = dt;
-      }
     } else {
       for (int d = threadIdx.x; d < D; d += 32 * GR) {
         qs[d] = pr[mx.oq + h * D + d] * mx.qscale;
@@ -168,14 +156,12 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       }
       m_prev = m;
     }
-    float v = is_n ? 1.f : 0.f;
-    if (is_v) v = KIND == KIND_SSD ? conv_silu<TAPS>(mx, sq.z, sq.x + t, t, sq.w + t, h * V + col) : pr[mx.ov + h * V + col];
-    const float x = v;
+    float v = is_v ? pr[mx.ov + h * V + col] : (is_n ? 1.f : 0.f);
     __syncthreads();
     float part = 0.f;
     if (KIND != KIND_GLA) {
-      const float a = KIND == KIND_RETENTION ? decay : s_sc[0];
-      if (KIND != KIND_RETENTION) v *= s_sc[1];
+      const float a = KIND == KIND_MLSTM ? s_sc[0] : decay;
+      if (KIND == KIND_MLSTM) v *= s_sc[1];
 #pragma unroll
       for (int j = 0; j < RPT; ++j) {
         const int d = g + j * GR;
@@ -200,7 +186,6 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       float o = 0.f;
 #pragma unroll
       for (int i = 0; i < GR; ++i) o += red[i * 33 + lane];
-      if (KIND == KIND_SSD) o = fmaf(mx.skip[h], x, o);
       if (is_n) raw.nq[(size_t)(sq.x + t) * mx.H + h] = o;
       else raw.o[((size_t)(sq.x + t) * mx.H + h) * V + col] = o;
     }
@@ -885,56 +870,7 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
     for (int v = H * V + tid; v < ldo; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
 }
 
-// State space: y silu(z), normed in `parts` equal parts of the heads' outputs laid end to end, times norm_w [H * V]. One block per
-// (part, row); columns from H * V up to `width` are set to zero. behind[row]: tokens of the same portion after the row; the
-// last rows of a portion leave their inputs in the convolution's ring.
-template <typename OutT>
-__global__ void __launch_bounds__(1024) ssd_out_kernel(const Mixer mx, const Raw raw, const float* norm_w, float eps, const int* slots, const int* behind,
-                                                       const int* pos, OutT* out, int ldo, int width) {
-  pdl_trigger();
-  pdl_wait();
-  __shared__ float scratch[33];
-  constexpr int KEEP = 4;
-  const int g = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
-  const int inner = mx.H * mx.V, n = inner / gridDim.x;
-  if (behind[t] < mx.taps - 1) {
-    const int CD = ssd_channels(mx), step = gridDim.x * nt;
-    const float* src = mx.proj + (size_t)t * mx.ld + mx.ov;
-    float* ring = mx.Cs + ((size_t)slots[t] * (mx.taps - 1) + pos[t] % (mx.taps - 1)) * CD;
-    for (int ch = g * nt + tid; ch < CD; ch += 4 * step) {
-      float in[4];
-#pragma unroll
-      for (int i = 0; i < 4; ++i) in[i] = ch + i * step < CD ? src[ch + i * step] : 0.f;
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-        if (ch + i * step < CD) ring[ch + i * step] = in[i];
-    }
-  }
-  const float* o = raw.o + (size_t)t * inner + g * n;
-  const float* gate = mx.proj + (size_t)t * mx.ld + mx.og + g * n;
-  float x[KEEP], ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < KEEP; ++i) {
-    const int v = tid + i * nt;
-    x[i] = v < n ? o[v] * silu_exact(gate[v]) : 0.f;
-    ss = fmaf(x[i], x[i], ss);
-  }
-  for (int v = tid + KEEP * nt; v < n; v += nt) {
-    const float y = o[v] * silu_exact(gate[v]);
-    ss = fmaf(y, y, ss);
-  }
-  const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
-  OutT* dst = out + (size_t)t * ldo + g * n;
-  const float* w = norm_w + g * n;
-#pragma unroll
-  for (int i = 0; i < KEEP; ++i)
-    if (tid + i * nt < n) dst[tid + i * nt] = (OutT)(x[i] * r * w[tid + i * nt]);
-  for (int v = tid + KEEP * nt; v < n; v += nt) dst[v] = (OutT)(o[v] * silu_exact(gate[v]) * r * w[v]);
-  if (g == gridDim.x - 1)
-    for (int v = inner + tid; v < width; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
-}
-
-template <int KIND, int TAPS = 0>
+template <int KIND>
 int launch_rows(const Mixer& mx, const Raw& raw, const int4* seqs, int nseq, cudaStream_t stream) {
   const int cols = mx.V + (KIND == KIND_MLSTM ? 1 : 0);
   const dim3 grid((cols + 31) / 32, mx.H, nseq);
@@ -942,7 +878,7 @@ int launch_rows(const Mixer& mx, const Raw& raw, const int4* seqs, int nseq, cud
   const int rpt = (mx.D + GR - 1) / GR;
 #define PK_ROWS_CASE(n)                                                                             \
   if (rpt <= n) {                                                                                   \
-    PK_LAUNCH_PDL((state_rows_kernel<KIND, n, TAPS>), grid, dim3(32 * GR), smem, stream, mx, raw, seqs);  \
+    PK_LAUNCH_PDL((state_rows_kernel<KIND, n>), grid, dim3(32 * GR), smem, stream, mx, raw, seqs);  \
     return PK_OK;                                                                                   \
   }
   PK_ROWS_CASE(4)
@@ -1013,10 +949,7 @@ PK_API int pk_state_rows(const PkStateMixer* d, const void* seqs, int nseq, cuda
   if (!unpack(d, mx, raw) || seqs == nullptr || nseq < 1) return PK_ERR_BAD_ARG;
   switch (d->kind) {
     case KIND_GLA: return launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream);
-    case KIND_SSD:
-      if (mx.taps == 4) return launch_rows<KIND_SSD, 4>(mx, raw, (const int4*)seqs, nseq, stream);
-      if (mx.taps == 3) return launch_rows<KIND_SSD, 3>(mx, raw, (const int4*)seqs, nseq, stream);
-      return launch_rows<KIND_SSD>(mx, raw, (const int4*)seqs, nseq, stream);
+    case KIND_SSD: return PK_ERR_UNSUPPORTED;      // pk_ssd_rows
     case KIND_MLSTM: return launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
     default: return launch_rows<KIND_RETENTION>(mx, raw, (const int4*)seqs, nseq, stream);
   }
@@ -1101,21 +1034,5 @@ PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head
     if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
     else PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
   }
-  return PK_OK;
-}
-
-// State space: gate, norm in `parts` parts, output rows [rows, ldo] of which `width` columns are this layer's; the last inputs of
-// every portion go into the convolution's ring (slots, behind and pos per row).
-PK_API int pk_ssd_out(const PkStateMixer* d, const float* norm_w, int parts, float eps, const int* slots, const int* behind, const int* pos, int rows,
-                      void* out, int ldo, int width, int out_f32, cudaStream_t stream) {
-  Mixer mx;
-  Raw raw;
-  if (!unpack(d, mx, raw) || d->kind != KIND_SSD || norm_w == nullptr || slots == nullptr || behind == nullptr || pos == nullptr || rows < 1 ||
-      rows > 65535 || out == nullptr || parts < 1 || mx.H * mx.V % parts != 0 || width < mx.H * mx.V || ldo < width)
-    return PK_ERR_BAD_ARG;
-  const int n = mx.H * mx.V / parts, nt = (n + 31) / 32 * 32;
-  const dim3 grid(parts, rows), block(nt <= 256 ? nt : n > 2048 ? 1024 : 256);
-  if (out_f32) PK_LAUNCH_PDL(ssd_out_kernel<float>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, slots, behind, pos, (float*)out, ldo, width);
-  else PK_LAUNCH_PDL(ssd_out_kernel<pk::bf16>, grid, block, (size_t)0, stream, mx, raw, norm_w, eps, slots, behind, pos, (pk::bf16*)out, ldo, width);
   return PK_OK;
 }

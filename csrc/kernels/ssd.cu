@@ -1,5 +1,10 @@
-// State-space recurrence of long portions on the 5th-generation tensor cores (bf16 models): tiles of 128 tokens, the same
-// chunked form as in linear_state.cu,
+// State-space recurrence of Mamba-2 (linear_state.cu has its equations and the fp32 chunk form).
+//
+// Rows form (decode, portions of a few tokens): one block per (sequence, head, 32 or 64 value columns), the state slice in
+// registers, tokens in order; the convolution is part of it. A last kernel gates and norms the outputs of all rows and keeps
+// the inputs that later convolutions need.
+//
+// Tiles (long portions of bf16 models) on the 5th-generation tensor cores: the chunked form over 128 tokens,
 //   y_i = e^{G_i} C_i S_c + sum_{j <= i} (C_i . B_j) e^{G_i - G_j} dt_j x_j + D x_i,     S_{c+1} = e^{G_end} S_c + sum_j B_j (dt_j e^{G_end - G_j} x_j)^T
 // with G the running log decay. x, B and C behind their convolution are bf16; what the recurrence makes of them is not: the
 // state, the factors and the sums are fp32, and a fp32 operand enters a product as the sum of two bf16 terms (16 significant
@@ -19,6 +24,237 @@ namespace {
 
 using namespace pk;
 using namespace pk::sm100;
+
+// ---------------------------------------------------------------------------------------
+// rows
+
+constexpr int GR = 8;   // row groups (warps) of a block
+
+template <int RPT, int TAPS, int VW>      // state rows per thread, taps (0: any number), adjacent value columns per thread
+__global__ void __launch_bounds__(32 * GR) ssd_rows_kernel(const PkStateMixer m, const int4* seqs) {
+  pdl_trigger();
+  pdl_wait();
+  constexpr int W = 32 * VW;
+  extern __shared__ float sm[];
+  float* qs = sm;                 // [D] C
+  float* ks = qs + m.D;           // [D] B
+  float* xs = ks + m.D;           // [W] x
+  float* red = xs + W;            // [GR][W]
+  __shared__ float s_sc[2];
+  const int4 sq = seqs[blockIdx.z];          // first row, tokens, slot, first position
+  const int h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, g = tid >> 5;
+  const int D = m.D, V = m.V, col0 = blockIdx.x * W, col = col0 + lane * VW;
+  const bool live = col < V;                 // VW 2: V is even
+  float* Sp = m.S + ((size_t)sq.z * m.H + h) * D * V + col;
+  float s[RPT][VW];
+#pragma unroll
+  for (int j = 0; j < RPT; ++j) {
+    const int d = g + j * GR;
+#pragma unroll
+    for (int k = 0; k < VW; ++k) s[j][k] = 0.f;
+    if (live && d < D && sq.w > 0) {
+      if (VW == 2) {
+        const float2 v = *reinterpret_cast<const float2*>(Sp + (size_t)d * V);
+        s[j][0] = v.x;
+        s[j][1 % VW] = v.y;
+      } else {
+        s[j][0] = Sp[(size_t)d * V];
+      }
+    }
+  }
+  const int b0 = m.H * V + h / (m.H / m.groups) * D;
+  const float skip = m.skip[h];
+  for (int t = 0; t < sq.y; ++t) {
+    const int row = sq.x + t, pos = sq.w + t;
+    for (int i = tid; i < 2 * D; i += 32 * GR) {
+      const bool is_q = i >= D;
+      const int d = is_q ? i - D : i;
+      (is_q ? qs : ks)[d] = conv_silu<TAPS>(m, sq.z, row, t, pos, b0 + (is_q ? m.groups * D : 0) + d);
+    }
+    if (tid < W && col0 + tid < V) xs[tid] = conv_silu<TAPS>(m, sq.z, row, t, pos, h * V + col0 + tid);
+    if (tid == 32 * GR - 1) {
+      const float dt = softplus(m.proj[(size_t)row * m.ld + m.odt + h] + m.dtb[h]);
+      s_sc[0] = expf(m.A[h] * dt);
+      s_sc[1] = dt;
+    }
+    __syncthreads();
+    float v[VW], part[VW];
+#pragma unroll
+    for (int k = 0; k < VW; ++k) {
+      v[k] = live ? xs[lane * VW + k] * s_sc[1] : 0.f;
+      part[k] = 0.f;
+    }
+    const float a = s_sc[0];
+#pragma unroll
+    for (int j = 0; j < RPT; ++j) {
+      const int d = g + j * GR;
+      if (d < D) {
+        const float kd = ks[d], qd = qs[d];
+#pragma unroll
+        for (int k = 0; k < VW; ++k) {
+          s[j][k] = fmaf(a, s[j][k], kd * v[k]);
+          part[k] = fmaf(s[j][k], qd, part[k]);
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < VW; ++k) red[g * W + lane * VW + k] = part[k];
+    __syncthreads();
+    if (tid < W && col0 + tid < V) {
+      float o = skip * xs[tid];
+#pragma unroll
+      for (int i = 0; i < GR; ++i) o += red[i * W + tid];
+      m.o[((size_t)row * m.H + h) * V + col0 + tid] = o;
+    }
+    if (t + 1 < sq.y) __syncthreads();
+  }
+  if (live) {
+#pragma unroll
+    for (int j = 0; j < RPT; ++j) {
+      const int d = g + j * GR;
+      if (d < D) {
+        if (VW == 2) *reinterpret_cast<float2*>(Sp + (size_t)d * V) = make_float2(s[j][0], s[j][1 % VW]);
+        else Sp[(size_t)d * V] = s[j][0];
+      }
+    }
+  }
+}
+
+template <int TAPS, int VW>
+int launch_rows(const PkStateMixer& m, const int4* seqs, int nseq, cudaStream_t stream) {
+  const dim3 grid((m.V + 32 * VW - 1) / (32 * VW), m.H, nseq);
+  const size_t smem = (size_t)(2 * m.D + (GR + 1) * 32 * VW) * sizeof(float);
+  const int rpt = (m.D + GR - 1) / GR;
+#define PK_ROWS_CASE(n)                                                                           \
+  if (rpt <= n) {                                                                                 \
+    PK_LAUNCH_PDL((ssd_rows_kernel<n, TAPS, VW>), grid, dim3(32 * GR), smem, stream, m, seqs);    \
+    return PK_OK;                                                                                 \
+  }
+  PK_ROWS_CASE(4)
+  PK_ROWS_CASE(8)
+  PK_ROWS_CASE(16)
+  PK_ROWS_CASE(32)
+  PK_ROWS_CASE(64)
+#undef PK_ROWS_CASE
+  return PK_ERR_UNSUPPORTED;
+}
+
+template <int VW>
+int launch_rows(const PkStateMixer& m, const int4* seqs, int nseq, cudaStream_t stream) {
+  if (m.taps == 4) return launch_rows<4, VW>(m, seqs, nseq, stream);
+  if (m.taps == 3) return launch_rows<3, VW>(m, seqs, nseq, stream);
+  return launch_rows<0, VW>(m, seqs, nseq, stream);
+}
+
+// ---------------------------------------------------------------------------------------
+// gate, norm
+
+template <int VW>
+__device__ __forceinline__ void load_f32(const float* p, float (&v)[VW]) {
+  if (VW == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1 % VW] = x.y; v[2 % VW] = x.z; v[3 % VW] = x.w;
+  } else {
+    v[0] = *p;
+  }
+}
+template <int VW>
+__device__ __forceinline__ void store(float* p, const float (&v)[VW]) {
+  if (VW == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % VW], v[2 % VW], v[3 % VW]);
+  else *p = v[0];
+}
+template <int VW>
+__device__ __forceinline__ void store(bf16* p, const float (&v)[VW]) {
+  if (VW == 4) {
+    const bf162 a = __floats2bfloat162_rn(v[0], v[1 % VW]), b = __floats2bfloat162_rn(v[2 % VW], v[3 % VW]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16(v[0]);
+  }
+}
+
+// y silu(z), normed in gridDim.x equal parts of the heads' outputs laid end to end, times norm_w [H * V]. One block per (part,
+// row); columns from H * V up to `width` are set to zero. behind[row]: tokens of the same portion after the row; the last rows of
+// a portion leave their inputs in the convolution's ring.
+template <typename OutT, int VW>
+__global__ void __launch_bounds__(1024) ssd_out_kernel(const PkStateMixer m, const float* norm_w, float eps, const int* slots, const int* behind, const int* pos,
+                                                       OutT* out, int ldo, int width) {
+  pdl_trigger();
+  pdl_wait();
+  __shared__ float scratch[33];
+  constexpr int KEEP = 4;
+  const int g = blockIdx.x, t = blockIdx.y, tid = threadIdx.x, nt = blockDim.x;
+  const int inner = m.H * m.V, n = inner / gridDim.x;
+  if (behind[t] < m.taps - 1) {
+    const int CD = ssd_channels(m), step = gridDim.x * nt;
+    const float* src = m.proj + (size_t)t * m.ld + m.ov;
+    float* ring = m.Cs + ((size_t)slots[t] * (m.taps - 1) + pos[t] % (m.taps - 1)) * CD;
+    for (int ch = g * nt + tid; ch < CD; ch += 4 * step) {
+      float in[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) in[i] = ch + i * step < CD ? src[ch + i * step] : 0.f;
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+        if (ch + i * step < CD) ring[ch + i * step] = in[i];
+    }
+  }
+  const float* o = m.o + (size_t)t * inner + g * n;
+  const float* gate = m.proj + (size_t)t * m.ld + m.og + g * n;
+  auto gated = [&](int v, float (&x)[VW]) {
+    float z[VW];
+    load_f32<VW>(o + v, x);
+    load_f32<VW>(gate + v, z);
+#pragma unroll
+    for (int k = 0; k < VW; ++k) x[k] *= silu_exact(z[k]);
+  };
+  float x[KEEP][VW], ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i) {
+    const int v = (tid + i * nt) * VW;
+    if (v >= n) continue;
+    gated(v, x[i]);
+#pragma unroll
+    for (int k = 0; k < VW; ++k) ss = fmaf(x[i][k], x[i][k], ss);
+  }
+  for (int v = (tid + KEEP * nt) * VW; v < n; v += nt * VW) {
+    float y[VW];
+    gated(v, y);
+#pragma unroll
+    for (int k = 0; k < VW; ++k) ss = fmaf(y[k], y[k], ss);
+  }
+  const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  OutT* dst = out + (size_t)t * ldo + g * n;
+  auto put = [&](int v, float (&y)[VW]) {
+    float w[VW];
+    load_f32<VW>(norm_w + g * n + v, w);
+#pragma unroll
+    for (int k = 0; k < VW; ++k) y[k] *= r * w[k];
+    store<VW>(dst + v, y);
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; ++i)
+    if ((tid + i * nt) * VW < n) put((tid + i * nt) * VW, x[i]);
+  for (int v = (tid + KEEP * nt) * VW; v < n; v += nt * VW) {
+    float y[VW];
+    gated(v, y);
+    put(v, y);
+  }
+  if (g == gridDim.x - 1)
+    for (int v = inner + tid; v < width; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
+}
+
+template <typename OutT, int VW>
+int launch_out(const PkStateMixer& m, const float* norm_w, int parts, float eps, const int* slots, const int* behind, const int* pos, int rows, OutT* out, int ldo,
+               int width, cudaStream_t stream) {
+  const int groups = (m.H * m.V / parts + VW - 1) / VW, per = rows > 64 ? 2 : 1;
+  int nt = ((groups + per - 1) / per + 31) / 32 * 32;
+  if (nt > 1024) nt = 1024;
+  PK_LAUNCH_PDL((ssd_out_kernel<OutT, VW>), dim3(parts, rows), dim3(nt), (size_t)0, stream, m, norm_w, eps, slots, behind, pos, out, ldo, width);
+  return PK_OK;
+}
+
+// ---------------------------------------------------------------------------------------
+// tiles
 
 constexpr int L = 128;               // tokens of a tile
 constexpr int NP = 128;              // padded state dimension
@@ -157,10 +393,13 @@ __global__ void __launch_bounds__(128) ssd_tile_kv_kernel(const __grid_constant_
     const float2 g = p.G[unit * L + tid], e = p.G[unit * L + L - 1];
     const float w = p.dt[unit * L + tid] * expf((e.x - g.x) + (e.y - g.y));
     const uint4* src = reinterpret_cast<const uint4*>(p.xbc + ((size_t)c * L + tid) * p.cols + h * VP);
+    uint4 raw[VP / 8];
+#pragma unroll
+    for (int k = 0; k < VP / 8; ++k) raw[k] = src[k];
 #pragma unroll
     for (int k = 0; k < VP / 8; ++k) {
       float f[8];
-      unpack8(src[k], f);
+      unpack8(raw[k], f);
       uint32_t hi[4], lo[4];
 #pragma unroll
       for (int i = 0; i < 4; ++i) split2(f[2 * i] * w, f[2 * i + 1] * w, hi[i], lo[i]);
@@ -288,36 +527,44 @@ __global__ void __launch_bounds__(128) ssd_tile_out_kernel(const __grid_constant
   gs[tid] = p.G[unit * L + tid];
   dts[tid] = p.dt[unit * L + tid];
   {
-    // state rows (one per state dimension) as two terms; 8 columns at a time, neighbouring threads on neighbouring pieces
+    // state rows (one per state dimension) as two terms; 8 columns at a time, neighbouring threads on neighbouring pieces,
+    // four pieces of a thread in flight
     const float* S = p.KV + unit * m.D * m.V;
     const bool v4 = (m.V & 3) == 0;
-    constexpr int PIECES = VP / 8;
-    for (int i = tid; i < NP * PIECES; i += 128) {
-      const int n = i / PIECES, k = i % PIECES;
-      float f[8];
+    constexpr int PIECES = VP / 8, AHEAD = 4;
+#pragma unroll 1
+    for (int i0 = tid; i0 < NP * PIECES; i0 += 128 * AHEAD) {
+      float f[AHEAD][8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) f[e] = 0.f;
-      if (n < m.D) {
+      for (int a = 0; a < AHEAD; ++a) {
+        const int n = (i0 + a * 128) / PIECES, k = (i0 + a * 128) % PIECES;
         const float* src = S + (size_t)n * m.V + k * 8;
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[a][e] = 0.f;
+        if (n >= m.D) continue;
         if (v4) {
 #pragma unroll
           for (int q = 0; q < 2; ++q)
             if (k * 8 + q * 4 < m.V) {
               const float4 x = *reinterpret_cast<const float4*>(src + q * 4);
-              f[q * 4] = x.x; f[q * 4 + 1] = x.y; f[q * 4 + 2] = x.z; f[q * 4 + 3] = x.w;
+              f[a][q * 4] = x.x; f[a][q * 4 + 1] = x.y; f[a][q * 4 + 2] = x.z; f[a][q * 4 + 3] = x.w;
             }
         } else {
 #pragma unroll
           for (int e = 0; e < 8; ++e)
-            if (k * 8 + e < m.V) f[e] = src[e];
+            if (k * 8 + e < m.V) f[a][e] = src[e];
         }
       }
-      uint32_t hi[4], lo[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) split2(f[2 * e], f[2 * e + 1], hi[e], lo[e]);
-      uint8_t* dst = ss + (k >> 3) * kPanel + n * 128 + (((k & 7) ^ (n & 7)) << 4);
-      *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-      *reinterpret_cast<uint4*>(dst + NV * kPanel) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      for (int a = 0; a < AHEAD; ++a) {
+        const int n = (i0 + a * 128) / PIECES, k = (i0 + a * 128) % PIECES;
+        uint32_t hi[4], lo[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) split2(f[a][2 * e], f[a][2 * e + 1], hi[e], lo[e]);
+        uint8_t* dst = ss + (k >> 3) * kPanel + n * 128 + (((k & 7) ^ (n & 7)) << 4);
+        *reinterpret_cast<uint4*>(dst) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+        *reinterpret_cast<uint4*>(dst + NV * kPanel) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+      }
     }
   }
   fence_proxy_async_smem();
@@ -485,7 +732,7 @@ int launch(const CUtensorMap& map, const Params& p, int ntiles, int nseq, cudaSt
   }
   const PkStateMixer& m = p.m;
   const int cb = (p.cols + 255) / 256;
-  const dim3 in_grid(ntiles, cb + (m.H + 7) / 8, 4);
+  const dim3 in_grid(ntiles, cb + (m.H + 7) / 8, 8);      // 16 rows per block
   if (m.taps == 2) ssd_tile_inputs_kernel<2><<<in_grid, 256, 0, stream>>>(p, cb);
   else if (m.taps == 3) ssd_tile_inputs_kernel<3><<<in_grid, 256, 0, stream>>>(p, cb);
   else if (m.taps == 4) ssd_tile_inputs_kernel<4><<<in_grid, 256, 0, stream>>>(p, cb);
@@ -502,6 +749,11 @@ int launch(const CUtensorMap& map, const Params& p, int ntiles, int nseq, cudaSt
   return PK_OK;
 }
 
+bool ssd_ok(const PkStateMixer* d) {
+  return d != nullptr && d->proj != nullptr && d->S != nullptr && d->o != nullptr && d->cw != nullptr && d->cb != nullptr && d->dtb != nullptr && d->A != nullptr &&
+         d->skip != nullptr && d->H >= 1 && d->D >= 1 && d->V >= 1 && d->groups >= 1 && d->H % d->groups == 0 && d->taps >= 1 && (d->taps == 1 || d->Cs != nullptr);
+}
+
 }  // namespace
 
 // Workspace floats of pk_ssd_tiles; 0 when the shape does not fit it.
@@ -516,9 +768,7 @@ PK_API size_t pk_ssd_tile_workspace(const PkStateMixer* d, int ntiles) {
 // [ntiles] = {first row, rows (1..128), portion, unused}, those of a portion one after the other from tile0[portion] on.
 PK_API int pk_ssd_tiles(const PkStateMixer* d, const void* seqs, int nseq, const void* tiles, const int* tile0, int ntiles, float* ws, uint32_t* status,
                         cudaStream_t stream) {
-  if (d == nullptr || d->proj == nullptr || d->S == nullptr || d->o == nullptr || d->cw == nullptr || d->cb == nullptr || d->dtb == nullptr || d->A == nullptr ||
-      d->skip == nullptr || d->Cs == nullptr || d->H < 1 || d->D < 1 || d->V < 1 || d->groups < 1 || d->H % d->groups != 0 || d->taps < 1 || seqs == nullptr ||
-      tiles == nullptr || tile0 == nullptr || nseq < 1 || ntiles < nseq || ntiles > 65535 || ws == nullptr || ((uintptr_t)ws & 255) != 0 ||
+  if (!ssd_ok(d) || seqs == nullptr || tiles == nullptr || tile0 == nullptr || nseq < 1 || ntiles < nseq || ntiles > 65535 || ws == nullptr || ((uintptr_t)ws & 255) != 0 ||
       ((uintptr_t)d->o & 15) != 0)
     return PK_ERR_BAD_ARG;
   if (d->D > NP || d->V > 128) return PK_ERR_UNSUPPORTED;
@@ -538,4 +788,30 @@ PK_API int pk_ssd_tiles(const PkStateMixer* d, const void* seqs, int nseq, const
              CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
     return PK_ERR_CUDA;
   return p.vp == 64 ? launch<64>(map, p, ntiles, nseq, stream) : launch<128>(map, p, ntiles, nseq, stream);
+}
+
+// Tokens of short portions, one after the other: outputs in `o`, states. seqs as above.
+PK_API int pk_ssd_rows(const PkStateMixer* d, const void* seqs, int nseq, int sm_count, cudaStream_t stream) {
+  if (!ssd_ok(d) || seqs == nullptr || nseq < 1 || d->D > 512) return PK_ERR_BAD_ARG;
+  const long long blocks = (long long)((d->V + 31) / 32) * d->H * nseq;      // narrow ones, while the machine is not full
+  if ((d->V & 1) == 0 && ((uintptr_t)d->S & 7) == 0 && blocks > 2LL * (sm_count > 0 ? sm_count : 148) && d->V > 32)
+    return launch_rows<2>(*d, (const int4*)seqs, nseq, stream);
+  return launch_rows<1>(*d, (const int4*)seqs, nseq, stream);
+}
+
+// Gate, norm in `parts` parts, output rows [rows, ldo] of which `width` columns are this layer's; the last inputs of every
+// portion go into the convolution's ring (slots, behind and pos per row).
+PK_API int pk_ssd_out(const PkStateMixer* d, const float* norm_w, int parts, float eps, const int* slots, const int* behind, const int* pos, int rows,
+                      void* out, int ldo, int width, int out_f32, cudaStream_t stream) {
+  if (!ssd_ok(d) || norm_w == nullptr || slots == nullptr || behind == nullptr || pos == nullptr || rows < 1 || rows > 65535 || out == nullptr || parts < 1 ||
+      d->H * d->V % parts != 0 || width < d->H * d->V || ldo < width)
+    return PK_ERR_BAD_ARG;
+  const bool v4 = (d->H * d->V / parts & 3) == 0 && (d->ld & 3) == 0 && (d->og & 3) == 0 && ((uintptr_t)d->proj & 15) == 0 && ((uintptr_t)d->o & 15) == 0 &&
+                  ((uintptr_t)norm_w & 15) == 0 && (ldo & 3) == 0 && ((uintptr_t)out & 15) == 0;
+  float* f = (float*)out;
+  pk::bf16* b = (pk::bf16*)out;
+  if (v4) return out_f32 ? launch_out<float, 4>(*d, norm_w, parts, eps, slots, behind, pos, rows, f, ldo, width, stream)
+                         : launch_out<pk::bf16, 4>(*d, norm_w, parts, eps, slots, behind, pos, rows, b, ldo, width, stream);
+  return out_f32 ? launch_out<float, 1>(*d, norm_w, parts, eps, slots, behind, pos, rows, f, ldo, width, stream)
+                 : launch_out<pk::bf16, 1>(*d, norm_w, parts, eps, slots, behind, pos, rows, b, ldo, width, stream);
 }

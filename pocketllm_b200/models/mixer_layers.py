@@ -74,16 +74,16 @@ class StepContext:
 
 class FusedLinear:
     """Row blocks of several matrices that share their input as one [N, K] matrix, padded with zeros to what the kernels
-    take; `at[name]` is the first output column of a block."""
+    take; `at[name]` is the first output column of a block (a multiple of `align`)."""
 
-    def __init__(self, blocks: list[tuple[str, torch.Tensor]], dtype: torch.dtype, device, k_pad: int | None = None):
+    def __init__(self, blocks: list[tuple[str, torch.Tensor]], dtype: torch.dtype, device, k_pad: int | None = None, align: int = 1):
         K = blocks[0][1].shape[1]
         self.K = k_pad or pad_to(K, 64)
         self.at, n = {}, 0
         for name, w in blocks:
             if w.shape[1] != K:
                 raise ValueError(f"{name}: {w.shape[1]} input columns, the others have {K}")
-            self.at[name] = n
+            self.at[name] = n = pad_to(n, align)
             n += w.shape[0]
         self.N = pad_to(n, 8)
         w = torch.zeros(self.N, self.K, dtype=dtype)
@@ -229,7 +229,7 @@ class StateSpaceMixer:
         o = ws.flat("raw_o", ctx.T * self.H * self.V, torch.float32)
         d = mo.StateMixer(proj=p.data_ptr(), ld=p.stride(0), o=o.data_ptr(), **self.desc)
         if ctx.n_short:
-            mo.state_rows(d, ctx.short, ctx.n_short)
+            mo.ssd_rows(d, ctx.short, ctx.n_short)
         if ctx.n_long:
             n = mo.ssd_tile_workspace(d, ctx.n_tiles) if self.dtype == torch.bfloat16 else 0
             if n:
@@ -472,7 +472,7 @@ class ParallelMixer:
 
     def __init__(self, left: GroupedAttention, right: StateSpaceMixer, w_left: dict, w_right: dict, dtype, device):
         self.left, self.right, self.dtype = left, right, dtype
-        self.proj = FusedLinear([("left." + n, t) for n, t in left.blocks(w_left)] + [("right", w_right["in"])], dtype, device)
+        self.proj = FusedLinear([("left." + n, t) for n, t in left.blocks(w_left)] + [("right", w_right["in"])], dtype, device, align=4)
         left.at(self.proj.at, "left.")
         right.at(self.proj.at["right"])
         n = left.H * left.V

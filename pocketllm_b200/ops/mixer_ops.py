@@ -54,7 +54,7 @@ def sm_count() -> int:
 _SIGNATURES = {
     "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
     "pk_sandwich_norm": "pppifipipifpiippp" "iipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
-    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii", "pk_ssd_tiles": "ppippipp",
+    "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii", "pk_ssd_tiles": "ppippipp", "pk_ssd_rows": "ppii",
     "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipi",
     "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipi", "pk_latent_prefill": "pipipippiiiiifppip",
     "pk_paged_prep": "pi", "pk_paged_rows": "ppi", "pk_paged_merge": "ppi", "pk_paged_prefill": "piipip",
@@ -147,6 +147,11 @@ def state_chunks(d: StateMixer, seqs: torch.Tensor, nseq: int, chunks: torch.Ten
 def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
     """Head norm + output gate of `rows` rows; norm_w [H * V], [V] when `per_head`, or None."""
     _call("pk_state_out", byref(d), norm_w, int(per_head), eps, last_slot, rows, out, out.stride(0), int(out.dtype == torch.float32))
+
+
+def ssd_rows(d: StateMixer, seqs: torch.Tensor, nseq: int) -> None:
+    """Recurrence of short portions of a state-space layer, its convolution included."""
+    _call("pk_ssd_rows", byref(d), seqs, nseq, sm_count())
 
 
 def ssd_tile_workspace(d: StateMixer, ntiles: int) -> int:

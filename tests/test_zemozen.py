@@ -83,7 +83,7 @@ def test_layers_of_the_model():
     assert left.const["sink"].tolist() == [0.0] * 4 and left.desc["post"] == 1.0 and m.layers[0].mixer.left.desc["post"] == pytest.approx(0.7)
     assert left.const["freq"].tolist() == pytest.approx([700.0 ** (-2 * i / 40) / 2.0 for i in range(20)])
     a = p.proj.at
-    assert (left.desc["oq"], left.desc["ok"], left.desc["ov"]) == (0, 4 * 40, 5 * 40) and a["right"] == 5 * 40 + 130
+    assert (left.desc["oq"], left.desc["ok"], left.desc["ov"]) == (0, 4 * 40, 5 * 40) and a["right"] == 5 * 40 + 132
     assert (right.desc["og"], right.desc["ov"], right.desc["odt"]) == (a["right"], a["right"] + 132, a["right"] + 2 * 132 + 140)
     assert right.S.shape == (3, 4, 70, 33) and right.ring.shape == (3, 2, 132 + 140) and left.cache.shape == (5, 64, 40 + 136)
     assert p.split == 520 and torch.equal(p.out.w[:88, 520:520 + 132], t["l3.mix.right.o"]) and (p.out.w[:, 652:] == 0).all()
