@@ -24,6 +24,7 @@ struct PkStateMixer {
   const float* A;
   const float* skip;
   float* Cs;
+  const float* low;
   int kind, ld, oq, ok, ov, og, oi, of, oa, H, D, V, rank, rot, groups, taps, odt;
   float qscale, cap, inv_tau;
 };

@@ -1,6 +1,8 @@
 // Latent attention over a paged cache: a cached row is [latent c (rms-normed) | rotated key part | zero padding], shared by
 // all heads; per head the unrotated key is W_uk c and the value W_uv c. Causal with an optional sliding window and an
-// optional learned sink per head (a score without key and value that counts once in the denominator).
+// optional learned sink per head (a score without key and value that counts once in the denominator). The rotated part may be
+// empty; queries may come from a latent of their own (normed by prep, expanded by a product behind it); the heads' outputs may be
+// multiplied with a sigmoid gate, element by element.
 //
 //   prep     per row: norm of the latent, rotation (rotate-half, any frequency table) of key part and queries, cache
 //            append, queries for the tensor-core kernel
@@ -48,9 +50,24 @@ struct PrepParams {
   float* qx;              // [rows, H, row]: columns K .. K + R <- rotated query, the padding <- 0 (null: skip)
   bf16* qf;               // [rows, H, qf_ld]: whole rotated query, padding <- 0 (null: skip)
   int qf_ld;
+  // queries from a latent: QK columns at oq -> normed rows for the product that expands them
+  int QK;                 // 0: the queries themselves are in proj
+  const float* q_norm;    // [QK]
+  void* ql;               // [rows, ql_ld], the cache's type, padding <- 0
+  int ql_ld;
 };
 
-// Block (row, group of eight heads), one warp per head; the first group also writes the cache row.
+// dst[0 .. n) = normed src times w, zeros up to `padded`. Whole block.
+template <typename T>
+__device__ __forceinline__ void norm_row(const float* src, int n, const float* w, float eps, T* dst, int padded, float* scratch) {
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+  const float r = 1.f / sqrtf(block_sum(ss, scratch) / (float)n + eps);
+  for (int i = threadIdx.x; i < padded; i += blockDim.x) dst[i] = (T)(i < n ? src[i] * r * w[i] : 0.f);
+}
+
+// Block (row, group of eight heads), one warp per head; the first group also writes the cache row. Queries from a latent: the second
+// block of a row norms it.
 template <typename CT>
 __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
   pdl_trigger();
@@ -60,6 +77,10 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
   const int warp = tid >> 5, lane = tid & 31;
   pdl_wait();
   const float* pr = p.proj + (size_t)t * p.ld;
+  if (p.QK > 0 && blockIdx.y == 1) {
+    norm_row<CT>(pr + p.oq, p.QK, p.q_norm, p.eps, reinterpret_cast<CT*>(p.ql) + (size_t)t * p.ql_ld, p.ql_ld, scratch);
+    return;
+  }
   const int pos = p.pos[t];
   float* cs = sm;
   float* sn = sm + half;
@@ -91,7 +112,7 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const PrepParams p) {
     __syncthreads();
   }
   const int h = blockIdx.y * 8 + warp;
-  if (h >= p.H) return;
+  if (h >= p.H || p.QK > 0) return;
   const float* q = pr + p.oq + h * (p.D + p.R);
   const float* qr = q + p.D;
   auto rotated = [&](int j) {
@@ -120,9 +141,10 @@ __global__ void __launch_bounds__(128) latent_gather_kernel(const Paged c, const
   }
 }
 
-// qx[row, h, 0 .. K) = W_uk[h]^T q[h]. Block: 128 latent columns of one head, up to 8 rows, 4 groups over the head dim.
+// qx[row, h, 0 .. K) = W_uk[h]^T q[h], zeros up to K_pad (what lies behind belongs to prep). Block: 128 latent columns of one head,
+// up to 8 rows, 4 groups over the head dim.
 template <typename WT>
-__global__ void __launch_bounds__(512) latent_absorb_kernel(const float* proj, int ld, int oq, int H, int D, int R, int K, const WT* uk,
+__global__ void __launch_bounds__(512) latent_absorb_kernel(const float* proj, int ld, int oq, int H, int D, int R, int K, int K_pad, const WT* uk,
                                                            const int* rows, int nrows, float* qx, int row) {
   pdl_trigger();
   pdl_wait();
@@ -153,7 +175,7 @@ __global__ void __launch_bounds__(512) latent_absorb_kernel(const float* proj, i
   __syncthreads();
   for (int i = threadIdx.x; i < nr * 128; i += 512) {
     const int r = i >> 7, c = i & 127;
-    if (blockIdx.y * 128 + c < K)
+    if (blockIdx.y * 128 + c < K_pad)      // columns behind K have summed nothing
       qx[((size_t)rows[r0 + r] * H + h) * row + blockIdx.y * 128 + c] =
           red[r * 128 + c] + red[(8 + r) * 128 + c] + red[(16 + r) * 128 + c] + red[(24 + r) * 128 + c];
   }
@@ -297,6 +319,8 @@ struct OutParams {
   int nrows;
   void* out;              // [rows of the step, ldo]
   int ldo;
+  const float* gate;      // [rows of the step, ldg] logits of the gate, head h at h V (null: none)
+  int ldg;
 };
 
 // o~[row, h, k] = sum over the splits, divided by the whole denominator (sink included). Written over split 0.
@@ -361,8 +385,12 @@ __global__ void __launch_bounds__(256) latent_out_kernel(const OutParams p, cons
 #pragma unroll
     for (int r = 0; r < 8; ++r) {
       if (r >= nr) break;
-      const float s = warp_sum(acc[r]);
-      if (lane == 0) out[(size_t)p.rows[r0 + r] * p.ldo + h * p.V + v] = (OutT)s;
+      float s = warp_sum(acc[r]);
+      if (lane == 0) {
+        const size_t row = p.rows[r0 + r];
+        if (p.gate) s /= 1.f + expf(-p.gate[row * p.ldg + h * p.V + v]);
+        out[row * p.ldo + h * p.V + v] = (OutT)s;
+      }
     }
   }
   if (h == p.H - 1 && blockIdx.z == 0)
@@ -395,15 +423,17 @@ int launch_rows(const RowsParams& p, int nrows, size_t smem, cudaStream_t stream
 
 }  // namespace
 
-// See PrepParams. row (elements per cached position) is a multiple of 8 and at least K + R; R even.
+// See PrepParams. row (elements per cached position) is a multiple of 8 and at least K + R; R even. QK > 0: no rotated part, qx and
+// qf are not written (the expanded queries are another product's output).
 PK_API int pk_latent_prep(const float* proj, int ld, int oq, int oc, int M, int H, int D, int R, int K, const float* c_norm, float eps,
                           const double* freq, float mag, const int* pos, const int* slot, void* cache, const int* table, int table_ld,
-                          int row, int cache_f32, float* qx, void* qf, int qf_ld, cudaStream_t stream) {
+                          int row, int cache_f32, float* qx, void* qf, int qf_ld, int QK, const float* q_norm, void* ql, int ql_ld, cudaStream_t stream) {
   if (M < 1 || H < 1 || D < 1 || R < 0 || (R & 1) != 0 || K < 1 || row < K + R || (row & 7) != 0 || cache == nullptr || table == nullptr) return PK_ERR_BAD_ARG;
   if (qf != nullptr && qf_ld < D + R) return PK_ERR_BAD_ARG;
-  PrepParams p{proj, ld, oq, oc, H, D, R, K, c_norm, eps, freq, mag, pos, slot, Paged{cache, table, table_ld, row}, qx, (pk::bf16*)qf, qf_ld};
+  if (QK < 0 || (QK > 0 && (q_norm == nullptr || ql == nullptr || ql_ld < QK || R != 0))) return PK_ERR_BAD_ARG;
+  PrepParams p{proj, ld, oq, oc, H, D, R, K, c_norm, eps, freq, mag, pos, slot, Paged{cache, table, table_ld, row}, qx, (pk::bf16*)qf, qf_ld, QK, q_norm, ql, ql_ld};
   const size_t smem = (size_t)(R + 2) * sizeof(float);
-  const dim3 grid(M, (qx != nullptr || qf != nullptr) ? (H + 7) / 8 : 1);
+  const dim3 grid(M, QK > 0 ? 2 : (qx != nullptr || qf != nullptr) ? (H + 7) / 8 : 1);
   if (cache_f32) PK_LAUNCH_PDL(latent_prep_kernel<float>, grid, dim3(256), smem, stream, p);
   else PK_LAUNCH_PDL(latent_prep_kernel<pk::bf16>, grid, dim3(256), smem, stream, p);
   return PK_OK;
@@ -420,14 +450,15 @@ PK_API int pk_latent_gather(const void* cache, const int* table, int table_ld, i
   return PK_OK;
 }
 
+// rows [nrows] of the step: qx columns 0 .. K_pad of their heads; R: what lies between the heads' D query columns.
 PK_API int pk_latent_absorb(const float* proj, int ld, int oq, int H, int D, int R, int K, const void* uk, int w_f32, const int* rows, int nrows,
-                            float* qx, int row, cudaStream_t stream) {
-  if (nrows < 1 || H < 1 || D < 1 || K < 1 || qx == nullptr || rows == nullptr) return PK_ERR_BAD_ARG;
+                            float* qx, int row, int K_pad, cudaStream_t stream) {
+  if (nrows < 1 || H < 1 || D < 1 || K < 1 || K_pad < K || row < K_pad || qx == nullptr || rows == nullptr) return PK_ERR_BAD_ARG;
   const size_t smem = (size_t)(8 * D + 4 * 8 * 128) * sizeof(float);
   if (smem > 48 * 1024) return PK_ERR_UNSUPPORTED;
-  const dim3 grid(H, (K + 127) / 128, (nrows + 7) / 8);
-  if (w_f32) PK_LAUNCH_PDL(latent_absorb_kernel<float>, grid, dim3(512), smem, stream, proj, ld, oq, H, D, R, K, (const float*)uk, rows, nrows, qx, row);
-  else PK_LAUNCH_PDL(latent_absorb_kernel<pk::bf16>, grid, dim3(512), smem, stream, proj, ld, oq, H, D, R, K, (const pk::bf16*)uk, rows, nrows, qx, row);
+  const dim3 grid(H, (K_pad + 127) / 128, (nrows + 7) / 8);
+  if (w_f32) PK_LAUNCH_PDL(latent_absorb_kernel<float>, grid, dim3(512), smem, stream, proj, ld, oq, H, D, R, K, K_pad, (const float*)uk, rows, nrows, qx, row);
+  else PK_LAUNCH_PDL(latent_absorb_kernel<pk::bf16>, grid, dim3(512), smem, stream, proj, ld, oq, H, D, R, K, K_pad, (const pk::bf16*)uk, rows, nrows, qx, row);
   return PK_OK;
 }
 
@@ -452,12 +483,12 @@ PK_API int pk_latent_rows(const float* qx, const int* rows, int nrows, const int
   return PK_ERR_UNSUPPORTED;
 }
 
-// Merge of the splits (in place), then W_uv. sink [H] or null.
+// Merge of the splits (in place), then W_uv and the gate. sink [H], gate [rows of the step, ldg] or null.
 PK_API int pk_latent_out(float* part_o, const float* part_ml, int nsplit, int H, int K, int V, const float* sink, const int* rows, int nrows,
-                         const void* uv, int f32, void* out, int ldo, cudaStream_t stream) {
-  if (nrows < 1 || nsplit < 1 || H < 1 || K < 1 || V < 1 || ldo < H * V) return PK_ERR_BAD_ARG;
+                         const void* uv, int f32, void* out, int ldo, const float* gate, int ldg, cudaStream_t stream) {
+  if ((gate != nullptr && ldg < H * V) || nrows < 1 || nsplit < 1 || H < 1 || K < 1 || V < 1 || ldo < H * V) return PK_ERR_BAD_ARG;
   PK_LAUNCH_PDL(latent_merge_kernel, dim3(nrows, H, (K + 127) / 128), dim3(128), (size_t)nsplit * sizeof(float), stream, part_o, part_ml, nsplit, H, K, sink);
-  OutParams p{part_o, nsplit, H, K, V, rows, nrows, out, ldo};
+  OutParams p{part_o, nsplit, H, K, V, rows, nrows, out, ldo, gate, ldg};
   const size_t smem = (size_t)8 * K * sizeof(float);
   const dim3 grid(H, (nrows + 7) / 8, (V + 15) / 16);
   if (f32) {

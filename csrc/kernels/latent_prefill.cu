@@ -1,6 +1,6 @@
 // Prefill attention of long portions on the 5th-generation tensor cores, for latent attention with expanded keys and
 // values (and any attention whose keys and values lie in contiguous rows): causal, optional sliding window, optional
-// learned sink per head, key width a multiple of 64 up to 256, value width a multiple of 64 in slices of up to 128.
+// learned sink per head, optional sigmoid gate on the outputs, key width a multiple of 64 up to 256, value width a multiple of 64 in slices of up to 128.
 //
 // One CTA works one (head, tile of up to 128 query rows of one portion, slice of the value dim). For every 64 positions
 // between the window's first and the causal limit:
@@ -34,6 +34,8 @@ struct Params {
   const float* sink;       // [H] or null
   bf16* out;               // [rows, ldo]
   int ldo;
+  const float* gate;       // [rows, ldg] logits of a sigmoid gate on the outputs, head h at h V (null: none)
+  int ldg;
   uint32_t* status;
 };
 
@@ -240,6 +242,26 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       const float inv = den > 0.f ? f / den : 0.f;
       bf16* dst = p.out + (size_t)(tile.x + r) * p.ldo + h * p.V + vs * 128;
       const int nv = min(VP, p.V - vs * 128);
+#pragma unroll
+      for (int v = 0; v < VP; ++v) o[v] *= inv;
+      if (p.gate) {
+        const float* g = p.gate + (size_t)(tile.x + r) * p.ldg + h * p.V + vs * 128;
+        if ((p.V & 3) == 0 && (p.ldg & 3) == 0 && ((uintptr_t)p.gate & 15) == 0) {
+#pragma unroll
+          for (int v = 0; v < VP / 4; ++v)
+            if (v * 4 < nv) {
+              const float4 x = *reinterpret_cast<const float4*>(g + v * 4);
+              o[v * 4] /= 1.f + __expf(-x.x);
+              o[v * 4 + 1] /= 1.f + __expf(-x.y);
+              o[v * 4 + 2] /= 1.f + __expf(-x.z);
+              o[v * 4 + 3] /= 1.f + __expf(-x.w);
+            }
+        } else {
+#pragma unroll
+          for (int v = 0; v < VP; ++v)
+            if (v < nv) o[v] /= 1.f + __expf(-g[v]);
+        }
+      }
       if ((p.V & 7) == 0) {
 #pragma unroll
         for (int v = 0; v < VP / 8; ++v) {
@@ -247,7 +269,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
             uint32_t w[4];
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-              const __nv_bfloat162 pr = __floats2bfloat162_rn(o[v * 8 + e * 2] * inv, o[v * 8 + e * 2 + 1] * inv);
+              const __nv_bfloat162 pr = __floats2bfloat162_rn(o[v * 8 + e * 2], o[v * 8 + e * 2 + 1]);
               w[e] = *reinterpret_cast<const uint32_t*>(&pr);
             }
             *reinterpret_cast<uint4*>(dst + v * 8) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -256,7 +278,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_c
       } else {
 #pragma unroll
         for (int v = 0; v < VP; ++v)
-          if (v < nv) dst[v] = __float2bfloat16(o[v] * inv);
+          if (v < nv) dst[v] = __float2bfloat16(o[v]);
       }
       if (h == p.H - 1 && vs == 0)
         for (int i = p.H * p.V; i < p.ldo; ++i) p.out[(size_t)(tile.x + r) * p.ldo + i] = __float2bfloat16(0.f);
@@ -315,11 +337,11 @@ int launch(const CUtensorMap& tq, const CUtensorMap& tkv, const Params& p, dim3 
 }  // namespace
 
 // q [rows, H, qk_panels * 64] bf16; kv [kv_rows, H * qk_panels * 64 | H * v_panels * 64] bf16; tiles [ntiles], seqs, gather
-// as in Params; out [rows, ldo] bf16, head h at h * V. window <= 0: full causal.
+// as in Params; out [rows, ldo] bf16, head h at h * V; gate [rows, ldg] or null. window <= 0: full causal.
 PK_API int pk_latent_prefill(const void* q, int rows, const void* kv, int kv_rows, const void* tiles, int ntiles, const void* seqs,
                              const void* gather, int H, int qk_panels, int v_panels, int V, int window, float scale, const float* sink,
-                             void* out, int ldo, uint32_t* status, cudaStream_t stream) {
-  if (rows < 1 || kv_rows < 1 || ntiles < 1 || H < 1 || V < 1 || V > v_panels * 64 || ldo < H * V || (ldo & 7) != 0) return PK_ERR_BAD_ARG;
+                             void* out, int ldo, const float* gate, int ldg, uint32_t* status, cudaStream_t stream) {
+  if ((gate != nullptr && ldg < H * V) || rows < 1 || kv_rows < 1 || ntiles < 1 || H < 1 || V < 1 || V > v_panels * 64 || ldo < H * V || (ldo & 7) != 0) return PK_ERR_BAD_ARG;
   if (qk_panels < 1 || qk_panels > 4 || v_panels < 1) return PK_ERR_UNSUPPORTED;
   if (((uintptr_t)q & 15) != 0 || ((uintptr_t)kv & 15) != 0 || ((uintptr_t)out & 15) != 0) return PK_ERR_BAD_ARG;
   if (v_panels > 1 && (v_panels & 1) != 0) return PK_ERR_UNSUPPORTED;
@@ -329,7 +351,7 @@ PK_API int pk_latent_prefill(const void* q, int rows, const void* kv, int kv_row
   if (!encode_rows64(encode, &tq, q, (uint64_t)H * qk_panels * 64, (uint64_t)rows)) return PK_ERR_CUDA;
   if (!encode_rows64(encode, &tkv, kv, (uint64_t)H * (qk_panels + v_panels) * 64, (uint64_t)kv_rows)) return PK_ERR_CUDA;
   Params p{(const int4*)tiles, (const int4*)seqs, (const int2*)gather, H, qk_panels, v_panels, V, window, scale * 1.4426950408889634f, sink,
-           (pk::bf16*)out, ldo, status};
+           (pk::bf16*)out, ldo, gate, ldg, status};
   if (v_panels == 1) return launch<64>(tq, tkv, p, dim3(ntiles, H, 1), stream);
   return launch<128>(tq, tkv, p, dim3(ntiles, H, v_panels / 2), stream);
 }

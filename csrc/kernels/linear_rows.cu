@@ -1,7 +1,8 @@
 // bf16 linear layers of one to eight rows (decode): the weights are streamed once, y[M, N] = x[M, K] W[N, K]^T with fp32
 // accumulation, fp32 / bf16 output or a SiLU(gate) * up epilogue. A warp owns two weight rows (a gate and its up row for
 // SwiGLU) and, when there are too few rows to fill the machine, a slice of K; the slices of a block are added in a fixed
-// order. The first weights are requested before the wait for the previous kernel.
+// order. The first weights are requested before the wait for the previous kernel. Weight rows from `split` on may have an input of
+// their own: two products whose inputs come from the same step in one launch.
 #include "../common/pk_common.cuh"
 
 namespace {
@@ -13,7 +14,8 @@ constexpr int WARPS = 8;
 
 struct RowsParams {
   const bf16* x;
-  int ldx;
+  const bf16* x2;           // input of weight rows from `split` (even) on
+  int split, ldx;
   const bf16* w;
   int N, K, epi, ksplit;    // ksplit: warps of a block that share a row pair (1, 2, 4, 8)
   void* y;
@@ -41,6 +43,7 @@ __global__ void __launch_bounds__(32 * WARPS) linear_rows_kernel(const RowsParam
   const int n1 = p.epi == OUT_SWIGLU ? g + groups : min(2 * g + 1, p.N - 1);
   const bf16* w0 = p.w + (size_t)(live ? n0 : 0) * p.K;
   const bf16* w1 = p.w + (size_t)(live ? n1 : 0) * p.K;
+  const bf16* x = n0 < p.split ? p.x : p.x2;
   const int stride = 256 * ks;
   int k = sl * 256 + lane * 8;
   uint4 a[U], b[U];
@@ -74,7 +77,7 @@ __global__ void __launch_bounds__(32 * WARPS) linear_rows_kernel(const RowsParam
 #pragma unroll
         for (int m = 0; m < M; ++m) {
           float fx[8];
-          unpack8(*reinterpret_cast<const uint4*>(p.x + (size_t)m * p.ldx + kk), fx);
+          unpack8(*reinterpret_cast<const uint4*>(x + (size_t)m * p.ldx + kk), fx);
 #pragma unroll
           for (int e = 0; e < 8; ++e) {
             acc0[m] = fmaf(fa[e], fx[e], acc0[m]);
@@ -128,9 +131,10 @@ __global__ void __launch_bounds__(32 * WARPS) linear_rows_kernel(const RowsParam
 
 }  // namespace
 
-// x [M <= 8, K] bf16 rows (stride ldx, K and ldx multiples of 8, 16-byte aligned), W [N, K] bf16. epi 0 bf16, 1 SwiGLU (N / 2
-// gate rows, then N / 2 up rows; bf16 out), 2 fp32.
-PK_API int pk_linear_rows(const void* x, int ldx, const void* w, int M, int N, int K, int epi, void* y, int ldy, int sm_count, cudaStream_t stream) {
+// As pk_linear_rows; x2 has the same stride and is the input of the weight rows from `split` (a multiple of 2) on.
+PK_API int pk_linear_rows2(const void* x, const void* x2, int split, int ldx, const void* w, int M, int N, int K, int epi, void* y, int ldy, int sm_count,
+                           cudaStream_t stream) {
+  if (x2 == nullptr || ((uintptr_t)x2 & 15) != 0 || split < 0 || (split & 1) != 0 || (epi == OUT_SWIGLU && split < N)) return PK_ERR_BAD_ARG;
   if (M < 1 || M > 8 || N < 1 || K < 8 || (K & 7) != 0 || (ldx & 7) != 0 || ldx < K || epi < 0 || epi > 2) return PK_ERR_BAD_ARG;
   if (((uintptr_t)x & 15) != 0 || ((uintptr_t)w & 15) != 0 || (epi == OUT_SWIGLU && (N & 1) != 0)) return PK_ERR_BAD_ARG;
   if (ldy < (epi == OUT_SWIGLU ? N / 2 : N)) return PK_ERR_BAD_ARG;
@@ -138,7 +142,7 @@ PK_API int pk_linear_rows(const void* x, int ldx, const void* w, int M, int N, i
   const int want = (sm_count > 0 ? sm_count : 148) * 16;      // warps that keep enough loads in flight
   int ks = 1;
   while (ks < WARPS && groups * ks < want && K >= 512 * ks * 2) ks *= 2;
-  RowsParams p{(const pk::bf16*)x, ldx, (const pk::bf16*)w, N, K, epi, ks, y, ldy};
+  RowsParams p{(const pk::bf16*)x, (const pk::bf16*)x2, split, ldx, (const pk::bf16*)w, N, K, epi, ks, y, ldy};
   const dim3 grid((groups + WARPS / ks - 1) / (WARPS / ks)), block(32 * WARPS);
   switch (M) {
     case 1: PK_LAUNCH_PDL((linear_rows_kernel<1, 4>), grid, block, (size_t)0, stream, p); break;
@@ -151,4 +155,10 @@ PK_API int pk_linear_rows(const void* x, int ldx, const void* w, int M, int N, i
     default: PK_LAUNCH_PDL((linear_rows_kernel<8, 2>), grid, block, (size_t)0, stream, p); break;
   }
   return PK_OK;
+}
+
+// x [M <= 8, K] bf16 rows (stride ldx, K and ldx multiples of 8, 16-byte aligned), W [N, K] bf16. epi 0 bf16, 1 SwiGLU (N / 2
+// gate rows, then N / 2 up rows; bf16 out), 2 fp32.
+PK_API int pk_linear_rows(const void* x, int ldx, const void* w, int M, int N, int K, int epi, void* y, int ldy, int sm_count, cudaStream_t stream) {
+  return pk_linear_rows2(x, x, (N + 1) & ~1, ldx, w, M, N, K, epi, y, ldy, sm_count, stream);
 }

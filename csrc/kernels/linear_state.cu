@@ -1,12 +1,13 @@
 // Recurrent mixers with an outer-product state: gated linear attention (a decay per key channel), the matrix memory of
-// xLSTM (scalar gates with a running maximum), retention (a constant decay per head, rotated queries and keys) and the
-// state-space recurrence of Mamba-2 (a scalar decay per token and head). All are
+// xLSTM (scalar gates with a running maximum), retention (a constant decay per head, rotated queries and keys), the state-space
+// recurrence of Mamba-2 (a scalar decay per token and head) and HGRN2 (a forget gate per key channel which is also the key). All are
 //   S_t = diag(a_t) S_{t-1} + b_t k_t v_t^T,    o_t = S_t^T q_t          S: [key dim, value dim], fp32
 // with a_t a vector (GLA: a = sigmoid(z)^(1/tau), b = 1) or a scalar (mLSTM: a = exp(f + m_{t-1} - m_t), b = exp(i - m_t),
 // m_t = max(f + m_{t-1}, i), m_0 = 0, and a normaliser n updated like a column of S with v = 1; retention: a = const, b = 1;
 // state space: k = B, q = C, v = x, a = exp(A dt), b = dt, dt = softplus(z + bias), B and C shared by a group of heads, and
 // o_t gets D x_t). The state-space inputs x, B and C pass a short causal convolution per channel and SiLU first; its last
-// inputs are part of a request's state, a ring [slot][position modulo (taps - 1)][channel].
+// inputs are part of a request's state, a ring [slot][position modulo (taps - 1)][channel]. HGRN2: a = f = l + (1 - l) sigmoid(z +
+// bias) with a lower bound l per channel, k = 1 - f, b = 1, q = silu(.).
 // Everything here is fp32: gates, decays, states and products.
 //
 // State lives in slots [slot][head][key][value] so that requests of one batch keep theirs anywhere; a portion that starts
@@ -14,7 +15,7 @@
 //   * rows (decode, portions of a few tokens): one block per (sequence, head, 32 value columns), the state slice in
 //     registers, tokens in order;
 //   * chunks of 64 tokens (prefill). The recurrence is linear in S, so only an elementwise scan over chunks is serial:
-//       gates   per token: log decays (GLA), or log f, i and the running maximum m (mLSTM: an associative (+, max) scan)
+//       gates   per token: log decays (GLA; HGRN2's are made inside the next kernel), or log f, i and the running maximum m (mLSTM: an associative (+, max) scan)
 //       intra   per (chunk, head): P_ij = sum_d q_i k_j exp(G_i - G_j) (j <= i), q~ = q exp(G_i), k~ = k exp(G_C - G_j)
 //       kv      per (chunk, head, tile): k~^T V
 //       scan    state before every chunk
@@ -32,23 +33,31 @@ namespace {
 
 using namespace pk;
 
-enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_RETENTION = 2, KIND_SSD = 3 };
+enum { KIND_GLA = 0, KIND_MLSTM = 1, KIND_RETENTION = 2, KIND_SSD = 3, KIND_HGRN = 4 };
+__host__ __device__ constexpr bool vector_decay(int kind) { return kind == KIND_GLA || kind == KIND_HGRN; }
 constexpr int CH = 64;    // chunk
 constexpr int SB = 16;    // sub-chunk
 
 __device__ __forceinline__ float log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+// HGRN2: the forget gate f of a channel and what it drops, 1 - f, each without a cancellation.
+__device__ __forceinline__ void forget_gate(float z, float low, float& f, float& drop) {
+  const float e = expf(-fabsf(z)), big = 1.f / (1.f + e), small = e / (1.f + e);
+  f = low + (1.f - low) * (z >= 0.f ? big : small);
+  drop = (1.f - low) * (z >= 0.f ? small : big);
+}
+__device__ __forceinline__ float log_forget(float f, float drop) { return f < 0.5f ? logf(fmaxf(f, 1e-37f)) : log1pf(-drop); }
 __device__ __forceinline__ float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
 
 // Columns of the fused input projection and the constants of one layer.
 struct Mixer {
-  const float* proj;   // [rows, ld]: q | k | v | gate | (i | f) or (low-rank decay input)
+  const float* proj;   // [rows, ld]: q | k | v | gate | (i | f) or (low-rank decay input); HGRN2: q | f | v
   int ld;
   int oq, ok, ov, og, oi, of, oa;
   int H, D, V;
   float qscale;
   // mLSTM
   const float* bi;
-  const float* bf;
+  const float* bf;     // [H]; HGRN2: [H * D]
   float cap;
   // GLA
   const float* a2;     // [rank, H * D] (transposed low-rank up projection)
@@ -67,6 +76,8 @@ struct Mixer {
   const float* skip;   // [H]
   float* Cs;           // [slots, taps - 1, channels] last inputs of the convolution, by position modulo (taps - 1)
   int groups, taps, odt;
+  // HGRN2
+  const float* low;    // [H * D] lower bounds
   // state
   float* S;            // [slots, H, D, V]
   float* N;            // [slots, H, D]      (mLSTM)
@@ -92,7 +103,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
   extern __shared__ float sm[];
   float* qs = sm;                 // [D]
   float* ks = qs + mx.D;          // [D]
-  float* as = ks + mx.D;          // [D] (GLA)
+  float* as = ks + mx.D;          // [D] (GLA, HGRN2)
   float* red = as + mx.D;         // [GR][33]
   __shared__ float s_sc[3];
   const int4 sq = seqs[blockIdx.z];          // first row, tokens, slot, first position
@@ -134,6 +145,11 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
           ks[i + half] = k[i + half];
         }
       }
+    } else if (KIND == KIND_HGRN) {
+      for (int d = threadIdx.x; d < D; d += 32 * GR) {
+        qs[d] = silu_exact(pr[mx.oq + h * D + d]);
+        forget_gate(pr[mx.of + h * D + d] + mx.bf[h * D + d], mx.low[h * D + d], as[d], ks[d]);
+      }
     } else {
       for (int d = threadIdx.x; d < D; d += 32 * GR) {
         qs[d] = pr[mx.oq + h * D + d] * mx.qscale;
@@ -159,7 +175,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
     float v = is_v ? pr[mx.ov + h * V + col] : (is_n ? 1.f : 0.f);
     __syncthreads();
     float part = 0.f;
-    if (KIND != KIND_GLA) {
+    if (!vector_decay(KIND)) {
       const float a = KIND == KIND_MLSTM ? s_sc[0] : decay;
       if (KIND == KIND_MLSTM) v *= s_sc[1];
 #pragma unroll
@@ -521,8 +537,9 @@ __global__ void __launch_bounds__(256) ssd_scores_kernel(const Mixer mx, const C
     *reinterpret_cast<float4*>(wk.P + (((size_t)c * mx.groups + g) * CH + ty * 4 + i) * CH + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
 }
 
-// GLA intra-chunk part. One block per (chunk, head); 32 channels at a time. Thread (ti, tj) owns the entries
+// Intra-chunk part of GLA and HGRN2. One block per (chunk, head); 32 channels at a time. Thread (ti, tj) owns the entries
 // (16 a + ti, 16 b + tj) for all sub-chunk pairs b <= a.
+template <int KIND>
 __global__ void __launch_bounds__(256) gla_intra_kernel(const Mixer mx, const Chunks ck, const Work wk) {
   constexpr int DT = 32, LD = DT + 1;
   __shared__ float q[CH][LD], k[CH][LD], g[CH][LD];     // g: running log decay inside the sub-chunk
@@ -542,9 +559,16 @@ __global__ void __launch_bounds__(256) gla_intra_kernel(const Mixer mx, const Ch
       float qv = 0.f, kv = 0.f, lv = 0.f;
       if (d < nd && r < len) {
         const float* pr = mx.proj + (size_t)(cd.x + r) * mx.ld + h * D + d0 + d;
-        qv = pr[mx.oq] * mx.qscale;
-        kv = pr[mx.ok];
-        lv = wk.logd[((size_t)c * CH + r) * HD + h * D + d0 + d];
+        if (KIND == KIND_HGRN) {
+          float f;
+          qv = silu_exact(pr[mx.oq]);
+          forget_gate(pr[mx.of] + mx.bf[h * D + d0 + d], mx.low[h * D + d0 + d], f, kv);
+          lv = log_forget(f, kv);
+        } else {
+          qv = pr[mx.oq] * mx.qscale;
+          kv = pr[mx.ok];
+          lv = wk.logd[((size_t)c * CH + r) * HD + h * D + d0 + d];
+        }
       }
       q[r][d] = qv;
       k[r][d] = kv;
@@ -845,7 +869,7 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
   for (int i = 0; i < KEEP; ++i) {
     const int v = tid + i * nt;
     x[i] = v < V ? o[v] : 0.f;
-    z[i] = v < V ? gate[v] : 0.f;
+    z[i] = KIND != KIND_HGRN && v < V ? gate[v] : 0.f;
   }
   if (KIND == KIND_MLSTM) {
     const float m = raw.m[unit];
@@ -860,12 +884,12 @@ __global__ void __launch_bounds__(256) state_out_kernel(const Mixer mx, const Ra
   const float* w = norm_w ? norm_w + (per_head ? 0 : h * V) : nullptr;
   auto put = [&](int v, float xv, float zv) {
     const float s = 1.f / (1.f + expf(-zv));
-    dst[v] = (OutT)(xv * r * (w ? w[v] : 1.f) * (KIND == KIND_MLSTM ? s : zv * s));
+    dst[v] = (OutT)(xv * r * (w ? w[v] : 1.f) * (KIND == KIND_HGRN ? 1.f : KIND == KIND_MLSTM ? s : zv * s));
   };
 #pragma unroll
   for (int i = 0; i < KEEP; ++i)
     if (tid + i * nt < V) put(tid + i * nt, x[i], z[i]);
-  for (int v = tid + KEEP * nt; v < V; v += nt) put(v, o[v], gate[v]);
+  for (int v = tid + KEEP * nt; v < V; v += nt) put(v, o[v], KIND != KIND_HGRN ? gate[v] : 0.f);
   if (h == H - 1)
     for (int v = H * V + tid; v < ldo; v += nt) out[(size_t)t * ldo + v] = (OutT)0.f;
 }
@@ -934,10 +958,11 @@ static bool unpack(const PkStateMixer* d, Mixer& mx, Raw& raw) {
   if (d->kind == KIND_SSD && (!d->cw || !d->cb || !d->dtb || !d->A || !d->skip || d->groups < 1 || d->H % d->groups != 0 || d->taps < 1 ||
                               (d->taps > 1 && !d->Cs)))
     return false;
-  if (d->kind < KIND_GLA || d->kind > KIND_SSD) return false;
+  if (d->kind == KIND_HGRN && (!d->bf || !d->low)) return false;
+  if (d->kind < KIND_GLA || d->kind > KIND_HGRN) return false;
   mx = Mixer{d->proj, d->ld, d->oq, d->ok, d->ov, d->og, d->oi, d->of, d->oa, d->H, d->D, d->V, d->qscale, d->bi, d->bf,
              d->cap, d->a2, d->a2b, d->rank, d->inv_tau, d->freq, d->rot, d->pw, d->cw, d->cb, d->dtb, d->A, d->skip, d->Cs,
-             d->groups, d->taps, d->odt, d->S, d->N, d->Ms};
+             d->groups, d->taps, d->odt, d->low, d->S, d->N, d->Ms};
   raw = Raw{d->o, d->nq, d->m};
   return true;
 }
@@ -951,6 +976,7 @@ PK_API int pk_state_rows(const PkStateMixer* d, const void* seqs, int nseq, cuda
     case KIND_GLA: return launch_rows<KIND_GLA>(mx, raw, (const int4*)seqs, nseq, stream);
     case KIND_SSD: return PK_ERR_UNSUPPORTED;      // pk_ssd_rows
     case KIND_MLSTM: return launch_rows<KIND_MLSTM>(mx, raw, (const int4*)seqs, nseq, stream);
+    case KIND_HGRN: return launch_rows<KIND_HGRN>(mx, raw, (const int4*)seqs, nseq, stream);
     default: return launch_rows<KIND_RETENTION>(mx, raw, (const int4*)seqs, nseq, stream);
   }
 }
@@ -984,7 +1010,9 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
     const int z = (H * mx.D + 255) / 256;
     gla_gates_kernel<<<dim3(nchunks, CH / 8, z < 16 ? z : 16), 256, (size_t)8 * mx.rank * sizeof(float), stream>>>(mx, ck, wk);
     PK_CHECK_LAUNCH();
-    gla_intra_kernel<<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
+    gla_intra_kernel<KIND_GLA><<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
+  } else if (d->kind == KIND_HGRN) {
+    gla_intra_kernel<KIND_HGRN><<<dim3(nchunks, H), 256, 0, stream>>>(mx, ck, wk);
   } else if (d->kind == KIND_SSD) {
     const int cb = (ssd_channels(mx) + 255) / 256;
     const dim3 grid(nchunks, cb + (H + 7) / 8);
@@ -1018,7 +1046,7 @@ PK_API int pk_state_chunks(const PkStateMixer* d, const void* seqs, int nseq, co
   return PK_OK;
 }
 
-// Head norm, output gate (SiLU; mLSTM: sigmoid) and running-maximum write-back for all rows of a step. norm_w null: no weight.
+// Head norm, output gate (SiLU; mLSTM: sigmoid; HGRN2: none) and running-maximum write-back for all rows of a step. norm_w null: no weight.
 PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head, float eps, const int* last_slot, int rows, void* out,
                         int ldo, int out_f32, cudaStream_t stream) {
   Mixer mx;
@@ -1027,12 +1055,12 @@ PK_API int pk_state_out(const PkStateMixer* d, const float* norm_w, int per_head
   if (rows > 65535) return PK_ERR_BAD_ARG;
   const int nt = (mx.V + 31) / 32 * 32;
   const dim3 grid(mx.H, rows), block(nt < 256 ? nt : 256);
-  if (d->kind != KIND_MLSTM) {
-    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
-    else PK_LAUNCH_PDL((state_out_kernel<KIND_GLA, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
-  } else {
-    if (out_f32) PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);
-    else PK_LAUNCH_PDL((state_out_kernel<KIND_MLSTM, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo);
-  }
+#define PK_OUT_CASE(kind)                                                                                                                                     \
+  if (out_f32) PK_LAUNCH_PDL((state_out_kernel<kind, float>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (float*)out, ldo);   \
+  else PK_LAUNCH_PDL((state_out_kernel<kind, pk::bf16>), grid, block, (size_t)0, stream, mx, raw, norm_w, per_head, eps, last_slot, (pk::bf16*)out, ldo)
+  if (d->kind == KIND_MLSTM) PK_OUT_CASE(KIND_MLSTM);
+  else if (d->kind == KIND_HGRN) PK_OUT_CASE(KIND_HGRN);
+  else PK_OUT_CASE(KIND_GLA);
+#undef PK_OUT_CASE
   return PK_OK;
 }

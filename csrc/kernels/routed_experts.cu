@@ -1,5 +1,5 @@
-// Routed experts: every token takes the `top` experts with the largest router scores (an optional correction per expert counts
-// for the choice alone); an expert is W_down act(W_up x) with act = max(., 0)^2, or W_down (silu(W_gate x) * (W_up x)), and the
+// Routed experts: every token takes the `top` experts with the largest router scores (an optional bias is part of the logits, an
+// optional correction per expert counts for the choice alone); an expert is W_down act(W_up x) with act = max(., 0)^2, or W_down (silu(W_gate x) * (W_up x)), and the
 // routing weight multiplies either its input (as a factor on the products, which is the same) or its output (as a factor
 // behind the activation). The last of the experts may be identities: they have no weights and return their input; what they
 // add up to, one factor per token, is left to the norm that follows (sandwich_norm.cu).
@@ -24,6 +24,7 @@ struct Router {
   float scale;
   const float* correction;             // [E] added to the scores for the choice (null: none)
   int real;                            // the first `real` experts have weights
+  const float* bias;                   // [E] added to the logits (null: none)
 };
 
 // One warp, up to 32 PER experts. Lane j < top gets the j-th best expert and its weight (ties: the lower index first).
@@ -35,7 +36,7 @@ __device__ __forceinline__ void select_experts(const Router& r, int token, int l
   for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
     v[i] = -INFINITY;
-    if (i * 32 < r.E && e < r.E) v[i] = fmaxf(z[e], -3.0e38f);
+    if (i * 32 < r.E && e < r.E) v[i] = fmaxf(z[e] + (r.bias ? r.bias[e] : 0.f), -3.0e38f);
   }
   float zmax = 0.f, den = 1.f, sc[PER];      // v: what the choice compares; sc: scores (kept apart when they differ)
   if (r.score == SCORE_SOFTMAX) {
@@ -355,13 +356,13 @@ int pick_slices(long long pairs, int K, int vec, int sm_count) {
 
 // Hidden rows of T tokens' experts. logits [T, ldz]; x [T, ldx] and w_up [E - identity, N, K] (gated: N gate rows, then N up
 // rows each) bf16, or fp32 when `f32`; hidden [T * top, ldh] of the same type; ids [T, top] out. K a multiple of 8, rows
-// 16-byte aligned. score 0 sigmoid, 1 softmax; correction [E] or null; renorm: the chosen weights are divided by their sum;
+// 16-byte aligned. score 0 sigmoid, 1 softmax; correction, bias [E] or null; renorm: the chosen weights are divided by their sum;
 // scale: factor on them; scale_after: weight on the output instead of the input; identity: how many of the E experts are
 // identities (skip_w [T] out, the sum of their weights).
-PK_API int pk_expert_up_rows(const float* logits, int ldz, int E, int top, int score, int renorm, float scale, const float* correction, int identity,
+PK_API int pk_expert_up_rows(const float* logits, int ldz, int E, int top, int score, int renorm, float scale, const float* correction, const float* bias, int identity,
                              float* skip_w, int scale_after, int gated, const void* x, int ldx, int T, const void* w_up, int N, int K, int f32,
                              int* ids, void* hidden, int ldh, int sm_count, cudaStream_t stream) {
-  Router r{logits, ldz, E, top, score, renorm, scale, correction, E - identity};
+  Router r{logits, ldz, E, top, score, renorm, scale, correction, E - identity, bias};
   if (!router_ok(r) || T < 1 || N < 1 || K < 8 || (K & 7) != 0 || ldx < K || (ldx & 7) != 0 || ldh < N || x == nullptr || w_up == nullptr || ids == nullptr ||
       hidden == nullptr || ((uintptr_t)x & 15) != 0 || ((uintptr_t)w_up & 15) != 0 || identity < 0 || (identity > 0 && skip_w == nullptr))
     return PK_ERR_BAD_ARG;
@@ -384,7 +385,7 @@ PK_API int pk_expert_down_rows(const int* ids, int top, int real, const void* hi
   if (ids == nullptr || top < 1 || top > kMaxTop || T < 1 || N < 1 || w_rows < N || K < 8 || (K & 7) != 0 || ldh < K || (ldh & 7) != 0 || ldy < N ||
       hidden == nullptr || w_down == nullptr || y == nullptr || ((uintptr_t)hidden & 15) != 0 || ((uintptr_t)w_down & 15) != 0)
     return PK_ERR_BAD_ARG;
-  RowsParams p{Router{nullptr, 0, 0, top, 0, 0, 0.f, nullptr, real}, hidden, ldh, w_down, N, K, w_rows, 1, 0, 0, (int*)ids, nullptr, y, ldy};
+  RowsParams p{Router{nullptr, 0, 0, top, 0, 0, 0.f, nullptr, real, nullptr}, hidden, ldh, w_down, N, K, w_rows, 1, 0, 0, (int*)ids, nullptr, y, ldy};
   const int pairs = (N + 1) / 2;
   p.slices = pick_slices((long long)pairs * T, K, f32 ? 4 : 8, sm_count);
   const dim3 grid(T, (pairs + WARPS / p.slices - 1) / (WARPS / p.slices));
@@ -396,10 +397,10 @@ PK_API int pk_expert_down_rows(const int* ids, int top, int real, const void* hi
 
 // Routes of T tokens grouped by expert: ids, weights [T, top]; seg [E - identity + 1]; place [T, top]; row_scale [T * top];
 // rows [T * top, K] bf16 = the tokens' x in expert order (K a multiple of 8); skip_w as above.
-PK_API int pk_expert_group(const float* logits, int ldz, int E, int top, int score, int renorm, float scale, const float* correction, int identity,
+PK_API int pk_expert_group(const float* logits, int ldz, int E, int top, int score, int renorm, float scale, const float* correction, const float* bias, int identity,
                            float* skip_w, int T, int* ids, float* weights, int* seg, int* place, float* row_scale, const void* x, int ldx, int K,
                            void* rows, cudaStream_t stream) {
-  Router r{logits, ldz, E, top, score, renorm, scale, correction, E - identity};
+  Router r{logits, ldz, E, top, score, renorm, scale, correction, E - identity, bias};
   if (!router_ok(r) || T < 1 || identity < 0 || (identity > 0 && skip_w == nullptr) || ids == nullptr || weights == nullptr || seg == nullptr ||
       place == nullptr || row_scale == nullptr || x == nullptr || rows == nullptr || K < 8 || (K & 7) != 0 || (ldx & 7) != 0 || ldx < K || ((uintptr_t)x & 15) != 0 || ((uintptr_t)rows & 15) != 0)
     return PK_ERR_BAD_ARG;

@@ -19,6 +19,7 @@
 // TMA loads have no multicast. Every wait is bounded (status word + CTA-wide abort flag).
 #include "../common/pk_sm100.cuh"
 #include "../common/pk_state.cuh"
+#include "../common/pk_vec.cuh"
 
 namespace {
 
@@ -148,30 +149,6 @@ int launch_rows(const PkStateMixer& m, const int4* seqs, int nseq, cudaStream_t 
 
 // ---------------------------------------------------------------------------------------
 // gate, norm
-
-template <int VW>
-__device__ __forceinline__ void load_f32(const float* p, float (&v)[VW]) {
-  if (VW == 4) {
-    const float4 x = *reinterpret_cast<const float4*>(p);
-    v[0] = x.x; v[1 % VW] = x.y; v[2 % VW] = x.z; v[3 % VW] = x.w;
-  } else {
-    v[0] = *p;
-  }
-}
-template <int VW>
-__device__ __forceinline__ void store(float* p, const float (&v)[VW]) {
-  if (VW == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % VW], v[2 % VW], v[3 % VW]);
-  else *p = v[0];
-}
-template <int VW>
-__device__ __forceinline__ void store(bf16* p, const float (&v)[VW]) {
-  if (VW == 4) {
-    const bf162 a = __floats2bfloat162_rn(v[0], v[1 % VW]), b = __floats2bfloat162_rn(v[2 % VW], v[3 % VW]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-  } else {
-    *p = __float2bfloat16(v[0]);
-  }
-}
 
 // y silu(z), normed in gridDim.x equal parts of the heads' outputs laid end to end, times norm_w [H * V]. One block per (part,
 // row); columns from H * V up to `width` are set to zero. behind[row]: tokens of the same portion after the row; the last rows of

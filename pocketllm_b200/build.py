@@ -43,7 +43,7 @@ COMMON = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "-Xcompiler",
 
 # translation units behind `ops.mixer_ops`
 KERNEL_SETS = {
-    "mixer": ["kernels/sandwich_norm.cu", "kernels/linear_f32.cu", "kernels/linear_rows.cu", "kernels/linear_state.cu", "kernels/ssd.cu",
+    "mixer": ["kernels/sandwich_norm.cu", "kernels/post_norm.cu", "kernels/linear_f32.cu", "kernels/linear_rows.cu", "kernels/linear_state.cu", "kernels/ssd.cu", "kernels/selective_scan.cu",
               "kernels/latent_attention.cu", "kernels/latent_prefill.cu", "kernels/paged_attention.cu", "kernels/paged_prefill.cu",
               "kernels/routed_experts.cu", "kernels/gemm_bf16.cu", "kernels/misc.cu", "common/pk_status.cu"],
 }

@@ -74,25 +74,32 @@ class StepContext:
 
 class FusedLinear:
     """Row blocks of several matrices that share their input as one [N, K] matrix, padded with zeros to what the kernels
-    take; `at[name]` is the first output column of a block (a multiple of `align`)."""
+    take; `at[name]` is the first output column of a block (a multiple of `align`). The blocks of `beside` come first and have an
+    input of their own."""
 
-    def __init__(self, blocks: list[tuple[str, torch.Tensor]], dtype: torch.dtype, device, k_pad: int | None = None, align: int = 1):
+    def __init__(self, blocks: list[tuple[str, torch.Tensor]], dtype: torch.dtype, device, k_pad: int | None = None, align: int = 1,
+                 beside: list[tuple[str, torch.Tensor]] | None = None):
         K = blocks[0][1].shape[1]
         self.K = k_pad or pad_to(K, 64)
         self.at, n = {}, 0
-        for name, w in blocks:
-            if w.shape[1] != K:
-                raise ValueError(f"{name}: {w.shape[1]} input columns, the others have {K}")
-            self.at[name] = n = pad_to(n, align)
-            n += w.shape[0]
+        self.split = 0
+        for part in (beside or [], blocks):
+            self.split = n = pad_to(n, 8)
+            for name, w in part:
+                if w.shape[1] != K:
+                    raise ValueError(f"{name}: {w.shape[1]} input columns, the others have {K}")
+                self.at[name] = n = pad_to(n, align)
+                n += w.shape[0]
         self.N = pad_to(n, 8)
         w = torch.zeros(self.N, self.K, dtype=dtype)
-        for name, b in blocks:
+        for name, b in (beside or []) + blocks:
             w[self.at[name]:self.at[name] + b.shape[0], :K] = b.to(dtype)
         self.w = w.to(device)
 
-    def __call__(self, ctx: StepContext, x: torch.Tensor, name: str, dtype: torch.dtype) -> torch.Tensor:
+    def __call__(self, ctx: StepContext, x: torch.Tensor, name: str, dtype: torch.dtype, beside: torch.Tensor | None = None) -> torch.Tensor:
         out = ctx.ws.rows(name, x.shape[0], self.N, dtype)
+        if self.split:
+            return mo.linear2(beside, x, self.split, self.w, out, ctx.status)
         return mo.linear(x, self.w, out, ctx.status)
 
 
@@ -101,24 +108,26 @@ def _f32(t: torch.Tensor, device) -> torch.Tensor:
 
 
 class RecurrentMixer:
-    """Base of the mixers with an outer-product state per head. Subclasses fill `self.desc` with what is theirs."""
+    """Base of the mixers with an outer-product state per head. Subclasses fill `self.desc` with what is theirs. `beside`: matrices
+    that the projection carries along for its owner (see `FusedLinear`)."""
     per_head_norm = False
+    inputs = ("q", "k", "v", "g")
 
-    def __init__(self, kind: int, w: dict, extra: list[str], heads: int, dim: int, vdim: int, eps: float, dtype, device, slots: int):
+    def __init__(self, kind: int, w: dict, extra: list[str], heads: int, dim: int, vdim: int, eps: float, dtype, device, slots: int, beside=None):
         if dim > 512:
             raise ValueError("recurrent mixers take key dims up to 512")
         self.H, self.D, self.V, self.eps, self.dtype = heads, dim, vdim, eps, dtype
-        for n, r in (("q", heads * dim), ("k", heads * dim), ("v", heads * vdim), ("g", heads * vdim)):
-            if w[n].shape[0] != r:
+        for n, r in (("q", heads * dim), ("k", heads * dim), ("f", heads * dim), ("v", heads * vdim), ("g", heads * vdim)):
+            if n in self.inputs and w[n].shape[0] != r:
                 raise ValueError(f"{n}: {w[n].shape[0]} rows, expected {r}")
-        self.proj = FusedLinear([(n, w[n]) for n in ["q", "k", "v", "g"] + extra], dtype, device)
+        self.proj = FusedLinear([(n, w[n]) for n in [*self.inputs, *extra]], dtype, device, beside=beside)
         self.out = FusedLinear([("o", w["o"])], dtype, device)
         self.norm = _f32(w["norm"], device) if "norm" in w else None
         self.S = torch.zeros(slots, heads, dim, vdim, device=device)
         self.N = self.Ms = None
         a = self.proj.at
         self.keep: list[torch.Tensor] = []
-        self.desc = dict(kind=kind, H=heads, D=dim, V=vdim, oq=a["q"], ok=a["k"], ov=a["v"], og=a["g"], qscale=dim ** -0.5, S=self.S.data_ptr())
+        self.desc = dict(kind=kind, H=heads, D=dim, V=vdim, qscale=dim ** -0.5, S=self.S.data_ptr(), **{"o" + n: a[n] for n in self.inputs})
 
     def again(self):
         """The same weights with states of their own (a further pass over the layer)."""
@@ -134,9 +143,9 @@ class RecurrentMixer:
     def state_bytes(self) -> int:
         return sum(t.numel() * 4 for t in (self.S, self.N, self.Ms) if t is not None)
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+    def forward(self, ctx: StepContext, h: torch.Tensor, beside: torch.Tensor | None = None) -> torch.Tensor:
         T, ws = ctx.T, ctx.ws
-        p = self.proj(ctx, h, "proj", torch.float32)
+        p = self.proj(ctx, h, "proj", torch.float32, beside)
         o = ws.flat("raw_o", T * self.H * self.V, torch.float32)
         nq, m = ws.flat("raw_nq", T * self.H, torch.float32), ws.flat("raw_m", T * self.H, torch.float32)
         d = mo.StateMixer(proj=p.data_ptr(), ld=p.stride(0), o=o.data_ptr(), nq=nq.data_ptr(), m=m.data_ptr(), **self.desc)
@@ -191,6 +200,91 @@ class RetentionMixer(RecurrentMixer):
         powers = (decay[:, None] ** torch.arange(mo.CHUNK + 1, dtype=torch.float64)).float().to(device)
         self.keep += [freq, powers]
         self.desc.update(freq=freq.data_ptr() if rot["dims"] else None, rot=rot["dims"], pw=powers.data_ptr())
+
+
+class HGRN2Mixer(RecurrentMixer):
+    """Linear attention whose forget gate is also its key: a channel keeps f and is written with 1 - f, f = l + (1 - l) sigmoid(.) above
+    a lower bound l; queries pass SiLU; the head outputs are normed with one weight shared by the heads."""
+    per_head_norm = True
+    inputs = ("q", "f", "v")
+
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, slots: int, beside=None):
+        super().__init__(mo.KIND_HGRN, w, [], m["heads"], m["dim"], m["vdim"], eps, dtype, device, slots, beside)
+        bias, low = _f32(w["f.b"], device), _f32(w["lower"], device)
+        self.keep += [bias, low]
+        self.desc.update(qscale=1.0, bf=bias.data_ptr(), low=low.data_ptr())
+
+
+class SelectiveScanMixer:
+    """The selective scan of Mamba: x through a short convolution, step sizes (from a low-rank projection), B and C from x, a decay per
+    channel and state, SiLU gate."""
+
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, slots: int, beside=None):
+        inner, N, rank, taps = m["inner"], m["state"], m["dt_rank"], m["conv"]
+        self.inner, self.N, self.rank, self.taps, self.dtype = inner, N, rank, taps, dtype
+        if N > 256:
+            raise ValueError("selective scans take states up to 256")
+        for n, s in (("in", (2 * inner, None)), ("conv", (inner, taps)), ("conv.b", (inner,)), ("x", (rank + 2 * N, inner)), ("dt", (inner, rank)),
+                     ("dt.b", (inner,)), ("A_log", (inner, N)), ("D", (inner,)), ("o", (None, inner))):
+            if any(b is not None and a != b for a, b in zip(w[n].shape, s)):
+                raise ValueError(f"{n}: shape {tuple(w[n].shape)}, expected {s}")
+        self.proj = FusedLinear([("x", w["in"][:inner]), ("z", w["in"][inner:])], dtype, device, align=4, beside=beside)
+        self.dbc = FusedLinear([("dbc", w["x"])], dtype, device)
+        self.out = FusedLinear([("o", w["o"])], dtype, device)
+        # step sizes: few rows read the plain matrix, many rows multiply it with a two-term input in bf16
+        kw = pad_to(rank, 32)
+        wide = torch.zeros(inner, kw if dtype == torch.float32 else 2 * kw)
+        for a in range(0, wide.shape[1], kw):
+            wide[:, a:a + rank] = w["dt"]
+        self.dt = FusedLinear([("dt", wide)], dtype, device, k_pad=wide.shape[1])
+        self.kw = kw
+        f = lambda n: _f32(w[n], device)
+        decay = (-torch.exp(w["A_log"].double()) * math.log2(math.e)).float().contiguous().to(device)
+        self.const = {"cw": f("conv"), "cb": f("conv.b"), "dt_bias": f("dt.b"), "A": decay, "skip": f("D"), "w_dt": self.dt.w}
+        self.desc = dict(ox=self.proj.at["x"], oz=self.proj.at["z"], ldw=self.dt.K, inner=inner, N=N, rank=rank, taps=taps, f32=int(dtype == torch.float32),
+                         **{n: t.data_ptr() for n, t in self.const.items()})
+        self._memory(slots, device)
+
+    def _memory(self, slots: int, device) -> None:
+        self.S = torch.zeros(slots, self.inner, self.N, device=device)
+        self.ring = torch.zeros(slots, max(self.taps - 1, 1), self.inner, device=device)
+        self.desc = dict(self.desc, S=self.S.data_ptr(), ring=self.ring.data_ptr())
+
+    def again(self):
+        """The same weights with states of their own."""
+        o = copy.copy(self)
+        o._memory(self.S.shape[0], self.S.device)
+        return o
+
+    def state_bytes(self) -> int:
+        return (self.S.numel() + self.ring.numel()) * 4
+
+    def forward(self, ctx: StepContext, h: torch.Tensor, beside: torch.Tensor | None = None) -> torch.Tensor:
+        p = self.proj(ctx, h, "proj", torch.float32, beside)
+        mix = ctx.ws.rows("mix", ctx.T, self.out.K, self.dtype)
+        self.run(ctx, p, mix)
+        return self.out(ctx, mix, "y", torch.float32)
+
+    def run(self, ctx: StepContext, p: torch.Tensor, mix: torch.Tensor) -> None:
+        T, ws = ctx.T, ctx.ws
+        x = ws.rows("scan_x", T, self.dbc.K, self.dtype)
+        d = mo.SelectiveScan(proj=p.data_ptr(), ld=p.stride(0), xc=x.data_ptr(), ldx=x.stride(0), out=mix.data_ptr(), ldo=mix.stride(0),
+                             pos=ctx.pos.data_ptr(), slot=ctx.slot.data_ptr(), **self.desc)
+        mo.scan_conv(d, T)
+        dbc = self.dbc(ctx, x, "scan_dbc", torch.float32)
+        d.dbc, d.ldb = dbc.data_ptr(), dbc.stride(0)
+        if ctx.n_short:
+            mo.scan_rows(d, ctx.short, ctx.n_short)
+        if ctx.n_long:
+            terms = ws.rows("scan_d", T, self.dt.K, self.dtype)
+            if self.dtype == torch.bfloat16:
+                mo.scan_split(dbc, self.rank, terms)
+            else:
+                terms[:, self.rank:] = 0
+                terms[:, :self.rank] = dbc[:, :self.rank]
+            dt = self.dt(ctx, terms, "scan_dt", torch.float32)
+            d.dt, d.ldt = dt.data_ptr(), dt.stride(0)
+            mo.scan_tiles(d, ctx.long, ctx.n_long)
 
 
 class StateSpaceMixer:
@@ -259,21 +353,25 @@ def rotary_frequencies(dims: int, base: float, scaling: dict | None = None) -> t
 class LatentAttentionMixer:
     """Latent attention over pages of [latent | rotated key part], optional sliding window and sinks. Few rows (decode) score
     queries mapped into the latent space against the cached rows; long portions in bf16 expand the keys and values they can
-    see with one GEMM and run the tensor-core kernel."""
+    see with one GEMM and run the tensor-core kernel. Without a rotated part (`rot_dim` missing) the queries may come from a latent of
+    their own (`dq`, `dq.norm`, `uq` among the weights instead of `q`); `g` among the weights: a sigmoid gate on the heads' outputs."""
 
-    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int):
-        H, D, R, V, K = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    def __init__(self, w: dict, m: dict, eps: float, dtype, device, pages: int, context: int, beside=None):
+        H, D, R, V, K = m["heads"], m["dim"], m.get("rot_dim") or 0, m["vdim"], m["kv_rank"]
+        self.q_rank = w["dq"].shape[0] if "dq" in w else 0
         self.H, self.D, self.R, self.V, self.K, self.eps, self.dtype = H, D, R, V, K, eps, dtype
         self.scale = float(m["scale"])
         self.window = int((m.get("mask") or {}).get("size") or 0)
-        for n, shape in (("q", (H * (D + R), None)), ("dkv", (K + R, None)), ("uk", (H * D, K)), ("uv", (H * V, K))):
-            if w[n].shape[0] != shape[0] or (shape[1] is not None and w[n].shape[1] != shape[1]):
+        for n, shape in (("q", (H * (D + R), None)), ("uq", (H * D, self.q_rank)), ("dkv", (K + R, None)), ("uk", (H * D, K)), ("uv", (H * V, K)), ("g", (H * V, None))):
+            if n in w and (w[n].shape[0] != shape[0] or (shape[1] is not None and w[n].shape[1] != shape[1])):
                 raise ValueError(f"{n}: shape {tuple(w[n].shape)}, expected {shape}")
-        if m["rot"]["dims"] != R:
-            raise ValueError("the rotated dimensions are the rotated part of the head")
-        freq, self.mag = rotary_frequencies(R, m["rot"]["base"], m["rot"].get("scaling"))
+        rot = m.get("rot") or {"dims": 0, "base": 1.0}
+        if rot["dims"] != R or (R and self.q_rank):
+            raise ValueError("the rotated dimensions are the rotated part of the head; queries from a latent have none")
+        freq, self.mag = rotary_frequencies(R, rot["base"], rot.get("scaling"))
         self.freq = freq.to(device)
-        self.proj = FusedLinear([("q", w["q"]), ("dkv", w["dkv"])], dtype, device)
+        self.proj = FusedLinear([(n, w[n]) for n in ("q", "dq", "dkv", "g") if n in w], dtype, device, align=4, beside=beside)
+        self.gated = "g" in w
         self.out = FusedLinear([("o", w["o"])], dtype, device)
         self.c_norm = _f32(w["dkv.norm"], device)
         self.sink = _f32(w["sink"], device) if "sink" in w else None
@@ -287,6 +385,11 @@ class LatentAttentionMixer:
         if self.v_panels > 1:
             self.v_panels = pad_to(self.v_panels, 2)
         self.tensor_core = dtype == torch.bfloat16 and self.qk_panels <= 4
+        if self.q_rank:      # heads of the expanded queries start where the tensor-core kernel wants them
+            uq = torch.zeros(H, self.qk_panels * 64, self.q_rank, dtype=dtype)
+            uq[:, :D] = w["uq"].to(dtype).view(H, D, self.q_rank)
+            self.uq = FusedLinear([("q", uq.view(-1, self.q_rank))], dtype, device)
+            self.q_norm = _f32(w["dq.norm"], device)
         self.kv_w = None
         if self.tensor_core:
             qw, vw = self.qk_panels * 64, self.v_panels * 64
@@ -305,17 +408,26 @@ class LatentAttentionMixer:
     def cache_bytes(self) -> int:
         return self.cache.numel() * self.cache.element_size()
 
-    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+    def forward(self, ctx: StepContext, h: torch.Tensor, beside: torch.Tensor | None = None) -> torch.Tensor:
         T, ws, H, D, R, K, V = ctx.T, ctx.ws, self.H, self.D, self.R, self.K, self.V
-        p = self.proj(ctx, h, "proj", torch.float32)
-        oq, oc = self.proj.at["q"], self.proj.at["dkv"]
+        p = self.proj(ctx, h, "proj", torch.float32, beside)
+        at = self.proj.at
+        gate = p[:, at["g"]:] if self.gated else None
         # rows that attend one by one: those of short portions, or all of them when the tensor-core form does not apply
         long = ctx.n_long > 0 and self.tensor_core
         rows, nrows = (ctx.rows, ctx.n_rows) if long or not ctx.n_long else (ctx.all_rows, T)
         qx = ws.flat("qx", T * H * self.row, torch.float32) if nrows else None
         qw = self.qk_panels * 64
-        qf = ws.flat("qf", T * H * qw, torch.bfloat16) if long else None
-        mo.latent_prep(p, oq, oc, H, D, R, K, self.c_norm, self.eps, self.freq, self.mag, ctx.pos, ctx.slot, self.cache, ctx.table, qx, qf, qw)
+        if self.q_rank:
+            ql = ws.rows("lat_q", T, self.uq.K, self.dtype)
+            mo.latent_prep(p, at["dq"], at["dkv"], H, D, R, K, self.c_norm, self.eps, self.freq, self.mag, ctx.pos, ctx.slot, self.cache, ctx.table, None, None, 0,
+                           q_rank=self.q_rank, q_norm=self.q_norm, ql=ql)
+            qf = self.uq(ctx, ql, "qf", torch.bfloat16) if long else None
+            q, oq, gap, k_pad = (self.uq(ctx, ql, "q_rows", torch.float32) if nrows else None), 0, qw - D, self.row
+        else:
+            qf = ws.flat("qf", T * H * qw, torch.bfloat16) if long else None
+            mo.latent_prep(p, at["q"], at["dkv"], H, D, R, K, self.c_norm, self.eps, self.freq, self.mag, ctx.pos, ctx.slot, self.cache, ctx.table, qx, qf, qw)
+            q, oq, gap, k_pad = p, at["q"], R, K
         mix = ws.rows("mix", T, self.out.K, self.dtype)
         if long:
             gather, total, longest = ctx.gather[self.window]
@@ -324,16 +436,16 @@ class LatentAttentionMixer:
             kv = ws.rows("lat_kv", total, self.kv_w.shape[0], torch.bfloat16)
             mo.linear(c, self.kv_w, kv, ctx.status)
             mo.latent_prefill(qf, T, kv, total, ctx.tiles, ctx.n_tiles, ctx.long, gather, H, self.qk_panels, self.v_panels, V, self.window, self.scale,
-                              self.sink, mix, ctx.status)
+                              self.sink, mix, ctx.status, gate)
         if nrows:
-            mo.latent_absorb(p, oq, H, D, R, K, self.uk, rows, nrows, qx, self.row)
+            mo.latent_absorb(q, oq, H, D, gap, K, self.uk, rows, nrows, qx, self.row, k_pad)
             per = max(8, (64 << 20) // (self.nsplit * H * K))
             for a in range(0, nrows, per):
                 n = min(per, nrows - a)
                 po, pm = ws.flat("part_o", n * self.nsplit * H * K, torch.float32), ws.flat("part_ml", n * self.nsplit * H * 2, torch.float32)
                 r = rows[a:a + n]
                 mo.latent_rows(qx, r, n, ctx.pos, ctx.slot, self.cache, ctx.table, H, K, self.window, self.scale, self.nsplit, po, pm)
-                mo.latent_out(po, pm, self.nsplit, H, K, V, self.sink, r, n, self.uv, mix)
+                mo.latent_out(po, pm, self.nsplit, H, K, V, self.sink, r, n, self.uv, mix, gate)
         return self.out(ctx, mix, "y", torch.float32)
 
 
@@ -496,10 +608,11 @@ class ParallelMixer:
 
 
 class SwiGLU:
-    """W_down (silu(W_gate h) * (W_up h)); the hidden size is padded to what the GEMM's epilogue takes."""
+    """W_down (silu(W_gate h) * (W_up h)); the hidden size is padded to what the GEMM's epilogue takes. `name`: of its scratch."""
 
-    def __init__(self, w: dict, dtype, device):
+    def __init__(self, w: dict, dtype, device, name: str = ""):
         ff, K = w["gate"].shape
+        self.name = name
         self.ff, self.dtype = pad_to(ff, 128), dtype
         gu = torch.zeros(2 * self.ff, pad_to(K, 64), dtype=dtype)
         gu[:ff, :K], gu[self.ff:self.ff + ff, :K] = w["gate"].to(dtype), w["up"].to(dtype)
@@ -507,23 +620,26 @@ class SwiGLU:
         self.down = FusedLinear([("down", w["down"])], dtype, device, k_pad=self.ff)
 
     def forward(self, ctx: StepContext, h: torch.Tensor) -> dict:
-        mid = ctx.ws.rows("mid", ctx.T, self.ff, self.dtype)
+        mid = ctx.ws.rows("mid" + self.name, ctx.T, self.ff, self.dtype)
         mo.linear(h, self.gate_up, mid, ctx.status, swiglu=True)
-        return {"y": self.down(ctx, mid, "y", torch.float32)}
+        return {"y": self.down(ctx, mid, "y" + self.name, torch.float32)}
 
 
 class RoutedExperts:
     """Routed experts W_down max(W_up x, 0)^2, or with `gate` matrices W_down (silu(W_gate x) * (W_up x)). Few rows (and fp32) stream
     the chosen experts' weights; many rows are grouped by expert and multiplied on the tensor cores, and the sum over a token's
-    experts is left to the norm that follows, as is what experts that return their input add: `forward` returns what
-    `sandwich_norm` takes."""
+    experts is left to the norm that follows, as is what experts that return their input and a `shared` expert add: `forward` returns
+    what `sandwich_norm` or the step of a `PostSum` model takes. `out_gate`: the matrix of a gate on the result, whose logits come with the
+    router's."""
 
     def __init__(self, router_w: torch.Tensor, up: list[torch.Tensor], down: list[torch.Tensor], router: mo.Router, dtype, device,
-                 gate: list[torch.Tensor] | None = None, correction: torch.Tensor | None = None):
+                 gate: list[torch.Tensor] | None = None, correction: torch.Tensor | None = None, bias: torch.Tensor | None = None,
+                 shared: "SwiGLU | None" = None, out_gate: torch.Tensor | None = None):
         E, (ff, K), W = router.experts, up[0].shape, down[0].shape[0]
         self.route, self.W, self.dtype, self.gated = router, W, dtype, gate is not None
-        self.router = FusedLinear([("router", router_w)], dtype, device)
-        self.correction = None if correction is None else _f32(correction, device)
+        self.router = FusedLinear([("router", router_w)] + ([] if out_gate is None else [("gate", out_gate)]), dtype, device, align=4)
+        self.correction, self.bias = (None if t is None else _f32(t, device) for t in (correction, bias))
+        self.shared = shared
         self.ff, kp = pad_to(ff, 128), pad_to(K, 64)
         self.up = torch.zeros(E, self.ff * (2 if gate else 1), kp, dtype=dtype, device=device)
         self.down = torch.zeros(E, pad_to(W, 128), self.ff, dtype=dtype, device=device)
@@ -540,13 +656,17 @@ class RoutedExperts:
         ids = ws.flat("route_ids", R, torch.int32)
         hidden = ws.rows("mid", R, self.ff, self.dtype)
         skip_w = ws.flat("route_skip", T, torch.float32) if r.identity else None
-        skip = {"skip": h, "skip_w": skip_w} if r.identity else {}
-        kw = {"correction": self.correction, "skip_w": skip_w}
+        rest = {"skip": h, "skip_w": skip_w} if r.identity else {}
+        kw = {"correction": self.correction, "skip_w": skip_w, "bias": self.bias}
+        if "gate" in self.router.at:
+            rest["gate"] = z[:, self.router.at["gate"]:]
+        if self.shared is not None:
+            rest["y2"] = self.shared.forward(ctx, h)["y"]
         if T <= mo.ROWS_MAX or self.dtype == torch.float32:
             mo.expert_up_rows(r, z, h, self.up, ids, hidden, gated=self.gated, **kw)
             y = ws.rows("y", T, self.down.shape[1], torch.float32)
             mo.expert_down_rows(r, ids, hidden, self.down, self.W, y)
-            return {"y": y, **skip}
+            return {"y": y, **rest}
         place = ws.rows("route_place", T, r.top, torch.int32)
         seg, scale = ws.flat("route_seg", r.experts + 1, torch.int32), ws.flat("route_scale", R, torch.float32)
         x = ws.rows("route_x", R, self.up.shape[2], self.dtype)
@@ -554,12 +674,14 @@ class RoutedExperts:
         mo.grouped_linear(x, self.up, seg, hidden, ctx.status, relu2=not self.gated, swiglu=self.gated, row_scale=scale, scale_after=r.on_output)
         y = ws.rows("expert_y", R, self.down.shape[1], torch.float32)
         mo.grouped_linear(hidden, self.down, seg, y, ctx.status)
-        return {"y": y, "y_rows": place, **skip}
+        return {"y": y, "y_rows": place, **rest}
 
 
 @dataclass
 class MixerLayer:
-    """A mixer and an optional feed-forward, normed before and optionally (`norm1b`, `norm2b`) after."""
+    """A mixer and an optional feed-forward, normed before and optionally (`norm1b`, `norm2b`) after; in a `PostSum` model `norm1` and
+    `norm2` follow the sums, the mixer may read a mix of its input with the previous token's (`shift`), whose input is kept per slot
+    (`before`), and both sublayers may have a gate on their results (`gate_b`: its biases; the logits come with the projections)."""
     mixer: object
     norm1: torch.Tensor
     norm1b: torch.Tensor | None = None
@@ -567,10 +689,26 @@ class MixerLayer:
     norm2: torch.Tensor | None = None
     norm2b: torch.Tensor | None = None
     reinject: bool = False         # the embedding output is added to the residual stream before this layer
+    shift: torch.Tensor | None = None
+    before: torch.Tensor | None = None
+    gate_b: tuple = (None, None)
 
-    def again(self, reinject: bool) -> "MixerLayer":
+    def again(self, reinject: bool = False) -> "MixerLayer":
         """A further run of the layer: the same weights, a state or cache of its own."""
-        return replace(self, mixer=self.mixer.again(), reinject=reinject)
+        return replace(self, mixer=self.mixer.again(), reinject=reinject, before=None if self.before is None else torch.zeros_like(self.before))
+
+
+@dataclass
+class PostSum:
+    """Layers are normed behind their sums, x <- norm(alpha x + y), and read x itself; a sinusoid of the position is added to the
+    embedding. `freq`: its angular frequencies (float64)."""
+    alpha: float
+    freq: torch.Tensor
+
+
+def sinusoid_frequencies(width: int, base: float = 10000.0) -> torch.Tensor:
+    """Column 2i of a row is the sine, column 2i + 1 the cosine of position x frequency i."""
+    return torch.pow(torch.tensor(base, dtype=torch.float64), -2.0 * torch.arange((width + 1) // 2, dtype=torch.float64) / width)
 
 
 @dataclass
@@ -587,6 +725,7 @@ class MixerModel:
     plus_one: bool = True          # norm weights are stored around zero
     embed_scale: float = 1.0
     residual_scale: float = 1.0    # factor on every sublayer's output
+    post: PostSum | None = None    # norms behind the sums instead of before the sublayers
 
     def windows(self) -> set[int]:
         return {L.mixer.window for L in self.layers if isinstance(L.mixer, LatentAttentionMixer)}

@@ -77,3 +77,8 @@ def _load() -> None:
     def _zemozen(path, **kw):
         from . import zemozen
         return zemozen.build_runtime(path, **kw)
+
+    @register("Zarinex", folder=True)
+    def _zarinex(path, **kw):
+        from . import zarinex
+        return zarinex.build_runtime(path, **kw)

@@ -1,6 +1,6 @@
 """Bindings of the mixer-decoder kernels: norms on an fp32 residual stream, fp32 and few-row bf16 linears, recurrent
-outer-product states (gated linear attention, mLSTM, retention, state space), latent and grouped-query attention over a paged cache, routed
-experts.
+outer-product states (gated linear attention, mLSTM, retention, state space, HGRN2), selective scan, latent and grouped-query attention over a
+paged cache, routed experts.
 
 Every function launches on the current stream and writes into buffers its caller owns (so that a step can be captured in
 a CUDA graph); a non-zero status raises.
@@ -15,7 +15,7 @@ import torch
 from . import EPI_BF16, EPI_F32, EPI_SWIGLU, _check
 from . import lib as _lib
 
-KIND_GLA, KIND_MLSTM, KIND_RETENTION, KIND_SSD = 0, 1, 2, 3
+KIND_GLA, KIND_MLSTM, KIND_RETENTION, KIND_SSD, KIND_HGRN = 0, 1, 2, 3, 4
 SCORES = {"sigmoid": 0, "softmax": 1}      # router scores
 EPI_RELU2 = 5       # grouped GEMM: squared ReLU with a factor per row
 PAGE = 64           # tokens per cache page
@@ -26,7 +26,7 @@ ROWS_MAX = 8        # widest portion (and batch) of the few-row kernels
 class StateMixer(Structure):
     """`PkStateMixer`: columns of the fused projection, constants, state and raw outputs of one recurrent layer."""
     _fields_ = [(n, c_void_p) for n in ("proj", "bi", "bf", "a2", "a2b", "S", "N", "Ms", "o", "nq", "m", "freq", "pw", "cw", "cb", "dtb", "A", "skip",
-                                        "Cs")] + \
+                                        "Cs", "low")] + \
                [(n, c_int) for n in ("kind", "ld", "oq", "ok", "ov", "og", "oi", "of", "oa", "H", "D", "V", "rank", "rot", "groups", "taps", "odt")] + \
                [(n, c_float) for n in ("qscale", "cap", "inv_tau")]
 
@@ -38,6 +38,19 @@ class PagedAttention(Structure):
                [(n, c_int) for n in ("ld", "oq", "ok", "ov", "H", "G", "maps", "D", "V", "R", "dp", "vp", "row", "table_ld", "f32", "window", "chunk", "q_ld",
                                      "ldo", "nsplit", "head_norm", "neighbours", "v_mix", "gate", "width")] + \
                [(n, c_float) for n in ("scale", "lambda_", "post", "eps", "cap", "mix")]
+
+
+class SelectiveScan(Structure):
+    """`PkSelectiveScan`: one selective-scan layer over one batch."""
+    _fields_ = [(n, c_void_p) for n in ("proj", "xc", "dbc", "dt", "w_dt", "dt_bias", "A", "skip", "cw", "cb", "S", "ring", "out", "pos", "slot")] + \
+               [(n, c_int) for n in ("ld", "ox", "oz", "ldx", "ldb", "ldt", "ldw", "ldo", "inner", "N", "rank", "taps", "f32")]
+
+
+class PostNorm(Structure):
+    """`PkPostNorm`: one residual step with its norm behind the sum."""
+    _fields_ = [(n, c_void_p) for n in ("x", "x_out", "tokens", "embed", "freq", "y", "y_rows", "y2", "gate", "gate_b", "w", "w_out", "pos", "slot", "behind", "save",
+                                        "shift", "before", "rows", "out", "out_shift")] + \
+               [(n, c_int) for n in ("vocab", "ldy", "y_top", "ldy2", "ldg", "M", "width", "ldo", "out_f32")] + [(n, c_float) for n in ("alpha", "eps")]
 
 
 _sms: dict[int, int] = {}
@@ -52,13 +65,14 @@ def sm_count() -> int:
 
 # argument kinds of the launchers, the stream excepted: p pointer, i int, f float
 _SIGNATURES = {
-    "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
-    "pk_sandwich_norm": "pppifipipifpiippp" "iipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_argmax": "piiiiipppp",
+    "pk_linear_f32": "pipiiiipi", "pk_linear_rows": "pipiiiipii", "pk_linear_rows2": "ppiipiiiipii", "pk_gemm_bf16": "pipiiiippippi",
+    "pk_sandwich_norm": "pppifipipifpiippp" "iipifpii", "pk_feed_tokens": "pipppp" "ip", "pk_post_norm": "p", "pk_argmax": "piiiiipppp",
     "pk_state_rows": "ppi", "pk_state_chunks": "ppippip", "pk_state_out": "ppifpipii", "pk_ssd_out": "ppifpppipiii", "pk_ssd_tiles": "ppippipp", "pk_ssd_rows": "ppii",
-    "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipi",
-    "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipi", "pk_latent_prefill": "pipipippiiiiifppip",
+    "pk_scan_conv": "pi", "pk_scan_split": "piiiip", "pk_scan_rows": "ppi", "pk_scan_tiles": "ppi",
+    "pk_latent_prep": "piiiiiiiipfpfpppp" "iiippi" "ippi", "pk_latent_gather": "ppiippiip", "pk_latent_absorb": "piiiiiipipipii",
+    "pk_latent_rows": "ppippppiiiiiifipp", "pk_latent_out": "ppiiiippipipipi", "pk_latent_prefill": "pipipippiiiiifppipip",
     "pk_paged_prep": "pi", "pk_paged_rows": "ppi", "pk_paged_merge": "ppi", "pk_paged_prefill": "piipip",
-    "pk_expert_up_rows": "piiiiifpipiipiipiiippii", "pk_expert_down_rows": "piipiipiiiipii", "pk_expert_group": "piiiiifpipipppppp" "iip",
+    "pk_expert_up_rows": "piiiiifppipiipiipiiippii", "pk_expert_down_rows": "piipiipiiiipii", "pk_expert_group": "piiiiifppipipppppp" "iip",
     "pk_gemm_bf16_grouped_scaled": "pippiiiiipipipi",
 }
 _bound: dict[tuple[int, str], object] = {}
@@ -100,6 +114,17 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, status: torch.Te
     return out
 
 
+def linear2(x: torch.Tensor, x2: torch.Tensor, split: int, w: torch.Tensor, out: torch.Tensor, status: torch.Tensor) -> torch.Tensor:
+    """As `linear` (fp32 out), with `x2` as the input of the weight rows from `split` on; one launch up to eight rows of bf16."""
+    M, K = x.shape
+    if x.dtype == torch.float32 or M > ROWS_MAX:
+        linear(x, w[:split], out[:, :split], status)
+        linear(x2, w[split:], out[:, split:], status)
+    else:
+        _call("pk_linear_rows2", x, x2, split, x.stride(0), w, M, w.shape[0], K, 2, out, out.stride(0), sm_count())
+    return out
+
+
 def sandwich_norm(x: torch.Tensor, *, eps: float, out: torch.Tensor | None = None, w_pre: torch.Tensor | None = None,
                   tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0, embed_add: bool = False,
                   y: torch.Tensor | None = None, y_rows: torch.Tensor | None = None, y_scale: float = 1.0, skip: torch.Tensor | None = None,
@@ -113,6 +138,11 @@ def sandwich_norm(x: torch.Tensor, *, eps: float, out: torch.Tensor | None = Non
           y_rows, 0 if y_rows is None else y_rows.shape[1], y_scale, skip, 0 if skip is None else skip.stride(0),
           int(skip is not None and skip.dtype == torch.float32), skip_w, w_post, rows, M, x.shape[1], w_pre, int(plus_one), eps, out,
           0 if out is None else out.stride(0), int(out is not None and out.dtype == torch.float32))
+
+
+def post_norm(d: PostNorm) -> None:
+    """One step of a residual stream that is normed behind the sum (see post_norm.cu)."""
+    _call("pk_post_norm", byref(d))
 
 
 def feed_tokens(nxt: torch.Tensor, tokens: torch.Tensor, pos: torch.Tensor, seqs: torch.Tensor, hist: torch.Tensor, step: torch.Tensor) -> None:
@@ -141,7 +171,7 @@ def state_chunk_workspace(d: StateMixer, nchunks: int) -> int:
 def state_chunks(d: StateMixer, seqs: torch.Tensor, nseq: int, chunks: torch.Tensor, chunk0: torch.Tensor, nchunks: int, ws: torch.Tensor) -> None:
     global launches
     _call("pk_state_chunks", byref(d), seqs, nseq, chunks, chunk0, nchunks, ws)
-    launches -= int(d.kind == KIND_RETENTION)      # no gates
+    launches -= int(d.kind in (KIND_RETENTION, KIND_HGRN))      # no gates
 
 
 def state_out(d: StateMixer, norm_w: torch.Tensor | None, per_head: bool, eps: float, last_slot: torch.Tensor, rows: int, out: torch.Tensor) -> None:
@@ -173,11 +203,32 @@ def ssd_out(d: StateMixer, norm_w: torch.Tensor, parts: int, eps: float, slots: 
     _call("pk_ssd_out", byref(d), norm_w, parts, eps, slots, behind, pos, rows, out, out.stride(0), out.shape[1], int(out.dtype == torch.float32))
 
 
+def scan_conv(d: SelectiveScan, rows: int) -> None:
+    """Convolution and SiLU of a selective-scan layer, all rows of a step."""
+    _call("pk_scan_conv", byref(d), rows)
+
+
+def scan_split(d: torch.Tensor, rank: int, out: torch.Tensor) -> None:
+    """The first `rank` columns of d (fp32) as two bf16 terms side by side, out [rows, 2 x padded rank]."""
+    _call("pk_scan_split", d, d.stride(0), rank, out.shape[1] // 2, out.shape[0], out)
+
+
+def scan_rows(d: SelectiveScan, seqs: torch.Tensor, nseq: int) -> None:
+    """Recurrence, gate and ring of short portions, W_dt included."""
+    _call("pk_scan_rows", byref(d), seqs, nseq)
+
+
+def scan_tiles(d: SelectiveScan, seqs: torch.Tensor, nseq: int) -> None:
+    """Recurrence, gate and ring of long portions."""
+    _call("pk_scan_tiles", byref(d), seqs, nseq)
+
+
 def latent_prep(proj: torch.Tensor, oq: int, oc: int, H: int, D: int, R: int, K: int, c_norm: torch.Tensor, eps: float, freq: torch.Tensor,
                 mag: float, pos: torch.Tensor, slot: torch.Tensor, cache: torch.Tensor, table: torch.Tensor, qx: torch.Tensor | None,
-                qf: torch.Tensor | None, qf_ld: int) -> None:
+                qf: torch.Tensor | None, qf_ld: int, *, q_rank: int = 0, q_norm: torch.Tensor | None = None, ql: torch.Tensor | None = None) -> None:
+    """`q_rank`: the columns at `oq` are the queries' latent, normed into `ql` [rows, padded rank]."""
     _call("pk_latent_prep", proj, proj.stride(0), oq, oc, proj.shape[0], H, D, R, K, c_norm, eps, freq, mag, pos, slot, cache, table,
-          table.stride(0), cache.shape[-1], int(cache.dtype == torch.float32), qx, qf, qf_ld)
+          table.stride(0), cache.shape[-1], int(cache.dtype == torch.float32), qx, qf, qf_ld, q_rank, q_norm, ql, 0 if ql is None else ql.shape[1])
 
 
 def latent_gather(cache: torch.Tensor, table: torch.Tensor, seqs: torch.Tensor, gather: torch.Tensor, nseq: int, max_rows: int, out: torch.Tensor) -> None:
@@ -185,8 +236,9 @@ def latent_gather(cache: torch.Tensor, table: torch.Tensor, seqs: torch.Tensor, 
 
 
 def latent_absorb(proj: torch.Tensor, oq: int, H: int, D: int, R: int, K: int, uk: torch.Tensor, rows: torch.Tensor, nrows: int, qx: torch.Tensor,
-                  row: int) -> None:
-    _call("pk_latent_absorb", proj, proj.stride(0), oq, H, D, R, K, uk, int(uk.dtype == torch.float32), rows, nrows, qx, row)
+                  row: int, k_pad: int | None = None) -> None:
+    """`R`: query columns between the heads' unrotated parts; columns K .. `k_pad` of qx are set to zero."""
+    _call("pk_latent_absorb", proj, proj.stride(0), oq, H, D, R, K, uk, int(uk.dtype == torch.float32), rows, nrows, qx, row, k_pad or K)
 
 
 def latent_rows(qx: torch.Tensor, rows: torch.Tensor, nrows: int, pos: torch.Tensor, slot: torch.Tensor, cache: torch.Tensor, table: torch.Tensor,
@@ -196,15 +248,16 @@ def latent_rows(qx: torch.Tensor, rows: torch.Tensor, nrows: int, pos: torch.Ten
 
 
 def latent_out(part_o: torch.Tensor, part_ml: torch.Tensor, nsplit: int, H: int, K: int, V: int, sink: torch.Tensor | None, rows: torch.Tensor,
-               nrows: int, uv: torch.Tensor, out: torch.Tensor) -> None:
-    _call("pk_latent_out", part_o, part_ml, nsplit, H, K, V, sink, rows, nrows, uv, int(uv.dtype == torch.float32), out, out.stride(0))
+               nrows: int, uv: torch.Tensor, out: torch.Tensor, gate: torch.Tensor | None = None) -> None:
+    _call("pk_latent_out", part_o, part_ml, nsplit, H, K, V, sink, rows, nrows, uv, int(uv.dtype == torch.float32), out, out.stride(0), gate,
+          0 if gate is None else gate.stride(0))
 
 
 def latent_prefill(q: torch.Tensor, nrows: int, kv: torch.Tensor, kv_rows: int, tiles: torch.Tensor, ntiles: int, seqs: torch.Tensor,
                    gather: torch.Tensor, H: int, qk_panels: int, v_panels: int, V: int, window: int, scale: float, sink: torch.Tensor | None,
-                   out: torch.Tensor, status: torch.Tensor) -> None:
+                   out: torch.Tensor, status: torch.Tensor, gate: torch.Tensor | None = None) -> None:
     _call("pk_latent_prefill", q, nrows, kv, kv_rows, tiles, ntiles, seqs, gather, H, qk_panels, v_panels, V, window, scale, sink, out,
-          out.stride(0), status)
+          out.stride(0), gate, 0 if gate is None else gate.stride(0), status)
 
 
 def paged_prep(a: PagedAttention, rows: int) -> None:
@@ -248,16 +301,18 @@ class Router:
     def outputs(self) -> int:
         return self.experts + self.identity
 
-    def args(self, correction: torch.Tensor | None, skip_w: torch.Tensor | None) -> tuple:
-        return self.outputs, self.top, SCORES[self.score], int(self.renorm), self.scale, correction, self.identity, skip_w
+    def args(self, correction: torch.Tensor | None, skip_w: torch.Tensor | None, bias: torch.Tensor | None) -> tuple:
+        return self.outputs, self.top, SCORES[self.score], int(self.renorm), self.scale, correction, bias, self.identity, skip_w
 
 
 def expert_up_rows(r: Router, logits: torch.Tensor, x: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, hidden: torch.Tensor, *, gated: bool = False,
-                   correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None) -> None:
+                   correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None,
+                   bias: torch.Tensor | None = None) -> None:
     """hidden [T * top, N] = squared ReLU of the chosen experts' up products, w [experts, N, K]; `gated`: silu(gate) * up, w [experts, N
-    gate rows and N up rows, K]. ids [T * top] out; `correction` [outputs] counts for the choice; skip_w [T] out (identities)."""
+    gate rows and N up rows, K]. ids [T * top] out; `correction` [outputs] counts for the choice, `bias` [outputs] is part of the
+    logits; skip_w [T] out (identities)."""
     E, N, K = w.shape
-    _call("pk_expert_up_rows", logits, logits.stride(0), *r.args(correction, skip_w), int(r.on_output), int(gated), x, x.stride(0), x.shape[0], w,
+    _call("pk_expert_up_rows", logits, logits.stride(0), *r.args(correction, skip_w, bias), int(r.on_output), int(gated), x, x.stride(0), x.shape[0], w,
           N // 2 if gated else N, K, int(w.dtype == torch.float32), ids, hidden, hidden.stride(0), sm_count())
 
 
@@ -269,9 +324,10 @@ def expert_down_rows(r: Router, ids: torch.Tensor, hidden: torch.Tensor, w: torc
 
 
 def expert_group(r: Router, logits: torch.Tensor, x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, seg: torch.Tensor, place: torch.Tensor,
-                 row_scale: torch.Tensor, rows: torch.Tensor, *, correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None) -> None:
+                 row_scale: torch.Tensor, rows: torch.Tensor, *, correction: torch.Tensor | None = None, skip_w: torch.Tensor | None = None,
+                   bias: torch.Tensor | None = None) -> None:
     """Routes of the tokens grouped by expert, token rows gathered in that order (rows [T * top, K])."""
-    _call("pk_expert_group", logits, logits.stride(0), *r.args(correction, skip_w), x.shape[0], ids, weights, seg, place, row_scale, x, x.stride(0),
+    _call("pk_expert_group", logits, logits.stride(0), *r.args(correction, skip_w, bias), x.shape[0], ids, weights, seg, place, row_scale, x, x.stride(0),
           rows.shape[1], rows)
 
 

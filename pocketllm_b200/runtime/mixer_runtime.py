@@ -159,6 +159,8 @@ class MixerRuntime:
     def _forward(self, ctx: StepContext, want: torch.Tensor | None, n_want: int) -> torch.Tensor | None:
         """The model over one batch; logits of the rows in `want` (None: of every row)."""
         m, ws, T = self.model, ctx.ws, ctx.T
+        if m.post is not None:
+            return self._forward_post(ctx, want, n_want)
         hk = m.head.K                                                   # padded width of every sublayer's input
         x = ws.rows("x", T, m.width, torch.float32)
         h = ws.rows("h", T, hk, m.dtype)
@@ -188,6 +190,62 @@ class MixerRuntime:
             return None
         hf = ws.rows("h_final", n, hk, m.dtype)
         mo.sandwich_norm(x, rows=want, count=n, w_pre=m.final_norm, out=hf, **y, **kw)
+        return m.head(ctx, hf, "logits", torch.float32)
+
+    def _forward_post(self, ctx: StepContext, want: torch.Tensor | None, n_want: int) -> torch.Tensor | None:
+        """The same for a model whose norms follow the sums. The residual stream alternates between two buffers, since a step looks at
+        the row before its own."""
+        m, ws, T = self.model, ctx.ws, ctx.T
+        hk, n = m.head.K, T if want is None else n_want
+        old, new = ws.rows("x", T, m.width, torch.float32), ws.rows("x_other", T, m.width, torch.float32)
+        h, hs, hf = ws.rows("h", T, hk, m.dtype), ws.rows("h_shift", T, hk, m.dtype), ws.rows("h_final", max(n, 1), hk, m.dtype)
+        batch = dict(pos=ctx.pos.data_ptr(), slot=ctx.slot.data_ptr(), behind=ctx.behind.data_ptr(), M=T, width=m.width, ldo=hk,
+                     out_f32=int(m.dtype == torch.float32), alpha=m.post.alpha, eps=m.eps)
+
+        def entering(i: int) -> dict:                                   # what layer i reads
+            L = m.layers[i]
+            if L.shift is None:
+                return dict(out=h)
+            return dict(out=h, out_shift=hs, shift=L.shift, before=L.before)
+
+        def step(**kw) -> None:
+            nonlocal old, new
+            y, gate = kw.get("y"), kw.get("gate")
+            for name, key in (("y", "ldy"), ("y2", "ldy2"), ("gate", "ldg")):
+                if kw.get(name) is not None:
+                    kw[key] = kw[name].stride(0)
+            if y is not None:
+                kw.update(x=old, y_top=kw["y_rows"].shape[1] if "y_rows" in kw else 0)
+            if gate is None:
+                kw.pop("gate_b", None)
+            mo.post_norm(mo.PostNorm(**{**batch, **{k: v.data_ptr() if isinstance(v, torch.Tensor) else v for k, v in kw.items()}}))
+            old, new = new, old
+
+        step(x_out=new, tokens=ctx.tokens, embed=m.embed, vocab=m.embed.shape[0], freq=m.post.freq, **entering(0))
+        finished = False
+        for i, L in enumerate(m.layers):
+            last = i + 1 == len(m.layers)
+            after = {} if last else entering(i + 1)
+            y = dict(y=L.mixer.forward(ctx, h if L.shift is None else hs, h), w=L.norm1, gate_b=L.gate_b[0], save=L.before)
+            if L.gate_b[0] is not None:
+                y["gate"] = ws.rows("proj", T, L.mixer.proj.N, torch.float32)[:, L.mixer.proj.at["gate"]:]
+            if L.mlp is None:
+                step(x_out=new, **y, **after)
+            else:
+                step(x_out=new, out=h, **y)
+                y = dict(w=L.norm2, gate_b=L.gate_b[1], **L.mlp.forward(ctx, h))
+                if last and self.launch_layers is None:
+                    finished = True
+                    if n:
+                        step(**y, rows=want, M=n, w_out=m.final_norm, out=hf)
+                else:
+                    step(x_out=new, **y, **after)
+            if self.launch_layers is not None:
+                self.launch_layers.append(old.clone())
+        if n == 0:
+            return None
+        if not finished:
+            mo.sandwich_norm(old, rows=want, count=n, w_pre=m.final_norm, out=hf, eps=m.eps, plus_one=False)
         return m.head(ctx, hf, "logits", torch.float32)
 
     def _mixed(self, entries: Sequence[StepEntry]) -> torch.Tensor:
