@@ -103,7 +103,7 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
   extern __shared__ float sm[];
   float* qs = sm;                 // [D]
   float* ks = qs + mx.D;          // [D]
-  float* as = ks + mx.D;          // [D] (GLA, HGRN2)
+  float* as = ks + mx.D;          // [D] (GLA)
   float* red = as + mx.D;         // [GR][33]
   __shared__ float s_sc[3];
   const int4 sq = seqs[blockIdx.z];          // first row, tokens, slot, first position
@@ -148,7 +148,8 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
     } else if (KIND == KIND_HGRN) {
       for (int d = threadIdx.x; d < D; d += 32 * GR) {
         qs[d] = silu_exact(pr[mx.oq + h * D + d]);
-        forget_gate(pr[mx.of + h * D + d] + mx.bf[h * D + d], mx.low[h * D + d], as[d], ks[d]);
+        float f;
+        forget_gate(pr[mx.of + h * D + d] + mx.bf[h * D + d], mx.low[h * D + d], f, ks[d]);
       }
     } else {
       for (int d = threadIdx.x; d < D; d += 32 * GR) {
@@ -191,7 +192,8 @@ __global__ void __launch_bounds__(32 * GR) state_rows_kernel(const Mixer mx, con
       for (int j = 0; j < RPT; ++j) {
         const int d = g + j * GR;
         if (d < D) {
-          s[j] = fmaf(as[d], s[j], ks[d] * v);
+          // HGRN2: what is dropped is replaced, which keeps the sum's digits when f is close to 1
+          s[j] = KIND == KIND_HGRN ? fmaf(ks[d], v - s[j], s[j]) : fmaf(as[d], s[j], ks[d] * v);
           part = fmaf(s[j], qs[d], part);
         }
       }

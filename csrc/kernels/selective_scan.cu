@@ -11,7 +11,8 @@
 //   tiles  long portions: the same lanes walk the tokens in tiles of 16 (8); the tile's B and C arrive by cp.async and its dt and x through
 //          registers while the tile before is worked on; the sums over a channel's lanes are taken for LN tokens at a time (every
 //          exchange halves the number of partial sums); the outputs of a tile are gated and stored together
-// Everything but x and W_dt is fp32.
+// Everything but x and W_dt is fp32. A decay close to 1 that is rounded to fp32 is off by the same few 2^-25 at every step of a long
+// memory; fp32 models therefore take what a state loses, exp(.) - 1, instead.
 #include "../common/pk_vec.cuh"
 
 // Plain data mirrored by the Python bindings.
@@ -22,7 +23,7 @@ struct PkSelectiveScan {
   const float* dt;         // [rows, ldt] W_dt d (tiles)
   const void* w_dt;        // [inner, ldw] (rows): `rank` columns, zeros up to a multiple of 8
   const float* dt_bias;    // [inner]
-  const float* A;          // [inner, N], negative, times log2(e)
+  const float* A;          // [inner, N], negative; times log2(e) when the model is in bf16
   const float* skip;       // [inner]
   const float* cw;         // [inner, taps], the last tap is the current token's
   const float* cb;         // [inner]
@@ -58,6 +59,12 @@ __device__ __forceinline__ float softplus_series(float z) {
   p = fmaf(p, q, 1.f / 3.f);
   p = fmaf(p * q, s, s);
   return fmaxf(z, 0.f) + 2.f * p;
+}
+
+// s exp(dt A)
+template <typename T>
+__device__ __forceinline__ float decayed(float dt, float a, float s) {
+  return sizeof(T) == 4 ? fmaf(expm1f(dt * a), s, s) : ex2(dt * a) * s;
 }
 
 template <typename T>
@@ -268,7 +275,7 @@ __global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveSca
     float y = 0.f;
 #pragma unroll
     for (int k = 0; k < NP; ++k) {
-      s[k] = fmaf(ex2(dt * a[k]), s[k], u * B[n0 + k]);
+      s[k] = fmaf(u, B[n0 + k], decayed<T>(dt, a[k], s[k]));
       y = fmaf(s[k], C[n0 + k], y);
     }
 #pragma unroll
@@ -390,7 +397,7 @@ __global__ void __launch_bounds__(THREADS) scan_tiles_kernel(const PkSelectiveSc
         y[i] = 0.f;
 #pragma unroll
         for (int k = 0; k < NP; ++k) {
-          s[k] = fmaf(ex2(q.x * a[k]), s[k], q.y * B[k]);
+          s[k] = fmaf(q.y, B[k], decayed<T>(q.x, a[k], s[k]));
           y[i] = fmaf(s[k], C[k], y[i]);
         }
       }

@@ -239,7 +239,7 @@ class SelectiveScanMixer:
         self.dt = FusedLinear([("dt", wide)], dtype, device, k_pad=wide.shape[1])
         self.kw = kw
         f = lambda n: _f32(w[n], device)
-        decay = (-torch.exp(w["A_log"].double()) * math.log2(math.e)).float().contiguous().to(device)
+        decay = (-torch.exp(w["A_log"].double()) * (math.log2(math.e) if dtype == torch.bfloat16 else 1.0)).float().contiguous().to(device)
         self.const = {"cw": f("conv"), "cb": f("conv.b"), "dt_bias": f("dt.b"), "A": decay, "skip": f("D"), "w_dt": self.dt.w}
         self.desc = dict(ox=self.proj.at["x"], oz=self.proj.at["z"], ldw=self.dt.K, inner=inner, N=N, rank=rank, taps=taps, f32=int(dtype == torch.float32),
                          **{n: t.data_ptr() for n, t in self.const.items()})
@@ -639,7 +639,7 @@ class RoutedExperts:
         self.route, self.W, self.dtype, self.gated = router, W, dtype, gate is not None
         self.router = FusedLinear([("router", router_w)] + ([] if out_gate is None else [("gate", out_gate)]), dtype, device, align=4)
         self.correction, self.bias = (None if t is None else _f32(t, device) for t in (correction, bias))
-        self.shared = shared
+        self.shared, self.gate_at = shared, self.router.at.get("gate")
         self.ff, kp = pad_to(ff, 128), pad_to(K, 64)
         self.up = torch.zeros(E, self.ff * (2 if gate else 1), kp, dtype=dtype, device=device)
         self.down = torch.zeros(E, pad_to(W, 128), self.ff, dtype=dtype, device=device)
@@ -658,8 +658,8 @@ class RoutedExperts:
         skip_w = ws.flat("route_skip", T, torch.float32) if r.identity else None
         rest = {"skip": h, "skip_w": skip_w} if r.identity else {}
         kw = {"correction": self.correction, "skip_w": skip_w, "bias": self.bias}
-        if "gate" in self.router.at:
-            rest["gate"] = z[:, self.router.at["gate"]:]
+        if self.gate_at is not None:
+            rest["gate"] = z[:, self.gate_at:]
         if self.shared is not None:
             rest["y2"] = self.shared.forward(ctx, h)["y"]
         if T <= mo.ROWS_MAX or self.dtype == torch.float32:
