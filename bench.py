@@ -282,8 +282,8 @@ def run_minimax(args) -> dict:
 def run_mixer(args) -> dict:
     """Prefill and decode throughput of a mixer decoder (Gidisun: mLSTM, GLA and windowed latent attention with SwiGLU; Pezarax:
     retention and chunked differential attention with routed experts; Zemozen: windowed attention, and attention beside a
-    state-space recurrence, with routed experts) at a size that resembles a real model's layers, beside
-    the closest other model at equal size. One step = one request: prefill of `--prompt-len` tokens, then `--decode-len` greedy
+    state-space recurrence, with routed experts; Zarinex: selective scan, gated latent attention and HGRN2, norms behind the sums,
+    routed experts beside a shared one) at a size that resembles a real model's layers, beside the closest other model at equal size. One step = one request: prefill of `--prompt-len` tokens, then `--decode-len` greedy
     tokens; a second figure decodes `--batch` requests together."""
     import torch
     from pocketllm_b200.utils import bench_mixers as bm
@@ -302,7 +302,8 @@ def run_mixer(args) -> dict:
     if args.model == "gidisun":
         like = bm.closest_model(args.size, n, d, k)
     else:
-        like = {"pezarax": bm.closest_to_pezarax, "zemozen": bm.closest_to_zemozen}[args.model](args.size, prompts, n, d, args.warmup, B)
+        like = {"pezarax": bm.closest_to_pezarax, "zemozen": bm.closest_to_zemozen,
+                "zarinex": bm.closest_to_zarinex}[args.model](args.size, prompts, n, d, args.warmup, B)
     value = k * d / r["decode_ms"] * 1e3
     return {"metric": f"single-request decode tok/s ({args.model.capitalize()}, {layers} layers of width {width}, {n}-token prompt, {d} greedy steps)",
             "value": round(value, 2), "unit": "tok/s", "n_gpus": 1, "steps": k, "warmup": args.warmup,
@@ -336,9 +337,9 @@ def main() -> int:
     ap.add_argument("--prompt-len", type=int, default=512)
     ap.add_argument("--decode-len", type=int, default=256)
     ap.add_argument("--prefill-chunk", type=int, default=512)
-    ap.add_argument("--model", default="qwen27b", choices=["qwen27b", "tiny", "minimax-m2", "gidisun", "pezarax", "zemozen"])
-    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="gidisun, pezarax, zemozen: width of the layers")
-    ap.add_argument("--batch", type=int, default=8, help="gidisun, pezarax, zemozen: requests decoded together for the second decode figure")
+    ap.add_argument("--model", default="qwen27b", choices=["qwen27b", "tiny", "minimax-m2", "gidisun", "pezarax", "zemozen", "zarinex"])
+    ap.add_argument("--size", default="4k", choices=["2k", "4k"], help="gidisun, pezarax, zemozen, zarinex: width of the layers")
+    ap.add_argument("--batch", type=int, default=8, help="gidisun, pezarax, zemozen, zarinex: requests decoded together for the second decode figure")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
@@ -347,7 +348,7 @@ def main() -> int:
         res = reference_arm.run(args)
     elif args.model == "minimax-m2":
         res = run_minimax(args)
-    elif args.model in ("gidisun", "pezarax", "zemozen"):
+    elif args.model in ("gidisun", "pezarax", "zemozen", "zarinex"):
         res = run_mixer(args)
     else:
         res = run_ours(args)

@@ -7,10 +7,12 @@
 //
 //   conv   x of all rows, into the type of the model (the operand of the product that yields d, B, C)
 //   split  d as the sum of two bf16 terms side by side, so that W_dt d of many rows on the tensor cores keeps 16 bits of d
-//   rows   portions of a few tokens: LN lanes per channel with NP states each, W_dt d in the same kernel (fp32 sums)
-//   tiles  long portions: the same lanes walk the tokens in tiles of 16 (8); the tile's B and C arrive by cp.async and its dt and x through
-//          registers while the tile before is worked on; the sums over a channel's lanes are taken for LN tokens at a time (every
-//          exchange halves the number of partial sums); the outputs of a tile are gated and stored together
+//   rows   portions of a few tokens: LN lanes per channel with NP states each, W_dt d in the same kernel (fp32 sums); a block takes a
+//          few portions, which share its rows of W_dt
+//   tiles  long portions: the same lanes walk the tokens in tiles of 16 (8), two states per instruction. Between two barriers a block
+//          requests tile i + 3 (cp.async), makes dt and dt x of tile i + 1, runs the recurrence over tile i, and gates and stores the
+//          outputs of tile i - 1: independent work that fills the waits of the recurrence. The sums over a channel's lanes are taken for
+//          LN tokens at a time (every exchange halves the number of partial sums)
 // Everything but x and W_dt is fp32. A decay close to 1 that is rounded to fp32 is off by the same few 2^-25 at every step of a long
 // memory; fp32 models therefore take what a state loses, exp(.) - 1, instead.
 #include "../common/pk_vec.cuh"
@@ -19,7 +21,7 @@
 struct PkSelectiveScan {
   const float* proj;       // [rows, ld]: x at column ox, z at oz
   const void* xc;          // [rows, ldx] x behind its convolution (model's type); conv writes it
-  const float* dbc;        // [rows, ldb]: d | B | C
+  const float* dbc;        // [rows, ldb]: d, B at column oB, C at oC
   const float* dt;         // [rows, ldt] W_dt d (tiles)
   const void* w_dt;        // [inner, ldw] (rows): `rank` columns, zeros up to a multiple of 8
   const float* dt_bias;    // [inner]
@@ -32,7 +34,7 @@ struct PkSelectiveScan {
   void* out;               // [rows, ldo], columns from inner on zero
   const int* pos;
   const int* slot;
-  int ld, ox, oz, ldx, ldb, ldt, ldw, ldo, inner, N, rank, taps, f32;
+  int ld, ox, oz, ldx, ldb, ldt, ldw, ldo, oB, oC, inner, N, rank, taps, f32;
 };
 
 namespace {
@@ -209,18 +211,14 @@ __device__ __forceinline__ void store_states(float* row, int n0, int N, const fl
   }
 }
 
-// Block: THREADS / LN channels of one short portion.
-template <typename T, int NP, int LN>
-__global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveScan p, const int4* seqs) {
-  constexpr int CB = THREADS / LN, VE = 16 / sizeof(T), AHEAD = 4;
+// Block: THREADS / LN channels of up to SQ short portions.
+template <typename T, int NP, int LN, int SQ>
+__global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveScan p, const int4* seqs, int nseq) {
+  constexpr int CB = THREADS / LN, NS = LN * NP, VE = 16 / sizeof(T), AHEAD = SQ == 1 ? 4 : 8;
   extern __shared__ float sm[];
-  const int4 sq = seqs[blockIdx.y];            // first row, tokens, slot, first position
   const int tid = threadIdx.x, l = tid % LN, c = blockIdx.x * CB + tid / LN, n0 = l * NP;
   const bool live = c < p.inner;
-  const int kw = (p.rank + 7) & ~7;
-  float* d = sm;                               // [kw] input of W_dt
-  float* B = d + kw;                           // [LN * NP] each
-  float* C = B + LN * NP;
+  const int kw = (p.rank + 7) & ~7, unit = kw + 2 * NS;      // per portion: d [kw], B, C [NS]
   // weights first: no kernel writes them
   const T* wrow = (const T*)p.w_dt + (size_t)(live ? c : 0) * p.ldw;
   uint4 first[AHEAD];
@@ -236,60 +234,86 @@ __global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveSca
   const float bias = live ? p.dt_bias[c] : 0.f, skip = live ? p.skip[c] : 0.f;
   pdl_trigger();
   pdl_wait();
-  float s[NP];
+  int4 sq[SQ];                                               // first row, tokens, slot, first position
+  float s[SQ][NP];
+  int most = 0;
 #pragma unroll
-  for (int k = 0; k < NP; ++k) s[k] = 0.f;
-  float* Sp = p.S + ((size_t)sq.z * p.inner + (live ? c : 0)) * p.N;
-  if (live && sq.w > 0) load_states<NP>(Sp, n0, p.N, s);
-  for (int t = 0; t < sq.y; ++t) {
-    const size_t row = (size_t)sq.x + t;
-    const float* src = p.dbc + row * p.ldb;
-    for (int i = tid; i < kw; i += THREADS) d[i] = i < p.rank ? src[i] : 0.f;
-    for (int i = tid; i < LN * NP; i += THREADS) {
-      B[i] = i < p.N ? src[p.rank + i] : 0.f;
-      C[i] = i < p.N ? src[p.rank + p.N + i] : 0.f;
-    }
-    const float x = live ? to_f<T>(((const T*)p.xc)[row * p.ldx + c]) : 0.f;
-    float z = 0.f, in = 0.f;
-    if (live && l == 0) {
-      z = p.proj[row * p.ld + p.oz + c];
-      if (sq.y - 1 - t < p.taps - 1) in = p.proj[row * p.ld + p.ox + c];
+  for (int q = 0; q < SQ; ++q) {
+    const int at = blockIdx.y * SQ + q;
+    sq[q] = at < nseq ? seqs[at] : make_int4(0, 0, 0, 0);
+    most = max(most, sq[q].y);
+#pragma unroll
+    for (int k = 0; k < NP; ++k) s[q][k] = 0.f;
+    if (live && sq[q].w > 0) load_states<NP>(p.S + ((size_t)sq[q].z * p.inner + c) * p.N, n0, p.N, s[q]);
+  }
+  for (int t = 0; t < most; ++t) {
+    float x[SQ], z[SQ], in[SQ];
+#pragma unroll
+    for (int q = 0; q < SQ; ++q) {
+      const bool on = t < sq[q].y;
+      const size_t row = (size_t)sq[q].x + t;
+      const float* src = p.dbc + row * p.ldb;
+      float* d = sm + q * unit;
+      if (on) {
+        for (int i = tid; i < kw; i += THREADS) d[i] = i < p.rank ? src[i] : 0.f;
+        for (int i = tid; i < NS; i += THREADS) {
+          d[kw + i] = i < p.N ? src[p.oB + i] : 0.f;
+          d[kw + NS + i] = i < p.N ? src[p.oC + i] : 0.f;
+        }
+      }
+      x[q] = on && live ? to_f<T>(((const T*)p.xc)[row * p.ldx + c]) : 0.f;
+      z[q] = in[q] = 0.f;
+      if (on && live && l == 0) {
+        z[q] = p.proj[row * p.ld + p.oz + c];
+        if (sq[q].y - 1 - t < p.taps - 1) in[q] = p.proj[row * p.ld + p.ox + c];
+      }
     }
     __syncthreads();
-    float dot = 0.f;
+    float dot[SQ];
+#pragma unroll
+    for (int q = 0; q < SQ; ++q) dot[q] = 0.f;
     auto add = [&](const uint4& u, int k) {
       const T* e = reinterpret_cast<const T*>(&u);
 #pragma unroll
-      for (int i = 0; i < VE; ++i) dot = fmaf(to_f<T>(e[i]), d[k + i], dot);
+      for (int q = 0; q < SQ; ++q)
+#pragma unroll
+        for (int i = 0; i < VE; ++i) dot[q] = fmaf(to_f<T>(e[i]), sm[q * unit + k + i], dot[q]);
     };
     if (live) {
 #pragma unroll
       for (int i = 0; i < AHEAD; ++i)
         if ((l + i * LN) * VE < kw) add(first[i], (l + i * LN) * VE);
-#pragma unroll 4
       for (int k = (l + AHEAD * LN) * VE; k < kw; k += LN * VE) add(*reinterpret_cast<const uint4*>(wrow + k), k);
     }
 #pragma unroll
-    for (int o = LN / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-    const float dt = softplus_series(dot + bias), u = dt * x;
-    float y = 0.f;
+    for (int q = 0; q < SQ; ++q) {
 #pragma unroll
-    for (int k = 0; k < NP; ++k) {
-      s[k] = fmaf(u, B[n0 + k], decayed<T>(dt, a[k], s[k]));
-      y = fmaf(s[k], C[n0 + k], y);
-    }
+      for (int o = LN / 2; o > 0; o >>= 1) dot[q] += __shfl_xor_sync(0xffffffffu, dot[q], o);
+      if (t >= sq[q].y) continue;
+      const float* B = sm + q * unit + kw;
+      const float dt = softplus_series(dot[q] + bias), u = dt * x[q];
+      float y = 0.f;
 #pragma unroll
-    for (int o = LN / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-    if (live && l == 0) {
+      for (int k = 0; k < NP; ++k) {
+        s[q][k] = fmaf(u, B[n0 + k], decayed<T>(dt, a[k], s[q][k]));
+        y = fmaf(s[q][k], B[NS + n0 + k], y);
+      }
+#pragma unroll
+      for (int o = LN / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+      const size_t row = (size_t)sq[q].x + t;
       T* out = (T*)p.out + row * p.ldo;
-      out[c] = (T)(fmaf(skip, x, y) * silu_of<T>(z));
-      if (sq.y - 1 - t < p.taps - 1) ring_at(p, sq.z, sq.w + t)[c] = in;
+      if (live && l == 0) {
+        out[c] = (T)(fmaf(skip, x[q], y) * silu_of<T>(z[q]));
+        if (sq[q].y - 1 - t < p.taps - 1) ring_at(p, sq[q].z, sq[q].w + t)[c] = in[q];
+      }
+      if (blockIdx.x == gridDim.x - 1)
+        for (int i = p.inner + tid; i < p.ldo; i += THREADS) out[i] = (T)0.f;
     }
-    if (blockIdx.x == gridDim.x - 1)
-      for (int i = p.inner + tid; i < p.ldo; i += THREADS) ((T*)p.out)[row * p.ldo + i] = (T)0.f;
-    if (t + 1 < sq.y) __syncthreads();
+    if (t + 1 < most) __syncthreads();
   }
-  if (live) store_states<NP>(Sp, n0, p.N, s);
+#pragma unroll
+  for (int q = 0; q < SQ; ++q)
+    if (live && sq[q].y > 0) store_states<NP>(p.S + ((size_t)sq[q].z * p.inner + c) * p.N, n0, p.N, s[q]);
 }
 
 // Sums of v[i] over the lanes of a group of G for i < G: lane l of the group gets the sum of v[l].
@@ -307,135 +331,253 @@ __device__ __forceinline__ float group_sums(float (&v)[G], int l) {
   return v[0];
 }
 
-__device__ __forceinline__ void async_f32(float* dst, const float* src, bool in) {      // 4 bytes, or zero
+template <int BYTES>
+__device__ __forceinline__ void async_copy(void* dst, const void* src, int bytes) {      // the rest of BYTES is zero
   const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(a), "l"(src), "r"(in ? 4 : 0) : "memory");
+  if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
 }
+
+typedef unsigned long long f32x2;
+__device__ __forceinline__ f32x2 pack2(float x, float y) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(x), "f"(y));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& x, float& y) { asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(v)); }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+
+// One step of NP states of a channel; what their lane adds to y.
+template <typename T, int NP>
+struct States {
+  float a[NP], s[NP];
+  __device__ __forceinline__ void start() {}
+  __device__ __forceinline__ float step(float dt, float u, const float* B, const float* C) {
+    float y = 0.f;
+#pragma unroll
+    for (int k = 0; k < NP; ++k) {
+      s[k] = fmaf(u, B[k], decayed<T>(dt, a[k], s[k]));
+      y = fmaf(s[k], C[k], y);
+    }
+    return y;
+  }
+  __device__ __forceinline__ void finish() {}
+};
+template <int NP>
+struct States<bf16, NP> {
+  float a[NP], s[NP];
+  f32x2 a2[NP / 2], s2[NP / 2];
+  __device__ __forceinline__ void start() {
+#pragma unroll
+    for (int k = 0; k < NP / 2; ++k) {
+      a2[k] = pack2(a[2 * k], a[2 * k + 1]);
+      s2[k] = pack2(s[2 * k], s[2 * k + 1]);
+    }
+  }
+  __device__ __forceinline__ float step(float dt, float u, const float* B, const float* C) {
+    const f32x2 dt2 = pack2(dt, dt), u2 = pack2(u, u);
+    f32x2 y = 0;
+#pragma unroll
+    for (int k = 0; k < NP / 4; ++k) {
+      const ulonglong2 b = reinterpret_cast<const ulonglong2*>(B)[k], c = reinterpret_cast<const ulonglong2*>(C)[k];
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        float x0, x1;
+        unpack2(mul2(dt2, a2[2 * k + j]), x0, x1);
+        s2[2 * k + j] = fma2(pack2(ex2(x0), ex2(x1)), s2[2 * k + j], mul2(u2, j ? b.y : b.x));
+        y = fma2(s2[2 * k + j], j ? c.y : c.x, y);
+      }
+    }
+    float y0, y1;
+    unpack2(y, y0, y1);
+    return y0 + y1;
+  }
+  __device__ __forceinline__ void finish() {
+#pragma unroll
+    for (int k = 0; k < NP / 2; ++k) unpack2(s2[k], s[2 * k], s[2 * k + 1]);
+  }
+};
+
+// Shared memory of a tiles block: STAGES raw tiles, then two tiles of (dt, dt x) and of sums.
+template <typename T, int NP, int LN>
+struct TileShape {
+  static constexpr int CB = THREADS / LN, NS = LN * NP, TT = NS > 128 ? 8 : 16, STAGES = 5;
+  static constexpr int YS = CB + 8;                            // row of the sums: lanes of a group store to different banks
+  static constexpr int DT = 0, Z = DT + TT * CB * 4, X = Z + TT * CB * 4, B = X + TT * CB * (int)sizeof(T), C = B + TT * NS * 4, RAW = C + TT * NS * 4;
+  static constexpr int DU = STAGES * RAW, Y = DU + 2 * TT * CB * 8, BYTES = Y + 2 * TT * YS * 4;
+};
 
 // Block: THREADS / LN channels of one long portion, all its tokens.
 template <typename T, int NP, int LN>
 __global__ void __launch_bounds__(THREADS) scan_tiles_kernel(const PkSelectiveScan p, const int4* seqs) {
   pdl_trigger();
   pdl_wait();
-  constexpr int CB = THREADS / LN, NS = LN * NP, TT = NS > 128 ? 8 : 16, G = LN < TT ? LN : TT;      // TT: tokens of a tile
-  constexpr int ITEMS = (TT * CB + THREADS - 1) / THREADS;      // (token, channel) pairs of a tile per thread
-  __shared__ __align__(16) float Bs[2][TT][NS], Cs[2][TT][NS];
-  __shared__ float2 du[TT][CB];                                 // dt, dt x
-  __shared__ float ys[TT][CB];
+  using Sh = TileShape<T, NP, LN>;
+  constexpr int CB = Sh::CB, NS = Sh::NS, TT = Sh::TT, G = LN < TT ? LN : TT, QC = CB / 4, QN = NS / 4;
+  extern __shared__ __align__(16) uint8_t smem[];
   const int4 sq = seqs[blockIdx.y];
   const int tid = threadIdx.x, l = tid % LN, ch = tid / LN, c0 = blockIdx.x * CB, c = c0 + ch, n0 = l * NP;
   const bool live = c < p.inner;
-  const int n = sq.y;
-  float a[NP], s[NP];
+  const int n = sq.y, tiles = (n + TT - 1) / TT;
+  States<T, NP> st;
 #pragma unroll
-  for (int k = 0; k < NP; ++k) a[k] = s[k] = 0.f;
+  for (int k = 0; k < NP; ++k) st.a[k] = st.s[k] = 0.f;
   float* Sp = p.S + ((size_t)sq.z * p.inner + (live ? c : 0)) * p.N;
   if (live) {
-    load_states<NP>(p.A + (size_t)c * p.N, n0, p.N, a);
-    if (sq.w > 0) load_states<NP>(Sp, n0, p.N, s);
+    load_states<NP>(p.A + (size_t)c * p.N, n0, p.N, st.a);
+    if (sq.w > 0) load_states<NP>(Sp, n0, p.N, st.s);
   }
-  // what a thread stages of a tile: dt and x (and z, the raw x for its epilogue) of its pairs
-  float dt[ITEMS], x[ITEMS], z[ITEMS], x_now[ITEMS], z_now[ITEMS];
-  auto fetch = [&](int t0) {
-#pragma unroll
-    for (int i = 0; i < ITEMS; ++i) {
-      const int e = tid + i * THREADS, t = t0 + e / CB, cc = c0 + e % CB;
-      dt[i] = x[i] = z[i] = 0.f;
-      if (e < TT * CB && t < n && cc < p.inner) {
-        const size_t row = (size_t)sq.x + t;
-        dt[i] = p.dt[row * p.ldt + cc];
-        x[i] = to_f<T>(((const T*)p.xc)[row * p.ldx + cc]);
-        z[i] = p.proj[row * p.ld + p.oz + cc];
+  st.start();
+  auto raw = [&](int i) { return smem + (i % Sh::STAGES) * Sh::RAW; };
+  auto du = [&](int i) { return reinterpret_cast<float4*>(smem + Sh::DU) + (i & 1) * TT * CB / 2; };       // two channels per float4
+  auto ys = [&](int i) { return reinterpret_cast<float*>(smem + Sh::Y) + (i & 1) * TT * Sh::YS; };
+  auto request = [&](int i) {
+    if (i < tiles) {
+      uint8_t* dst = raw(i);
+      for (int e = tid; e < TT * QC; e += THREADS) {
+        const int t = i * TT + e / QC, cc = c0 + e % QC * 4;
+        const bool in = t < n && cc < p.inner;
+        const size_t row = (size_t)sq.x + (in ? t : 0);
+        const int col = in ? cc : 0, bytes = in ? min(16, (p.inner - cc) * 4) : 0;
+        async_copy<16>(dst + Sh::DT + e * 16, p.dt + row * p.ldt + col, bytes);
+        async_copy<16>(dst + Sh::Z + e * 16, p.proj + row * p.ld + p.oz + col, bytes);
+        async_copy<4 * sizeof(T)>(dst + Sh::X + e * 4 * sizeof(T), (const T*)p.xc + row * p.ldx + col, in ? 4 * (int)sizeof(T) : 0);
       }
-    }
-  };
-  auto fetch_bc = [&](int t0, int b) {
-    for (int e = tid; e < TT * NS; e += THREADS) {
-      const int t = e / NS, k = e % NS;
-      const bool in = t0 + t < n && k < p.N;
-      const float* src = p.dbc + ((size_t)sq.x + min(t0 + t, n - 1)) * p.ldb + p.rank + min(k, p.N - 1);
-      async_f32(&Bs[b][t][k], src, in);
-      async_f32(&Cs[b][t][k], src + p.N, in);
+      for (int e = tid; e < TT * QN; e += THREADS) {
+        const int t = i * TT + e / QN, k = e % QN * 4;
+        const bool in = t < n && k < p.N;
+        const float* src = p.dbc + ((size_t)sq.x + (in ? t : 0)) * p.ldb;
+        const int bytes = in ? min(16, (p.N - k) * 4) : 0;
+        async_copy<16>(dst + Sh::B + e * 16, src + p.oB + (in ? k : 0), bytes);
+        async_copy<16>(dst + Sh::C + e * 16, src + p.oC + (in ? k : 0), bytes);
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  float bias[ITEMS], skip[ITEMS];
+  auto load_x = [&](const uint8_t* tile, int e, float (&x)[4]) { load_any<4>(tile + Sh::X, (size_t)e * 4, sizeof(T) == 4, x); };
+  // a thread's groups of four channels have one place in a row
+  float bias[4], skip[4];
+  const int cq = c0 + tid % QC * 4;
 #pragma unroll
-  for (int i = 0; i < ITEMS; ++i) {
-    const int cc = c0 + (tid + i * THREADS) % CB;
-    bias[i] = cc < p.inner ? p.dt_bias[cc] : 0.f;
-    skip[i] = cc < p.inner ? p.skip[cc] : 0.f;
+  for (int k = 0; k < 4; ++k) {
+    bias[k] = cq + k < p.inner ? p.dt_bias[cq + k] : 0.f;
+    skip[k] = cq + k < p.inner ? p.skip[cq + k] : 0.f;
   }
-  fetch_bc(0, 0);
-  fetch(0);
-  for (int t0 = 0, b = 0; t0 < n; t0 += TT, b ^= 1) {
+  auto prepare = [&](int i) {                                 // dt and dt x; a token behind the end changes nothing
+    const uint8_t* tile = raw(i);
+    for (int e = tid; e < TT * QC; e += THREADS) {
+      const float4 v = reinterpret_cast<const float4*>(tile + Sh::DT)[e];
+      const float d[4] = {v.x, v.y, v.z, v.w};
+      float x[4], dt[4];
+      load_x(tile, e, x);
+      const bool in = i * TT + e / QC < n;
 #pragma unroll
-    for (int i = 0; i < ITEMS; ++i) {
-      const int e = tid + i * THREADS;
-      x_now[i] = x[i];
-      z_now[i] = z[i];
-      if (e < TT * CB) {
-        const float d = t0 + e / CB < n ? softplus_series(dt[i] + bias[i]) : 0.f;      // a token behind the end changes nothing
-        du[e / CB][e % CB] = make_float2(d, d * x[i]);
+      for (int k = 0; k < 4; ++k) dt[k] = in ? softplus_series(d[k] + bias[k]) : 0.f;
+      du(i)[2 * e] = make_float4(dt[0], dt[0] * x[0], dt[1], dt[1] * x[1]);
+      du(i)[2 * e + 1] = make_float4(dt[2], dt[2] * x[2], dt[3], dt[3] * x[3]);
+    }
+  };
+  auto finish = [&](int i) {                                  // skip, gate, store, ring
+    const uint8_t* tile = raw(i);
+    for (int e = tid; e < TT * QC; e += THREADS) {
+      const int t = i * TT + e / QC;
+      if (t >= n || cq >= p.inner) continue;
+      const float4 y4 = *reinterpret_cast<const float4*>(ys(i) + e / QC * Sh::YS + e % QC * 4), z4 = reinterpret_cast<const float4*>(tile + Sh::Z)[e];
+      const float y[4] = {y4.x, y4.y, y4.z, y4.w}, z[4] = {z4.x, z4.y, z4.z, z4.w};
+      float x[4], o[4];
+      load_x(tile, e, x);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) o[k] = fmaf(skip[k], x[k], y[k]) * silu_of<T>(z[k]);
+      const size_t row = (size_t)sq.x + t;
+      T* out = (T*)p.out + row * p.ldo + cq;
+      if (cq + 4 <= p.inner) {
+        store<4>(out, o);
+      } else {
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          if (cq + k < p.inner) out[k] = (T)o[k];
       }
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    if (t0 + TT < n) {
-      fetch_bc(t0 + TT, b ^ 1);
-      fetch(t0 + TT);
-    }
-#pragma unroll 1
-    for (int tg = 0; tg < TT; tg += G) {
-      float y[G];
+      if (n - 1 - t < p.taps - 1) {
+        float* ring = ring_at(p, sq.z, sq.w + t) + cq;
+        const float* in = p.proj + row * p.ld + p.ox + cq;
 #pragma unroll
-      for (int i = 0; i < G; ++i) {
-        const float2 q = du[tg + i][ch];
-        float B[NP], C[NP];
-        load_states<NP>(Bs[b][tg + i], n0, NS, B);
-        load_states<NP>(Cs[b][tg + i], n0, NS, C);
-        y[i] = 0.f;
-#pragma unroll
-        for (int k = 0; k < NP; ++k) {
-          s[k] = fmaf(q.y, B[k], decayed<T>(q.x, a[k], s[k]));
-          y[i] = fmaf(s[k], C[k], y[i]);
-        }
-      }
-      float sum = group_sums<G>(y, l);
-#pragma unroll
-      for (int o = G; o < LN; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      if (l < G) ys[tg + l][ch] = sum;
-    }
-    __syncthreads();
-#pragma unroll
-    for (int i = 0; i < ITEMS; ++i) {
-      const int e = tid + i * THREADS, t = t0 + e / CB, cc = c0 + e % CB;
-      if (e < TT * CB && t < n && cc < p.inner) {
-        const size_t row = (size_t)sq.x + t;
-        ((T*)p.out)[row * p.ldo + cc] = (T)(fmaf(skip[i], x_now[i], ys[e / CB][e % CB]) * silu_of<T>(z_now[i]));
-        if (n - 1 - t < p.taps - 1) ring_at(p, sq.z, sq.w + t)[cc] = p.proj[row * p.ld + p.ox + cc];
+        for (int k = 0; k < 4; ++k)
+          if (cq + k < p.inner) ring[k] = in[k];
       }
     }
     if (blockIdx.x == gridDim.x - 1 && p.ldo > p.inner) {
       const int pad = p.ldo - p.inner;
       for (int e = tid; e < TT * pad; e += THREADS)
-        if (t0 + e / pad < n) ((T*)p.out)[((size_t)sq.x + t0 + e / pad) * p.ldo + p.inner + e % pad] = (T)0.f;
+        if (i * TT + e / pad < n) ((T*)p.out)[((size_t)sq.x + i * TT + e / pad) * p.ldo + p.inner + e % pad] = (T)0.f;
     }
+  };
+  request(0);
+  request(1);
+  request(2);
+  asm volatile("cp.async.wait_group 2;" ::: "memory");
+  __syncthreads();
+  prepare(0);
+  for (int i = 0; i < tiles; ++i) {
+    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();                                          // dt of tile i, sums of tile i - 1, raw tile i + 1; tile i - 2 is done with
+    request(i + 3);
+    if (i + 1 < tiles) prepare(i + 1);
+    const float* B = reinterpret_cast<const float*>(raw(i) + Sh::B) + n0;
+    const float* C = reinterpret_cast<const float*>(raw(i) + Sh::C) + n0;
+    const float2* q = reinterpret_cast<const float2*>(du(i)) + ch;
+    float* sums = ys(i) + ch;
+#pragma unroll
+    for (int tg = 0; tg < TT; tg += G) {
+      float y[G];
+#pragma unroll
+      for (int j = 0; j < G; ++j) {
+        const float2 v = q[(tg + j) * CB];
+        y[j] = st.step(v.x, v.y, B + (tg + j) * NS, C + (tg + j) * NS);
+      }
+      float sum = group_sums<G>(y, l);
+#pragma unroll
+      for (int o = G; o < LN; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      if (l < G) sums[(tg + l) * Sh::YS] = sum;
+    }
+    if (i > 0) finish(i - 1);
   }
-  if (live) store_states<NP>(Sp, n0, p.N, s);
+  __syncthreads();
+  finish(tiles - 1);
+  st.finish();
+  if (live) store_states<NP>(Sp, n0, p.N, st.s);
+}
+
+template <typename T, int NP, int LN, int SQ>
+int launch_rows(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream_t stream) {
+  const size_t smem = (size_t)SQ * (((p.rank + 7) & ~7) + 2 * NP * LN) * sizeof(float);
+  if (smem > 48 * 1024) return PK_ERR_UNSUPPORTED;
+  const dim3 grid((p.inner + THREADS / LN - 1) / (THREADS / LN), (nseq + SQ - 1) / SQ);
+  PK_LAUNCH_PDL((scan_rows_kernel<T, NP, LN, SQ>), grid, dim3(THREADS), smem, stream, p, seqs, nseq);
+  return PK_OK;
 }
 
 template <typename T, int NP, int LN>
 int launch_scan(const PkSelectiveScan& p, const int4* seqs, int nseq, bool tiles, cudaStream_t stream) {
-  constexpr int CB = THREADS / LN;
-  const dim3 grid((p.inner + CB - 1) / CB, nseq);
-  if (tiles) {
-    PK_LAUNCH_PDL((scan_tiles_kernel<T, NP, LN>), grid, dim3(THREADS), (size_t)0, stream, p, seqs);
-  } else {
-    const size_t smem = (size_t)(((p.rank + 7) & ~7) + 2 * NP * LN) * sizeof(float);
-    if (smem > 48 * 1024) return PK_ERR_UNSUPPORTED;
-    PK_LAUNCH_PDL((scan_rows_kernel<T, NP, LN>), grid, dim3(THREADS), smem, stream, p, seqs);
+  if (!tiles) return nseq == 1 || p.rank > 1024 ? launch_rows<T, NP, LN, 1>(p, seqs, nseq, stream) : launch_rows<T, NP, LN, 4>(p, seqs, nseq, stream);
+  using Sh = TileShape<T, NP, LN>;
+  static PkDeviceOnce once;
+  if (PkDeviceOnceGuard g{once}; g.needed()) {
+    if (cudaFuncSetAttribute((const void*)scan_tiles_kernel<T, NP, LN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Sh::BYTES) != cudaSuccess) {
+      pk_set_last_cuda_error((int)cudaGetLastError());
+      return PK_ERR_CUDA;
+    }
+    g.done();
   }
+  PK_LAUNCH_PDL((scan_tiles_kernel<T, NP, LN>), dim3((p.inner + Sh::CB - 1) / Sh::CB, nseq), dim3(THREADS), (size_t)Sh::BYTES, stream, p, seqs);
   return PK_OK;
 }
 
@@ -477,7 +619,7 @@ bool scan_ok(const PkSelectiveScan* d) {
 }
 
 bool recurrence_ok(const PkSelectiveScan* d, const void* seqs, int nseq) {
-  return scan_ok(d) && seqs != nullptr && nseq >= 1 && nseq <= 65535 && d->dbc != nullptr && d->ldb >= d->rank + 2 * d->N && d->dt_bias != nullptr && d->A != nullptr &&
+  return scan_ok(d) && seqs != nullptr && nseq >= 1 && nseq <= 65535 && d->dbc != nullptr && d->oB >= d->rank && d->oC >= d->oB + d->N && d->ldb >= d->oC + d->N && d->dt_bias != nullptr && d->A != nullptr &&
          d->skip != nullptr && d->S != nullptr && d->out != nullptr && d->ldo >= d->inner &&
          ((d->N & 3) != 0 || (((uintptr_t)d->A & 15) == 0 && ((uintptr_t)d->S & 15) == 0));
 }
@@ -504,8 +646,12 @@ PK_API int pk_scan_rows(const PkSelectiveScan* d, const void* seqs, int nseq, cu
   return d->f32 ? launch_scan<float>(*d, (const int4*)seqs, nseq, false, stream) : launch_scan<pk::bf16>(*d, (const int4*)seqs, nseq, false, stream);
 }
 
-// Long portions, W_dt d given.
+// Long portions, W_dt d given. Rows of dt, dbc and proj, and the columns oB, oC and oz, start on 16 bytes, rows of xc and out on four
+// elements; xc is zero from inner on.
 PK_API int pk_scan_tiles(const PkSelectiveScan* d, const void* seqs, int nseq, cudaStream_t stream) {
   if (!recurrence_ok(d, seqs, nseq) || d->dt == nullptr || d->ldt < d->inner) return PK_ERR_BAD_ARG;
+  if (((d->ldt | d->ld | d->ldb | d->oB | d->oC | d->oz | d->ldx | d->ldo) & 3) != 0 || d->ldx < ((d->inner + 3) & ~3) || ((uintptr_t)d->dt & 15) != 0 ||
+      ((uintptr_t)d->proj & 15) != 0 || ((uintptr_t)d->dbc & 15) != 0 || ((uintptr_t)d->xc & 15) != 0 || ((uintptr_t)d->out & 15) != 0)
+    return PK_ERR_BAD_ARG;
   return d->f32 ? launch_scan<float>(*d, (const int4*)seqs, nseq, true, stream) : launch_scan<pk::bf16>(*d, (const int4*)seqs, nseq, true, stream);
 }

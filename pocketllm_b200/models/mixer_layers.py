@@ -229,7 +229,7 @@ class SelectiveScanMixer:
             if any(b is not None and a != b for a, b in zip(w[n].shape, s)):
                 raise ValueError(f"{n}: shape {tuple(w[n].shape)}, expected {s}")
         self.proj = FusedLinear([("x", w["in"][:inner]), ("z", w["in"][inner:])], dtype, device, align=4, beside=beside)
-        self.dbc = FusedLinear([("dbc", w["x"])], dtype, device)
+        self.dbc = FusedLinear([("d", w["x"][:rank]), ("B", w["x"][rank:rank + N]), ("C", w["x"][rank + N:])], dtype, device, align=4)
         self.out = FusedLinear([("o", w["o"])], dtype, device)
         # step sizes: few rows read the plain matrix, many rows multiply it with a two-term input in bf16
         kw = pad_to(rank, 32)
@@ -241,7 +241,7 @@ class SelectiveScanMixer:
         f = lambda n: _f32(w[n], device)
         decay = (-torch.exp(w["A_log"].double()) * (math.log2(math.e) if dtype == torch.bfloat16 else 1.0)).float().contiguous().to(device)
         self.const = {"cw": f("conv"), "cb": f("conv.b"), "dt_bias": f("dt.b"), "A": decay, "skip": f("D"), "w_dt": self.dt.w}
-        self.desc = dict(ox=self.proj.at["x"], oz=self.proj.at["z"], ldw=self.dt.K, inner=inner, N=N, rank=rank, taps=taps, f32=int(dtype == torch.float32),
+        self.desc = dict(ox=self.proj.at["x"], oz=self.proj.at["z"], oB=self.dbc.at["B"], oC=self.dbc.at["C"], ldw=self.dt.K, inner=inner, N=N, rank=rank, taps=taps, f32=int(dtype == torch.float32),
                          **{n: t.data_ptr() for n, t in self.const.items()})
         self._memory(slots, device)
 

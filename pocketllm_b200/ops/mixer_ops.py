@@ -43,7 +43,7 @@ class PagedAttention(Structure):
 class SelectiveScan(Structure):
     """`PkSelectiveScan`: one selective-scan layer over one batch."""
     _fields_ = [(n, c_void_p) for n in ("proj", "xc", "dbc", "dt", "w_dt", "dt_bias", "A", "skip", "cw", "cb", "S", "ring", "out", "pos", "slot")] + \
-               [(n, c_int) for n in ("ld", "ox", "oz", "ldx", "ldb", "ldt", "ldw", "ldo", "inner", "N", "rank", "taps", "f32")]
+               [(n, c_int) for n in ("ld", "ox", "oz", "ldx", "ldb", "ldt", "ldw", "ldo", "oB", "oC", "inner", "N", "rank", "taps", "f32")]
 
 
 class PostNorm(Structure):

@@ -1,10 +1,11 @@
 """Throughput of mixer decoders at sizes that resemble a real model's layers, beside the closest other model at equal size
 (Gidisun: the Qwen hybrid, DeltaNet + GQA with the same width, feed-forward, depth and vocabulary; Pezarax: Gidisun with the
 same width, heads, depth and as many weights per token in its feed-forward; Zemozen: Pezarax with the same width, depth, number
-of experts and weights per expert), and the time of each design's kernels beside the like kernels of the other families.
+of experts and weights per expert; Zarinex: Zemozen with the same width, depth, number of experts and weights per expert), and the time
+of each design's kernels beside the like kernels of the other families.
 
-    python -m pocketllm_b200.utils.bench_mixers --kernels [gidisun|pezarax|zemozen]
-    python bench.py --model gidisun|pezarax|zemozen [--size 2k|4k]
+    python -m pocketllm_b200.utils.bench_mixers --kernels [gidisun|pezarax|zemozen|zarinex]
+    python bench.py --model gidisun|pezarax|zemozen|zarinex [--size 2k|4k]
 
 Random weights; every weight set is larger than L2. Device times by CUDA events.
 """
@@ -17,6 +18,7 @@ import torch
 
 from ..models import gidisun as gd
 from ..models import pezarax as pz
+from ..models import zarinex as zx
 from ..models import zemozen as zm
 
 VOCAB = 32000
@@ -60,6 +62,22 @@ def zemozen_config(size: str) -> zm.ZemozenConfig:
                                        "residual_mult": 0.7, "layers": [{"type": t, "mixer": mix[t], "mlp": mlp} for t in ZEMOZEN_PATTERN]})
 
 
+#                  width  scan (inner, state, dt rank)  latent (heads, dim, vdim, query rank, rank)  HGRN2 (heads, dim, vdim)  experts (number, top, ff, shared ff)
+ZARINEX_SIZES = {"2k": (2048, (4096, 16, 128), (16, 128, 128, 768, 512), (16, 128, 128), (32, 2, 1024, 1024)),
+                 "4k": (4096, (8192, 16, 256), (32, 128, 128, 1536, 512), (32, 128, 128), (32, 2, 2048, 2048))}
+ZARINEX_PATTERN = ("mamba1", "latent_attention", "mamba1", "hgrn2", "mamba1", "latent_attention", "hgrn2", "mamba1")
+
+
+def zarinex_config(size: str) -> zx.ZarinexConfig:
+    W, s, a, h, e = ZARINEX_SIZES[size]
+    mix = {"mamba1": {"inner": s[0], "state": s[1], "dt_rank": s[2], "conv": 4},
+           "latent_attention": {"heads": a[0], "dim": a[1], "vdim": a[2], "q_rank": a[3], "kv_rank": a[4], "scale": a[1] ** -0.5},
+           "hgrn2": {"heads": h[0], "dim": h[1], "vdim": h[2]}}
+    mlp = {"kind": "moe", "expert": {"ff": e[2]}, "router": {"experts": e[0], "top": e[1]}, "shared": {"ff": e[3]}}
+    return zx.ZarinexConfig.from_dict({"architecture": zx.ARCH, "vocab": VOCAB, "width": W, "norm": {"eps": 1e-5}, "postln_alpha": 2.0,
+                                       "layers": [{"type": t, "mixer": mix[t], "mlp": mlp} for t in ZARINEX_PATTERN]})
+
+
 def config(size: str, ff: int | None = None) -> gd.GidisunConfig:
     W, dense_ff, m, g, a = SIZES[size]
     ff = ff or dense_ff
@@ -75,7 +93,8 @@ def config(size: str, ff: int | None = None) -> gd.GidisunConfig:
 def build(design: str, size: str, batch: int, context: int, ff: int | None = None):
     """(runtime with random weights, bytes of weights that one decoded token streams)."""
     from ..runtime.mixer_runtime import MixerRuntime
-    mod, c = {"gidisun": lambda: (gd, config(size, ff)), "pezarax": lambda: (pz, pezarax_config(size)), "zemozen": lambda: (zm, zemozen_config(size))}[design]()
+    mod, c = {"gidisun": lambda: (gd, config(size, ff)), "pezarax": lambda: (pz, pezarax_config(size)), "zemozen": lambda: (zm, zemozen_config(size)),
+              "zarinex": lambda: (zx, zarinex_config(size))}[design]()
     t = mod.random_tensors(c, 0, device="cuda")
     pages = batch * (-(-context // 64))
     streamed = 0.0
@@ -84,7 +103,7 @@ def build(design: str, size: str, batch: int, context: int, ff: int | None = Non
         if ".mlp.e" in n:
             L = c.layers[int(n[1:n.index(".")])]
             share = L.top / (L.experts + getattr(L, "identity", 0))
-        streamed += v.numel() * 2 * share if n != "embed" else 0.0
+        streamed += v.numel() * 2 * share if n != "embed" or "head" not in t else 0.0
     rt = MixerRuntime(mod.build_model(c, t, slots=batch, pages=pages), max_requests=batch, pages=pages)
     return rt, streamed
 
@@ -155,6 +174,15 @@ def closest_to_zemozen(size: str, prompts, n: int, d: int, warmup: int, batch: i
     rt, streamed = build("pezarax", size, batch, n + d + 64)
     r, k = requests(rt, prompts, n, d, warmup, batch), len(prompts) - warmup
     return {"model": "Pezarax (retention, differential attention, routed experts; bf16 weights)", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
+            "decode_tok_s": round(k * d / r["decode_ms"] * 1e3, 1), "decode_tok_s_batch": round(k * d * batch / r["batch_ms"] * 1e3, 1),
+            "weight_gb_per_token": round(streamed / 1e9, 2), "decode_weight_gbs": round(streamed * k * d / r["decode_ms"] / 1e6, 1)}
+
+
+def closest_to_zarinex(size: str, prompts, n: int, d: int, warmup: int, batch: int) -> dict:
+    """Zemozen with as many experts of as many weights."""
+    rt, streamed = build("zemozen", size, batch, n + d + 64)
+    r, k = requests(rt, prompts, n, d, warmup, batch), len(prompts) - warmup
+    return {"model": "Zemozen (windowed attention beside a state-space recurrence, routed experts; bf16 weights)", "prefill_tok_s": round(k * n / r["prefill_ms"] * 1e3, 1),
             "decode_tok_s": round(k * d / r["decode_ms"] * 1e3, 1), "decode_tok_s_batch": round(k * d * batch / r["batch_ms"] * 1e3, 1),
             "weight_gb_per_token": round(streamed / 1e9, 2), "decode_weight_gbs": round(streamed * k * d / r["decode_ms"] / 1e6, 1)}
 
@@ -248,6 +276,9 @@ def _state(kind: str, dims, T: int, singles: bool):
     elif kind == "mlstm":
         w.update({"i": r(H, W), "f": r(H, W), "i.b": torch.zeros(H), "f.b": torch.full((H,), 3.0), "norm": torch.ones(H * V)})
         m = ml.MLSTMMixer(w, {"heads": H, "dim": D, "vdim": V, "gate_cap": 12.0}, 1e-5, torch.bfloat16, "cuda", b.slots)
+    elif kind == "hgrn2":
+        w.update({"f": r(H * D, W), "f.b": torch.full((H * D,), 3.0), "lower": torch.full((H * D,), 0.3), "norm": torch.ones(V)})
+        m = ml.HGRN2Mixer(w, {"heads": H, "dim": D, "vdim": V}, 1e-5, torch.bfloat16, "cuda", b.slots)
     else:
         w.update({"a1": r(16, W), "a2": r(H * D, 16), "a2.b": torch.full((H * D,), 2.0), "norm": torch.ones(V)})
         m = ml.GLAMixer(w, {"heads": H, "dim": D, "vdim": V, "tau": 14.0}, 1e-5, torch.bfloat16, "cuda", b.slots)
@@ -612,13 +643,148 @@ def zemozen_kernels() -> None:
                                                                                T * 4096 * 18.0), T=T)
 
 
+def _selective_scan(dims, T: int, singles: bool, dtype=torch.bfloat16) -> dict:
+    """One selective-scan layer between its input and output projections: {kernel: (call, flops, bytes)}. Flops of the recurrence: two
+    products, a decay and two sums per channel and state."""
+    from ..models import mixer_layers as ml
+    from ..ops import mixer_ops as mo
+    inner, N, rank = dims
+    W, es = 64, 2 if dtype == torch.bfloat16 else 4
+    b = _Batch(T, 4096, 64, singles=singles)
+    g = torch.Generator().manual_seed(0)
+    r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
+    w = {"in": r(2 * inner, W), "conv": r(inner, 4), "conv.b": torch.zeros(inner), "x": r(rank + 2 * N, inner), "dt": r(inner, rank), "dt.b": torch.full((inner,), -3.0),
+         "A_log": torch.log(torch.arange(1, N + 1).float()).repeat(inner, 1), "D": torch.ones(inner), "o": r(W, inner)}
+    m = ml.SelectiveScanMixer(w, {"inner": inner, "state": N, "dt_rank": rank, "conv": 4}, 1e-5, dtype, "cuda", b.slots)
+    ctx, ws = b.ctx, b.ctx.ws
+    p = m.proj(ctx, torch.randn(T, W, device="cuda").to(dtype), "proj", torch.float32)
+    mix = ws.rows("mix", T, m.out.K, dtype)
+    m.run(ctx, p, mix)
+    x, dbc = ws.rows("scan_x", T, m.dbc.K, dtype), ws.rows("scan_dbc", T, m.dbc.N, torch.float32)
+    d = mo.SelectiveScan(proj=p.data_ptr(), ld=p.stride(0), xc=x.data_ptr(), ldx=x.stride(0), out=mix.data_ptr(), ldo=mix.stride(0), pos=ctx.pos.data_ptr(),
+                         slot=ctx.slot.data_ptr(), dbc=dbc.data_ptr(), ldb=dbc.stride(0), **m.desc)
+    keep = (m, b, p, mix, x, dbc)
+    flops = 5.0 * T * inner * N
+    out = {"all between the projections": (lambda k=keep: m.run(ctx, p, mix), 0, 0),
+           "convolution": (lambda k=keep: mo.scan_conv(d, T), 0, T * inner * (4.0 + es))}
+    if singles:
+        out["rows form (step sizes, gate included)"] = (lambda k=keep: mo.scan_rows(d, ctx.short, ctx.n_short), 0, T * inner * N * 8.0 + inner * (m.dt.K // 2 * es + N * 4))
+        return out
+    terms, dt = ws.rows("scan_d", T, m.dt.K, dtype), ws.rows("scan_dt", T, m.dt.N, torch.float32)
+    d.dt, d.ldt = dt.data_ptr(), dt.stride(0)
+    if dtype == torch.bfloat16:
+        out["step sizes (split and product)"] = (lambda k=(keep, terms): (mo.scan_split(dbc, m.rank, terms), m.dt(ctx, terms, "scan_dt", torch.float32)),
+                                                 2.0 * T * inner * m.dt.K, T * inner * 4.0)
+    out["recurrence (gate included)"] = (lambda k=(keep, dt): mo.scan_tiles(d, ctx.long, ctx.n_long), flops, T * inner * (8.0 + 2 * es))
+    return out
+
+
+def _gated_latent(dims, T: int, start: int, singles: bool):
+    """Latent attention with queries from a latent and gated outputs, as `_latent`."""
+    from ..models import mixer_layers as ml
+    from ..ops import mixer_ops as mo
+    H, D, V, Q, K = dims
+    W = 64
+    b = _Batch(T, start, start + T, singles=singles)
+    g = torch.Generator().manual_seed(0)
+    r = lambda *s: torch.randn(*s, generator=g) * s[-1] ** -0.5
+    m = ml.LatentAttentionMixer({"dq": r(Q, W), "dq.norm": torch.ones(Q), "uq": r(H * D, Q), "dkv": r(K, W), "dkv.norm": torch.ones(K), "uk": r(H * D, K),
+                                 "uv": r(H * V, K), "g": r(H * V, W), "o": r(W, H * V)},
+                                {"heads": H, "dim": D, "vdim": V, "kv_rank": K, "scale": D ** -0.5}, 1e-5, torch.bfloat16, "cuda", b.pages, start + T)
+    m.cache.normal_()
+    ctx, ws = b.ctx, b.ctx.ws
+    p = m.proj(ctx, torch.randn(T, m.proj.K, device="cuda").to(torch.bfloat16), "proj", torch.float32)
+    at, qw = m.proj.at, m.qk_panels * 64
+    gate, ql, mix = p[:, at["g"]:], ws.rows("lat_q", T, m.uq.K, torch.bfloat16), ws.rows("mix", T, m.out.K, torch.bfloat16)
+    span = sum(start + i + 1 for i in range(T)) if not singles else T * (start + 1)
+    prep = lambda k=(m, b, p): mo.latent_prep(p, at["dq"], at["dkv"], H, D, 0, K, m.c_norm, 1e-5, m.freq, 1.0, ctx.pos, ctx.slot, m.cache, ctx.table, None, None, 0,
+                                              q_rank=Q, q_norm=m.q_norm, ql=ql)
+    prep_bytes = T * ((Q + K) * 4.0 + (m.row + m.uq.K) * 2)
+    if singles:
+        q, qx = m.uq(ctx, ql, "q_rows", torch.float32), ws.flat("qx", T * H * m.row, torch.float32)
+        po, pm = ws.flat("po", T * m.nsplit * H * K, torch.float32), ws.flat("pm", T * m.nsplit * H * 2, torch.float32)
+        return {"prep": (prep, 0, prep_bytes),
+                "absorb": (lambda: mo.latent_absorb(q, 0, H, D, qw - D, K, m.uk, ctx.rows, T, qx, m.row, m.row), 2.0 * T * H * D * K, H * D * K * 2.0),
+                "rows": (lambda: mo.latent_rows(qx, ctx.rows, T, ctx.pos, ctx.slot, m.cache, ctx.table, H, K, 0, m.scale, m.nsplit, po, pm),
+                         2.0 * span * H * (m.row + K), span * m.row * 2.0),
+                "merge + values + gate": (lambda: mo.latent_out(po, pm, m.nsplit, H, K, V, None, ctx.rows, T, m.uv, mix, gate), 2.0 * T * H * V * K, H * V * K * 2.0)}
+    qf = m.uq(ctx, ql, "qf", torch.bfloat16)
+    gather, total, longest = ctx.gather[0]
+    c, kv = ws.rows("c", total, m.row, torch.bfloat16), ws.rows("kv", total, m.kv_w.shape[0], torch.bfloat16)
+    return {"prep": (prep, 0, prep_bytes),
+            "gather": (lambda: mo.latent_gather(m.cache, ctx.table, ctx.long, gather, 1, longest, c), 0, total * m.row * 4.0),
+            "expand": (lambda: mo.linear(c, m.kv_w, kv, ctx.status), 2.0 * total * m.row * kv.shape[1], 0),
+            "attention": (lambda: mo.latent_prefill(qf, T, kv, total, ctx.tiles, ctx.n_tiles, ctx.long, gather, H, m.qk_panels, m.v_panels, V, 0, m.scale, None, mix,
+                                                    ctx.status, gate), 2.0 * span * H * (D + V), 0)}
+
+
+def zarinex_kernels() -> None:
+    """The new kernels and variants, each followed by the like kernel of Zemozen or Gidisun in the same run."""
+    from ..ops import mixer_ops as mo
+    show = lambda name, d, **kw: print(json.dumps({"kernel": name, **kw, **d}), flush=True)
+    dims, space = (8192, 16, 256), (64, 64, 128, 8)
+    for T in (512, 2048):
+        for k, (f, fl, nb) in _selective_scan(dims, T, False).items():
+            show("selective scan: " + k, _roof(timed(f), fl, nb), T=T, dims=dims)
+        for k, (f, fl, nb) in _selective_scan(dims, T, False, torch.float32).items():
+            show("selective scan, fp32: " + k, _roof(timed(f), fl, nb), T=T, dims=dims)
+        f, fl, _ = _state_space(space, T, False)
+        show("like kernel: state space prefill, tensor cores", _roof(timed(f), fl), T=T, dims=space)
+    for B in (1, 8):
+        for k, (f, fl, nb) in _selective_scan(dims, B, True).items():
+            show("selective scan: " + k, _roof(timed(f), fl, nb), B=B, dims=dims)
+        f, _, nb = _state_space(space, B, True)
+        show("like kernel: state space rows form", _roof(timed(f), 0, nb), B=B, dims=space)
+    head = (32, 128, 128)
+    for T in (512, 2048):
+        for kind in ("hgrn2", "gla"):
+            f, fl, _ = _state(kind, head, T, False)
+            show(("like kernel: " if kind == "gla" else "") + f"{kind} chunk form + head norm", _roof(timed(f), fl), T=T, dims=head)
+    for B in (1, 8):
+        for kind in ("hgrn2", "gla"):
+            f, _, nb = _state(kind, head, B, True)
+            show(("like kernel: " if kind == "gla" else "") + f"{kind} rows form + head norm", _roof(timed(f), 0, nb), B=B, dims=head)
+    for T in (512, 2048):
+        for k, (f, fl, nb) in _gated_latent((32, 128, 128, 1536, 512), T, 8192 - T, False).items():
+            show("gated latent prefill: " + k, _roof(timed(f), fl, nb), T=T, context=8192)
+        for k, (f, fl, nb) in _latent((32, 128, 64, 128, 512, 0), T, 8192 - T, False).items():
+            show("like kernel: latent prefill: " + k, _roof(timed(f), fl, nb), T=T, context=8192)
+    for B in (1, 8):
+        for k, (f, fl, nb) in _gated_latent((32, 128, 128, 1536, 512), B, 1500, True).items():
+            show("gated latent rows: " + k, _roof(timed(f), fl, nb), B=B)
+        for k, (f, fl, nb) in _latent((32, 128, 64, 128, 512, 0), B, 1500, True).items():
+            show("like kernel: latent rows: " + k, _roof(timed(f), fl, nb), B=B)
+    W = 4096
+    for T in (1, 8, 512, 2048):
+        x, y, w = torch.randn(T, W, device="cuda"), torch.randn(2 * T, W, device="cuda"), torch.randn(W, device="cuda")
+        xo, gate, y2, before = torch.empty_like(x), torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda"), torch.randn(T, W, device="cuda")
+        o, o2 = (torch.empty(T, W, device="cuda", dtype=torch.bfloat16) for _ in range(2))
+        place = torch.randperm(2 * T, device="cuda").to(torch.int32).view(T, 2)
+        b = _Batch(T, 64, 64, singles=T <= mo.ROWS_MAX).ctx
+        base = dict(x=x, x_out=xo, gate=gate, ldg=W, gate_b=w, w=w, y=y, ldy=W, pos=b.pos, slot=b.slot, behind=b.behind, M=T, width=W, ldo=W, alpha=2.0, eps=1e-5, out=o)
+        other = dict(shift=w, before=before, out_shift=o2)
+        call = lambda **kw: mo.post_norm(mo.PostNorm(**{k: v.data_ptr() if isinstance(v, torch.Tensor) else v for k, v in (base | kw).items()}))
+        show("gate + sum + norm, input kept", _roof(timed(lambda: call(save=before)), 0, T * W * 18.0), T=T)
+        show("expert rows + shared expert + gate + sum + norm + token shift", _roof(timed(lambda: call(y_rows=place, y_top=2, y2=y2, ldy2=W, **other)),
+                                                                                   0, T * W * 28.0), T=T)
+        show("like kernel: residual add + norm", _roof(timed(lambda: mo.sandwich_norm(x, y=y, w_pre=w, out=o, eps=1e-5)), 0, T * W * 14.0), T=T)
+        show("like kernel: sum of two expert rows + residual add + norm", _roof(timed(lambda: mo.sandwich_norm(x, y=y, y_rows=place, w_pre=w, out=o, eps=1e-5)), 0, T * W * 18.0), T=T)
+    for M in (1, 8):
+        for N, split in ((20480, 4096), (12288, 4096)):
+            ws = [torch.randn(N, W, device="cuda").to(torch.bfloat16) for _ in range(3)]
+            x, x2 = (torch.randn(M, W, device="cuda").to(torch.bfloat16) for _ in range(2))
+            y, s = torch.empty(M, N, device="cuda"), torch.zeros(1, dtype=torch.int32, device="cuda")
+            show("few-row linear with two inputs", _roof(timed(lambda: [mo.linear2(x, x2, split, w, y, s) for w in ws], reps=8) / 3, 0, N * W * 2.0), M=M, N=N)
+            show("like kernel: few-row linear", _roof(timed(lambda: [mo.linear(x, w, y, s) for w in ws], reps=8) / 3, 0, N * W * 2.0), M=M, N=N)
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernels", nargs="?", const="gidisun", choices=["gidisun", "pezarax", "zemozen"], help="time the design's kernels beside the like kernels")
+    ap.add_argument("--kernels", nargs="?", const="gidisun", choices=["gidisun", "pezarax", "zemozen", "zarinex"], help="time the design's kernels beside the like kernels")
     ap.add_argument("--size", default="2k", choices=sorted(SIZES))
     args = ap.parse_args()
     if args.kernels:
-        {"gidisun": kernels, "pezarax": pezarax_kernels, "zemozen": zemozen_kernels}[args.kernels]()
+        {"gidisun": kernels, "pezarax": pezarax_kernels, "zemozen": zemozen_kernels, "zarinex": zarinex_kernels}[args.kernels]()
     else:
         print(json.dumps(closest_model(args.size, 512, 64, 3)))
     return 0
