@@ -43,31 +43,33 @@ namespace {
 
 using namespace pk;
 
-template <typename OutT, int PT, int VW, int THREADS>
-__global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, int per_block) {
+// PT groups of VW values per thread. One group (few rows): the weights, which no kernel writes, are fetched before the wait. Several
+// groups (many rows): they are read where they are used, which leaves registers for more blocks.
+template <typename OutT, int PT, int VW, int THREADS, bool SHIFT>
+__global__ void __launch_bounds__(THREADS, PT == 2 ? 2 : 1) post_norm_kernel(const PkPostNorm p, int per_block) {
+  constexpr bool EARLY = PT == 1;
   pdl_trigger();
   __shared__ float scratch[33];
   const int tid = threadIdx.x, nt = blockDim.x;
-  // weights are not written by any kernel: fetched before the wait
-  float wn[PT][VW], gb[PT][VW], sh[PT][VW], prev[PT][VW];
+  float wn[VW], gb[VW], sh[VW], prev[SHIFT ? PT : 1][VW];
 #pragma unroll
-  for (int i = 0; i < PT; ++i) {
-    const int c = (tid + i * nt) * VW;
-#pragma unroll
-    for (int j = 0; j < VW; ++j) wn[i][j] = gb[i][j] = sh[i][j] = prev[i][j] = 0.f;
-    if (c < p.width) {
-      if (p.w) load_f32<VW>(p.w + c, wn[i]);
-      if (p.gate) load_f32<VW>(p.gate_b + c, gb[i]);
-      if (p.shift) load_f32<VW>(p.shift + c, sh[i]);
-    }
+  for (int j = 0; j < VW; ++j) wn[j] = gb[j] = sh[j] = 0.f;
+  if (EARLY && tid * VW < p.width) {
+    if (p.w) load_f32<VW>(p.w + tid * VW, wn);
+    if (p.gate) load_f32<VW>(p.gate_b + tid * VW, gb);
+    if (SHIFT) load_f32<VW>(p.shift + tid * VW, sh);
   }
   pdl_wait();
   const int r0 = blockIdx.x * per_block, r1 = min(r0 + per_block, p.M);
-  const bool again = p.shift && r0 > 0 && p.behind[r0 - 1] > 0;      // the row before is of the same portion
+  const bool again = SHIFT && r0 > 0 && p.behind[r0 - 1] > 0;      // the row before is of the same portion
   for (int r = r0 - (again ? 1 : 0); r < r1; ++r) {
     const bool own = r >= r0;
     const int row = p.rows ? p.rows[r] : r;
     float v[PT][VW];
+#pragma unroll
+    for (int i = 0; i < PT; ++i)
+#pragma unroll
+      for (int j = 0; j < VW; ++j) v[i][j] = 0.f;
     if (p.x == nullptr) {
       int t = p.tokens[row];
       t = t < 0 ? 0 : (t >= p.vocab ? p.vocab - 1 : t);
@@ -75,8 +77,6 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, 
 #pragma unroll
       for (int i = 0; i < PT; ++i) {
         const int c = (tid + i * nt) * VW;
-#pragma unroll
-        for (int j = 0; j < VW; ++j) v[i][j] = 0.f;
         if (c >= p.width) continue;
         load_any<VW>(p.embed, (size_t)t * p.width + c, false, v[i]);
         if (p.freq) {
@@ -96,50 +96,65 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, 
         }
       }
     } else {
-      const float* xr = p.x + (size_t)row * p.width;
+      const size_t at = (size_t)row * p.width;
       const bool keep = own && p.save && p.behind[row] == 0;
-      float* kept = keep ? p.save + (size_t)p.slot[row] * p.width : nullptr;
+      // all loads of a row are in flight together
+      float u[PT][VW], g[PT][VW];
+#pragma unroll
+      for (int i = 0; i < PT; ++i) {
+        const int c = (tid + i * nt) * VW;
+#pragma unroll
+        for (int j = 0; j < VW; ++j) u[i][j] = g[i][j] = 0.f;
+        if (c >= p.width) continue;
+        load_f32<VW>(p.x + at + c, v[i]);
+        if (p.gate) load_f32<VW>(p.gate + (size_t)row * p.ldg + c, g[i]);
+        if (!p.y_rows) load_f32<VW>(p.y + (size_t)row * p.ldy + c, u[i]);
+      }
+      auto add_row = [&](const float* y) {
+        float a[PT][VW];
+#pragma unroll
+        for (int i = 0; i < PT; ++i) {
+#pragma unroll
+          for (int j = 0; j < VW; ++j) a[i][j] = 0.f;
+          if ((tid + i * nt) * VW < p.width) load_f32<VW>(y + (tid + i * nt) * VW, a[i]);
+        }
+#pragma unroll
+        for (int i = 0; i < PT; ++i)
+#pragma unroll
+          for (int j = 0; j < VW; ++j) u[i][j] += a[i][j];
+      };
+      if (p.y_rows) {
+        const int* from = p.y_rows + (size_t)row * p.y_top;
+        for (int k = 0; k < p.y_top; k += 2) {
+          const int f0 = from[k], f1 = k + 1 < p.y_top ? from[k + 1] : -1;
+          if (f0 >= 0) add_row(p.y + (size_t)f0 * p.ldy);
+          if (f1 >= 0) add_row(p.y + (size_t)f1 * p.ldy);
+        }
+      }
+      if (p.y2) add_row(p.y2 + (size_t)row * p.ldy2);
       float ss = 0.f;
 #pragma unroll
       for (int i = 0; i < PT; ++i) {
         const int c = (tid + i * nt) * VW;
-        float u[VW], g[VW];
-#pragma unroll
-        for (int j = 0; j < VW; ++j) v[i][j] = u[j] = g[j] = 0.f;
         if (c >= p.width) continue;
-        load_f32<VW>(xr + c, v[i]);
-        if (p.gate) load_f32<VW>(p.gate + (size_t)row * p.ldg + c, g);
-        if (p.y_rows) {
-          for (int k = 0; k < p.y_top; ++k) {
-            float a[VW];
-            const int from = p.y_rows[(size_t)row * p.y_top + k];
-            if (from < 0) continue;
-            load_f32<VW>(p.y + (size_t)from * p.ldy + c, a);
-#pragma unroll
-            for (int j = 0; j < VW; ++j) u[j] += a[j];
-          }
-        } else {
-          load_f32<VW>(p.y + (size_t)row * p.ldy + c, u);
-        }
-        if (p.y2) {
-          float a[VW];
-          load_f32<VW>(p.y2 + (size_t)row * p.ldy2 + c, a);
-#pragma unroll
-          for (int j = 0; j < VW; ++j) u[j] += a[j];
-        }
-        if (keep) store<VW>(kept + c, v[i]);
+        if (keep) store<VW>(p.save + (size_t)p.slot[row] * p.width + c, v[i]);
+        if (!EARLY && p.gate) load_f32<VW>(p.gate_b + c, gb);
 #pragma unroll
         for (int j = 0; j < VW; ++j) {
-          const float f = p.gate ? 1.f / (1.f + expf(-(g[j] + gb[i][j]))) : 1.f;
-          v[i][j] = fmaf(p.alpha, v[i][j], f * u[j]);
+          const float f = p.gate ? 1.f / (1.f + expf(-(g[i][j] + gb[j]))) : 1.f;
+          v[i][j] = fmaf(p.alpha, v[i][j], f * u[i][j]);
           ss = fmaf(v[i][j], v[i][j], ss);
         }
       }
       const float rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
 #pragma unroll
-      for (int i = 0; i < PT; ++i)
+      for (int i = 0; i < PT; ++i) {
+        const int c = (tid + i * nt) * VW;
+        if (c >= p.width) continue;
+        if (!EARLY) load_f32<VW>(p.w + c, wn);
 #pragma unroll
-        for (int j = 0; j < VW; ++j) v[i][j] = v[i][j] * rr * wn[i][j];
+        for (int j = 0; j < VW; ++j) v[i][j] = v[i][j] * rr * wn[j];
+      }
     }
     if (own) {
       float rr = 1.f;
@@ -152,7 +167,7 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, 
         rr = 1.f / sqrtf(block_sum(ss, scratch) / (float)p.width + p.eps);
       }
       const float* from = nullptr;      // x of the token before, when it is not carried
-      const bool first = p.shift && (r == 0 || p.behind[r - 1] == 0);
+      const bool first = SHIFT && (r == 0 || p.behind[r - 1] == 0);
       if (first && p.pos[row] > 0) from = p.before + (size_t)p.slot[row] * p.width;
 #pragma unroll
       for (int i = 0; i < PT; ++i) {
@@ -166,24 +181,25 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, 
           for (int j = 0; j < VW; ++j) o[j] = p.w_out ? v[i][j] * rr * o[j] : v[i][j];
           store<VW>(reinterpret_cast<OutT*>(p.out) + (size_t)r * p.ldo + c, o);
         }
-        if (p.shift) {
+        if (SHIFT) {
           float o[VW];
+          if (!EARLY) load_f32<VW>(p.shift + c, sh);
           if (first) {
 #pragma unroll
             for (int j = 0; j < VW; ++j) prev[i][j] = 0.f;
             if (from) load_f32<VW>(from + c, prev[i]);
           }
 #pragma unroll
-          for (int j = 0; j < VW; ++j) o[j] = fmaf(prev[i][j] - v[i][j], sh[i][j], v[i][j]);
+          for (int j = 0; j < VW; ++j) o[j] = fmaf(prev[i][j] - v[i][j], sh[j], v[i][j]);
           store<VW>(reinterpret_cast<OutT*>(p.out_shift) + (size_t)r * p.ldo + c, o);
         }
       }
       for (int c = p.width + tid; c < p.ldo; c += nt) {
         if (p.out) reinterpret_cast<OutT*>(p.out)[(size_t)r * p.ldo + c] = (OutT)0.f;
-        if (p.shift) reinterpret_cast<OutT*>(p.out_shift)[(size_t)r * p.ldo + c] = (OutT)0.f;
+        if (SHIFT) reinterpret_cast<OutT*>(p.out_shift)[(size_t)r * p.ldo + c] = (OutT)0.f;
       }
     }
-    if (p.shift) {
+    if (SHIFT) {
 #pragma unroll
       for (int i = 0; i < PT; ++i)
 #pragma unroll
@@ -192,30 +208,35 @@ __global__ void __launch_bounds__(THREADS) post_norm_kernel(const PkPostNorm p, 
   }
 }
 
-template <typename OutT, int VW>
+template <typename OutT, int VW, bool SHIFT>
 int launch_norm(const PkPostNorm& p, cudaStream_t stream) {
   const int groups = (p.width + VW - 1) / VW;
-  // few rows: as many threads as help their latency; many rows: smaller blocks with a few groups per thread, and a few rows per
-  // block so that fewer rows are computed twice
-  const int cap = p.M <= 64 && groups <= 2048 ? 1024 : 512;
-  const int nt = groups >= cap ? cap : ((groups + 31) / 32) * 32;
+  // few rows: as many threads as help their latency; many rows: two groups per thread, and a few rows per block so that fewer rows are
+  // computed twice
+  const int want = groups > 1024 ? 512 : p.M <= 64 ? groups : (groups + 1) / 2;
+  const int nt = (want + 31) / 32 * 32;
   const int per = (groups + nt - 1) / nt;
-  int rows = p.shift && !p.rows ? p.M / 592 : 1;
+  int rows = SHIFT ? p.M / 592 : 1;
   rows = rows < 1 ? 1 : rows > 4 ? 4 : rows;
   const dim3 grid((p.M + rows - 1) / rows);
-#define PK_NORM_CASE(n, threads)                                                                                     \
-  if (per <= n && nt <= threads) {                                                                                   \
-    PK_LAUNCH_PDL((post_norm_kernel<OutT, n, VW, threads>), grid, dim3(nt), (size_t)0, stream, p, rows);             \
-    return PK_OK;                                                                                                    \
+#define PK_NORM_CASE(n, threads)                                                                                            \
+  if (per <= n && nt <= threads) {                                                                                          \
+    PK_LAUNCH_PDL((post_norm_kernel<OutT, n, VW, threads, SHIFT>), grid, dim3(nt), (size_t)0, stream, p, rows);             \
+    return PK_OK;                                                                                                           \
   }
+  PK_NORM_CASE(1, 256)
   PK_NORM_CASE(1, 1024)
   PK_NORM_CASE(2, 512)
-  PK_NORM_CASE(2, 1024)
   PK_NORM_CASE(4, 512)
   PK_NORM_CASE(8, 512)
   PK_NORM_CASE(16, 512)
 #undef PK_NORM_CASE
   return PK_ERR_UNSUPPORTED;
+}
+
+template <typename OutT, int VW>
+int launch_norm(const PkPostNorm& p, cudaStream_t stream) {
+  return p.shift ? launch_norm<OutT, VW, true>(p, stream) : launch_norm<OutT, VW, false>(p, stream);
 }
 
 bool aligned(const void* p, int ld = 0) { return ((uintptr_t)p & 15) == 0 && (ld & 3) == 0; }

@@ -9,8 +9,8 @@
 //   split  d as the sum of two bf16 terms side by side, so that W_dt d of many rows on the tensor cores keeps 16 bits of d
 //   rows   portions of a few tokens: LN lanes per channel with NP states each, W_dt d in the same kernel (fp32 sums); a block takes a
 //          few portions, which share its rows of W_dt
-//   tiles  long portions: the same lanes walk the tokens in tiles of 16 (8), two states per instruction. Between two barriers a block
-//          requests tile i + 3 (cp.async), makes dt and dt x of tile i + 1, runs the recurrence over tile i, and gates and stores the
+//   tiles  long portions: the same lanes walk the tokens in tiles of 8 to 32, two states per instruction. Between two barriers a block
+//          requests tile i + 2 (cp.async), makes dt and dt x of tile i + 1, runs the recurrence over tile i, and gates and stores the
 //          outputs of tile i - 1: independent work that fills the waits of the recurrence. The sums over a channel's lanes are taken for
 //          LN tokens at a time (every exchange halves the number of partial sums)
 // Everything but x and W_dt is fp32. A decay close to 1 that is rounded to fp32 is off by the same few 2^-25 at every step of a long
@@ -211,11 +211,18 @@ __device__ __forceinline__ void store_states(float* row, int n0, int N, const fl
   }
 }
 
+template <int BYTES>
+__device__ __forceinline__ void async_copy(void* dst, const void* src, int bytes) {      // the rest of BYTES is zero
+  const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
+  if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
+}
+
 // Block: THREADS / LN channels of up to SQ short portions.
 template <typename T, int NP, int LN, int SQ>
-__global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveScan p, const int4* seqs, int nseq) {
-  constexpr int CB = THREADS / LN, NS = LN * NP, VE = 16 / sizeof(T), AHEAD = SQ == 1 ? 4 : 8;
-  extern __shared__ float sm[];
+__global__ void __launch_bounds__(THREADS, 4) scan_rows_kernel(const PkSelectiveScan p, const int4* seqs, int nseq) {
+  constexpr int CB = THREADS / LN, NS = LN * NP, VE = 16 / sizeof(T), AHEAD = 4;
+  extern __shared__ __align__(16) float sm[];
   const int tid = threadIdx.x, l = tid % LN, c = blockIdx.x * CB + tid / LN, n0 = l * NP;
   const bool live = c < p.inner;
   const int kw = (p.rank + 7) & ~7, unit = kw + 2 * NS;      // per portion: d [kw], B, C [NS]
@@ -246,28 +253,35 @@ __global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveSca
     for (int k = 0; k < NP; ++k) s[q][k] = 0.f;
     if (live && sq[q].w > 0) load_states<NP>(p.S + ((size_t)sq[q].z * p.inner + c) * p.N, n0, p.N, s[q]);
   }
+  const int dq = kw / 4, nq = dq + 2 * NS / 4;              // 16-byte pieces of a portion's d, and of d, B and C
   for (int t = 0; t < most; ++t) {
+    // all of the tokens' loads are in flight together
+    for (int e = tid; e < SQ * nq; e += THREADS) {
+      int q = 0;
+#pragma unroll
+      for (int j = 1; j < SQ; ++j) q += e >= j * nq;
+      int4 own = sq[0];
+#pragma unroll
+      for (int j = 1; j < SQ; ++j)
+        if (q == j) own = sq[j];
+      const int i = e - q * nq, part = i < dq ? 0 : i < dq + NS / 4 ? 1 : 2;
+      const int k = (i - (part == 0 ? 0 : part == 1 ? dq : dq + NS / 4)) * 4, len = part == 0 ? p.rank : p.N;
+      const bool in = t < own.y && k < len;
+      const float* src = p.dbc + ((size_t)own.x + (in ? t : 0)) * p.ldb + (part == 0 ? 0 : part == 1 ? p.oB : p.oC) + (in ? k : 0);
+      async_copy<16>(sm + q * unit + i * 4, src, in ? min(16, (len - k) * 4) : 0);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
     float x[SQ], z[SQ], in[SQ];
 #pragma unroll
     for (int q = 0; q < SQ; ++q) {
-      const bool on = t < sq[q].y;
-      const size_t row = (size_t)sq[q].x + t;
-      const float* src = p.dbc + row * p.ldb;
-      float* d = sm + q * unit;
-      if (on) {
-        for (int i = tid; i < kw; i += THREADS) d[i] = i < p.rank ? src[i] : 0.f;
-        for (int i = tid; i < NS; i += THREADS) {
-          d[kw + i] = i < p.N ? src[p.oB + i] : 0.f;
-          d[kw + NS + i] = i < p.N ? src[p.oC + i] : 0.f;
-        }
-      }
-      x[q] = on && live ? to_f<T>(((const T*)p.xc)[row * p.ldx + c]) : 0.f;
-      z[q] = in[q] = 0.f;
-      if (on && live && l == 0) {
-        z[q] = p.proj[row * p.ld + p.oz + c];
-        if (sq[q].y - 1 - t < p.taps - 1) in[q] = p.proj[row * p.ld + p.ox + c];
-      }
+      const bool on = t < sq[q].y && live;
+      const size_t row = (size_t)sq[q].x + (on ? t : 0);
+      const int col = live ? c : 0;
+      x[q] = to_f<T>(((const T*)p.xc)[row * p.ldx + col]);
+      z[q] = p.proj[row * p.ld + p.oz + col];
+      in[q] = p.proj[row * p.ld + p.ox + col];
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     float dot[SQ];
 #pragma unroll
@@ -275,35 +289,47 @@ __global__ void __launch_bounds__(THREADS) scan_rows_kernel(const PkSelectiveSca
     auto add = [&](const uint4& u, int k) {
       const T* e = reinterpret_cast<const T*>(&u);
 #pragma unroll
-      for (int q = 0; q < SQ; ++q)
+      for (int i = 0; i < VE; i += 4)
 #pragma unroll
-        for (int i = 0; i < VE; ++i) dot[q] = fmaf(to_f<T>(e[i]), sm[q * unit + k + i], dot[q]);
+        for (int q = 0; q < SQ; ++q) {
+          const float4 d = *reinterpret_cast<const float4*>(sm + q * unit + k + i);
+          dot[q] = fmaf(to_f<T>(e[i]), d.x, fmaf(to_f<T>(e[i + 1]), d.y, dot[q]));
+          dot[q] = fmaf(to_f<T>(e[i + 2]), d.z, fmaf(to_f<T>(e[i + 3]), d.w, dot[q]));
+        }
     };
     if (live) {
 #pragma unroll
       for (int i = 0; i < AHEAD; ++i)
         if ((l + i * LN) * VE < kw) add(first[i], (l + i * LN) * VE);
+#pragma unroll 2
       for (int k = (l + AHEAD * LN) * VE; k < kw; k += LN * VE) add(*reinterpret_cast<const uint4*>(wrow + k), k);
     }
 #pragma unroll
-    for (int q = 0; q < SQ; ++q) {
+    for (int o = LN / 2; o > 0; o >>= 1)
 #pragma unroll
-      for (int o = LN / 2; o > 0; o >>= 1) dot[q] += __shfl_xor_sync(0xffffffffu, dot[q], o);
-      if (t >= sq[q].y) continue;
-      const float* B = sm + q * unit + kw;
-      const float dt = softplus_series(dot[q] + bias), u = dt * x[q];
-      float y = 0.f;
+      for (int q = 0; q < SQ; ++q) dot[q] += __shfl_xor_sync(0xffffffffu, dot[q], o);
+    float y[SQ];
+#pragma unroll
+    for (int q = 0; q < SQ; ++q) {      // a portion that has ended: dt 0 changes nothing
+      const float* B = sm + q * unit + kw + n0;
+      const float dt = t < sq[q].y ? softplus_series(dot[q] + bias) : 0.f, u = dt * x[q];
+      y[q] = 0.f;
 #pragma unroll
       for (int k = 0; k < NP; ++k) {
-        s[q][k] = fmaf(u, B[n0 + k], decayed<T>(dt, a[k], s[q][k]));
-        y = fmaf(s[q][k], B[NS + n0 + k], y);
+        s[q][k] = fmaf(u, B[k], decayed<T>(dt, a[k], s[q][k]));
+        y[q] = fmaf(s[q][k], B[NS + k], y[q]);
       }
+    }
 #pragma unroll
-      for (int o = LN / 2; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-      const size_t row = (size_t)sq[q].x + t;
-      T* out = (T*)p.out + row * p.ldo;
+    for (int o = LN / 2; o > 0; o >>= 1)
+#pragma unroll
+      for (int q = 0; q < SQ; ++q) y[q] += __shfl_xor_sync(0xffffffffu, y[q], o);
+#pragma unroll
+    for (int q = 0; q < SQ; ++q) {
+      if (t >= sq[q].y) continue;
+      T* out = (T*)p.out + ((size_t)sq[q].x + t) * p.ldo;
       if (live && l == 0) {
-        out[c] = (T)(fmaf(skip, x[q], y) * silu_of<T>(z[q]));
+        out[c] = (T)(fmaf(skip, x[q], y[q]) * silu_of<T>(z[q]));
         if (sq[q].y - 1 - t < p.taps - 1) ring_at(p, sq[q].z, sq[q].w + t)[c] = in[q];
       }
       if (blockIdx.x == gridDim.x - 1)
@@ -331,13 +357,6 @@ __device__ __forceinline__ float group_sums(float (&v)[G], int l) {
   return v[0];
 }
 
-template <int BYTES>
-__device__ __forceinline__ void async_copy(void* dst, const void* src, int bytes) {      // the rest of BYTES is zero
-  const uint32_t a = (uint32_t)__cvta_generic_to_shared(dst);
-  if (BYTES == 16) asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(a), "l"(src), "r"(bytes) : "memory");
-}
-
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack2(float x, float y) {
   f32x2 r;
@@ -356,24 +375,33 @@ __device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
   return r;
 }
 
-// One step of NP states of a channel; what their lane adds to y.
+// What a lane needs of a token: dt, dt x, and B and C of its states.
+template <int NP>
+struct Token {
+  float2 du;
+  f32x2 B[NP / 2], C[NP / 2];
+  __device__ __forceinline__ void load(const float2* d, const float* b, const float* c) {
+    du = *d;
+    if (NP == 2) {
+      B[0] = *reinterpret_cast<const f32x2*>(b);
+      C[0] = *reinterpret_cast<const f32x2*>(c);
+      return;
+    }
+#pragma unroll
+    for (int k = 0; k < NP / 4; ++k) {
+      const ulonglong2 x = reinterpret_cast<const ulonglong2*>(b)[k], y = reinterpret_cast<const ulonglong2*>(c)[k];
+      B[2 * k] = x.x;
+      B[2 * k + 1] = x.y;
+      C[2 * k] = y.x;
+      C[2 * k + 1] = y.y;
+    }
+  }
+};
+
+// NP states of a channel over SUB tokens; y: what their lane adds to the outputs. Decays and inputs of all tokens come first, the
+// serial part is one product per token.
 template <typename T, int NP>
 struct States {
-  float a[NP], s[NP];
-  __device__ __forceinline__ void start() {}
-  __device__ __forceinline__ float step(float dt, float u, const float* B, const float* C) {
-    float y = 0.f;
-#pragma unroll
-    for (int k = 0; k < NP; ++k) {
-      s[k] = fmaf(u, B[k], decayed<T>(dt, a[k], s[k]));
-      y = fmaf(s[k], C[k], y);
-    }
-    return y;
-  }
-  __device__ __forceinline__ void finish() {}
-};
-template <int NP>
-struct States<bf16, NP> {
   float a[NP], s[NP];
   f32x2 a2[NP / 2], s2[NP / 2];
   __device__ __forceinline__ void start() {
@@ -383,23 +411,30 @@ struct States<bf16, NP> {
       s2[k] = pack2(s[2 * k], s[2 * k + 1]);
     }
   }
-  __device__ __forceinline__ float step(float dt, float u, const float* B, const float* C) {
-    const f32x2 dt2 = pack2(dt, dt), u2 = pack2(u, u);
-    f32x2 y = 0;
+  template <int SUB>
+  __device__ __forceinline__ void run(const Token<NP> (&t)[SUB], float* y) {
+    f32x2 e[SUB][NP / 2], in[SUB][NP / 2];
 #pragma unroll
-    for (int k = 0; k < NP / 4; ++k) {
-      const ulonglong2 b = reinterpret_cast<const ulonglong2*>(B)[k], c = reinterpret_cast<const ulonglong2*>(C)[k];
+    for (int i = 0; i < SUB; ++i)
 #pragma unroll
-      for (int j = 0; j < 2; ++j) {
+      for (int k = 0; k < NP / 2; ++k) {
         float x0, x1;
-        unpack2(mul2(dt2, a2[2 * k + j]), x0, x1);
-        s2[2 * k + j] = fma2(pack2(ex2(x0), ex2(x1)), s2[2 * k + j], mul2(u2, j ? b.y : b.x));
-        y = fma2(s2[2 * k + j], j ? c.y : c.x, y);
+        unpack2(mul2(pack2(t[i].du.x, t[i].du.x), a2[k]), x0, x1);
+        e[i][k] = sizeof(T) == 4 ? pack2(expm1f(x0), expm1f(x1)) : pack2(ex2(x0), ex2(x1));
+        in[i][k] = mul2(pack2(t[i].du.y, t[i].du.y), t[i].B[k]);
       }
+#pragma unroll
+    for (int i = 0; i < SUB; ++i) {
+      f32x2 sum = 0;
+#pragma unroll
+      for (int k = 0; k < NP / 2; ++k) {
+        s2[k] = sizeof(T) == 4 ? fma2(pack2(1.f, 1.f), fma2(e[i][k], s2[k], s2[k]), in[i][k]) : fma2(e[i][k], s2[k], in[i][k]);
+        sum = fma2(s2[k], t[i].C[k], sum);
+      }
+      float y0, y1;
+      unpack2(sum, y0, y1);
+      y[i] = y0 + y1;
     }
-    float y0, y1;
-    unpack2(y, y0, y1);
-    return y0 + y1;
   }
   __device__ __forceinline__ void finish() {
 #pragma unroll
@@ -410,7 +445,7 @@ struct States<bf16, NP> {
 // Shared memory of a tiles block: STAGES raw tiles, then two tiles of (dt, dt x) and of sums.
 template <typename T, int NP, int LN>
 struct TileShape {
-  static constexpr int CB = THREADS / LN, NS = LN * NP, TT = NS > 128 ? 8 : 16, STAGES = 5;
+  static constexpr int CB = THREADS / LN, NS = LN * NP, TT = NS > 128 ? 8 : LN >= 8 && NS <= 32 ? 32 : 16, STAGES = 4;
   static constexpr int YS = CB + 8;                            // row of the sums: lanes of a group store to different banks
   static constexpr int DT = 0, Z = DT + TT * CB * 4, X = Z + TT * CB * 4, B = X + TT * CB * (int)sizeof(T), C = B + TT * NS * 4, RAW = C + TT * NS * 4;
   static constexpr int DU = STAGES * RAW, Y = DU + 2 * TT * CB * 8, BYTES = Y + 2 * TT * YS * 4;
@@ -522,31 +557,43 @@ __global__ void __launch_bounds__(THREADS) scan_tiles_kernel(const PkSelectiveSc
   };
   request(0);
   request(1);
-  request(2);
-  asm volatile("cp.async.wait_group 2;" ::: "memory");
+  asm volatile("cp.async.wait_group 1;" ::: "memory");
   __syncthreads();
   prepare(0);
   for (int i = 0; i < tiles; ++i) {
-    asm volatile("cp.async.wait_group 1;" ::: "memory");
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();                                          // dt of tile i, sums of tile i - 1, raw tile i + 1; tile i - 2 is done with
-    request(i + 3);
+    request(i + 2);
     if (i + 1 < tiles) prepare(i + 1);
     const float* B = reinterpret_cast<const float*>(raw(i) + Sh::B) + n0;
     const float* C = reinterpret_cast<const float*>(raw(i) + Sh::C) + n0;
     const float2* q = reinterpret_cast<const float2*>(du(i)) + ch;
-    float* sums = ys(i) + ch;
+    constexpr int SUB = NP > 4 ? 2 : 4;                       // tokens whose operands are in registers together
+    Token<NP> tok[2][SUB];
+    float y[TT];
+    auto load = [&](int t) {
 #pragma unroll
-    for (int tg = 0; tg < TT; tg += G) {
-      float y[G];
+      for (int j = 0; j < SUB; ++j) tok[t / SUB & 1][j].load(q + (t + j) * CB, B + (t + j) * NS, C + (t + j) * NS);
+    };
+    load(0);
 #pragma unroll
-      for (int j = 0; j < G; ++j) {
-        const float2 v = q[(tg + j) * CB];
-        y[j] = st.step(v.x, v.y, B + (tg + j) * NS, C + (tg + j) * NS);
-      }
-      float sum = group_sums<G>(y, l);
+    for (int t = 0; t < TT; t += SUB) {
+      if (t + SUB < TT) load(t + SUB);
+      st.run(tok[t / SUB & 1], y + t);
+    }
+#pragma unroll
+    for (int t = 0; t < TT; t += G) {
+      float part[G];
+#pragma unroll
+      for (int j = 0; j < G; ++j) part[j] = y[t + j];
+      float sum = group_sums<G>(part, l);
 #pragma unroll
       for (int o = G; o < LN; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-      if (l < G) sums[(tg + l) * Sh::YS] = sum;
+      y[t] = sum;
+    }
+    if (l < G) {
+#pragma unroll
+      for (int t = 0; t < TT; t += G) ys(i)[(t + l) * Sh::YS + ch] = y[t];
     }
     if (i > 0) finish(i - 1);
   }
@@ -566,8 +613,15 @@ int launch_rows(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream
 }
 
 template <typename T, int NP, int LN>
-int launch_scan(const PkSelectiveScan& p, const int4* seqs, int nseq, bool tiles, cudaStream_t stream) {
-  if (!tiles) return nseq == 1 || p.rank > 1024 ? launch_rows<T, NP, LN, 1>(p, seqs, nseq, stream) : launch_rows<T, NP, LN, 4>(p, seqs, nseq, stream);
+int launch_rows(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream_t stream) {
+  const bool fits = (size_t)4 * (((p.rank + 7) & ~7) + 2 * NP * LN) * sizeof(float) <= 48 * 1024;
+  if (nseq == 1 || !fits) return launch_rows<T, NP, LN, 1>(p, seqs, nseq, stream);
+  if (nseq <= 4) return launch_rows<T, NP, LN, 2>(p, seqs, nseq, stream);
+  return launch_rows<T, NP, LN, 4>(p, seqs, nseq, stream);
+}
+
+template <typename T, int NP, int LN>
+int launch_tiles(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream_t stream) {
   using Sh = TileShape<T, NP, LN>;
   static PkDeviceOnce once;
   if (PkDeviceOnceGuard g{once}; g.needed()) {
@@ -582,14 +636,27 @@ int launch_scan(const PkSelectiveScan& p, const int4* seqs, int nseq, bool tiles
 }
 
 template <typename T>
-int launch_scan(const PkSelectiveScan& p, const int4* seqs, int nseq, bool tiles, cudaStream_t stream) {
-  if (p.N <= 4) return launch_scan<T, 4, 1>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 8) return launch_scan<T, 4, 2>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 16) return launch_scan<T, 4, 4>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 32) return launch_scan<T, 4, 8>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 64) return launch_scan<T, 4, 16>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 128) return launch_scan<T, 4, 32>(p, seqs, nseq, tiles, stream);
-  if (p.N <= 256) return launch_scan<T, 8, 32>(p, seqs, nseq, tiles, stream);
+int launch_rows(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream_t stream) {
+  if (p.N <= 4) return launch_rows<T, 4, 1>(p, seqs, nseq, stream);
+  if (p.N <= 8) return launch_rows<T, 4, 2>(p, seqs, nseq, stream);
+  if (p.N <= 16) return launch_rows<T, 4, 4>(p, seqs, nseq, stream);
+  if (p.N <= 32) return launch_rows<T, 4, 8>(p, seqs, nseq, stream);
+  if (p.N <= 64) return launch_rows<T, 4, 16>(p, seqs, nseq, stream);
+  if (p.N <= 128) return launch_rows<T, 4, 32>(p, seqs, nseq, stream);
+  if (p.N <= 256) return launch_rows<T, 8, 32>(p, seqs, nseq, stream);
+  return PK_ERR_UNSUPPORTED;
+}
+
+// Few states per thread: every scheduler needs several warps to fill the waits of a chain of tokens.
+template <typename T>
+int launch_tiles(const PkSelectiveScan& p, const int4* seqs, int nseq, cudaStream_t stream) {
+  if (p.N <= 4) return launch_tiles<T, 2, 2>(p, seqs, nseq, stream);
+  if (p.N <= 8) return launch_tiles<T, 2, 4>(p, seqs, nseq, stream);
+  if (p.N <= 16) return launch_tiles<T, 2, 8>(p, seqs, nseq, stream);
+  if (p.N <= 32) return launch_tiles<T, 4, 8>(p, seqs, nseq, stream);
+  if (p.N <= 64) return launch_tiles<T, 4, 16>(p, seqs, nseq, stream);
+  if (p.N <= 128) return launch_tiles<T, 4, 32>(p, seqs, nseq, stream);
+  if (p.N <= 256) return launch_tiles<T, 8, 32>(p, seqs, nseq, stream);
   return PK_ERR_UNSUPPORTED;
 }
 
@@ -597,7 +664,8 @@ template <typename T, int VW>
 int launch_conv(const PkSelectiveScan& p, int rows, cudaStream_t stream) {
   const int blocks = (p.ldx + THREADS * VW - 1) / (THREADS * VW);
   int per = (int)((long long)rows * blocks / (148 * 16));
-  per = per < 1 ? 1 : per > 32 ? 32 : per;
+  const int least = rows < 64 ? 1 : 8;      // a block's first row fetches the whole window
+  per = per < least ? least : per > 32 ? 32 : per;
   const dim3 grid((rows + per - 1) / per, blocks);
   if (p.taps == 2) PK_LAUNCH_PDL((conv_kernel<T, 2, VW>), grid, dim3(THREADS), (size_t)0, stream, p, rows, per);
   else if (p.taps == 3) PK_LAUNCH_PDL((conv_kernel<T, 3, VW>), grid, dim3(THREADS), (size_t)0, stream, p, rows, per);
@@ -619,7 +687,8 @@ bool scan_ok(const PkSelectiveScan* d) {
 }
 
 bool recurrence_ok(const PkSelectiveScan* d, const void* seqs, int nseq) {
-  return scan_ok(d) && seqs != nullptr && nseq >= 1 && nseq <= 65535 && d->dbc != nullptr && d->oB >= d->rank && d->oC >= d->oB + d->N && d->ldb >= d->oC + d->N && d->dt_bias != nullptr && d->A != nullptr &&
+  return scan_ok(d) && seqs != nullptr && nseq >= 1 && nseq <= 65535 && d->dbc != nullptr && d->oB >= d->rank && d->oC >= d->oB + d->N &&
+         d->ldb >= d->oC + d->N && ((d->ldb | d->oB | d->oC) & 3) == 0 && ((uintptr_t)d->dbc & 15) == 0 && d->dt_bias != nullptr && d->A != nullptr &&
          d->skip != nullptr && d->S != nullptr && d->out != nullptr && d->ldo >= d->inner &&
          ((d->N & 3) != 0 || (((uintptr_t)d->A & 15) == 0 && ((uintptr_t)d->S & 15) == 0));
 }
@@ -640,10 +709,11 @@ PK_API int pk_scan_split(const float* d, int ldd, int rank, int kp, int rows, vo
   return PK_OK;
 }
 
-// Short portions: seqs [nseq] = {first row, tokens, slot, first position}. w_dt rows 16-byte aligned, ldw a multiple of 8.
+// Short portions: seqs [nseq] = {first row, tokens, slot, first position}. w_dt rows 16-byte aligned, ldw a multiple of 8; rows of dbc
+// and the columns oB, oC start on 16 bytes.
 PK_API int pk_scan_rows(const PkSelectiveScan* d, const void* seqs, int nseq, cudaStream_t stream) {
   if (!recurrence_ok(d, seqs, nseq) || d->w_dt == nullptr || d->ldw < ((d->rank + 7) & ~7) || (d->ldw & 7) != 0 || ((uintptr_t)d->w_dt & 15) != 0) return PK_ERR_BAD_ARG;
-  return d->f32 ? launch_scan<float>(*d, (const int4*)seqs, nseq, false, stream) : launch_scan<pk::bf16>(*d, (const int4*)seqs, nseq, false, stream);
+  return d->f32 ? launch_rows<float>(*d, (const int4*)seqs, nseq, stream) : launch_rows<pk::bf16>(*d, (const int4*)seqs, nseq, stream);
 }
 
 // Long portions, W_dt d given. Rows of dt, dbc and proj, and the columns oB, oC and oz, start on 16 bytes, rows of xc and out on four
@@ -653,5 +723,5 @@ PK_API int pk_scan_tiles(const PkSelectiveScan* d, const void* seqs, int nseq, c
   if (((d->ldt | d->ld | d->ldb | d->oB | d->oC | d->oz | d->ldx | d->ldo) & 3) != 0 || d->ldx < ((d->inner + 3) & ~3) || ((uintptr_t)d->dt & 15) != 0 ||
       ((uintptr_t)d->proj & 15) != 0 || ((uintptr_t)d->dbc & 15) != 0 || ((uintptr_t)d->xc & 15) != 0 || ((uintptr_t)d->out & 15) != 0)
     return PK_ERR_BAD_ARG;
-  return d->f32 ? launch_scan<float>(*d, (const int4*)seqs, nseq, true, stream) : launch_scan<pk::bf16>(*d, (const int4*)seqs, nseq, true, stream);
+  return d->f32 ? launch_tiles<float>(*d, (const int4*)seqs, nseq, stream) : launch_tiles<pk::bf16>(*d, (const int4*)seqs, nseq, stream);
 }
