@@ -5,8 +5,8 @@
         [--max-new-tokens N] [--temperature T] [--top-p P] [--seed S] [--mtp] [--skip-special]
 
 `safetensors` directories hold a DeepSeek-V4 checkpoint (run by the DSV4 runtime, optionally with MTP speculative
-decoding) or one of a registered architecture such as Gidisun or Pezarax (chosen by config.json); `gguf` files go through the architecture registry (MiniMax-M2, GLM-DSA). Tokenizer: a directory with
-`tokenizer.json`, the GGUF's own metadata, or `chars` (one token per character, for tiny test models).
+decoding) or one of a registered architecture such as Gidisun, Pezarax, Zemozen or Zarinex (chosen by
+config.json); `gguf` files go through the architecture registry (MiniMax-M2, GLM-DSA). Tokenizer: a directory with `tokenizer.json`, the GGUF's own metadata, or `chars` (one token per character, for tiny test models).
 """
 from __future__ import annotations
 

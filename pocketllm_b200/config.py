@@ -18,7 +18,7 @@ from typing import Any
 class ModelConfig:
     path: str = ""
     format: str = "auto"                 # auto | safetensors | gguf
-    family: str = "auto"                 # auto | qwen_hybrid | deepseek_v4 | minimax-m2 | glm-dsa | Gidisun | Pezarax
+    family: str = "auto"                 # auto | qwen_hybrid | deepseek_v4 | minimax-m2 | glm-dsa | Gidisun | Pezarax | Zemozen | Zarinex
     tokenizer: str = ""                  # directory with tokenizer.json, a GGUF file, or "chars"
     chat_format: str = "auto"            # auto | qwen | dsv4 | glm | minimax
     max_context: int = 4096
