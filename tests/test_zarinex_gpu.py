@@ -366,6 +366,31 @@ def test_decode_batches(dtype):
 
 
 @pytest.mark.parametrize("dtype", [F32, BF16])
+def test_many_short_portions_in_one_batch(dtype):
+    """Seven requests whose portions of one to eight tokens share blocks of the scan, some of them resting."""
+    from pocketllm_b200.runtime.mixer_runtime import StepEntry
+    cfg = config([scan(), forget(), scan(inner=45, state=33, rank=50)])
+    t = tensors(cfg, 15)
+    seqs = [tokens(30 + 3 * i, cfg["vocab"], 110 + i) for i in range(7)]
+    rt = runtime(cfg, t, dtype, max_requests=7, pages=7)
+    at, got, k = [0] * 7, [[] for _ in seqs], 0
+    while any(a < len(s) for a, s in zip(at, seqs)):
+        e = [StepEntry(i, s[at[i]:at[i] + 1 + (3 * i + 5 * k) % 8], ()) for i, s in enumerate(seqs) if at[i] < len(s) and (i + k) % 4]
+        k += 1
+        for x in e:
+            x.want = range(len(x.tokens))
+        z = rt.step(e).double().cpu() if e else []
+        for x in e:
+            n = len(x.tokens)
+            got[x.rid].append(z[:n])
+            z = z[n:]
+            at[x.rid] += n
+    rt.check_status()
+    for i, s in enumerate(seqs):
+        check(torch.cat(got[i]), oracle(cfg, t, s, f"short {i}"), dtype)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF16])
 def test_one_key_at_page_borders(dtype):
     """One key stands out: at page borders, at the start of the sequence and far back, in prompts, short portions and single tokens."""
     cfg = config([latent(), latent(heads=1, dim=4, vdim=13)])
