@@ -283,8 +283,8 @@ def run_mixer(args) -> dict:
     """Prefill and decode throughput of a mixer decoder (Gidisun: mLSTM, GLA and windowed latent attention with SwiGLU; Pezarax:
     retention and chunked differential attention with routed experts; Zemozen: windowed attention, and attention beside a
     state-space recurrence, with routed experts; Zarinex: selective scan, gated latent attention and HGRN2, norms behind the sums,
-    routed experts beside a shared one) at a size that resembles a real model's layers, beside the closest other model at equal size. One step = one request: prefill of `--prompt-len` tokens, then `--decode-len` greedy
-    tokens; a second figure decodes `--batch` requests together."""
+    routed experts beside a shared one) at a size that resembles a real model's layers, beside the closest other model at equal
+    size. One step = one request: prefill of `--prompt-len` tokens, then `--decode-len` greedy tokens; a second figure decodes `--batch` requests together."""
     import torch
     from pocketllm_b200.utils import bench_mixers as bm
     if args.gpus != 1:
